@@ -26,10 +26,13 @@ _UNSUPPORTED_KW = ("num_beams", "penalty_alpha", "num_return_sequences", "constr
 
 def supports(model, kwargs) -> bool:
     fam = family_for(model)
-    if fam is None or fam.engine not in ("llama", "mixtral"):
+    if fam is None or fam.engine not in ("llama", "mixtral", "latent"):
         return False
     if getattr(model, "_ipex_engine_disabled", False):
         return False
+    if fam.engine == "latent":
+        # every size and weight format of the family runs on its engine; only the request can rule it out
+        return not any(kwargs.get(k) not in (None, False, 1) for k in _UNSUPPORTED_KW)
     if getattr(getattr(model, "config", None), "ipex_alibi", False):
         return False            # linear attention biases instead of rotary positions: module path
     from .. import config as _cfg
@@ -69,12 +72,25 @@ def supports(model, kwargs) -> bool:
     return True
 
 
+def engine_class(model):
+    fam = family_for(model)
+    if fam is not None and fam.engine == "latent":
+        from .latent_engine import LatentEngine
+        return LatentEngine
+    return DecoderEngine
+
+
+def takes_stopping_criteria(model) -> bool:
+    """Engines that keep ragged batches also run the callers' stopping criteria (served batches come with both)."""
+    return getattr(engine_class(model), "ragged", False)
+
+
 def get_engine(model, batch: int, need_len: int) -> DecoderEngine:
     eng = getattr(model, "_ipex_engine", None)
     if eng is None or eng.max_batch < batch or eng.max_len < need_len:
         max_len = max(need_len, 2048)
         max_len = (max_len + 255) // 256 * 256
-        eng = DecoderEngine(model, max_batch=max(batch, 1), max_len=max_len)
+        eng = engine_class(model)(model, max_batch=max(batch, 1), max_len=max_len)
         model._ipex_engine = eng
     return eng
 
@@ -98,7 +114,8 @@ def _sample(logits, do_sample, temperature, top_k, top_p):
 
 
 @torch.no_grad()
-def engine_generate(model, input_ids, generation_config=None, streamer=None, attention_mask=None, **kwargs):
+def engine_generate(model, input_ids, generation_config=None, streamer=None, attention_mask=None,
+                    stopping_criteria=None, **kwargs):
     gc = generation_config or model.generation_config
     max_new = kwargs.get("max_new_tokens", None)
     if max_new is None:
@@ -116,7 +133,8 @@ def engine_generate(model, input_ids, generation_config=None, streamer=None, att
     if pad is None:
         pad = eos_ids[0] if eos_ids else 0
     B, S = input_ids.shape
-    if attention_mask is not None and not bool(attention_mask.all()):
+    padded = attention_mask is not None and not bool(attention_mask.all())
+    if padded and not getattr(engine_class(model), "ragged", False):
         # left-padded batches need per-row positions: use the module path
         model._ipex_engine_disabled = True
         try:
@@ -129,7 +147,7 @@ def engine_generate(model, input_ids, generation_config=None, streamer=None, att
     torch.cuda.synchronize()
     t0 = time.perf_counter()
     with nvtx_range("ipex_llm.prefill"):
-        logits = eng.prefill(input_ids)
+        logits = eng.prefill(input_ids, attention_mask) if padded else eng.prefill(input_ids)
     if rep_pen and rep_pen != 1.0:
         cuda_ops.repetition_penalty_inplace(logits, input_ids, rep_pen)
     nxt = _sample(logits, do_sample, temperature, top_k, top_p)
@@ -140,6 +158,8 @@ def engine_generate(model, input_ids, generation_config=None, streamer=None, att
     eos_t = torch.tensor(eos_ids, device=input_ids.device) if eos_ids else None
     if eos_t is not None and min_new <= 1:
         finished |= torch.isin(nxt, eos_t)
+    if stopping_criteria:
+        finished |= stopping_criteria(out[:, :S + 1], None)
     if streamer is not None:
         streamer.put(input_ids.cpu())
         streamer.put(nxt.cpu())
@@ -151,8 +171,11 @@ def engine_generate(model, input_ids, generation_config=None, streamer=None, att
     n_gen = 1
     graph_greedy = not do_sample and not (rep_pen and rep_pen != 1.0)
     step_times = []
-    check_every = 16 if streamer is None else 1
+    check_every = 16 if streamer is None and not stopping_criteria else 1
+    ends = eos_t is not None or bool(stopping_criteria)
     while n_gen < max_new:
+        if stopping_criteria and bool(finished.all()):
+            break
         ts = time.perf_counter()
         with nvtx_range("ipex_llm.decode_step"):
             eng.decode_step(B)
@@ -164,15 +187,17 @@ def engine_generate(model, input_ids, generation_config=None, streamer=None, att
                 cuda_ops.repetition_penalty_inplace(lg, out[:, :S + n_gen], rep_pen)
             nxt = _sample(lg, do_sample, temperature, top_k, top_p)
             eng.tokens[:B] = nxt
-        if eos_t is not None:
+        if ends:
             nxt = torch.where(finished, torch.full_like(nxt, pad), nxt)
-            if n_gen + 1 > min_new:
+            if eos_t is not None and n_gen + 1 > min_new:
                 finished = finished | torch.isin(nxt, eos_t)
         out[:, S + n_gen] = nxt
         n_gen += 1
+        if stopping_criteria:
+            finished = finished | stopping_criteria(out[:, :S + n_gen], None)
         if streamer is not None:
             streamer.put(nxt.cpu())
-        if eos_t is not None and (n_gen % check_every == 0) and bool(finished.all()):
+        if ends and (n_gen % check_every == 0) and bool(finished.all()):
             break
         step_times.append(time.perf_counter() - ts)
     torch.cuda.synchronize()

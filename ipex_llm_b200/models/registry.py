@@ -146,6 +146,8 @@ FAMILIES = {
        for mt, prefix in (("t5", "T5"), ("mt5", "MT5"), ("umt5", "UMT5"))},
     "rwkv": Family(pre=[R.rescale_before_quantization],
                    post=[("RwkvSelfAttention", R.rwkv4_attention_forward), ("RwkvFeedForward", R.rwkv4_ffn_forward)]),
+    # multi-head latent attention on a 32-bit residual stream: the package's own model class, all of it on its engine
+    "dobetar": Family(engine="latent"),
     # LayerNorm families without a dedicated forward file: low-bit linears + the fused LayerNorm kernel
     "gpt_neox": Family(post=[("LayerNorm", C.layer_norm_forward)]),
     "bloom": Family(post=[("LayerNorm", C.layer_norm_forward)]),

@@ -33,6 +33,13 @@ QUANTIZE_BIN = os.path.join(BIN_DIR, "ipex-quantize")
 HOST_LIB = os.path.join(HERE, "libipex_quant_core.so")
 CUDA_LIB = os.path.join(HERE, "libipex_llm_cuda.so")
 
+# Parts of the kernel library that stand on their own.  A process that needs one of them and finds no complete library
+# compiles just these sources (seconds instead of minutes); ``build_cuda`` always builds everything.
+COMPONENTS = {
+    "stream": ("elementwise.cu", "gemm_stream_tcgen05.cu", "gemv_dense.cu", "latent_attn.cu",
+               "latent_prefill_tcgen05.cu", "stream_ops.cu"),
+}
+
 NVCC_ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]
 
 
@@ -112,22 +119,35 @@ def cuda_flags(verbose=False):
     return flags
 
 
+def component_lib(name: str) -> str:
+    return os.path.join(HERE, f"libipex_llm_cuda_{name}.so")
+
+
+def build_component(name: str, force=False, verbose=False):
+    """The library of one entry of ``COMPONENTS``."""
+    return _build_cuda([os.path.join(CUDA_DIR, f) for f in COMPONENTS[name]], component_lib(name), force, verbose)
+
+
 def build_cuda(force=False, verbose=False):
+    return _build_cuda(_sources(CUDA_DIR, (".cu",)), CUDA_LIB, force, verbose)
+
+
+def _build_cuda(srcs, out, force, verbose):
     nvcc = _nvcc()
     if nvcc is None:
         raise RuntimeError("nvcc not found: cannot build the sm_100a kernels")
-    srcs = _sources(CUDA_DIR, (".cu",))
-    deps = _sources(CUDA_DIR, (".cu", ".cuh", ".h"))
+    deps = srcs + _sources(CUDA_DIR, (".cuh", ".h"))
     flags = cuda_flags(verbose)
     digest = _hash_files(deps, " ".join(f for f in flags if f != CUDA_DIR and f != "-v" and f != "-Xptxas"))
-    if not force and _stamp_ok(CUDA_LIB, digest):
-        return CUDA_LIB
+    if not force and _stamp_ok(out, digest):
+        return out
     os.makedirs(OBJ_DIR, exist_ok=True)
 
     def compile_one(src):
         obj = os.path.join(OBJ_DIR, os.path.basename(src)[:-3] + ".o")
         # per-file incremental rebuild: hash of this file + every header
-        fdig = _hash_files([src] + [d for d in deps if not d.endswith(".cu")], " ".join(flags))
+        fdig = _hash_files([src] + [d for d in deps if not d.endswith(".cu")],
+                           " ".join(f for f in flags if f != CUDA_DIR))
         if not force and os.path.exists(obj) and _stamp_ok(obj, fdig):
             return obj, ""
         cmd = [nvcc, *flags, "-c", src, "-o", obj]
@@ -144,10 +164,11 @@ def build_cuda(force=False, verbose=False):
         for (_, log), s in zip(results, srcs):
             if log:
                 print(f"== {os.path.basename(s)}\n{log}")
-    cmd = [nvcc, *NVCC_ARCH, "-shared", "-o", CUDA_LIB, *objs, "-lcuda"]
-    subprocess.check_call(cmd)
-    _write_stamp(CUDA_LIB, digest)
-    return CUDA_LIB
+    part = f"{out}.{os.getpid()}"
+    subprocess.check_call([nvcc, *NVCC_ARCH, "-shared", "-o", part, *objs, "-lcuda"])
+    os.replace(part, out)
+    _write_stamp(out, digest)
+    return out
 
 
 def build_all(force=False, verbose=False):

@@ -1,0 +1,465 @@
+// Few-row products with dense 16-bit or 32-bit weights for decoders that keep a 32-bit residual stream, sm_100a.
+//
+//   gemv_rows    y[M <= 8, N] = act( x . W[N, K]^T )   with x either activations in the weight dtype or the fp32
+//                residual stream, RMS-normed while it is staged in shared memory; the result goes out in the weight
+//                dtype, is added to an fp32 residual, or leaves as fp32 with an optional tanh soft-cap (logits)
+//   moe_router   norm + router scores in fp32 + sigmoid + top-k of one token per CTA
+//   moe_glu      per (token, choice) slot: clamped gated unit of the chosen expert, the routing weight applied to the
+//                expert's input
+//   moe_down     residual[t] += sum over the token's choices of down_e(y)
+//
+// All products are fp32 FMAs over 16-byte weight loads: with up to eight rows the weights are the traffic, and eight
+// rows of FMAs still fit under the memory time.  A warp owns R weight rows and walks K in steps of 32 vectors with
+// several loads in flight per lane.  With programmatic dependent launch the rows a warp touches first are pulled
+// into L2 while the previous kernel drains.
+#include "common/utils.cuh"
+
+namespace {
+
+constexpr int kThreads = 512;
+constexpr int kWarps = kThreads / 32;
+
+template <typename T> struct Vec {
+  static constexpr int n = 16 / sizeof(T);
+};
+
+template <typename T>
+__device__ __forceinline__ void unpack(const uint4& v, float (&f)[Vec<T>::n]) {
+  if constexpr (sizeof(T) == 4) {
+    f[0] = __uint_as_float(v.x); f[1] = __uint_as_float(v.y); f[2] = __uint_as_float(v.z); f[3] = __uint_as_float(v.w);
+  } else if constexpr (std::is_same<T, __nv_bfloat16>::value) {
+    const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      f[2 * i] = __uint_as_float(w[i] << 16);
+      f[2 * i + 1] = __uint_as_float(w[i] & 0xFFFF0000u);
+    }
+  } else {
+    const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float2 t = __half22float2(*reinterpret_cast<const __half2*>(&w[i]));
+      f[2 * i] = t.x;
+      f[2 * i + 1] = t.y;
+    }
+  }
+}
+
+// acc[m][r] += sum_k x[m][k] * w[r][k]; x in shared memory (row stride kp elements, zero-filled past K), weight rows
+// in global memory.  `vec`: K is a multiple of the vector width and the rows are 16-byte aligned.
+template <typename T, int M, int R>
+__device__ __forceinline__ void dot_rows(const T* const (&w)[R], const T* sx, int kp, int K, bool vec, int lane,
+                                         float (&acc)[M][R]) {
+  constexpr int VN = Vec<T>::n;
+  constexpr int U = R >= 4 ? 2 : 4;
+  if (vec) {
+    const int nv = K / VN;
+    for (int v0 = 0; v0 < nv; v0 += 32 * U) {
+      uint4 raw[U][R];
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int v = v0 + u * 32 + lane;
+#pragma unroll
+        for (int r = 0; r < R; ++r)
+          raw[u][r] = v < nv ? ldg_nc_v4(reinterpret_cast<const uint4*>(w[r]) + v) : make_uint4(0, 0, 0, 0);
+      }
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int v = v0 + u * 32 + lane;
+        if (v >= nv) break;
+        float wf[R][VN];
+#pragma unroll
+        for (int r = 0; r < R; ++r) unpack<T>(raw[u][r], wf[r]);
+#pragma unroll
+        for (int m = 0; m < M; ++m) {
+          float xf[VN];
+          unpack<T>(*reinterpret_cast<const uint4*>(sx + (size_t)m * kp + v * VN), xf);
+#pragma unroll
+          for (int r = 0; r < R; ++r)
+#pragma unroll
+            for (int i = 0; i < VN; ++i) acc[m][r] = fmaf(xf[i], wf[r][i], acc[m][r]);
+        }
+      }
+    }
+  } else {
+    for (int k = lane; k < K; k += 32) {
+#pragma unroll
+      for (int r = 0; r < R; ++r) {
+        const float wv = DT<T>::to_f(w[r][k]);
+#pragma unroll
+        for (int m = 0; m < M; ++m) acc[m][r] = fmaf(DT<T>::to_f(sx[(size_t)m * kp + k]), wv, acc[m][r]);
+      }
+    }
+  }
+#pragma unroll
+  for (int m = 0; m < M; ++m)
+#pragma unroll
+    for (int r = 0; r < R; ++r) acc[m][r] = warp_sum(acc[m][r]);
+}
+
+// block-wide sum (every thread gets it)
+__device__ __forceinline__ float block_sum(float v, float* red) {
+  v = warp_sum(v);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  __syncthreads();
+  if (lane == 0) red[warp] = v;
+  __syncthreads();
+  float t = lane < (int)(blockDim.x >> 5) ? red[lane] : 0.f;
+  return warp_sum(t);
+}
+
+// Stage `rows` rows: plain copy of T rows, or RMS norm of fp32 rows.  Zero fill up to kp.
+template <typename T>
+__device__ __forceinline__ void stage_rows(T* sx, int kp, const void* x, int64_t ldx, const T* norm_w, float eps,
+                                           int rows, int K, float* red) {
+  for (int m = 0; m < rows; ++m) {
+    T* dst = sx + (size_t)m * kp;
+    if (norm_w != nullptr) {
+      const float* src = reinterpret_cast<const float*>(x) + (int64_t)m * ldx;
+      float s = 0.f;
+      for (int k = threadIdx.x; k < K; k += blockDim.x) s = fmaf(src[k], src[k], s);
+      s = block_sum(s, red);
+      const float inv = 1.0f / sqrtf(s / (float)K + eps);
+      for (int k = threadIdx.x; k < K; k += blockDim.x)
+        dst[k] = DT<T>::from_f(src[k] * inv * DT<T>::to_f(norm_w[k]));
+    } else {
+      const T* src = reinterpret_cast<const T*>(x) + (int64_t)m * ldx;
+      for (int k = threadIdx.x; k < K; k += blockDim.x) dst[k] = src[k];
+    }
+    for (int k = K + threadIdx.x; k < kp; k += blockDim.x) dst[k] = DT<T>::from_f(0.f);
+  }
+  __syncthreads();
+}
+
+struct GemvRowsArgs {
+  const void* w;         // [N, K], row stride ldw
+  const void* x;         // T [M, K] or fp32 [M, K] (norm_w != null), row stride ldx
+  const void* norm_w;    // T [K] or null
+  void* out;             // out_mode 0: T [M, N]; 1: fp32, accumulated into; 2: fp32 written (soft-capped)
+  int64_t ldw, ldx, ldo;
+  float eps, softcap;
+  int M, N, K, kp;
+  int out_mode, act;     // act 1: square of relu
+  int vec;
+};
+
+template <typename T, int M, int R>
+__global__ void __launch_bounds__(kThreads) gemv_rows_kernel(GemvRowsArgs a) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  __shared__ float red[kWarps];
+  T* sx = reinterpret_cast<T*>(smem);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const T* W = reinterpret_cast<const T*>(a.w);
+  const int ntask = (a.N + R - 1) / R;
+  const int t0 = blockIdx.x * kWarps + warp;
+  pdl_launch_dependents();
+  if (a.vec && t0 < ntask && lane < R && t0 * R + lane < a.N)
+    prefetch_l2_bulk(W + (int64_t)(t0 * R + lane) * a.ldw, (uint32_t)(a.K * sizeof(T)));
+  pdl_wait();
+  stage_rows<T>(sx, a.kp, a.x, a.ldx, reinterpret_cast<const T*>(a.norm_w), a.eps, a.M, a.K, red);
+  for (int t = t0; t < ntask; t += gridDim.x * kWarps) {
+    const T* w[R];
+#pragma unroll
+    for (int r = 0; r < R; ++r) w[r] = W + (int64_t)min(t * R + r, a.N - 1) * a.ldw;
+    float acc[M][R] = {};
+    dot_rows<T, M, R>(w, sx, a.kp, a.K, a.vec != 0, lane, acc);
+#pragma unroll
+    for (int m = 0; m < M; ++m)
+#pragma unroll
+      for (int r = 0; r < R; ++r) {
+        const int n = t * R + r;
+        if (lane == ((m * R + r) & 31) && m < a.M && n < a.N) {
+          float v = acc[m][r];
+          if (a.act == 1) v = v > 0.f ? v * v : 0.f;
+          if (a.out_mode == 0) {
+            reinterpret_cast<T*>(a.out)[(int64_t)m * a.ldo + n] = DT<T>::from_f(v);
+          } else {
+            float* o = reinterpret_cast<float*>(a.out) + (int64_t)m * a.ldo + n;
+            if (a.out_mode == 1) *o += v;
+            else *o = a.softcap > 0.f ? a.softcap * tanhf(v / a.softcap) : v;
+          }
+        }
+      }
+  }
+}
+
+int sm_count() {
+  static int sms = [] {
+    int dev = 0, n = 148;
+    cudaGetDevice(&dev);
+    cudaDeviceGetAttribute(&n, cudaDevAttrMultiProcessorCount, dev);
+    return n;
+  }();
+  return sms;
+}
+
+template <typename T, int M, int R>
+cudaError_t launch_gemv(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
+  auto kern = gemv_rows_kernel<T, M, R>;
+  const size_t smem = (size_t)M * a.kp * sizeof(T);      // rows past a.M are read (and dropped), never used
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return e;
+  }
+  const int ntask = (a.N + R - 1) / R;
+  const int per_sm = smem > 100 * 1024 ? 1 : 2;
+  const int want = (ntask + kWarps - 1) / kWarps, cap = sm_count() * per_sm;
+  return launch_kernel(kern, dim3(want < cap ? want : cap), dim3(kThreads), smem, st, pdl, a);
+}
+
+template <typename T, int M>
+cudaError_t pick_rows(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
+  const int warps = sm_count() * kWarps;
+  if (a.N >= 4 * warps) return launch_gemv<T, M, 4>(a, pdl, st);
+  if (a.N >= warps) return launch_gemv<T, M, 2>(a, pdl, st);
+  return launch_gemv<T, M, 1>(a, pdl, st);
+}
+
+template <typename T>
+cudaError_t pick_m(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
+  if (a.M == 1) return pick_rows<T, 1>(a, pdl, st);
+  if (a.M == 2) return pick_rows<T, 2>(a, pdl, st);
+  if (a.M <= 4) return pick_rows<T, 4>(a, pdl, st);
+  return pick_rows<T, 8>(a, pdl, st);
+}
+
+// ------------------------------------------------------------------------------------------------ mixture of experts
+struct RouterArgs {
+  const float* x;        // residual stream [tokens, K]
+  const void* norm_w;
+  const void* w;         // [E, K]
+  float* weights;        // [tokens, k]
+  int64_t* idx;          // [tokens, k]
+  int64_t ldx;
+  float eps;
+  int K, E, k;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(kThreads) moe_router_kernel(RouterArgs a) {
+  extern __shared__ __align__(16) float sh[];      // [K] normed row, [E] scores
+  __shared__ float red[kWarps];
+  float* h = sh;
+  float* sc = sh + a.K;
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  pdl_launch_dependents();
+  pdl_wait();
+  const float* src = a.x + (int64_t)t * a.ldx;
+  float s = 0.f;
+  for (int k = threadIdx.x; k < a.K; k += kThreads) {
+    const float v = src[k];
+    h[k] = v;
+    s = fmaf(v, v, s);
+  }
+  s = block_sum(s, red);
+  const float inv = 1.0f / sqrtf(s / (float)a.K + a.eps);
+  const T* nw = reinterpret_cast<const T*>(a.norm_w);
+  for (int k = threadIdx.x; k < a.K; k += kThreads) h[k] *= inv * DT<T>::to_f(nw[k]);
+  __syncthreads();
+  for (int e = warp; e < a.E; e += kWarps) {
+    const T* w = reinterpret_cast<const T*>(a.w) + (int64_t)e * a.K;
+    float acc = 0.f;
+    for (int k = lane; k < a.K; k += 32) acc = fmaf(h[k], DT<T>::to_f(w[k]), acc);
+    acc = warp_sum(acc);
+    if (lane == 0) sc[e] = 1.0f / (1.0f + expf(-acc));
+  }
+  __syncthreads();
+  if (warp == 0) {
+    for (int r = 0; r < a.k; ++r) {
+      float best = -1.f;
+      int bi = 0x7fffffff;
+      for (int e = lane; e < a.E; e += 32)
+        if (sc[e] > best) { best = sc[e]; bi = e; }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+        if (ov > best || (ov == best && oi < bi)) { best = ov; bi = oi; }
+      }
+      if (bi >= a.E) { bi = 0; best = 0.f; }       // scores that are not numbers
+      if (lane == 0) {
+        a.weights[(int64_t)t * a.k + r] = best;
+        a.idx[(int64_t)t * a.k + r] = bi;
+        sc[bi] = -2.f;
+      }
+      __syncwarp();
+    }
+  }
+}
+
+struct MoeArgs {
+  const float* x;          // glu: residual stream [tokens, K]
+  const void* norm_w;
+  const void* w;           // glu: [E, 2I, K]; down: [E, N, I]
+  const void* y_in;        // down: [tokens * k, I]
+  void* out;               // glu: T [tokens * k, I]; down: fp32 residual [tokens, N], accumulated into
+  const float* weights;    // [tokens, k]
+  const int64_t* idx;      // [tokens, k]
+  int64_t ldx, ldo;
+  float eps, limit, alpha;
+  int K, I, E, k, kp;
+  int interleaved;         // gate / up rows in alternating 16-row tiles, else gate rows then up rows
+  int vec;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(kThreads) moe_glu_kernel(MoeArgs a) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  __shared__ float red[kWarps];
+  T* sx = reinterpret_cast<T*>(smem);
+  const int slot = blockIdx.y, t = slot / a.k;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int e = (int)a.idx[slot];
+  stage_rows<T>(sx, a.kp, a.x + (int64_t)t * a.ldx, 0, reinterpret_cast<const T*>(a.norm_w), a.eps, 1, a.K, red);
+  const T* W = reinterpret_cast<const T*>(a.w) + (int64_t)e * 2 * a.I * a.K;
+  const float rw = a.weights[slot];
+  for (int i = blockIdx.x * kWarps + warp; i < a.I; i += gridDim.x * kWarps) {
+    const int g = a.interleaved ? (i >> 4) * 32 + (i & 15) : i;
+    const int u = a.interleaved ? g + 16 : a.I + i;
+    const T* w[2] = {W + (int64_t)g * a.K, W + (int64_t)u * a.K};
+    float acc[1][2] = {};
+    dot_rows<T, 1, 2>(w, sx, a.kp, a.K, a.vec != 0, lane, acc);
+    if (lane == 0) {
+      const float gv = fminf(acc[0][0] * rw, a.limit);
+      const float uv = fminf(fmaxf(acc[0][1] * rw, -a.limit), a.limit);
+      const float y = gv / (1.0f + expf(-a.alpha * gv)) * (uv + 1.0f);
+      reinterpret_cast<T*>(a.out)[(int64_t)slot * a.I + i] = DT<T>::from_f(y);
+    }
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kThreads) moe_down_kernel(MoeArgs a) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  __shared__ float red[kWarps];
+  T* sx = reinterpret_cast<T*>(smem);
+  const int t = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  pdl_launch_dependents();
+  pdl_wait();
+  stage_rows<T>(sx, a.kp, reinterpret_cast<const T*>(a.y_in) + (int64_t)t * a.k * a.I, a.I, (const T*)nullptr, 0.f,
+                a.k, a.I, red);
+  const int N = a.K;
+  for (int n2 = blockIdx.x * kWarps + warp; n2 * 2 < N; n2 += gridDim.x * kWarps) {
+    const int n = n2 * 2;
+    float s0 = 0.f, s1 = 0.f;
+    for (int j = 0; j < a.k; ++j) {
+      const int64_t e = a.idx[(int64_t)t * a.k + j];
+      const T* We = reinterpret_cast<const T*>(a.w) + e * (int64_t)N * a.I;
+      const T* w[2] = {We + (int64_t)n * a.I, We + (int64_t)min(n + 1, N - 1) * a.I};
+      float acc[1][2] = {};
+      dot_rows<T, 1, 2>(w, sx + (size_t)j * a.kp, a.kp, a.I, a.vec != 0, lane, acc);
+      s0 += acc[0][0];
+      s1 += acc[0][1];
+    }
+    float* o = reinterpret_cast<float*>(a.out) + (int64_t)t * a.ldo + n;
+    if (lane == 0) o[0] += s0;
+    if (lane == 1 && n + 1 < N) o[1] += s1;
+  }
+}
+
+template <typename T>
+int padded(int K) { return (K + Vec<T>::n - 1) / Vec<T>::n * Vec<T>::n; }
+
+template <typename T>
+int vec_ok(const void* p, int64_t ld, int K) {
+  return (reinterpret_cast<uintptr_t>(p) & 15) == 0 && ld % Vec<T>::n == 0 && K % Vec<T>::n == 0;
+}
+
+template <typename K>
+cudaError_t allow_smem(K kern, size_t smem) {
+  if (smem <= 48 * 1024) return cudaSuccess;
+  if (smem > 226 * 1024) return cudaErrorInvalidValue;
+  return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+}
+
+template <typename F>
+int by_dtype(int dtype, F&& f) {
+  if (dtype == DT_F16) return (int)f((__half*)nullptr);
+  if (dtype == DT_BF16) return (int)f((__nv_bfloat16*)nullptr);
+  if (dtype == DT_F32) return (int)f((float*)nullptr);
+  return (int)cudaErrorInvalidValue;
+}
+
+}  // namespace
+
+// Rows of x one call may take: the staged rows must fit shared memory.
+IPEX_API int ipex_gemv_rows_max(int K, int dtype) {
+  const int64_t row = ((int64_t)K + 8) * (dtype == DT_F32 ? 4 : 2);
+  const int64_t m = (200 * 1024) / row;
+  return m >= 8 ? 8 : m >= 4 ? 4 : m >= 2 ? 2 : (int)m;
+}
+
+// y = act(x . W^T): see GemvRowsArgs.  M <= ipex_gemv_rows_max(K, dtype).
+IPEX_API int ipex_gemv_rows(const void* w, int64_t ldw, const void* x, int64_t ldx, const void* norm_w, float eps,
+                            void* out, int64_t ldo, int M, int N, int K, int out_mode, int act, float softcap, int dtype,
+                            int pdl, void* stream) {
+  if (M < 1 || N < 1 || K < 1 || out_mode < 0 || out_mode > 2 || M > ipex_gemv_rows_max(K, dtype))
+    return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    GemvRowsArgs a = {w, x, norm_w, out, ldw, ldx, ldo, eps, softcap, M, N, K, padded<T>(K), out_mode, act, 0};
+    a.vec = vec_ok<T>(w, ldw, K);
+    return pick_m<T>(a, pdl != 0, (cudaStream_t)stream);
+  });
+}
+
+// Router of `tokens` rows of the residual stream: weights = the k largest sigmoid scores, idx = their experts
+// (descending score, the lower index first among equals).
+IPEX_API int ipex_moe_router_sigmoid(const float* x, int64_t ldx, const void* norm_w, float eps, const void* w,
+                                     float* weights, int64_t* idx, int tokens, int K, int E, int k, int dtype, int pdl,
+                                     void* stream) {
+  if (tokens < 1 || K < 1 || E < 1 || k < 1 || k > E) return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    RouterArgs a = {x, norm_w, w, weights, idx, ldx, eps, K, E, k};
+    const size_t smem = ((size_t)K + E) * sizeof(float);
+    cudaError_t e = allow_smem(moe_router_kernel<T>, smem);
+    if (e != cudaSuccess) return e;
+    return launch_kernel(moe_router_kernel<T>, dim3(tokens), dim3(kThreads), smem, (cudaStream_t)stream, pdl != 0, a);
+  });
+}
+
+// First half of the experts for `tokens` rows: y[token * k + j] = g * sigmoid(alpha g) * (u + 1), g = min(gate, limit),
+// u = clamp(up, +-limit), gate / up of expert idx[token, j] on weight * norm(x).
+IPEX_API int ipex_moe_glu_rows(const float* x, int64_t ldx, const void* norm_w, float eps, const void* w, void* y,
+                               const float* weights, const int64_t* idx, int tokens, int K, int I, int E, int k,
+                               float limit, float alpha, int interleaved, int dtype, int pdl, void* stream) {
+  if (tokens < 1 || K < 1 || I < 1 || k < 1 || (int64_t)tokens * k > 65535 || (interleaved && I % 16 != 0))
+    return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    MoeArgs a = {};
+    a.x = x; a.norm_w = norm_w; a.w = w; a.out = y; a.weights = weights; a.idx = idx; a.ldx = ldx; a.eps = eps;
+    a.limit = limit; a.alpha = alpha; a.K = K; a.I = I; a.E = E; a.k = k; a.kp = padded<T>(K);
+    a.interleaved = interleaved;
+    a.vec = vec_ok<T>(w, K, K);
+    const size_t smem = (size_t)a.kp * sizeof(T);
+    cudaError_t e = allow_smem(moe_glu_kernel<T>, smem);
+    if (e != cudaSuccess) return e;
+    const int slots = tokens * k, want = (I + kWarps - 1) / kWarps;
+    const int cap = (sm_count() * 4 + slots - 1) / slots;
+    return launch_kernel(moe_glu_kernel<T>, dim3(want < cap ? want : cap, slots), dim3(kThreads), smem,
+                         (cudaStream_t)stream, pdl != 0, a);
+  });
+}
+
+// Second half: residual[token] += sum_j down_{idx[token, j]}(y[token * k + j]).
+IPEX_API int ipex_moe_down_rows(const void* y, const void* w, float* residual, int64_t ldr, const int64_t* idx,
+                                int tokens, int N, int I, int E, int k, int dtype, int pdl, void* stream) {
+  if (tokens < 1 || tokens > 65535 || N < 1 || I < 1 || k < 1) return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    MoeArgs a = {};
+    a.y_in = y; a.w = w; a.out = residual; a.idx = idx; a.ldo = ldr; a.K = N; a.I = I; a.E = E; a.k = k;
+    a.kp = padded<T>(I);
+    a.vec = vec_ok<T>(w, I, I);
+    const size_t smem = (size_t)a.kp * k * sizeof(T);
+    cudaError_t e = allow_smem(moe_down_kernel<T>, smem);
+    if (e != cudaSuccess) return e;
+    const int want = (N / 2 + kWarps) / kWarps, cap = (sm_count() * 4 + tokens - 1) / tokens;
+    return launch_kernel(moe_down_kernel<T>, dim3(want < cap ? want : cap, tokens), dim3(kThreads), smem,
+                         (cudaStream_t)stream, pdl != 0, a);
+  });
+}

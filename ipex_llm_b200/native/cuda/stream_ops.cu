@@ -1,0 +1,397 @@
+// Element-wise and routing kernels of decoders with a 32-bit residual stream, sm_100a: embedding (scaled, with an
+// optional bigram table), RMS norm of the stream into the activation dtype, tanh soft-cap of fp32 logits, and the
+// data movement around a dense expert bank for prompts (slots grouped by expert on the device, row gather, clamped
+// gated unit, combination into the stream), plus a plain tiled product for sizes the tensor-core kernels do not take
+// and for 32-bit models.
+#include "common/utils.cuh"
+
+namespace {
+
+template <typename F>
+int by_dtype(int dtype, F&& f) {
+  if (dtype == DT_F16) return (int)f((__half*)nullptr);
+  if (dtype == DT_BF16) return (int)f((__nv_bfloat16*)nullptr);
+  if (dtype == DT_F32) return (int)f((float*)nullptr);
+  return (int)cudaErrorInvalidValue;
+}
+
+__device__ __forceinline__ float block_sum(float v, float* red) {
+  v = warp_sum(v);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  __syncthreads();
+  if (lane == 0) red[warp] = v;
+  __syncthreads();
+  float t = lane < (int)(blockDim.x >> 5) ? red[lane] : 0.f;
+  return warp_sum(t);
+}
+
+// One CTA per token.  The token id is filed in the history [slots, cap] at its position; the bigram row needs the
+// token before it, which is either the neighbouring entry of this launch or already in the history.
+template <typename T>
+__global__ void embed_stream_kernel(const int64_t* __restrict__ tokens, const int* __restrict__ slot,
+                                    const int* __restrict__ pos, const int* __restrict__ start, int* history,
+                                    int64_t cap, const T* __restrict__ table, const T* __restrict__ bigram,
+                                    float* __restrict__ out, int W, int64_t vocab, float scale, int64_t buckets,
+                                    int64_t mul_prev, int64_t mul_cur) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x;
+  int64_t tok = tokens[t];
+  tok = tok < 0 ? 0 : (tok >= vocab ? vocab - 1 : tok);
+  const int s = slot[t], p = pos[t];
+  int64_t row = -1;
+  if (bigram != nullptr) {
+    row = buckets;
+    if (p > start[s]) {
+      int64_t prev;
+      if (t > 0 && slot[t - 1] == s && pos[t - 1] == p - 1) prev = tokens[t - 1];
+      else prev = history[(int64_t)s * cap + p - 1];
+      row = (prev * mul_prev + tok * mul_cur) % buckets;
+      if (row < 0) row += buckets;
+    }
+  }
+  if (threadIdx.x == 0) history[(int64_t)s * cap + p] = (int)tok;
+  const T* e = table + tok * W;
+  const T* b = bigram + (row < 0 ? 0 : row) * W;
+  float* o = out + (int64_t)t * W;
+  for (int i = threadIdx.x; i < W; i += blockDim.x) {
+    float v = DT<T>::to_f(e[i]) * scale;
+    if (row >= 0) v += DT<T>::to_f(b[i]);
+    o[i] = v;
+  }
+}
+
+template <typename T>
+__global__ void norm_stream_kernel(const float* __restrict__ x, int64_t ldx, const T* __restrict__ w,
+                                   T* __restrict__ out, int64_t ldo, const int* __restrict__ rows, int K, float eps) {
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t r = rows != nullptr ? rows[blockIdx.x] : (int)blockIdx.x;
+  const float* src = x + r * ldx;
+  T* dst = out + (int64_t)blockIdx.x * ldo;
+  float s = 0.f;
+  const bool v4 = K % 4 == 0 && ldx % 4 == 0;
+  if (v4) {
+    for (int k = threadIdx.x; k < K / 4; k += blockDim.x) {
+      const float4 f = reinterpret_cast<const float4*>(src)[k];
+      s += f.x * f.x + f.y * f.y + f.z * f.z + f.w * f.w;
+    }
+  } else {
+    for (int k = threadIdx.x; k < K; k += blockDim.x) s = fmaf(src[k], src[k], s);
+  }
+  s = block_sum(s, red);
+  const float inv = 1.0f / sqrtf(s / (float)K + eps);
+  if (v4 && ldo % 4 == 0) {
+    for (int k = threadIdx.x; k < K / 4; k += blockDim.x) {
+      const float4 f = reinterpret_cast<const float4*>(src)[k];
+      __align__(16) T o[4];
+      o[0] = DT<T>::from_f(f.x * inv * DT<T>::to_f(w[4 * k]));
+      o[1] = DT<T>::from_f(f.y * inv * DT<T>::to_f(w[4 * k + 1]));
+      o[2] = DT<T>::from_f(f.z * inv * DT<T>::to_f(w[4 * k + 2]));
+      o[3] = DT<T>::from_f(f.w * inv * DT<T>::to_f(w[4 * k + 3]));
+      if constexpr (sizeof(T) == 2) reinterpret_cast<uint2*>(dst)[k] = *reinterpret_cast<const uint2*>(o);
+      else reinterpret_cast<uint4*>(dst)[k] = *reinterpret_cast<const uint4*>(o);
+    }
+  } else {
+    for (int k = threadIdx.x; k < K; k += blockDim.x) dst[k] = DT<T>::from_f(src[k] * inv * DT<T>::to_f(w[k]));
+  }
+}
+
+__global__ void softcap_kernel(float* x, int64_t n, float cap) {
+  const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < n) x[i] = cap * tanhf(x[i] / cap);
+}
+
+// x += y for a row-major y of the activation dtype (packed-weight projections, whose kernels write 16 bits)
+template <typename T>
+__global__ void add_stream_kernel(float* __restrict__ x, const T* __restrict__ y, int64_t n) {
+  const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < n) x[i] += DT<T>::to_f(y[i]);
+}
+
+template <typename T>
+__global__ void relu2_kernel(T* x, int64_t n) {
+  const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < n) {
+    const float v = fmaxf(DT<T>::to_f(x[i]), 0.f);
+    x[i] = DT<T>::from_f(v * v);
+  }
+}
+
+// ---------------------------------------------------------------------------------------------- routing for prompts
+// fp32 router logits [tokens, E] -> the k largest sigmoid scores and their experts; a warp per token.
+__global__ void sigmoid_topk_kernel(const float* __restrict__ logits, int64_t ld, float* __restrict__ w,
+                                    int64_t* __restrict__ idx, int tokens, int E, int k) {
+  extern __shared__ float sh[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, wpb = blockDim.x >> 5;
+  const int t = blockIdx.x * wpb + warp;
+  if (t >= tokens) return;
+  float* sc = sh + (size_t)warp * E;
+  for (int e = lane; e < E; e += 32) sc[e] = 1.0f / (1.0f + expf(-logits[(int64_t)t * ld + e]));
+  __syncwarp();
+  for (int r = 0; r < k; ++r) {
+    float best = -1.f;
+    int bi = 0x7fffffff;
+    for (int e = lane; e < E; e += 32)
+      if (sc[e] > best) { best = sc[e]; bi = e; }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, best, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (ov > best || (ov == best && oi < bi)) { best = ov; bi = oi; }
+    }
+    if (bi >= E) { bi = 0; best = 0.f; }
+    if (lane == 0) {
+      w[(int64_t)t * k + r] = best;
+      idx[(int64_t)t * k + r] = bi;
+      sc[bi] = -2.f;
+    }
+    __syncwarp();
+  }
+}
+
+// (token, choice) slots grouped by expert, one CTA: order[pos] = slot, inverse[slot] = pos, ranges[e] = (first, count).
+// The order inside an expert is arbitrary (every row is computed on its own).
+__global__ void __launch_bounds__(1024) group_slots_kernel(const int64_t* __restrict__ ids, int slots, int E,
+                                                           int* __restrict__ order, int* __restrict__ inverse,
+                                                           int* __restrict__ ranges) {
+  extern __shared__ int cnt[];        // [E] counts, then next free position
+  for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
+  __syncthreads();
+  for (int s = threadIdx.x; s < slots; s += blockDim.x) atomicAdd(&cnt[(int)ids[s]], 1);
+  __syncthreads();
+  if (threadIdx.x < 32) {             // exclusive prefix over the experts, one warp
+    int run = 0;
+    for (int e0 = 0; e0 < E; e0 += 32) {
+      const int e = e0 + threadIdx.x;
+      const int c = e < E ? cnt[e] : 0;
+      int p = c;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int v = __shfl_up_sync(0xffffffffu, p, o);
+        if ((int)threadIdx.x >= o) p += v;
+      }
+      if (e < E) {
+        ranges[2 * e] = run + p - c;
+        ranges[2 * e + 1] = c;
+        cnt[e] = run + p - c;
+      }
+      run += __shfl_sync(0xffffffffu, p, 31);
+    }
+  }
+  __syncthreads();
+  for (int s = threadIdx.x; s < slots; s += blockDim.x) {
+    const int p = atomicAdd(&cnt[(int)ids[s]], 1);
+    order[p] = s;
+    inverse[s] = p;
+  }
+}
+
+// xs[pos] = x[order[pos] / k], ws[pos] = w[order[pos]]
+template <typename T>
+__global__ void gather_slots_kernel(const T* __restrict__ x, const float* __restrict__ w, const int* __restrict__ order,
+                                    T* __restrict__ xs, float* __restrict__ ws, int K, int k) {
+  const int p = blockIdx.x, s = order[p];
+  const T* src = x + (int64_t)(s / k) * K;
+  T* dst = xs + (int64_t)p * K;
+  if (K % (16 / (int)sizeof(T)) == 0) {
+    const int nv = K * (int)sizeof(T) / 16;
+    for (int i = threadIdx.x; i < nv; i += blockDim.x)
+      reinterpret_cast<uint4*>(dst)[i] = reinterpret_cast<const uint4*>(src)[i];
+  } else {
+    for (int i = threadIdx.x; i < K; i += blockDim.x) dst[i] = src[i];
+  }
+  if (threadIdx.x == 0) ws[p] = w[s];
+}
+
+// y = g * sigmoid(alpha g) * (u + 1) with g = min(ws * gate, limit), u = clamp(ws * up, +-limit); gu fp32 [rows, 2I]
+template <typename T>
+__global__ void glu_rows_kernel(const float* __restrict__ gu, const float* __restrict__ ws, T* __restrict__ y, int I,
+                                float limit, float alpha, int interleaved) {
+  const int r = blockIdx.x;
+  const float w = ws[r];
+  const float* row = gu + (int64_t)r * 2 * I;
+  for (int i = threadIdx.x; i < I; i += blockDim.x) {
+    const int gi = interleaved ? (i >> 4) * 32 + (i & 15) : i;
+    const int ui = interleaved ? gi + 16 : I + i;
+    const float g = fminf(row[gi] * w, limit);
+    const float u = fminf(fmaxf(row[ui] * w, -limit), limit);
+    y[(int64_t)r * I + i] = DT<T>::from_f(g / (1.0f + expf(-alpha * g)) * (u + 1.0f));
+  }
+}
+
+// residual[t] += sum_j y[inverse[t * k + j]]
+template <typename T>
+__global__ void combine_slots_kernel(const T* __restrict__ y, const int* __restrict__ inverse,
+                                     float* __restrict__ residual, int N, int k) {
+  const int t = blockIdx.x;
+  float* o = residual + (int64_t)t * N;
+  for (int n = threadIdx.x; n < N; n += blockDim.x) {
+    float s = 0.f;
+    for (int j = 0; j < k; ++j) s += DT<T>::to_f(y[(int64_t)inverse[(int64_t)t * k + j] * N + n]);
+    o[n] += s;
+  }
+}
+
+// ------------------------------------------------------------------------------------------- plain tiled product
+// out[m, n] (fp32 or T) = sum_k x[m, k] w[n, k], 64 x 64 tiles, fp32 FMAs; with ranges, group g multiplies its rows
+// [ranges[g][0], + ranges[g][1]) of x by weight matrix g.
+template <typename T, typename TO>
+__global__ void __launch_bounds__(256) gemm_plain_kernel(const T* __restrict__ x, const T* __restrict__ w,
+                                                         TO* __restrict__ out, const int* __restrict__ ranges, int M,
+                                                         int N, int K) {
+  __shared__ float sa[16][65], sb[16][65];
+  int row0 = 0;
+  if (ranges != nullptr) {
+    row0 = ranges[2 * blockIdx.z];
+    M = ranges[2 * blockIdx.z + 1];
+    w += (int64_t)blockIdx.z * N * K;
+  }
+  const int n0 = blockIdx.x * 64, tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  for (int m0 = blockIdx.y * 64; m0 < M; m0 += gridDim.y * 64) {
+    float acc[4][4] = {};
+    for (int k0 = 0; k0 < K; k0 += 16) {
+      for (int i = threadIdx.x; i < 1024; i += 256) {
+        const int kk = i & 15, r = i >> 4;
+        const int k = k0 + kk;
+        sa[kk][r] = (m0 + r < M && k < K) ? DT<T>::to_f(x[(int64_t)(row0 + m0 + r) * K + k]) : 0.f;
+        sb[kk][r] = (n0 + r < N && k < K) ? DT<T>::to_f(w[(int64_t)(n0 + r) * K + k]) : 0.f;
+      }
+      __syncthreads();
+#pragma unroll
+      for (int kk = 0; kk < 16; ++kk) {
+        float av[4], bv[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) { av[i] = sa[kk][ty + 16 * i]; bv[i] = sb[kk][tx + 16 * i]; }
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
+      }
+      __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int m = m0 + ty + 16 * i, n = n0 + tx + 16 * j;
+        if (m < M && n < N) out[(int64_t)(row0 + m) * N + n] = DT<TO>::from_f(acc[i][j]);
+      }
+  }
+}
+
+}  // namespace
+
+// out[t] = table[token] * scale (+ bigram row), fp32.  history: int32 [slots, cap]; start: int32 [slots], the position
+// of each sequence's first token.  bigram may be null (buckets etc. are ignored then).
+IPEX_API int ipex_embed_stream(const int64_t* tokens, const int* slot, const int* pos, const int* start, int* history,
+                               int64_t cap, const void* table, const void* bigram, float* out, int n, int W,
+                               int64_t vocab, float scale, int64_t buckets, int64_t mul_prev, int64_t mul_cur, int dtype,
+                               int pdl, void* stream) {
+  if (n < 1 || W < 1 || (bigram != nullptr && buckets < 1)) return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    return launch_kernel(embed_stream_kernel<T>, dim3(n), dim3(256), 0, (cudaStream_t)stream, pdl != 0, tokens, slot,
+                         pos, start, history, cap, (const T*)table, (const T*)bigram, out, W, vocab, scale, buckets,
+                         mul_prev, mul_cur);
+  });
+}
+
+// out[i] = RMS norm of row rows[i] (or i) of the fp32 stream, in the activation dtype.
+IPEX_API int ipex_norm_stream(const float* x, int64_t ldx, const void* w, void* out, int64_t ldo, const int* rows, int n,
+                              int K, float eps, int dtype, int pdl, void* stream) {
+  if (n < 1 || K < 1) return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    return launch_kernel(norm_stream_kernel<T>, dim3(n), dim3(256), 0, (cudaStream_t)stream, pdl != 0, x, ldx,
+                         (const T*)w, (T*)out, ldo, rows, K, eps);
+  });
+}
+
+IPEX_API int ipex_softcap_f32(float* x, int64_t n, float cap, void* stream) {
+  if (n < 1 || !(cap > 0.f)) return (int)cudaErrorInvalidValue;
+  softcap_kernel<<<(unsigned)((n + 255) / 256), 256, 0, (cudaStream_t)stream>>>(x, n, cap);
+  return (int)cudaGetLastError();
+}
+
+IPEX_API int ipex_add_stream(float* x, const void* y, int64_t n, int dtype, void* stream) {
+  if (n < 1) return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    add_stream_kernel<T><<<(unsigned)((n + 255) / 256), 256, 0, (cudaStream_t)stream>>>(x, (const T*)y, n);
+    return cudaGetLastError();
+  });
+}
+
+IPEX_API int ipex_relu2_inplace(void* x, int64_t n, int dtype, void* stream) {
+  if (n < 1) return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    relu2_kernel<T><<<(unsigned)((n + 255) / 256), 256, 0, (cudaStream_t)stream>>>((T*)x, n);
+    return cudaGetLastError();
+  });
+}
+
+IPEX_API int ipex_moe_sigmoid_topk(const float* logits, int64_t ld, float* w, int64_t* idx, int tokens, int E, int k,
+                                   void* stream) {
+  if (tokens < 1 || E < 1 || E > 3000 || k < 1 || k > E) return (int)cudaErrorInvalidValue;
+  sigmoid_topk_kernel<<<(tokens + 3) / 4, 128, (size_t)4 * E * sizeof(float), (cudaStream_t)stream>>>(
+      logits, ld, w, idx, tokens, E, k);
+  return (int)cudaGetLastError();
+}
+
+// Expert ids must lie in [0, E).
+IPEX_API int ipex_moe_group_slots(const int64_t* ids, int slots, int E, int* order, int* inverse, int* ranges,
+                                  void* stream) {
+  if (slots < 1 || E < 1 || E > 12000) return (int)cudaErrorInvalidValue;
+  group_slots_kernel<<<1, 1024, (size_t)E * sizeof(int), (cudaStream_t)stream>>>(ids, slots, E, order, inverse, ranges);
+  return (int)cudaGetLastError();
+}
+
+IPEX_API int ipex_moe_gather_slots(const void* x, const float* w, const int* order, void* xs, float* ws, int slots,
+                                   int K, int k, int dtype, void* stream) {
+  if (slots < 1 || K < 1 || k < 1) return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    gather_slots_kernel<T><<<slots, 128, 0, (cudaStream_t)stream>>>((const T*)x, w, order, (T*)xs, ws, K, k);
+    return cudaGetLastError();
+  });
+}
+
+IPEX_API int ipex_moe_glu_from_gu(const float* gu, const float* ws, void* y, int rows, int I, float limit, float alpha,
+                                  int interleaved, int dtype, void* stream) {
+  if (rows < 1 || I < 1 || (interleaved && I % 16 != 0)) return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    glu_rows_kernel<T><<<rows, 128, 0, (cudaStream_t)stream>>>(gu, ws, (T*)y, I, limit, alpha, interleaved);
+    return cudaGetLastError();
+  });
+}
+
+IPEX_API int ipex_moe_combine_slots(const void* y, const int* inverse, float* residual, int tokens, int N, int k,
+                                    int dtype, void* stream) {
+  if (tokens < 1 || N < 1 || k < 1) return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    combine_slots_kernel<T><<<tokens, 256, 0, (cudaStream_t)stream>>>((const T*)y, inverse, residual, N, k);
+    return cudaGetLastError();
+  });
+}
+
+// out = x . w^T with contiguous operands; ranges (device, [groups][2]) may be null (groups = 1).  out_f32: fp32 output.
+IPEX_API int ipex_gemm_plain(const void* x, const void* w, void* out, const int* ranges, int groups, int M, int N, int K,
+                             int out_f32, int dtype, void* stream) {
+  if (M < 1 || N < 1 || K < 1 || groups < 1 || groups > 65535) return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    const int mt = (M + 63) / 64;
+    dim3 grid((N + 63) / 64, mt < 1024 ? mt : 1024, groups);
+    cudaStream_t st = (cudaStream_t)stream;
+    if (out_f32)
+      gemm_plain_kernel<T, float><<<grid, 256, 0, st>>>((const T*)x, (const T*)w, (float*)out, ranges, M, N, K);
+    else
+      gemm_plain_kernel<T, T><<<grid, 256, 0, st>>>((const T*)x, (const T*)w, (T*)out, ranges, M, N, K);
+    return cudaGetLastError();
+  });
+}

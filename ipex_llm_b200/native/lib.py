@@ -19,6 +19,7 @@ from . import build as _build
 _lock = threading.Lock()
 _host = None
 _cuda = None
+_stream = None
 
 c_void_p = ctypes.c_void_p
 c_int = ctypes.c_int
@@ -91,6 +92,24 @@ def cuda_lib() -> ctypes.CDLL:
                 cuda_api.declare(lib)
                 _cuda = lib
     return _cuda
+
+
+def stream_lib() -> ctypes.CDLL:
+    """The kernels of the "stream" component: the complete library when it is there and has them, else the component's
+    own library, built on first use."""
+    global _stream
+    if _stream is None:
+        if os.path.exists(os.environ.get("IPEX_LLM_CUDA_LIB") or _build.CUDA_LIB):
+            lib = cuda_lib()
+        else:
+            lib = None
+        if lib is None or not hasattr(lib, "ipex_gemm_stream"):
+            with _lock:
+                lib = ctypes.CDLL(_build.build_component("stream"))
+        from . import cuda_api
+        cuda_api.declare_stream(lib)
+        _stream = lib
+    return _stream
 
 
 def ptr(t) -> ctypes.c_void_p:

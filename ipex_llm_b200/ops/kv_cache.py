@@ -320,6 +320,132 @@ class DynamicCompressFp8Cache(_BlockCache):
     layer_cls = CompressFp8Layer
 
 
+class LatentLayer(NormalLayer):
+    """Latents of multi-head latent attention: one row per token that serves as key and value of every head, held as
+    ``_k [B, 1, capacity, row]`` (latent, shared rotated key part, zeros up to the kernels' row size); there is no
+    separate value storage.  Rows are zero-filled because the kernels read whole rows."""
+
+    def _alloc(self, bsz, heads, cap, dk, dv, dtype, device):
+        return (torch.zeros(bsz, heads, cap, dk, dtype=dtype, device=device),
+                torch.zeros(bsz, heads, cap, 0, dtype=dtype, device=device))
+
+
+class LatentCache(_BlockCache):
+    """Cache of a decoder with latent attention, plus what else a sequence carries along: the history of its token
+    ids (``history [slots, capacity]``, the previous token of an embedding over token pairs) and the row of its first
+    token (``start [slots]``; later rows of a left-padded batch are not the first).
+
+    Rows of the batch dimension are slots: a sequence takes one (``acquire``), keeps it however the batch around it
+    changes, and gives it back (``release``); ``lengths`` counts the tokens each slot holds."""
+    layer_cls = LatentLayer
+
+    def __init__(self, config=None, **kwargs):
+        super().__init__(config)
+        self.history = None
+        self.start = None
+        self.lengths = []
+        self._free = []
+        self._first = []         # host copy of ``start``
+
+    # -- storage ----------------------------------------------------------------------------------------------
+    @property
+    def slots(self) -> int:
+        return 0 if self.history is None else self.history.shape[0]
+
+    @property
+    def capacity(self) -> int:
+        return 0 if self.history is None else self.history.shape[1]
+
+    def allocate(self, slots: int, capacity: int, row_widths, dtype, device) -> bool:
+        """Room for ``slots`` sequences of ``capacity`` tokens; ``row_widths``: one cache row width per layer.  What the
+        cache holds already is kept.  True when the storage moved."""
+        if slots <= self.slots and capacity <= self.capacity:
+            return False
+        old_slots = self.slots
+        slots, capacity = max(slots, old_slots), max(capacity, self.capacity)
+        while len(self.layers) < len(row_widths):
+            self.layers.append(self.layer_class_to_replicate())
+        for layer, row in zip(self.layers, row_widths):
+            prev, n = layer._k, layer.length
+            layer.preallocate(slots, 1, capacity, row, 0, dtype, device)
+            if prev is not None:
+                layer._k[:prev.shape[0], :, :prev.shape[2]] = prev
+                layer.set_length(n)
+        history = torch.zeros(slots, capacity, dtype=torch.int32, device=device)
+        start = torch.zeros(slots, dtype=torch.int32, device=device)
+        if self.history is not None:
+            history[:old_slots, :self.history.shape[1]] = self.history
+            start[:old_slots] = self.start
+        self.history, self.start = history, start
+        self.lengths += [0] * (slots - old_slots)
+        self._free += list(range(old_slots, slots))
+        return True
+
+    # -- slots ------------------------------------------------------------------------------------------------
+    def acquire(self) -> int:
+        if not self._free:
+            raise RuntimeError("no free cache slot: release a finished sequence or allocate more")
+        slot = self._free.pop(0)
+        self.lengths[slot] = 0
+        return slot
+
+    def release(self, slot: int):
+        if slot in self._free or not 0 <= slot < self.slots:
+            raise ValueError(f"slot {slot} is not in use")
+        self.lengths[slot] = 0
+        self._free.append(slot)
+        self._free.sort()
+
+    def first_row(self, slot: int) -> int:
+        return self._first[slot] if slot < len(self._first) else 0
+
+    def set_first_rows(self, rows):
+        """First-token rows of slots ``0 ..`` (left-padded batches)."""
+        self._first = [int(r) for r in rows]
+        self.start[:len(rows)] = torch.tensor(self._first, dtype=torch.int32, device=self.start.device)
+
+    def advance_all(self, length: int):
+        """Every slot of a padded batch now reaches to row ``length``."""
+        self._free = []
+        self.lengths = [length] * self.slots
+        for layer in self.layers:
+            layer.set_length(length)
+
+    def release_all(self):
+        self._first = []
+        self._free = list(range(self.slots))
+        self.lengths = [0] * self.slots
+        if self.start is not None:
+            self.start.zero_()
+        for layer in self.layers:
+            layer.set_length(0)
+
+    # -- batch surgery of the transformers generation loop -----------------------------------------------------
+    def _reindex(self, fn):
+        if self.history is not None:
+            self.history, self.start = fn(self.history), fn(self.start)
+            self.lengths = fn(torch.tensor(self.lengths)).tolist()
+            self._first = self.start.tolist()
+            self._free = []
+
+    def reorder_cache(self, beam_idx):
+        super().reorder_cache(beam_idx)
+        self._reindex(lambda t: t.index_select(0, beam_idx.to(t.device)))
+
+    def batch_repeat_interleave(self, repeats: int):
+        super().batch_repeat_interleave(repeats)
+        self._reindex(lambda t: t.repeat_interleave(repeats, dim=0))
+
+    def batch_select_indices(self, indices):
+        super().batch_select_indices(indices)
+        self._reindex(lambda t: t[indices.to(t.device) if isinstance(indices, torch.Tensor) else indices])
+
+    def crop(self, max_length: int):
+        super().crop(max_length)
+        n = self.get_seq_length()
+        self.lengths = [min(x, n) for x in self.lengths]
+
+
 def is_fp8_cache(cache) -> bool:
     return isinstance(cache, (DynamicFp8Cache, DynamicCompressFp8Cache))
 

@@ -50,10 +50,14 @@ def ipex_generate(self, inputs=None, generation_config=None, logits_processor=No
         from .speculative import speculative_generate
         return speculative_generate(self, inputs=inputs, draft_model=self.draft_model,
                                     generation_config=generation_config, streamer=streamer, **kwargs)
-    if logits_processor is None and stopping_criteria is None and prefix_allowed_tokens_fn is None \
-            and assistant_model is None and _engine_ok(self, inputs, kwargs):
-        from ..engine import engine_generate
-        return engine_generate(self, inputs, generation_config=generation_config, streamer=streamer, **kwargs)
+    if logits_processor is None and prefix_allowed_tokens_fn is None and assistant_model is None \
+            and _engine_ok(self, inputs, kwargs):
+        from ..engine import engine_generate, takes_stopping_criteria
+        if stopping_criteria is None:
+            return engine_generate(self, inputs, generation_config=generation_config, streamer=streamer, **kwargs)
+        if takes_stopping_criteria(self):
+            return engine_generate(self, inputs, generation_config=generation_config, streamer=streamer,
+                                   stopping_criteria=stopping_criteria, **kwargs)
     # only what the caller actually gave: some generate() overrides (Whisper) test for the presence of a keyword
     optional = dict(generation_config=generation_config, logits_processor=logits_processor,
                     stopping_criteria=stopping_criteria, prefix_allowed_tokens_fn=prefix_allowed_tokens_fn,

@@ -30,6 +30,9 @@ from ..quant.params import FP4Params
 from ..quant.policy import load_imatrix_data
 from ..utils.common import invalidInputError
 from .convert import ggml_convert_low_bit
+from .remote_archs import register_native_archs
+
+register_native_archs()
 
 logger = logging.getLogger(__name__)
 

@@ -334,6 +334,24 @@ def _minicpm3(c: dict):
     return cfg, convert
 
 
+# Architectures that neither transformers nor a remote modeling file implements: the package's own model classes.  Their
+# raw checkpoints carry an ``architecture`` field instead of a ``model_type`` (one written back by ``save_pretrained`` or
+# ``save_low_bit`` has both, and loads through the Auto classes the module registers).
+NATIVE_ARCHS: Dict[str, str] = {"Dobetar": "dobetar"}
+
+
+def register_native_archs():
+    import importlib
+    for name in NATIVE_ARCHS.values():
+        importlib.import_module(f"..models.{name}", __package__).register()
+
+
+def _load_native_arch(c: dict, path: str, torch_dtype):
+    import importlib
+    mod = importlib.import_module(f"..models.{NATIVE_ARCHS[c['architecture']]}", __package__)
+    return mod.build(c, _read_state_dict(path), torch_dtype)
+
+
 REMOTE_ARCHS: Dict[str, Callable[[dict], Optional[Tuple[object, Callable]]]] = {
     "chatglm": _chatglm, "baichuan": _baichuan, "internlm": _internlm, "internlm2": _internlm2, "qwen": _qwen,
     "minicpm": _minicpm, "minicpm3": _minicpm3, "aquila": _aquila,
@@ -348,6 +366,8 @@ def maybe_load_remote_arch(path, torch_dtype=None):
     with open(os.path.join(path, "config.json")) as f:
         c = json.load(f)
     mt = c.get("model_type")
+    if mt is None and c.get("architecture") in NATIVE_ARCHS:
+        return _load_native_arch(c, str(path), torch_dtype)
     if mt not in REMOTE_ARCHS:
         return None
     from transformers import AutoModelForCausalLM
