@@ -55,31 +55,34 @@ def window_visible(n, size):
     return (d >= 0) & (d < size) if size else d >= 0
 
 
-def latent_attention(w, pre, m, h, eps, faults=()):
-    """Multi-head latent attention of one sequence ``h [n, width]`` (already normed); returns the mixer's output."""
-    n = h.shape[0]
+def latent_mix(q, kv, w_norm, w_uk, w_uv, m, eps, faults=()):
+    """Attention of one sequence from its projections: ``q [n, H, dim + rot_dim]``, ``kv [n, kv_rank + rot_dim]``.
+    Returns the heads' outputs ``[n, H, vdim]``."""
+    n = q.shape[0]
     H, dim, rd, vd, R = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
     pos = torch.arange(n)
-    q = (h @ w[pre + "q"].T).view(n, H, dim + rd)
-    kv = h @ w[pre + "dkv"].T
-    c = rms_norm(kv[:, :R], w[pre + "dkv.norm"], eps)
-    k_rot = kv[:, R:]
+    c = rms_norm(kv[:, :R], w_norm, eps)
+    q_rot, k_rot = q[:, :, dim:], kv[:, R:]
     rot = m.get("rot")
-    q_rot = q[:, :, dim:]
     if rot and rd:
         q_rot = rotate_half_pairs(q_rot, pos, float(rot["base"]), rot["dims"])
         k_rot = rotate_half_pairs(k_rot, pos, float(rot["base"]), rot["dims"])
-    k = (c @ w[pre + "uk"].T).view(n, H, dim)
-    v = (c @ w[pre + "uv"].T).view(n, H, vd)
+    k = (c @ w_uk.T).view(n, H, dim)
+    v = (c @ w_uv.T).view(n, H, vd)
     size = (m.get("mask") or {}).get("size")
-    if "window_plus_one" in faults and size:
-        size = size + 1
-    if "window_minus_one" in faults and size:
-        size = size - 1
+    if size:
+        size += ("window_plus_one" in faults) - ("window_minus_one" in faults)
     s = torch.einsum("ihd,jhd->hij", q[:, :, :dim], k) + torch.einsum("ihd,jd->hij", q_rot, k_rot)
     s = (s * m["scale"]).masked_fill(~window_visible(n, size), -math.inf)
-    o = torch.einsum("hij,jhd->ihd", torch.softmax(s, -1), v)
-    return o.reshape(n, H * vd) @ w[pre + "o"].T
+    return torch.einsum("hij,jhd->ihd", torch.softmax(s, -1), v)
+
+
+def latent_attention(w, pre, m, h, eps, faults=()):
+    """Multi-head latent attention of one sequence ``h [n, width]`` (already normed); returns the mixer's output."""
+    n = h.shape[0]
+    q = (h @ w[pre + "q"].T).view(n, m["heads"], m["dim"] + m["rot_dim"])
+    o = latent_mix(q, h @ w[pre + "dkv"].T, w[pre + "dkv.norm"], w[pre + "uk"], w[pre + "uv"], m, eps, faults)
+    return o.reshape(n, -1) @ w[pre + "o"].T
 
 
 def squared_relu_mlp(w, pre, h):
@@ -134,3 +137,70 @@ def forward(weights, cfg, tokens, dtype=F64, faults=(), trace=None):
         if trace is not None:
             trace.append(x.clone())
     return softcap(rms_norm(x, w["final.norm"], eps) @ w["head"].T, cfg.get("logit_softcap"))
+
+
+def greedy(weights, cfg, tokens, n):
+    """``n`` greedy continuation tokens, every step recomputed from the whole sequence."""
+    seq = list(tokens)
+    for _ in range(n):
+        seq.append(int(forward(weights, cfg, seq)[-1].argmax()))
+    return seq[len(tokens):]
+
+
+# ------------------------------------------------------------------------------------------------
+# random models
+# ------------------------------------------------------------------------------------------------
+def latent_layer(heads=4, dim=32, rot_dim=16, vdim=24, kv_rank=64, window=11, base=10000.0, mlp=None, scale=None):
+    return {"type": "latent_attention", "mlp": mlp,
+            "mixer": {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank,
+                      "mask": {"size": window}, "rot": {"base": base, "dims": rot_dim},
+                      "scale": scale if scale is not None else (dim + rot_dim) ** -0.5}}
+
+
+def dense(ff):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe(ff, experts, top, limit=1.5):
+    return {"kind": "moe", "expert": {"ff": ff, "limit": limit}, "router": {"experts": experts, "top": top}}
+
+
+def random_weights(cfg, seed=0, sharp=2.5):
+    """Checkpoint tensors of ``cfg`` (bf16-representable fp32): projections keep unit variance, queries are scaled by
+    ``sharp`` so that the attention is far from uniform."""
+    g = torch.Generator().manual_seed(seed)
+    W = cfg["width"]
+
+    def mat(n, k, gain=1.0):
+        return (torch.randn(n, k, generator=g) * gain / math.sqrt(k)).bfloat16().float()
+
+    def norm(n):
+        return (1.0 + 0.2 * torch.randn(n, generator=g)).bfloat16().float()
+
+    w = {"embed": mat(cfg["vocab"], W, math.sqrt(W)), "final.norm": norm(W), "head": mat(cfg["vocab"], W, 2.0)}
+    b = cfg["embedding"].get("bigram")
+    if b:
+        w["bigram"] = mat(b["buckets"] + 1, W, 2.0 * math.sqrt(W))
+    for i, layer in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", layer["mixer"]
+        H, R = m["heads"], m["kv_rank"]
+        w[p + "norm1"] = norm(W)
+        w[p + "mix.q"] = mat(H * (m["dim"] + m["rot_dim"]), W, sharp)
+        w[p + "mix.dkv"] = mat(R + m["rot_dim"], W)
+        w[p + "mix.dkv.norm"] = norm(R)
+        w[p + "mix.uk"] = mat(H * m["dim"], R)
+        w[p + "mix.uv"] = mat(H * m["vdim"], R)
+        w[p + "mix.o"] = mat(W, H * m["vdim"])
+        f = layer.get("mlp")
+        if not f:
+            continue
+        w[p + "norm2"] = norm(W)
+        if f["kind"] == "dense":
+            w[p + "mlp.up"], w[p + "mlp.down"] = mat(f["ff"], W), mat(W, f["ff"])
+        else:
+            w[p + "mlp.router"] = mat(f["router"]["experts"], W, 2.0)
+            for e in range(f["router"]["experts"]):
+                q = f"{p}mlp.e{e}."
+                ff = f["expert"]["ff"]
+                w[q + "gate"], w[q + "up"], w[q + "down"] = mat(ff, W, 2.0), mat(ff, W, 2.0), mat(W, ff)
+    return w
