@@ -108,25 +108,71 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   return warp_sum(t);
 }
 
-// Stage `rows` rows: plain copy of T rows, or RMS norm of fp32 rows.  Zero fill up to kp.
+// Stage `rows` rows: plain copy of T rows, or RMS norm of fp32 rows.  Zero fill up to kp.  Whole block; `red` holds one
+// float per warp.
 template <typename T>
 __device__ __forceinline__ void stage_rows(T* sx, int kp, const void* x, int64_t ldx, const T* norm_w, float eps,
                                            int rows, int K, float* red) {
-  for (int m = 0; m < rows; ++m) {
-    T* dst = sx + (size_t)m * kp;
-    if (norm_w != nullptr) {
-      const float* src = reinterpret_cast<const float*>(x) + (int64_t)m * ldx;
-      float s = 0.f;
-      for (int k = threadIdx.x; k < K; k += blockDim.x) s = fmaf(src[k], src[k], s);
-      s = block_sum(s, red);
-      const float inv = 1.0f / sqrtf(s / (float)K + eps);
-      for (int k = threadIdx.x; k < K; k += blockDim.x)
-        dst[k] = DT<T>::from_f(src[k] * inv * DT<T>::to_f(norm_w[k]));
-    } else {
+  constexpr int VN = Vec<T>::n;
+  const int warps = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  for (int m = 0; m < rows; ++m)
+    for (int k = K + threadIdx.x; k < kp; k += blockDim.x) sx[(size_t)m * kp + k] = DT<T>::from_f(0.f);
+  if (norm_w == nullptr) {
+    for (int m = 0; m < rows; ++m) {
+      T* dst = sx + (size_t)m * kp;
       const T* src = reinterpret_cast<const T*>(x) + (int64_t)m * ldx;
-      for (int k = threadIdx.x; k < K; k += blockDim.x) dst[k] = src[k];
+      if (K % VN == 0 && (reinterpret_cast<uintptr_t>(src) & 15) == 0) {
+        for (int v = threadIdx.x; v < K / VN; v += blockDim.x)
+          reinterpret_cast<uint4*>(dst)[v] = reinterpret_cast<const uint4*>(src)[v];
+      } else {
+        for (int k = threadIdx.x; k < K; k += blockDim.x) dst[k] = src[k];
+      }
     }
-    for (int k = K + threadIdx.x; k < kp; k += blockDim.x) dst[k] = DT<T>::from_f(0.f);
+    __syncthreads();
+    return;
+  }
+  // `per` warps share a row: the sums of all rows meet in one barrier
+  const int per = rows >= warps ? 1 : warps / rows;
+  for (int m0 = 0; m0 < rows; m0 += warps / per) {
+    const int m = m0 + warp / per, sub = warp % per;
+    const bool on = m < rows && warp < warps / per * per;
+    const float* src = reinterpret_cast<const float*>(x) + (int64_t)(on ? m : 0) * ldx;
+    const bool v4 = K % 4 == 0 && (reinterpret_cast<uintptr_t>(src) & 15) == 0;
+    float s = 0.f;
+    if (on) {
+      if (v4) {
+#pragma unroll 4
+        for (int k = sub * 32 + lane; k < K / 4; k += per * 32) {
+          const float4 f = reinterpret_cast<const float4*>(src)[k];
+          s += f.x * f.x + f.y * f.y + f.z * f.z + f.w * f.w;
+        }
+      } else {
+        for (int k = sub * 32 + lane; k < K; k += per * 32) s = fmaf(src[k], src[k], s);
+      }
+    }
+    s = warp_sum(s);
+    __syncthreads();
+    if (lane == 0) red[warp] = s;
+    __syncthreads();
+    if (on) {
+      s = 0.f;
+      for (int i = 0; i < per; ++i) s += red[warp / per * per + i];
+      const float inv = 1.0f / sqrtf(s / (float)K + eps);
+      T* dst = sx + (size_t)m * kp;
+      if (v4) {
+#pragma unroll 4
+        for (int k = sub * 32 + lane; k < K / 4; k += per * 32) {
+          const float4 f = reinterpret_cast<const float4*>(src)[k];
+          dst[4 * k] = DT<T>::from_f(f.x * inv * DT<T>::to_f(norm_w[4 * k]));
+          dst[4 * k + 1] = DT<T>::from_f(f.y * inv * DT<T>::to_f(norm_w[4 * k + 1]));
+          dst[4 * k + 2] = DT<T>::from_f(f.z * inv * DT<T>::to_f(norm_w[4 * k + 2]));
+          dst[4 * k + 3] = DT<T>::from_f(f.w * inv * DT<T>::to_f(norm_w[4 * k + 3]));
+        }
+      } else {
+        for (int k = sub * 32 + lane; k < K; k += per * 32)
+          dst[k] = DT<T>::from_f(src[k] * inv * DT<T>::to_f(norm_w[k]));
+      }
+    }
   }
   __syncthreads();
 }
@@ -142,6 +188,20 @@ struct GemvRowsArgs {
   int out_mode, act;     // act 1: square of relu
   int vec;
 };
+
+__device__ __forceinline__ float finish(float v, int act) { return act == 1 ? (v > 0.f ? v * v : 0.f) : v; }
+
+template <typename T>
+__device__ __forceinline__ void store_row(const GemvRowsArgs& a, int m, int n, float v) {
+  v = finish(v, a.act);
+  if (a.out_mode == 0) {
+    reinterpret_cast<T*>(a.out)[(int64_t)m * a.ldo + n] = DT<T>::from_f(v);
+  } else {
+    float* o = reinterpret_cast<float*>(a.out) + (int64_t)m * a.ldo + n;
+    if (a.out_mode == 1) *o += v;
+    else *o = a.softcap > 0.f ? a.softcap * tanhf(v / a.softcap) : v;
+  }
+}
 
 template <typename T, int M, int R>
 __global__ void __launch_bounds__(kThreads) gemv_rows_kernel(GemvRowsArgs a) {
@@ -169,17 +229,123 @@ __global__ void __launch_bounds__(kThreads) gemv_rows_kernel(GemvRowsArgs a) {
       for (int r = 0; r < R; ++r) {
         const int n = t * R + r;
         if (lane == ((m * R + r) & 31) && m < a.M && n < a.N) {
-          float v = acc[m][r];
-          if (a.act == 1) v = v > 0.f ? v * v : 0.f;
-          if (a.out_mode == 0) {
-            reinterpret_cast<T*>(a.out)[(int64_t)m * a.ldo + n] = DT<T>::from_f(v);
-          } else {
-            float* o = reinterpret_cast<float*>(a.out) + (int64_t)m * a.ldo + n;
-            if (a.out_mode == 1) *o += v;
-            else *o = a.softcap > 0.f ? a.softcap * tanhf(v / a.softcap) : v;
+          store_row<T>(a, m, n, acc[m][r]);
+        }
+      }
+  }
+}
+
+template <typename T>
+__device__ __forceinline__ void mma16816(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0,
+                                         uint32_t b1) {
+  if constexpr (std::is_same<T, __nv_bfloat16>::value)
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+  else
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.f16.f16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+                 : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+// 16-bit weights on the tensor cores, NT * 8 tokens: a tile is 16 weight rows (the A operand, straight from global
+// memory), `split` warps of the CTA share its K range and meet once per tile in shared memory.  The k order inside a
+// 32-wide block is permuted alike for both operands, so that a lane's fragment is one 16-byte load: lane (g, t) holds
+// k = 8 t .. 8 t + 7 of rows g and g + 8, and of token g.  Normed rows are staged in shared memory; plain
+// activations are read where they are (a CTA reads each value about once).
+template <typename T, int NT>
+__global__ void __launch_bounds__(kThreads) gemv_mma_kernel(GemvRowsArgs a, int split) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  __shared__ float red[kWarps];
+  constexpr int U = NT == 1 ? 4 : 2;
+  float* part = reinterpret_cast<float*>(smem);                         // [2][kWarps][NT * 128]
+  T* sx = reinterpret_cast<T*>(smem + 2 * kWarps * NT * 128 * sizeof(float));
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+  const int tpc = kWarps / split, sub = warp % split;
+  const int ntile = (a.N + 15) / 16, nkb = (a.K + 31) / 32;
+  const int per = (nkb + split - 1) / split, kb0 = sub * per, kb1 = min(kb0 + per, nkb);
+  const T* W = reinterpret_cast<const T*>(a.w);
+  pdl_launch_dependents();
+  {
+    const int tile = blockIdx.x * tpc + warp / split, row = tile * 16 + lane;
+    const int k0 = kb0 * 32, bytes = (min(kb1 * 32, a.K) - k0) * (int)sizeof(T);
+    if (lane < 16 && row < a.N && bytes > 0) prefetch_l2_bulk(W + (int64_t)row * a.ldw + k0, (uint32_t)bytes);
+  }
+  pdl_wait();
+  const bool staged = a.norm_w != nullptr;
+  if (staged)
+    stage_rows<T>(sx, a.kp, a.x, a.ldx, reinterpret_cast<const T*>(a.norm_w), a.eps, a.M, a.K, red);
+  const T* xs[NT];
+  bool xon[NT];
+#pragma unroll
+  for (int n = 0; n < NT; ++n) {
+    const int m = n * 8 + g;
+    xon[n] = m < a.M;
+    xs[n] = (staged ? sx + (size_t)(xon[n] ? m : 0) * a.kp
+                    : reinterpret_cast<const T*>(a.x) + (int64_t)(xon[n] ? m : 0) * a.ldx) + t * 8;
+  }
+  int par = 0;
+  for (int base = blockIdx.x * tpc; base < ntile; base += gridDim.x * tpc, par ^= 1) {
+    const int tile = base + warp / split;
+    float acc[2][NT][4] = {};
+    if (tile < ntile) {
+      const T* w0 = W + (int64_t)min(tile * 16 + g, a.N - 1) * a.ldw + t * 8;
+      const T* w1 = W + (int64_t)min(tile * 16 + g + 8, a.N - 1) * a.ldw + t * 8;
+      for (int kb = kb0; kb < kb1; kb += U) {
+        uint4 r0[U], r1[U];
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          const int k = (kb + u) * 32;
+          const bool in = kb + u < kb1 && k + t * 8 < a.K;
+          r0[u] = in ? ldg_nc_v4(w0 + k) : make_uint4(0, 0, 0, 0);
+          r1[u] = in ? ldg_nc_v4(w1 + k) : make_uint4(0, 0, 0, 0);
+        }
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          const int k = (kb + u) * 32;
+          const bool in = kb + u < kb1 && k + t * 8 < a.K;
+#pragma unroll
+          for (int n = 0; n < NT; ++n) {
+            const uint4 x = in && xon[n] ? *reinterpret_cast<const uint4*>(xs[n] + k) : make_uint4(0, 0, 0, 0);
+            mma16816<T>(acc[0][n], r0[u].x, r1[u].x, r0[u].y, r1[u].y, x.x, x.y);
+            mma16816<T>(acc[1][n], r0[u].z, r1[u].z, r0[u].w, r1[u].w, x.z, x.w);
           }
         }
       }
+    }
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) acc[0][n][i] += acc[1][n][i];
+    // accumulator i of lane (g, t): weight row g + 8 * (i / 2), token n * 8 + 2 t + (i & 1)
+    if (split > 1) {
+      float* mine = part + ((size_t)par * kWarps + warp) * (NT * 128);
+#pragma unroll
+      for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) mine[(n * 4 + i) * 32 + lane] = acc[0][n][i];
+      __syncthreads();
+      // the group's warps share the sums: value (n, i) goes to warp (n * 4 + i) % split
+      const float* grp = part + ((size_t)par * kWarps + warp / split * split) * (NT * 128);
+#pragma unroll
+      for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+          if ((n * 4 + i) % split == sub) {
+            float v = 0.f;
+            for (int w = 0; w < split; ++w) v += grp[w * (NT * 128) + (n * 4 + i) * 32 + lane];
+            const int row = tile * 16 + g + 8 * (i >> 1), m = n * 8 + 2 * t + (i & 1);
+            if (tile < ntile && row < a.N && m < a.M) store_row<T>(a, m, row, v);
+          }
+    } else {
+#pragma unroll
+      for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int row = tile * 16 + g + 8 * (i >> 1), m = n * 8 + 2 * t + (i & 1);
+          if (tile < ntile && row < a.N && m < a.M) store_row<T>(a, m, row, acc[0][n][i]);
+        }
+    }
   }
 }
 
@@ -215,8 +381,37 @@ cudaError_t pick_rows(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
   return launch_gemv<T, M, 1>(a, pdl, st);
 }
 
+template <typename T, int NT>
+cudaError_t launch_gemv_mma(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
+  auto kern = gemv_mma_kernel<T, NT>;
+  a.kp = (a.K + 31) / 32 * 32 + 32;        // 64 bytes of skew between rows: neighbouring tokens in different banks
+  const size_t smem = (size_t)2 * kWarps * NT * 128 * sizeof(float) + (a.norm_w != nullptr ? (size_t)a.M * a.kp * sizeof(T) : 0);
+  if (smem > 226 * 1024) return cudaErrorInvalidValue;
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return e;
+  }
+  // enough warps for the machine, at least four k blocks each
+  const int ntile = (a.N + 15) / 16, nkb = (a.K + 31) / 32, want = sm_count() * 2 * kWarps;
+  int split = 1;
+  while (split < kWarps && ntile * split < want && nkb / (2 * split) >= 4) split *= 2;
+  const int tpc = kWarps / split, ctas = (ntile + tpc - 1) / tpc, cap = sm_count() * 2;
+  return launch_kernel(kern, dim3(ctas < cap ? ctas : cap), dim3(kThreads), smem, st, pdl, a, split);
+}
+
+int g_mma_from = 1;      // smallest row count that takes the tensor-core kernel
+bool mma_from(const GemvRowsArgs& a) { return a.M >= g_mma_from; }
+
 template <typename T>
 cudaError_t pick_m(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
+  if constexpr (sizeof(T) == 2) {
+    const bool direct = a.norm_w != nullptr || ((reinterpret_cast<uintptr_t>(a.x) & 15) == 0 && a.ldx % 8 == 0);
+    if (a.vec && direct && mma_from(a)) {
+      if (a.M <= 8) return launch_gemv_mma<T, 1>(a, pdl, st);
+      return launch_gemv_mma<T, 2>(a, pdl, st);
+    }
+  }
+  if (a.M > 8) return cudaErrorInvalidValue;
   if (a.M == 1) return pick_rows<T, 1>(a, pdl, st);
   if (a.M == 2) return pick_rows<T, 2>(a, pdl, st);
   if (a.M <= 4) return pick_rows<T, 4>(a, pdl, st);
@@ -259,7 +454,18 @@ __global__ void __launch_bounds__(kThreads) moe_router_kernel(RouterArgs a) {
   for (int e = warp; e < a.E; e += kWarps) {
     const T* w = reinterpret_cast<const T*>(a.w) + (int64_t)e * a.K;
     float acc = 0.f;
-    for (int k = lane; k < a.K; k += 32) acc = fmaf(h[k], DT<T>::to_f(w[k]), acc);
+    constexpr int VN = Vec<T>::n;
+    if (a.K % VN == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0) {
+#pragma unroll 4
+      for (int v = lane; v < a.K / VN; v += 32) {
+        float wf[VN];
+        unpack<T>(ldg_nc_v4(reinterpret_cast<const uint4*>(w) + v), wf);
+#pragma unroll
+        for (int i = 0; i < VN; ++i) acc = fmaf(h[v * VN + i], wf[i], acc);
+      }
+    } else {
+      for (int k = lane; k < a.K; k += 32) acc = fmaf(h[k], DT<T>::to_f(w[k]), acc);
+    }
     acc = warp_sum(acc);
     if (lane == 0) sc[e] = 1.0f / (1.0f + expf(-acc));
   }
@@ -384,12 +590,16 @@ int by_dtype(int dtype, F&& f) {
 
 }  // namespace
 
-// Rows of x one call may take: the staged rows must fit shared memory.
+// Rows of x one call may take.  Normed rows are staged in shared memory, which may allow fewer (the call says so).
 IPEX_API int ipex_gemv_rows_max(int K, int dtype) {
+  if (dtype != DT_F32 && K % 8 == 0) return 16;
   const int64_t row = ((int64_t)K + 8) * (dtype == DT_F32 ? 4 : 2);
   const int64_t m = (200 * 1024) / row;
   return m >= 8 ? 8 : m >= 4 ? 4 : m >= 2 ? 2 : (int)m;
 }
+
+// Timing sweeps: smallest row count of the tensor-core kernel (17: never).
+IPEX_API void ipex_gemv_rows_tune(int mma_from_rows) { g_mma_from = mma_from_rows; }
 
 // y = act(x . W^T): see GemvRowsArgs.  M <= ipex_gemv_rows_max(K, dtype).
 IPEX_API int ipex_gemv_rows(const void* w, int64_t ldw, const void* x, int64_t ldx, const void* norm_w, float eps,

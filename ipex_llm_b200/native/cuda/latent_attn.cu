@@ -304,20 +304,25 @@ __device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], 
                  : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-// MG groups of 16 heads per CTA (four warps each); RT: 8-column output tiles per warp (R <= 32 * RT).
-template <typename T, int MG, int RT>
-__global__ void __launch_bounds__(MG * 128) latent_attn_mma_kernel(LatentAttnArgs a) {
+// MG groups of 16 heads per CTA, eight warps each.
+//   scores  a warp owns a quarter of the row (k) for 16 of the tile's 32 keys; its part of the queries stays in
+//           registers for the whole loop, the four partial sums of a score meet in shared memory
+//   values  a warp owns RT 8-column tiles of the output for all heads of the CTA
+// KS: 16-wide k steps a warp holds (row <= 64 * KS values).
+template <typename T, int MG, int RT, int KS>
+__global__ void __launch_bounds__(MG * 256) latent_attn_mma_kernel(LatentAttnArgs a) {
   extern __shared__ __align__(16) uint8_t smem[];
-  constexpr int kHeads = MG * 16;
-  const int Dp = (int)a.ldc;                    // R + rd rounded up to a multiple of 32, zero-filled
+  constexpr int kHeads = MG * 16, kWarpsHere = MG * 8;
+  constexpr int kLdS = kKT + 4;
+  const int Dp = (int)a.ldc;                    // R + rd rounded up to a multiple of 64, zero-filled
   const int ld = Dp + 8;                        // shared-memory row: 16 bytes of skew between rows
-  T* sQ = reinterpret_cast<T*>(smem);           // [kHeads][ld]
-  T* sK = sQ + kHeads * ld;                     // [kStages][kKT][ld]
+  T* sK = reinterpret_cast<T*>(smem);           // [kStages][kKT][ld]
   T* sP = sK + kStages * kKT * ld;              // [kHeads][kKT + 8]
-  float* sS = reinterpret_cast<float*>(sP + kHeads * (kKT + 8));   // [kHeads][kKT + 4]
-  float* sC = sS + kHeads * (kKT + 4);          // [kHeads] rescale factors
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int wi = warp & 3, mg = warp >> 2;
+  float* sS = reinterpret_cast<float*>(sP + kHeads * (kKT + 8));   // [4][kHeads][kLdS]
+  float* sC = sS + 4 * kHeads * kLdS;           // [kHeads] rescale factors
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, tq = lane & 3;
+  const int mg = warp >> 3, kq = warp & 3, kh = (warp >> 2) & 1;
+  static_assert(kHeads <= kKT, "the queries pass through one stage");
   const int h0 = blockIdx.x * kHeads, split = blockIdx.y, m = blockIdx.z;
   pdl_launch_dependents();
   pdl_wait();
@@ -328,36 +333,37 @@ __global__ void __launch_bounds__(MG * 128) latent_attn_mma_kernel(LatentAttnArg
   const int vec_row = Dp / 8;
   auto load_tile = [&](int i) {
     T* dst = sK + (i % kStages) * kKT * ld;
-    for (int c = tid; c < kKT * vec_row; c += MG * 128) {
-      const int r = c / vec_row, v = c % vec_row;
-      const int j = min(lo + i * kKT + r, hi - 1);          // rows past the end repeat the last one (masked below)
-      cp_async16(dst + r * ld + v * 8, base + (int64_t)j * a.ldc + v * 8);
+    for (int r = warp; r < kKT; r += kWarpsHere) {
+      const T* src = base + (int64_t)min(lo + i * kKT + r, hi - 1) * a.ldc;   // past the end: the last row, masked below
+      for (int v = lane; v < vec_row; v += 32) cp_async16(dst + r * ld + v * 8, src + v * 8);
     }
   };
   for (int i = 0; i < kStages - 1; ++i) {
     if (i < ntile) load_tile(i);
     asm volatile("cp.async.commit_group;" ::: "memory");
   }
-  // queries: [absorbed | rotated | zeros], heads past H are zero
-  for (int i = tid; i < kHeads * Dp; i += MG * 128) {
-    const int r = i / Dp, c = i % Dp, h = h0 + r;
-    T v = DT<T>::from_f(0.f);
-    if (h < a.H) {
-      if (c < a.R) v = reinterpret_cast<const T*>(a.qabs)[((int64_t)m * a.H + h) * a.R + c];
-      else if (c < a.R + a.rd)
-        v = reinterpret_cast<const T*>(a.qkv)[(int64_t)m * a.ldq + (int64_t)h * (a.dim + a.rd) + a.dim + c - a.R];
-    }
-    sQ[r * ld + c] = v;
+  // queries [absorbed | rotated | zeros] (heads past H are zero) pass through the stage that the prologue left free
+  // into the warp's fragments
+  const int ks = Dp / 64, k0 = kq * (Dp / 4);
+  const int ar = lane & 15, ac = (lane >> 4) * 8;                   // ldmatrix address of an A fragment
+  T* sQ = sK + (kStages - 1) * kKT * ld;
+  for (int r = warp; r < kHeads; r += kWarpsHere) {
+    const int h = h0 + r;
+    const bool on = h < a.H;
+    const uint4* qv = reinterpret_cast<const uint4*>(reinterpret_cast<const T*>(a.qabs) +
+                                                     ((int64_t)m * a.H + (on ? h : 0)) * a.R);
+    const T* qr = reinterpret_cast<const T*>(a.qkv) + (int64_t)m * a.ldq + (int64_t)(on ? h : 0) * (a.dim + a.rd) + a.dim;
+    for (int v = lane; v < a.R / 8; v += 32)
+      reinterpret_cast<uint4*>(sQ + r * ld)[v] = on ? qv[v] : make_uint4(0, 0, 0, 0);
+    for (int i = lane; i < Dp - a.R; i += 32) sQ[r * ld + a.R + i] = on && i < a.rd ? qr[i] : DT<T>::from_f(0.f);
   }
-  float o[RT][4];
+  __syncthreads();
+  uint32_t qa[KS][4];
 #pragma unroll
-  for (int j = 0; j < RT; ++j)
-#pragma unroll
-    for (int i = 0; i < 4; ++i) o[j][i] = 0.f;
-  float mrow[4], lrow[4];                        // rows warp * 4 + i of the CTA, same value in every lane
-#pragma unroll
-  for (int i = 0; i < 4; ++i) { mrow[i] = -INFINITY; lrow[i] = 0.f; }
-  const int ar = (lane & 15), ac = (lane >> 4) * 8;         // ldmatrix address of an A fragment
+  for (int s = 0; s < KS; ++s)
+    if (s < ks) ldsm4(qa[s], sQ + (mg * 16 + ar) * ld + k0 + s * 16 + ac);
+  float o[MG][RT][4] = {};
+  float mrow[2] = {-INFINITY, -INFINITY}, lrow[2] = {0.f, 0.f};     // rows warp * 2 + i of the CTA
   for (int t = 0; t < ntile; ++t) {
     asm volatile("cp.async.wait_group %0;" ::"n"(kStages - 2) : "memory");
     __syncthreads();                              // tile t is in; everybody is done with tile t - 1
@@ -366,29 +372,31 @@ __global__ void __launch_bounds__(MG * 128) latent_attn_mma_kernel(LatentAttnArg
     const T* K = sK + (t % kStages) * kKT * ld;
     {
       float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
-      const T* qb = sQ + (mg * 16 + ar) * ld + ac;
-      const T* kb = K + (wi * 8 + (lane & 7)) * ld + (lane >> 3) * 8;
-#pragma unroll 4
-      for (int k = 0; k < Dp; k += 32) {
-        uint32_t a0[4], a1[4], b[4];
-        ldsm4(b, kb + k);
-        ldsm4(a0, qb + k);
-        ldsm4(a1, qb + k + 16);
-        mma16816<T>(c0, a0, b[0], b[1]);
-        mma16816<T>(c1, a1, b[2], b[3]);
+      // matrices of one x4: keys 0-7 at k and k + 8, keys 8-15 at k and k + 8
+      const T* kb = K + (kh * 16 + (lane & 7) + ((lane >> 4) << 3)) * ld + k0 + ((lane >> 3) & 1) * 8;
+#pragma unroll
+      for (int s = 0; s < KS; ++s) {
+        if (s < ks) {
+          uint32_t b[4];
+          ldsm4(b, kb + s * 16);
+          mma16816<T>(c0, qa[s], b[0], b[1]);
+          mma16816<T>(c1, qa[s], b[2], b[3]);
+        }
       }
-      float* s0 = sS + (mg * 16 + (lane >> 2)) * (kKT + 4) + wi * 8 + (lane & 3) * 2;
-      s0[0] = c0[0] + c1[0];
-      s0[1] = c0[1] + c1[1];
-      s0[8 * (kKT + 4)] = c0[2] + c1[2];
-      s0[8 * (kKT + 4) + 1] = c0[3] + c1[3];
+      float* s0 = sS + ((size_t)kq * kHeads + mg * 16 + g) * kLdS + kh * 16 + tq * 2;
+      *reinterpret_cast<float2*>(s0) = make_float2(c0[0], c0[1]);
+      *reinterpret_cast<float2*>(s0 + 8) = make_float2(c1[0], c1[1]);
+      *reinterpret_cast<float2*>(s0 + 8 * kLdS) = make_float2(c0[2], c0[3]);
+      *reinterpret_cast<float2*>(s0 + 8 * kLdS + 8) = make_float2(c1[2], c1[3]);
     }
     __syncthreads();
     const bool valid = lo + t * kKT + lane < hi;
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int r = warp * 4 + i;
-      const float s = valid ? sS[r * (kKT + 4) + lane] * a.scale_log2 : -INFINITY;
+    for (int i = 0; i < 2; ++i) {
+      const int r = warp * 2 + i;
+      const float* sr = sS + (size_t)r * kLdS + lane;
+      const float sum = (sr[0] + sr[kHeads * kLdS]) + (sr[2 * kHeads * kLdS] + sr[3 * kHeads * kLdS]);
+      const float s = valid ? sum * a.scale_log2 : -INFINITY;
       const float mn = fmaxf(mrow[i], warp_max(s));
       const float corr = ex2(mrow[i] - mn);       // first tile: 2^-inf = 0
       const float p = valid ? ex2(s - mn) : 0.f;
@@ -398,21 +406,27 @@ __global__ void __launch_bounds__(MG * 128) latent_attn_mma_kernel(LatentAttnArg
       if (lane == 0) sC[r] = corr;
     }
     __syncthreads();
-    {
-      uint32_t p0[4], p1[4];
-      const T* pb = sP + (mg * 16 + ar) * (kKT + 8) + ac;
-      ldsm4(p0, pb);
-      ldsm4(p1, pb + 16);
-      const float f0 = sC[mg * 16 + (lane >> 2)], f1 = sC[mg * 16 + (lane >> 2) + 8];
+    uint32_t p[MG][2][4];
+    float f[MG][2];
 #pragma unroll
-      for (int j = 0; j < RT; ++j) {
-        const int n = (wi + 4 * j) * 8;
-        if (n < a.R) {
-          uint32_t b[4];
-          ldsm4t(b, K + lane * ld + n);
-          o[j][0] *= f0; o[j][1] *= f0; o[j][2] *= f1; o[j][3] *= f1;
-          mma16816<T>(o[j], p0, b[0], b[1]);
-          mma16816<T>(o[j], p1, b[2], b[3]);
+    for (int i = 0; i < MG; ++i) {
+      const T* pb = sP + (i * 16 + ar) * (kKT + 8) + ac;
+      ldsm4(p[i][0], pb);
+      ldsm4(p[i][1], pb + 16);
+      f[i][0] = sC[i * 16 + g];
+      f[i][1] = sC[i * 16 + g + 8];
+    }
+#pragma unroll
+    for (int j = 0; j < RT; ++j) {
+      const int n = (warp + kWarpsHere * j) * 8;
+      if (n < a.R) {
+        uint32_t b[4];
+        ldsm4t(b, K + lane * ld + n);
+#pragma unroll
+        for (int i = 0; i < MG; ++i) {
+          o[i][j][0] *= f[i][0]; o[i][j][1] *= f[i][0]; o[i][j][2] *= f[i][1]; o[i][j][3] *= f[i][1];
+          mma16816<T>(o[i][j], p[i][0], b[0], b[1]);
+          mma16816<T>(o[i][j], p[i][1], b[2], b[3]);
         }
       }
     }
@@ -420,8 +434,8 @@ __global__ void __launch_bounds__(MG * 128) latent_attn_mma_kernel(LatentAttnArg
   asm volatile("cp.async.wait_group 0;" ::: "memory");
   const int64_t part0 = ((int64_t)m * a.nsplit + split) * a.H;
 #pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const int h = h0 + warp * 4 + i;
+  for (int i = 0; i < 2; ++i) {
+    const int h = h0 + warp * 2 + i;
     if (lane == 0 && h < a.H) {
       a.ml[(part0 + h) * 2] = mrow[i];
       a.ml[(part0 + h) * 2 + 1] = lrow[i];
@@ -430,35 +444,37 @@ __global__ void __launch_bounds__(MG * 128) latent_attn_mma_kernel(LatentAttnArg
   if (ntile == 0) return;                         // l = 0: the merge does not read this split's output
 #pragma unroll
   for (int j = 0; j < RT; ++j) {
-    const int n = (wi + 4 * j) * 8 + (lane & 3) * 2;
+    const int n = (warp + kWarpsHere * j) * 8 + tq * 2;
     if (n < a.R) {
 #pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        const int h = h0 + mg * 16 + (lane >> 2) + 8 * i;
-        if (h < a.H)
-          *reinterpret_cast<float2*>(a.o + (part0 + h) * a.R + n) = make_float2(o[j][2 * i], o[j][2 * i + 1]);
-      }
+      for (int i = 0; i < MG; ++i)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int h = h0 + i * 16 + g + 8 * e;
+          if (h < a.H)
+            *reinterpret_cast<float2*>(a.o + (part0 + h) * a.R + n) = make_float2(o[i][j][2 * e], o[i][j][2 * e + 1]);
+        }
     }
   }
 }
 
-template <typename T, int MG, int RT>
+template <typename T, int MG, int RT, int KS>
 cudaError_t launch_mma(const LatentAttnArgs& a, bool pdl, cudaStream_t st) {
-  auto kern = latent_attn_mma_kernel<T, MG, RT>;
+  auto kern = latent_attn_mma_kernel<T, MG, RT, KS>;
   const size_t ld = (size_t)a.ldc + 8;
-  const size_t smem = sizeof(T) * (MG * 16 * ld + kStages * kKT * ld + MG * 16 * (kKT + 8)) +
-                      sizeof(float) * (MG * 16 * (kKT + 4) + MG * 16);
+  const size_t smem = sizeof(T) * (kStages * kKT * ld + MG * 16 * (kKT + 8)) +
+                      sizeof(float) * (4 * MG * 16 * (kKT + 4) + MG * 16);
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return e;
   dim3 grid((a.H + MG * 16 - 1) / (MG * 16), a.nsplit, a.M);
-  return launch_kernel(kern, grid, dim3(MG * 128), smem, st, pdl, a);
+  return launch_kernel(kern, grid, dim3(MG * 256), smem, st, pdl, a);
 }
 
 template <typename T, int MG>
 cudaError_t dispatch_rt(const LatentAttnArgs& a, bool pdl, cudaStream_t st) {
-  if (a.R <= 128) return launch_mma<T, MG, 4>(a, pdl, st);
-  if (a.R <= 256) return launch_mma<T, MG, 8>(a, pdl, st);
-  return launch_mma<T, MG, 16>(a, pdl, st);
+  if (a.R <= 128 && a.ldc <= 320) return launch_mma<T, MG, 2 / MG, 5>(a, pdl, st);
+  if (a.R <= 256 && a.ldc <= 320) return launch_mma<T, MG, 4 / MG, 5>(a, pdl, st);
+  return launch_mma<T, MG, 8 / MG, 10>(a, pdl, st);
 }
 
 // ------------------------------------------------------------------------------------------------ merge + W_uv
@@ -474,67 +490,110 @@ struct UvArgs {
 constexpr int kUvThreads = 256;
 template <typename T, int V, int MT>
 __global__ void __launch_bounds__(kUvThreads) latent_uv_kernel(UvArgs a) {
-  extern __shared__ float sh[];          // [MT][R] merged latents, [MT][nsplit] weights
+  extern __shared__ __align__(16) float sh[];   // [MT][R4] merged latents, [MT][nsplit] weights
+  __shared__ int s_valid[MT];
+  const int R4 = (a.R + 3) / 4 * 4;
   float* so = sh;
-  float* sw = sh + MT * a.R;
+  float* sw = sh + MT * R4;
   const int h = blockIdx.x, m0 = blockIdx.z * MT, mn = min(MT, a.M - m0);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   pdl_launch_dependents();
   pdl_wait();
-  if (threadIdx.x < MT) {
-    const int m = m0 + threadIdx.x;
-    float* w = sw + threadIdx.x * a.nsplit;
-    if ((int)threadIdx.x < mn) {
+  if (warp < MT) {                              // a warp per token: weights of the splits (empty ones come last)
+    const int m = m0 + warp;
+    float* w = sw + warp * a.nsplit;
+    int nv = 0;
+    if (warp < mn) {
       float mx = -INFINITY, l = 0.f;
-      for (int s = 0; s < a.nsplit; ++s) mx = fmaxf(mx, a.ml[(((int64_t)m * a.nsplit + s) * a.H + h) * 2]);
-      for (int s = 0; s < a.nsplit; ++s) {
+      for (int s = lane; s < a.nsplit; s += 32) {
+        const float* e = a.ml + (((int64_t)m * a.nsplit + s) * a.H + h) * 2;
+        if (e[1] > 0.f) { mx = fmaxf(mx, e[0]); nv = s + 1; }
+      }
+      mx = warp_max(mx);
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) nv = max(nv, __shfl_xor_sync(0xffffffffu, nv, o));
+      for (int s = lane; s < a.nsplit; s += 32) {
         const float* e = a.ml + (((int64_t)m * a.nsplit + s) * a.H + h) * 2;
         const float f = e[1] > 0.f ? exp2f(e[0] - mx) : 0.f;
         w[s] = f;
         l += f * e[1];
       }
+      l = warp_sum(l);
       const float inv = l > 0.f ? 1.0f / l : 0.f;
-      for (int s = 0; s < a.nsplit; ++s) w[s] *= inv;
-    } else {
-      for (int s = 0; s < a.nsplit; ++s) w[s] = 0.f;
+      for (int s = lane; s < a.nsplit; s += 32) w[s] *= inv;
     }
+    if (lane == 0) s_valid[warp] = nv;
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < MT * a.R; i += kUvThreads) {
-    const int mm = i / a.R, r = i % a.R;
-    float v = 0.f;
-    for (int s = 0; s < a.nsplit; ++s) {
-      const float f = sw[mm * a.nsplit + s];
-      if (f != 0.f) v = fmaf(f, a.o[(((int64_t)(m0 + mm) * a.nsplit + s) * a.H + h) * a.R + r], v);
-    }
-    so[i] = v;
-  }
-  __syncthreads();
-  const int v0 = blockIdx.y * a.rows_per_block, v1 = min(v0 + a.rows_per_block, a.vd);
-  for (int v = v0 + warp; v < v1; v += kUvThreads / 32) {
-    const T* w = reinterpret_cast<const T*>(a.w_uv) + ((int64_t)h * a.vd + v) * a.R;
-    float acc[MT] = {};
-    for (int r = lane * V; r < a.R; r += 32 * V) {
-      float wf[V];
-      if constexpr (V > 1) {
-        const uint4 raw = ldg_nc_v4(w + r);
-        const T* e = reinterpret_cast<const T*>(&raw);
 #pragma unroll
-        for (int i = 0; i < V; ++i) wf[i] = DT<T>::to_f(e[i]);
-      } else {
-        wf[0] = DT<T>::to_f(w[r]);
+  for (int mm = 0; mm < MT; ++mm) {
+    const int nv = s_valid[mm];
+    const float* w = sw + mm * a.nsplit;
+    const float* src = a.o + ((int64_t)(m0 + mm) * a.nsplit * a.H + h) * a.R;
+    const int64_t step = (int64_t)a.H * a.R;
+    if (a.R % 2 == 0) {
+      for (int r = threadIdx.x * 2; r < a.R; r += kUvThreads * 2) {
+        float2 v = make_float2(0.f, 0.f);
+        for (int s0 = 0; s0 < nv; s0 += 16) {          // sixteen partial rows in flight
+          float2 x[16];
+#pragma unroll
+          for (int i = 0; i < 16; ++i)
+            x[i] = s0 + i < nv ? *reinterpret_cast<const float2*>(src + (s0 + i) * step + r) : make_float2(0.f, 0.f);
+#pragma unroll
+          for (int i = 0; i < 16; ++i) {
+            const float f = s0 + i < nv ? w[s0 + i] : 0.f;
+            v.x = fmaf(f, x[i].x, v.x);
+            v.y = fmaf(f, x[i].y, v.y);
+          }
+        }
+        so[mm * R4 + r] = v.x;
+        so[mm * R4 + r + 1] = v.y;
+      }
+    } else {
+      for (int r = threadIdx.x; r < a.R; r += kUvThreads) {
+        float v = 0.f;
+        for (int s = 0; s < nv; ++s) v = fmaf(w[s], src[s * step + r], v);
+        so[mm * R4 + r] = v;
+      }
+    }
+  }
+  __syncthreads();
+  constexpr int RW = 4;                          // value rows a warp works on at a time
+  const int v0 = blockIdx.y * a.rows_per_block, v1 = min(v0 + a.rows_per_block, a.vd);
+  for (int v = v0 + warp * RW; v < v1; v += kUvThreads / 32 * RW) {
+    const T* w = reinterpret_cast<const T*>(a.w_uv) + ((int64_t)h * a.vd + v) * a.R;
+    float acc[RW][MT] = {};
+    for (int r = lane * V; r < a.R; r += 32 * V) {
+      float wf[RW][V];
+#pragma unroll
+      for (int q = 0; q < RW; ++q) {
+        const T* wq = w + (int64_t)min(q, v1 - 1 - v) * a.R + r;
+        if constexpr (V > 1) {
+          const uint4 raw = ldg_nc_v4(wq);
+          const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+          for (int i = 0; i < V; ++i) wf[q][i] = DT<T>::to_f(e[i]);
+        } else {
+          wf[q][0] = DT<T>::to_f(*wq);
+        }
       }
 #pragma unroll
       for (int mm = 0; mm < MT; ++mm)
 #pragma unroll
-        for (int i = 0; i < V; ++i) acc[mm] = fmaf(so[mm * a.R + r + i], wf[i], acc[mm]);
+        for (int i = 0; i < V; ++i) {
+          const float x = so[mm * R4 + r + i];
+#pragma unroll
+          for (int q = 0; q < RW; ++q) acc[q][mm] = fmaf(x, wf[q][i], acc[q][mm]);
+        }
     }
 #pragma unroll
-    for (int mm = 0; mm < MT; ++mm) {
-      const float s = warp_sum(acc[mm]);
-      if (lane == 0 && mm < mn)
-        reinterpret_cast<T*>(a.out)[(int64_t)(m0 + mm) * a.ldo + (int64_t)h * a.vd + v] = DT<T>::from_f(s);
-    }
+    for (int q = 0; q < RW; ++q)
+#pragma unroll
+      for (int mm = 0; mm < MT; ++mm) {
+        const float s = warp_sum(acc[q][mm]);
+        if (lane == q * MT + mm && mm < mn && v + q < v1)
+          reinterpret_cast<T*>(a.out)[(int64_t)(m0 + mm) * a.ldo + (int64_t)h * a.vd + v + q] = DT<T>::from_f(s);
+      }
   }
 }
 
@@ -558,7 +617,7 @@ cudaError_t launch_prep(const PrepArgs& a, bool pdl, cudaStream_t st) {
 template <typename T, int V, int MT>
 cudaError_t launch_uv(UvArgs& a, int blocks_y, bool pdl, cudaStream_t st) {
   auto kern = latent_uv_kernel<T, V, MT>;
-  const size_t smem = (size_t)MT * (a.R + a.nsplit) * sizeof(float);
+  const size_t smem = (size_t)MT * ((a.R + 3) / 4 * 4 + a.nsplit) * sizeof(float);
   cudaError_t e = allow_smem(kern, smem);
   if (e != cudaSuccess) return e;
   return launch_kernel(kern, dim3(a.H, blocks_y, (a.M + MT - 1) / MT), dim3(kUvThreads), smem, st, pdl, a);
@@ -603,7 +662,7 @@ IPEX_API int ipex_latent_prompt_prep(void* qkv, int64_t ldq, const void* norm_w,
 
 // Cache row stride (elements) the attention kernels want for R + rd values.
 IPEX_API int ipex_latent_row(int R, int rd, int dtype) {
-  const int a = dtype == DT_F32 ? 4 : 32;
+  const int a = dtype == DT_F32 ? 4 : 64;
   return (R + rd + a - 1) / a * a;
 }
 
@@ -646,10 +705,10 @@ IPEX_API int ipex_latent_uv(const float* o, const float* ml, const void* w_uv, v
     using T = std::remove_pointer_t<decltype(tag)>;
     const int mt = M == 1 ? 1 : 4;
     if ((M + mt - 1) / mt > 65535) return cudaErrorInvalidValue;
-    // enough blocks for the machine, at least eight rows (one per warp) each
+    // enough blocks for the machine, at least four rows per warp each
     const int have = H * ((M + mt - 1) / mt);
     int by = (296 + have - 1) / have;
-    const int most = (vd + 7) / 8;
+    const int most = (vd + 31) / 32;
     by = by < 1 ? 1 : (by > most ? most : by);
     UvArgs a = {o, ml, w_uv, out, ldo, M, H, R, vd, nsplit, (vd + by - 1) / by};
     cudaStream_t st = (cudaStream_t)stream;

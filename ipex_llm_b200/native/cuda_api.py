@@ -97,6 +97,7 @@ _STREAM = {
 
 
 def declare_stream(lib: ctypes.CDLL):
+    lib.ipex_gemv_rows_tune.argtypes, lib.ipex_gemv_rows_tune.restype = [ci], None
     for name, args in _STREAM.items():
         fn = getattr(lib, name)
         fn.argtypes, fn.restype = args, ci

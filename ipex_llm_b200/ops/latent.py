@@ -42,8 +42,11 @@ def rows_max(K: int, dtype) -> int:
 
 
 def gemv_rows(w, x, out, mode: int, norm=None, eps: float = 0.0, act: int = 0, softcap: float = 0.0, pdl=False):
-    """``act(x @ w.T)`` for a few rows.  ``norm``: ``x`` is the stream and is RMS-normed with this weight on the way."""
+    """``act(x @ w.T)`` for a few rows.  ``norm``: ``x`` is the stream and is RMS-normed with this weight on the way
+    (inside the product for one or two rows; a CTA would spend longer on the norms of more rows than on its weights)."""
     M, N, K = x.shape[0], w.shape[0], w.shape[1]
+    if norm is not None and M > 2 and w.dtype != torch.float32:
+        x, norm = norm_stream(x, norm, eps, pdl=pdl), None
     rc = stream_lib().ipex_gemv_rows(ptr(w), w.stride(0), ptr(x), x.stride(0), ptr(norm), eps, ptr(out), out.stride(0),
                                      M, N, K, mode, act, softcap, _dt(w), int(pdl), current_stream())
     api.check(rc, "gemv_rows")
@@ -119,13 +122,13 @@ def embed_stream(tokens, slot, pos, cache, table, scale: float, bigram=None, buc
     return out
 
 
-def norm_stream(x, weight, eps: float, rows=None, out=None):
+def norm_stream(x, weight, eps: float, rows=None, out=None, pdl=False):
     """RMS norm of the stream (or of its rows ``rows``, int32) in the weight's dtype."""
     n, K = (x.shape[0] if rows is None else rows.shape[0]), x.shape[1]
     if out is None:
         out = torch.empty(n, K, dtype=weight.dtype, device=x.device)
     rc = stream_lib().ipex_norm_stream(ptr(x), x.stride(0), ptr(weight), ptr(out), out.stride(0), ptr(rows), n, K, eps,
-                                       _dt(weight), 0, current_stream())
+                                       _dt(weight), int(pdl), current_stream())
     api.check(rc, "norm_stream")
     return out
 
@@ -235,9 +238,10 @@ class LatentSpec:
 
 
 def pick_latent_splits(tokens: int, heads: int, visible: int, n_sm: int = 148) -> int:
-    """Parts the visible keys of a query token are split into: enough CTAs for one per SM, at least 32 keys each."""
+    """Parts the visible keys of a query token are split into: one CTA per SM in a single wave, at least 64 keys each
+    (every part costs the merge a read of its partial output)."""
     groups = -(-heads // 32)
-    return max(1, min(-(-n_sm // max(1, tokens * groups)), -(-visible // 32), 64))
+    return max(1, min(n_sm // max(1, tokens * groups), -(-visible // 64), 32))
 
 
 def latent_step(spec: LatentSpec, qkv, w_uk, w_uv, kv_norm, cos, sin, slot, pos, cache, layer_idx: int, out,
