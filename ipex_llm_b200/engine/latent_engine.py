@@ -229,6 +229,10 @@ class LatentStack:
     def forward_padded(self, input_ids, attention_mask, cache: LatentCache, logits_to_keep=0):
         B, S = input_ids.shape
         past = cache.get_seq_length()
+        if cache.layers and (cache.layers[0]._k.dtype != self.dtype or cache.slots != B or
+                             [layer._k.shape[-1] for layer in cache.layers] != self.row_widths):
+            raise TypeError(f"the cache was filled by another model or batch: {cache.slots} x {cache.layers[0]._k.dtype}"
+                            f", this call needs {B} x {self.dtype} of the same row widths")
         cache.allocate(B, self._grown(cache, past + S), self.row_widths, self.dtype, self.device)
         if past == 0:
             pads = [0] * B

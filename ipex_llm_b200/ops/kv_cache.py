@@ -381,6 +381,14 @@ class LatentCache(_BlockCache):
         self._free += list(range(old_slots, slots))
         return True
 
+    def reserve(self, extra_tokens: int):
+        """Room for ``extra_tokens`` behind what a padded batch holds."""
+        need = self.get_seq_length() + extra_tokens
+        if self.layers and need > self.capacity:
+            k = self.layers[0]._k
+            self.allocate(self.slots, need + KV_CACHE_ALLOC_BLOCK_LENGTH, [layer._k.shape[-1] for layer in self.layers],
+                          k.dtype, k.device)
+
     # -- slots ------------------------------------------------------------------------------------------------
     def acquire(self) -> int:
         if not self._free:

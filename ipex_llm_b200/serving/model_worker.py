@@ -189,7 +189,8 @@ class ModelWorker:
         for r, m in zip(batch, enc["attention_mask"]):
             r.prompt_tokens = int(m.sum())
         max_new = max(r.params.max_new_tokens for r in batch)
-        streamer = BatchTextIteratorStreamer(len(batch), tok, skip_prompt=True, skip_special_tokens=True)
+        streamer = BatchTextIteratorStreamer(len(batch), tok, skip_prompt=True, skip_special_tokens=True,
+                                             limits=[r.params.max_new_tokens for r in batch])
         done = [False] * len(batch)
         eos = tok.eos_token_id
 
@@ -232,7 +233,7 @@ class ModelWorker:
             for i, (r, piece) in enumerate(zip(batch, pieces)):
                 if done[i]:
                     continue
-                r.generated_tokens = streamer.generated_tokens[i]
+                r.generated_tokens = pieces.counts[i]
                 if piece:
                     r.text += piece
                     cut = _first_stop(r.text, r.params.stop)
@@ -254,6 +255,7 @@ class ModelWorker:
         out = result["ids"]
         for i, r in enumerate(batch):
             if not done[i]:
+                r.generated_tokens = streamer.generated_tokens[i]
                 new = out[i, ids.shape[1]:]
                 hit_eos = eos is not None and bool((new == eos).any())
                 self._finish(r, "stop" if hit_eos else "length")

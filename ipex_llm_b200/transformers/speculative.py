@@ -89,9 +89,11 @@ def _engine_pair(target, draft, need_len: int):
     if dev.type != "cuda" or next(draft.parameters()).device != dev:
         return None
     try:
-        from ..engine import DecoderEngine, supports
+        from ..engine import DecoderEngine, engine_class, supports
         if not supports(target, {}) or not supports(draft, {}):
             return None
+        if engine_class(target) is not DecoderEngine or engine_class(draft) is not DecoderEngine:
+            return None         # (an engine without multi-token verification: the module path drafts and verifies)
         max_len = (max(need_len, 2048) + 255) // 256 * 256
         pair = []
         for m, mb in ((target, 8), (draft, 1)):

@@ -74,6 +74,23 @@ def test_batch_streamer_incremental_text():
     assert "".join(c[0] for c in chunks) == "w5 w7" and "".join(c[1] for c in chunks) == "w6 w8"
 
 
+def test_batch_streamer_limits():
+    """A sequence at its limit releases its last word at once, ignores later tokens, and the counts travel with the text."""
+    from ipex_llm.transformers.streamer import BatchTextIteratorStreamer
+
+    class Tok:
+        def decode(self, ids, **kw):
+            return " ".join(f"w{i}" for i in ids)
+    s = BatchTextIteratorStreamer(2, Tok(), skip_prompt=True, limits=[1, 3])
+    s.put(torch.tensor([[1, 2], [3, 4]]))
+    for a, b in ((5, 6), (7, 8), (9, 10)):
+        s.put(torch.tensor([a, b]))
+    s.end()
+    chunks = list(s)
+    assert "".join(c[0] for c in chunks) == "w5" and "".join(c[1] for c in chunks) == "w6 w8 w10"
+    assert chunks[0].counts == [1, 1] and chunks[-1].counts == [1, 3] and s.generated_tokens == [1, 3]
+
+
 def test_generate_and_openai_endpoints(worker):
     from fastapi.testclient import TestClient
     from ipex_llm_b200.serving import FastApp
