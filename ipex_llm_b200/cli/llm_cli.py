@@ -2,6 +2,7 @@
 
     python -m ipex_llm_b200.cli.llm_cli -m <model dir or low-bit dir> -p "Once upon a time" -n 64 [-t sym_int4]
     python -m ipex_llm_b200.cli.llm_cli --chat -m <model dir>
+    python -m ipex_llm_b200.cli.llm_cli -m <dir without a tokenizer> -t bf16 --token-ids "12 7 90" -n 16
 
 The reference ships shell wrappers around per-family native binaries (``llm-cli -x llama -m model.bin -p ...``,
 python/llm/src/ipex_llm/cli/llm-cli:1-98); here the same flags drive the transformers-style API and ``-x`` is accepted
@@ -15,7 +16,7 @@ import sys
 import time
 
 
-def _load(path: str, low_bit: str, device: str):
+def _load(path: str, low_bit: str, device: str, tokenizer: bool = True):
     import torch
     from transformers import AutoTokenizer
     from ..transformers import AutoModel, AutoModelForCausalLM
@@ -28,7 +29,7 @@ def _load(path: str, low_bit: str, device: str):
     if path.endswith(".gguf"):
         model, tok = AutoModelForCausalLM.from_gguf(path, low_bit=low_bit)
     else:
-        tok = AutoTokenizer.from_pretrained(path, trust_remote_code=True)
+        tok = AutoTokenizer.from_pretrained(path, trust_remote_code=True) if tokenizer else None
         loader = (lambda c: c.load_low_bit(path, trust_remote_code=True)) if saved else \
             (lambda c: c.from_pretrained(path, load_in_low_bit=low_bit, trust_remote_code=True))
         try:
@@ -46,6 +47,8 @@ def build_parser():
     p.add_argument("-x", "--model_family", default=None, help="accepted for compatibility; read from the checkpoint")
     p.add_argument("-t", "--low-bit", default="sym_int4")
     p.add_argument("-p", "--prompt", default=None)
+    p.add_argument("--token-ids", default=None, help="prompt as token ids (\"12 7 90\"), answered with token ids; for "
+                   "checkpoints without a tokenizer")
     p.add_argument("-n", "--n_predict", type=int, default=128)
     p.add_argument("--temp", type=float, default=0.0)
     p.add_argument("--top_p", type=float, default=1.0)
@@ -71,9 +74,22 @@ def _generate(model, tok, prompt, n, temp, top_p, stream=True):
     return tok.decode(out[0][ids.shape[1]:], skip_special_tokens=True), new, dt
 
 
+def _generate_ids(model, ids, a):
+    import torch
+    kw = dict(max_new_tokens=a.n_predict, do_sample=a.temp > 0)
+    if a.temp > 0:
+        kw.update(temperature=a.temp, top_p=a.top_p)
+    with torch.no_grad():
+        out = model.generate(torch.tensor([ids], device=next(model.parameters()).device), **kw)
+    return out[0, len(ids):].tolist()
+
+
 def main(argv=None):
     a = build_parser().parse_args(argv)
-    model, tok = _load(a.model, a.low_bit, a.device)
+    model, tok = _load(a.model, a.low_bit, a.device, tokenizer=a.token_ids is None)
+    if a.token_ids is not None:
+        print(" ".join(map(str, _generate_ids(model, [int(t) for t in a.token_ids.replace(",", " ").split()], a))))
+        return 0
     if not a.chat:
         prompt = a.prompt if a.prompt is not None else sys.stdin.read()
         _, new, dt = _generate(model, tok, prompt, a.n_predict, a.temp, a.top_p)

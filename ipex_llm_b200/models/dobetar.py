@@ -101,7 +101,7 @@ class DenseExperts(nn.Module):
 
 
 class ClampedMoE(nn.Module):
-    """Sigmoid-routed experts: the routing weight multiplies the expert's input."""
+    """Sigmoid-routed experts, each of which reads its input scaled by the routing weight."""
 
     gate_alpha = 1.702           # slope of the gate's sigmoid, part of the design
 

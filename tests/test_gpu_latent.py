@@ -145,7 +145,8 @@ def bank_and_weights(dtype, W, I, E, top, limit, seed=0):
 @pytest.mark.parametrize("dtype", [F32, BF16])
 @pytest.mark.parametrize("W,I,E,top", [(64, 32, 6, 1), (72, 24, 5, 3), (50, 10, 4, 4), (128, 48, 40, 2)])
 def test_experts_both_paths(dtype, W, I, E, top):
-    """The routing weight multiplies the experts' input; the clamps bind (limit below the typical gate)."""
+    """Experts read scaled inputs (scaling outputs instead would show); the clamps bind: the limit is below the typical
+    gate."""
     from ipex_llm_b200.ops import latent as L
     bank, w, p = bank_and_weights(dtype, W, I, E, top, limit=0.8)
     nw = (1 + 0.2 * rnd(W, seed=7)).to(dtype).double()
@@ -296,7 +297,7 @@ def test_window_edges_with_a_key_that_stands_out(dtype, window):
     """The stand-out key at p decides every query that sees it, and none past p + window - 1; decoding one by one, in
     portions and (16-bit) as a prompt."""
     p, n = 13, 13 + window + 6
-    mx = Mixer(dtype, 8, 64, 16, 32, 96, window, n, standout=(p,))
+    mx = Mixer(dtype, 6, 48, 24, 32, 80, window, n, standout=(p,))
     want = mx.want()
     i, o = p + window - 1, p + window
     for fault, at in (("window_plus_one", o), ("window_minus_one", i)):
@@ -654,6 +655,22 @@ def test_served_batch_runs_on_the_engine():
         want = [words[t] for t in O.greedy(w, cfg, p, n)]
         want = [x for x in want if x not in ("<pad>", "<s>", "<unk>")]
         assert r.generated_tokens == n and r.text.split() == want
+
+
+def test_command_line_on_token_ids(tmp_path, capsys):
+    import json
+    from safetensors.torch import save_file
+    from ipex_llm_b200.cli import llm_cli
+    from ipex_llm_b200.transformers import AutoModelForCausalLM
+    cfg = cfg_plain()
+    (tmp_path / "config.json").write_text(json.dumps(cfg))
+    save_file({k: v.bfloat16().contiguous() for k, v in O.random_weights(cfg, seed=4).items()},
+              str(tmp_path / "model.safetensors"))
+    assert llm_cli.main(["-m", str(tmp_path), "-t", "bf16", "--token-ids", "3 9 4, 77", "-n", "6"]) == 0
+    got = [int(t) for t in capsys.readouterr().out.split()]
+    model = AutoModelForCausalLM.from_pretrained(str(tmp_path), load_in_low_bit="bf16", torch_dtype=BF16).to("cuda")
+    out = model.generate(torch.tensor([[3, 9, 4, 77]], device="cuda"), max_new_tokens=6, do_sample=False)
+    assert got == out[0, 4:].tolist() and len(got) == 6
 
 
 def test_trace_replay(tmp_path):
