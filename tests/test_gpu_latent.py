@@ -220,7 +220,7 @@ class Mixer:
         if len(standout):
             # every query shares a direction per head, and the stand-out rows' latents point along it for all heads
             d = rnd(heads, dim, seed=seed + 6)
-            q[:, :, :dim] = 0.4 * q[:, :, :dim] + d
+            q[:, :, :dim] = 0.4 * q[:, :, :dim] + 1.8 * d
             pull = torch.einsum("hd,hdr->r", d, self.uk.view(heads, dim, R))
             for i, p in enumerate(standout):
                 kv[p, :R] = 0.4 * kv[p, :R] + pull / pull.std() * (2.0 + i)
