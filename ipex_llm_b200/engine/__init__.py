@@ -24,13 +24,17 @@ _UNSUPPORTED_KW = ("num_beams", "penalty_alpha", "num_return_sequences", "constr
                    "inputs_embeds", "past_key_values")
 
 
+# engines of the package's own model classes, which run every size and weight format of their family
+_STREAM_ENGINES = {"latent": ("latent_engine", "LatentEngine"), "hybrid": ("hybrid_engine", "HybridEngine")}
+
+
 def supports(model, kwargs) -> bool:
     fam = family_for(model)
-    if fam is None or fam.engine not in ("llama", "mixtral", "latent"):
+    if fam is None or fam.engine not in ("llama", "mixtral", *_STREAM_ENGINES):
         return False
     if getattr(model, "_ipex_engine_disabled", False):
         return False
-    if fam.engine == "latent":
+    if fam.engine in _STREAM_ENGINES:
         # every size and weight format of the family runs on its engine; only the request can rule it out
         return not any(kwargs.get(k) not in (None, False, 1) for k in _UNSUPPORTED_KW)
     if getattr(getattr(model, "config", None), "ipex_alibi", False):
@@ -74,9 +78,10 @@ def supports(model, kwargs) -> bool:
 
 def engine_class(model):
     fam = family_for(model)
-    if fam is not None and fam.engine == "latent":
-        from .latent_engine import LatentEngine
-        return LatentEngine
+    if fam is not None and fam.engine in _STREAM_ENGINES:
+        import importlib
+        module, name = _STREAM_ENGINES[fam.engine]
+        return getattr(importlib.import_module(f".{module}", __package__), name)
     return DecoderEngine
 
 

@@ -510,6 +510,7 @@ class DecoderEngine:
             # warm up outside capture (lazy allocations, cudaFuncSetAttribute), restoring the state it advances
             saved_tok, saved_len = self.tokens.clone(), self.past_len.clone()
             saved_h = None if self.first_stage else self.h[0].clone()   # a later stage's input arrives in h[0]
+            saved_state = [(t, t.clone()) for t in self._step_state()]
             s = torch.cuda.Stream()
             s.wait_stream(torch.cuda.current_stream())
             with torch.cuda.stream(s):
@@ -519,6 +520,8 @@ class DecoderEngine:
             self.past_len.copy_(saved_len)
             if saved_h is not None:
                 self.h[0].copy_(saved_h)
+            for t, old in saved_state:
+                t.copy_(old)
             comm = self._tp_comm()
             parity = comm._parity if comm is not None else 0
             g = torch.cuda.CUDAGraph()
@@ -532,6 +535,10 @@ class DecoderEngine:
             # the buffer parity of the fused all-reduces is baked into the graph: realign (same on every rank)
             comm.barrier()
         entry[0].replay()
+
+    def _step_state(self):
+        """Tensors of the cache that a step changes in a way that running it again would not repeat."""
+        return []
 
     def _tp_comm(self):
         tp = self.layers[0].o.tp

@@ -168,11 +168,12 @@ class DobetarForCausalLM(PreTrainedModel, GenerationMixin):
         """Runs the latent engine's step on ``input_ids [B, S]`` behind whatever ``past_key_values`` holds.  Positions
         follow from the cache and the left padding that ``attention_mask`` shows on the first call, so
         ``position_ids`` is not read."""
-        from ..engine.latent_engine import stack_for
+        from ..engine.latent_engine import LatentStack
+        from ..engine.stream_engine import stack_for
         from ..ops.kv_cache import LatentCache
         if input_ids is None or inputs_embeds is not None:
             raise NotImplementedError("this architecture embeds token pairs: pass input_ids")
-        stack = stack_for(self)
+        stack = stack_for(self, LatentStack)
         cache = past_key_values if isinstance(past_key_values, LatentCache) else None
         if cache is None:
             if past_key_values is not None and past_key_values.get_seq_length() > 0:

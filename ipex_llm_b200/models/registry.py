@@ -148,6 +148,8 @@ FAMILIES = {
                    post=[("RwkvSelfAttention", R.rwkv4_attention_forward), ("RwkvFeedForward", R.rwkv4_ffn_forward)]),
     # multi-head latent attention on a 32-bit residual stream: the package's own model class, all of it on its engine
     "dobetar": Family(engine="latent"),
+    # windowed attention and gated-delta-rule layers on a 32-bit residual stream: likewise
+    "letarax": Family(engine="hybrid"),
     # LayerNorm families without a dedicated forward file: low-bit linears + the fused LayerNorm kernel
     "gpt_neox": Family(post=[("LayerNorm", C.layer_norm_forward)]),
     "bloom": Family(post=[("LayerNorm", C.layer_norm_forward)]),

@@ -36,8 +36,8 @@ CUDA_LIB = os.path.join(HERE, "libipex_llm_cuda.so")
 # Parts of the kernel library that stand on their own.  A process that needs one of them and finds no complete library
 # compiles just these sources (seconds instead of minutes); ``build_cuda`` always builds everything.
 COMPONENTS = {
-    "stream": ("elementwise.cu", "gemm_stream_tcgen05.cu", "gemv_dense.cu", "latent_attn.cu",
-               "latent_prefill_tcgen05.cu", "stream_ops.cu"),
+    "stream": ("delta_rule.cu", "elementwise.cu", "gemm_stream_tcgen05.cu", "gemv_dense.cu", "kv_attn.cu",
+               "latent_attn.cu", "latent_prefill_tcgen05.cu", "stream_ops.cu"),
 }
 
 NVCC_ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]

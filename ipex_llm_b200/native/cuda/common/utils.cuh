@@ -50,6 +50,13 @@ __device__ __forceinline__ float warp_max(float v) {
   return v;
 }
 
+// Tanh form of gelu, 0.5 z (1 + tanh(c (z + 0.044715 z^3))), through 0.5 (1 + tanh y) = 1 / (1 + e^(-2y)).
+__device__ __forceinline__ float gelu_tanh(float z) {
+  const float y = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+  return z / (1.0f + expf(-2.0f * y));
+}
+__device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
+
 // Programmatic dependent launch: a kernel launched with the programmatic-serialization attribute may start
 // while its predecessor in the stream is still running.  pdl_wait() blocks until the predecessor has
 // completed and its writes are visible; everything before it may only touch data the predecessor never

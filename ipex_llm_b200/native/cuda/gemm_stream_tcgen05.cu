@@ -1,8 +1,9 @@
 // Dense tcgen05 GEMM for decoders with a 32-bit residual stream and dense expert banks, sm_100a:
 //
-//     out = x[M, K] . W[N, K]^T      out_mode 0: 16-bit, optionally squared relu      1: added to an fp32 stream
-//                                    2: fp32 (router scores, logits)
+//     out = x[M, K] . W[N, K]^T (+ bias)  out_mode 0: 16-bit, optionally squared relu      1: added to an fp32 stream
+//                                         2: fp32 (router scores, logits)
 //     y = glu(row_scale * (x . W_gu^T))                    gate / up rows interleaved in 16-row tiles, N / 2 columns
+//     y = gelu_tanh(gate) * up, with biases                gate / up rows interleaved in 8-row tiles, N / 2 columns
 //
 // With `ranges` the launch covers a whole bank of weight matrices: group e multiplies its rows
 // [ranges[e][0], + ranges[e][1]) of x, read from DEVICE memory, so one launch serves all experts of a prompt and the
@@ -27,8 +28,9 @@ struct Args {
   int* err;
   int64_t ldo;
   int M, N, K, groups;
-  int out_mode, act;        // act 1: squared relu (out_mode 0); 2: clamped gated unit
+  int out_mode, act;        // act 1: squared relu (out_mode 0); 2: clamped gated unit; 3: gelu-gated unit
   float limit, alpha;
+  const void* bias;         // T [N] or null
 };
 
 template <int BT>
@@ -189,7 +191,20 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
         tmem_ld_32x32(tmem_base + (uint32_t(qd * 32) << 16) + acc * BT + c * 32, v);
         const int lim = min(32, rows - c * 32);
         const int64_t r0 = xrow + c * 32;
-        if (a.act == 2) {
+        const float bn = a.bias != nullptr && n < a.N ? to_float<T>(reinterpret_cast<const T*>(a.bias)[n]) : 0.f;
+        if (a.act == 3) {
+          // lanes with bit 3 clear hold gate rows, the lanes eight above them the matching up rows
+          const int n_out = (tl.nb * kBM + qd * 32) / 2 + (lane >> 4) * 8 + (lane & 7);
+          T* out = reinterpret_cast<T*>(a.out) + r0 * a.ldo + n_out;
+          const bool writer = (lane & 8) == 0 && n_out < a.N / 2;
+#pragma unroll
+          for (int j = 0; j < 32; ++j) {
+            const float sv = __uint_as_float(v[j]) + bn;
+            const float u = __shfl_down_sync(0xffffffffu, sv, 8);
+            const float y = 0.7978845608028654f * (sv + 0.044715f * sv * sv * sv);
+            if (writer && j < lim) out[(int64_t)j * a.ldo] = from_float<T>(sv / (1.0f + __expf(-2.0f * y)) * u);
+          }
+        } else if (a.act == 2) {
           // lanes 0..15 hold gate rows, lanes 16..31 the matching up rows
           const int n_out = (tl.nb * kBM + qd * 32) / 2 + (lane & 15);
           T* out = reinterpret_cast<T*>(a.out) + r0 * a.ldo + n_out;
@@ -208,7 +223,7 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
             T* out = reinterpret_cast<T*>(a.out) + r0 * a.ldo + n;
 #pragma unroll
             for (int j = 0; j < 32; ++j) {
-              float f = __uint_as_float(v[j]);
+              float f = __uint_as_float(v[j]) + bn;
               if (a.act == 1) f = f > 0.f ? f * f : 0.f;
               if (j < lim) out[(int64_t)j * a.ldo] = from_float<T>(f);
             }
@@ -220,11 +235,11 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
               for (int j = 0; j < 32; ++j) old[j] = j < lim ? out[(int64_t)j * a.ldo] : 0.f;
 #pragma unroll
               for (int j = 0; j < 32; ++j)
-                if (j < lim) out[(int64_t)j * a.ldo] = old[j] + __uint_as_float(v[j]);
+                if (j < lim) out[(int64_t)j * a.ldo] = old[j] + (__uint_as_float(v[j]) + bn);
             } else {
 #pragma unroll
               for (int j = 0; j < 32; ++j)
-                if (j < lim) out[(int64_t)j * a.ldo] = __uint_as_float(v[j]);
+                if (j < lim) out[(int64_t)j * a.ldo] = __uint_as_float(v[j]) + bn;
             }
           }
         }
@@ -283,20 +298,23 @@ int dispatch(int bt, const void* x, int64_t ldx, int x_rows, const void* w, int6
 }  // namespace
 
 // See the head of this file.  M: rows of x; with `ranges` the groups' rows partition them.  w: [groups * N, K].  bt:
-// token tile (32 / 64 / 128 / 256).  row_scale only with act 2 (then out_mode 0 and N a multiple of 32).
+// token tile (32 / 64 / 128 / 256).  row_scale only with act 2 (then out_mode 0 and N a multiple of 32).  act 3: out_mode
+// 0, N a multiple of 16.  bias (may be null) has N entries of the operands' type; not with act 2 or ranges.
 // Strides of x and w multiples of 8 elements, bases 16-byte aligned.  Returns a cudaError_t, or -1 when the
 // tensor-map encoder rejects the operands.
 IPEX_API int ipex_gemm_stream(const void* x, int64_t ldx, const void* w, int64_t ldw, void* out, int64_t ldo,
-                              const float* row_scale, const int* ranges, int groups, int M, int N, int K, int out_mode,
+                              const void* bias, const float* row_scale, const int* ranges, int groups, int M, int N, int K, int out_mode,
                               int act, float limit, float alpha, int bt, int dtype, int* err, void* stream) {
   if (M < 1 || N < 1 || K < 1 || groups < 1 || (ldx % 8) != 0 || (ldw % 8) != 0 || out_mode < 0 || out_mode > 2)
     return (int)cudaErrorInvalidValue;
   if ((groups > 1) != (ranges != nullptr) && ranges == nullptr) return (int)cudaErrorInvalidValue;
   if (act == 2 && (row_scale == nullptr || out_mode != 0 || (N % 32) != 0)) return (int)cudaErrorInvalidValue;
-  if (act < 0 || act > 2 || (act == 1 && out_mode != 0)) return (int)cudaErrorInvalidValue;
+  if (act < 0 || act > 3 || (act == 1 && out_mode != 0) || (act == 3 && (out_mode != 0 || (N % 16) != 0)) ||
+      (bias != nullptr && (act == 2 || ranges != nullptr)))
+    return (int)cudaErrorInvalidValue;
   if ((reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15)) return (int)cudaErrorInvalidValue;
   if ((int64_t)groups * N > 0x7fffffff) return (int)cudaErrorInvalidValue;
-  Args a = {out, row_scale, ranges, err, ldo, M, N, K, groups, out_mode, act, limit, alpha};
+  Args a = {out, row_scale, ranges, err, ldo, M, N, K, groups, out_mode, act, limit, alpha, bias};
   cudaStream_t st = (cudaStream_t)stream;
   if (dtype == DT_F16) return dispatch<__half>(bt, x, ldx, M, w, ldw, a, st);
   if (dtype == DT_BF16) return dispatch<__nv_bfloat16>(bt, x, ldx, M, w, ldw, a, st);

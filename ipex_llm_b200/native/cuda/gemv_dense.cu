@@ -1,8 +1,10 @@
 // Few-row products with dense 16-bit or 32-bit weights for decoders that keep a 32-bit residual stream, sm_100a.
 //
 //   gemv_rows    y[M <= 8, N] = act( x . W[N, K]^T )   with x either activations in the weight dtype or the fp32
-//                residual stream, RMS-normed while it is staged in shared memory; the result goes out in the weight
-//                dtype, is added to an fp32 residual, or leaves as fp32 with an optional tanh soft-cap (logits)
+//                residual stream, RMS-normed while it is staged in shared memory; the result (plus a bias) goes out in
+//                the weight dtype, is added to an fp32 residual, or leaves as fp32 with an optional tanh soft-cap
+//                (logits); gate and up rows may be joined to gelu_tanh(gate) * up, and the rows of a second matrix
+//                may ride along with fp32 results (gates of a recurrence beside its projections)
 //   moe_router   norm + router scores in fp32 + sigmoid + top-k of one token per CTA
 //   moe_glu      per (token, choice) slot: clamped gated unit of the chosen expert, the routing weight applied to the
 //                expert's input
@@ -185,15 +187,43 @@ struct GemvRowsArgs {
   int64_t ldw, ldx, ldo;
   float eps, softcap;
   int M, N, K, kp;
-  int out_mode, act;     // act 1: square of relu
+  int out_mode, act;     // act 1: square of relu; 3: gelu_tanh(gate) * up, N / 2 columns come out
   int vec;
+  const void* bias;      // T [N] or null
+  const void* w2;        // rows N1 .. N (row stride ldw), or null (then N1 = N)
+  float* out2;           // ... and their results, fp32
+  int64_t ldo2;
+  int N1;
+  int interleaved;       // act 3: gate and up rows alternate in blocks of eight, else gate rows before up rows
 };
 
 __device__ __forceinline__ float finish(float v, int act) { return act == 1 ? (v > 0.f ? v * v : 0.f) : v; }
 
 template <typename T>
+__device__ __forceinline__ const T* weight_row(const GemvRowsArgs& a, int n) {
+  return n < a.N1 ? reinterpret_cast<const T*>(a.w) + (int64_t)n * a.ldw
+                  : reinterpret_cast<const T*>(a.w2) + (int64_t)(n - a.N1) * a.ldw;
+}
+
+template <typename T>
+__device__ __forceinline__ float bias_of(const GemvRowsArgs& a, int n) {
+  return a.bias != nullptr ? DT<T>::to_f(reinterpret_cast<const T*>(a.bias)[n]) : 0.f;
+}
+
+// hidden unit i of token m from its two products (weight rows ng and nu)
+template <typename T>
+__device__ __forceinline__ void store_gated(const GemvRowsArgs& a, int m, int i, int ng, int nu, float g, float u) {
+  const float v = gelu_tanh(g + bias_of<T>(a, ng)) * (u + bias_of<T>(a, nu));
+  reinterpret_cast<T*>(a.out)[(int64_t)m * a.ldo + i] = DT<T>::from_f(v);
+}
+
+template <typename T>
 __device__ __forceinline__ void store_row(const GemvRowsArgs& a, int m, int n, float v) {
-  v = finish(v, a.act);
+  if (n >= a.N1) {
+    a.out2[(int64_t)m * a.ldo2 + n - a.N1] = v;
+    return;
+  }
+  v = finish(v + bias_of<T>(a, n), a.act);
   if (a.out_mode == 0) {
     reinterpret_cast<T*>(a.out)[(int64_t)m * a.ldo + n] = DT<T>::from_f(v);
   } else {
@@ -203,26 +233,36 @@ __device__ __forceinline__ void store_row(const GemvRowsArgs& a, int m, int n, f
   }
 }
 
-template <typename T, int M, int R>
+// GLU: a task is a hidden unit, its two rows are the gate's and the up product's.
+template <typename T, int M, int R, bool GLU>
 __global__ void __launch_bounds__(kThreads) gemv_rows_kernel(GemvRowsArgs a) {
   extern __shared__ __align__(16) uint8_t smem[];
   __shared__ float red[kWarps];
   T* sx = reinterpret_cast<T*>(smem);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const T* W = reinterpret_cast<const T*>(a.w);
   const int ntask = (a.N + R - 1) / R;
   const int t0 = blockIdx.x * kWarps + warp;
+  auto row_of = [&](int t, int r) {
+    if constexpr (GLU) return a.interleaved ? (t >> 3) * 16 + (t & 7) + 8 * r : t + r * (a.N / 2);
+    else return t * R + r;
+  };
   pdl_launch_dependents();
-  if (a.vec && t0 < ntask && lane < R && t0 * R + lane < a.N)
-    prefetch_l2_bulk(W + (int64_t)(t0 * R + lane) * a.ldw, (uint32_t)(a.K * sizeof(T)));
+  if (a.vec && t0 < ntask && lane < R && row_of(t0, lane) < a.N)
+    prefetch_l2_bulk(weight_row<T>(a, row_of(t0, lane)), (uint32_t)(a.K * sizeof(T)));
   pdl_wait();
   stage_rows<T>(sx, a.kp, a.x, a.ldx, reinterpret_cast<const T*>(a.norm_w), a.eps, a.M, a.K, red);
   for (int t = t0; t < ntask; t += gridDim.x * kWarps) {
     const T* w[R];
 #pragma unroll
-    for (int r = 0; r < R; ++r) w[r] = W + (int64_t)min(t * R + r, a.N - 1) * a.ldw;
+    for (int r = 0; r < R; ++r) w[r] = weight_row<T>(a, min(row_of(t, r), a.N - 1));
     float acc[M][R] = {};
     dot_rows<T, M, R>(w, sx, a.kp, a.K, a.vec != 0, lane, acc);
+    if constexpr (GLU) {
+#pragma unroll
+      for (int m = 0; m < M; ++m)
+        if (lane == m && m < a.M) store_gated<T>(a, m, t, row_of(t, 0), row_of(t, 1), acc[m][0], acc[m][1]);
+      continue;
+    }
 #pragma unroll
     for (int m = 0; m < M; ++m)
 #pragma unroll
@@ -264,12 +304,11 @@ __global__ void __launch_bounds__(kThreads) gemv_mma_kernel(GemvRowsArgs a, int 
   const int tpc = kWarps / split, sub = warp % split;
   const int ntile = (a.N + 15) / 16, nkb = (a.K + 31) / 32;
   const int per = (nkb + split - 1) / split, kb0 = sub * per, kb1 = min(kb0 + per, nkb);
-  const T* W = reinterpret_cast<const T*>(a.w);
   pdl_launch_dependents();
   {
     const int tile = blockIdx.x * tpc + warp / split, row = tile * 16 + lane;
     const int k0 = kb0 * 32, bytes = (min(kb1 * 32, a.K) - k0) * (int)sizeof(T);
-    if (lane < 16 && row < a.N && bytes > 0) prefetch_l2_bulk(W + (int64_t)row * a.ldw + k0, (uint32_t)bytes);
+    if (lane < 16 && row < a.N && bytes > 0) prefetch_l2_bulk(weight_row<T>(a, row) + k0, (uint32_t)bytes);
   }
   pdl_wait();
   const bool staged = a.norm_w != nullptr;
@@ -289,8 +328,8 @@ __global__ void __launch_bounds__(kThreads) gemv_mma_kernel(GemvRowsArgs a, int 
     const int tile = base + warp / split;
     float acc[2][NT][4] = {};
     if (tile < ntile) {
-      const T* w0 = W + (int64_t)min(tile * 16 + g, a.N - 1) * a.ldw + t * 8;
-      const T* w1 = W + (int64_t)min(tile * 16 + g + 8, a.N - 1) * a.ldw + t * 8;
+      const T* w0 = weight_row<T>(a, min(tile * 16 + g, a.N - 1)) + t * 8;
+      const T* w1 = weight_row<T>(a, min(tile * 16 + g + 8, a.N - 1)) + t * 8;
       for (int kb = kb0; kb < kb1; kb += U) {
         uint4 r0[U], r1[U];
 #pragma unroll
@@ -327,6 +366,22 @@ __global__ void __launch_bounds__(kThreads) gemv_mma_kernel(GemvRowsArgs a, int 
       __syncthreads();
       // the group's warps share the sums: value (n, i) goes to warp (n * 4 + i) % split
       const float* grp = part + ((size_t)par * kWarps + warp / split * split) * (NT * 128);
+      if (a.act == 3) {
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+          for (int i = 0; i < 2; ++i)
+            if ((n * 2 + i) % split == sub) {
+              float gv = 0.f, uv = 0.f;
+              for (int w = 0; w < split; ++w) {
+                gv += grp[w * (NT * 128) + (n * 4 + i) * 32 + lane];
+                uv += grp[w * (NT * 128) + (n * 4 + i + 2) * 32 + lane];
+              }
+              const int row = tile * 16 + g, m = n * 8 + 2 * t + i;
+              if (tile < ntile && m < a.M) store_gated<T>(a, m, tile * 8 + g, row, row + 8, gv, uv);
+            }
+        continue;
+      }
 #pragma unroll
       for (int n = 0; n < NT; ++n)
 #pragma unroll
@@ -337,6 +392,15 @@ __global__ void __launch_bounds__(kThreads) gemv_mma_kernel(GemvRowsArgs a, int 
             const int row = tile * 16 + g + 8 * (i >> 1), m = n * 8 + 2 * t + (i & 1);
             if (tile < ntile && row < a.N && m < a.M) store_row<T>(a, m, row, v);
           }
+    } else if (a.act == 3) {
+#pragma unroll
+      for (int n = 0; n < NT; ++n)
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+          const int row = tile * 16 + g, m = n * 8 + 2 * t + i;
+          if (tile < ntile && m < a.M)
+            store_gated<T>(a, m, tile * 8 + g, row, row + 8, acc[0][n][i], acc[0][n][i + 2]);
+        }
     } else {
 #pragma unroll
       for (int n = 0; n < NT; ++n)
@@ -359,9 +423,9 @@ int sm_count() {
   return sms;
 }
 
-template <typename T, int M, int R>
+template <typename T, int M, int R, bool GLU = false>
 cudaError_t launch_gemv(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
-  auto kern = gemv_rows_kernel<T, M, R>;
+  auto kern = gemv_rows_kernel<T, M, R, GLU>;
   const size_t smem = (size_t)M * a.kp * sizeof(T);      // rows past a.M are read (and dropped), never used
   if (smem > 48 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -376,6 +440,7 @@ cudaError_t launch_gemv(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
 template <typename T, int M>
 cudaError_t pick_rows(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
   const int warps = sm_count() * kWarps;
+  if (a.act == 3) return launch_gemv<T, M, 2, true>(a, pdl, st);
   if (a.N >= 4 * warps) return launch_gemv<T, M, 4>(a, pdl, st);
   if (a.N >= warps) return launch_gemv<T, M, 2>(a, pdl, st);
   return launch_gemv<T, M, 1>(a, pdl, st);
@@ -406,7 +471,7 @@ template <typename T>
 cudaError_t pick_m(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
   if constexpr (sizeof(T) == 2) {
     const bool direct = a.norm_w != nullptr || ((reinterpret_cast<uintptr_t>(a.x) & 15) == 0 && a.ldx % 8 == 0);
-    if (a.vec && direct && mma_from(a)) {
+    if (a.vec && direct && mma_from(a) && (a.act != 3 || a.interleaved)) {
       if (a.M <= 8) return launch_gemv_mma<T, 1>(a, pdl, st);
       return launch_gemv_mma<T, 2>(a, pdl, st);
     }
@@ -601,16 +666,31 @@ IPEX_API int ipex_gemv_rows_max(int K, int dtype) {
 // Timing sweeps: smallest row count of the tensor-core kernel (17: never).
 IPEX_API void ipex_gemv_rows_tune(int mma_from_rows) { g_mma_from = mma_from_rows; }
 
-// y = act(x . W^T): see GemvRowsArgs.  M <= ipex_gemv_rows_max(K, dtype).
+// y = act(x . W^T + bias): see GemvRowsArgs.  M <= ipex_gemv_rows_max(K, dtype).  w2 / out2 (may be null): N2 more
+// rows with the same row stride whose results go to out2 [M, ldo2] in fp32.  act 3: out_mode 0, N even (a multiple of
+// 16 when interleaved), no second matrix.
 IPEX_API int ipex_gemv_rows(const void* w, int64_t ldw, const void* x, int64_t ldx, const void* norm_w, float eps,
-                            void* out, int64_t ldo, int M, int N, int K, int out_mode, int act, float softcap, int dtype,
+                            const void* bias, void* out, int64_t ldo, const void* w2, int N2, float* out2, int64_t ldo2,
+                            int M, int N, int K, int out_mode, int act, int interleaved, float softcap, int dtype,
                             int pdl, void* stream) {
   if (M < 1 || N < 1 || K < 1 || out_mode < 0 || out_mode > 2 || M > ipex_gemv_rows_max(K, dtype))
+    return (int)cudaErrorInvalidValue;
+  if (act < 0 || act == 2 || act > 3 || (act == 3 && (out_mode != 0 || (N % 2) || (interleaved && (N % 16)) || w2 != nullptr)) ||
+      (w2 != nullptr && (N2 < 1 || out2 == nullptr)))
     return (int)cudaErrorInvalidValue;
   return by_dtype(dtype, [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
     GemvRowsArgs a = {w, x, norm_w, out, ldw, ldx, ldo, eps, softcap, M, N, K, padded<T>(K), out_mode, act, 0};
-    a.vec = vec_ok<T>(w, ldw, K);
+    a.bias = bias;
+    a.N1 = N;
+    a.interleaved = interleaved;
+    if (w2 != nullptr) {
+      a.w2 = w2;
+      a.out2 = out2;
+      a.ldo2 = ldo2;
+      a.N = N + N2;
+    }
+    a.vec = vec_ok<T>(w, ldw, K) && (w2 == nullptr || vec_ok<T>(w2, ldw, K));
     return pick_m<T>(a, pdl != 0, (cudaStream_t)stream);
   });
 }

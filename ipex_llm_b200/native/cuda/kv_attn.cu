@@ -1,0 +1,472 @@
+// Windowed attention over cached keys and values of different sizes, with an optional sink and mixed values, sm_100a.
+//
+//   kv_append   keys and values of the new tokens into the cache, the values mixed with those of an earlier layer;
+//               for prompts also the transposed values that the tcgen05 prompt attention reads
+//   kv_attn     attention of query tokens against what their slots hold: decoding (which appends its own row on the
+//               way), portions of prompts, and whole prompts of sizes or formats the tensor-core kernel does not take
+//
+// kv_attn: a cluster of up to eight CTAs shares the visible keys of one query token for up to RT query heads of one key
+// head.  A CTA walks its keys in tiles: eight lanes share a key for the scores (every lane has four keys in flight), the
+// tile's weights meet in shared memory, then threads own value columns and take turns over the keys.  The parts of a
+// cluster are merged through distributed shared memory, where the sink joins the denominator; nothing but the output is
+// written, so the step needs no scratch and no second launch.
+#include <cooperative_groups.h>
+
+#include "common/utils.cuh"
+
+namespace {
+
+namespace cg = cooperative_groups;
+
+constexpr int kThreads = 256;
+constexpr int kTile = 128;            // keys per tile
+
+template <typename F>
+int by_dtype(int dtype, F&& f) {
+  if (dtype == DT_F16) return (int)f((__half*)nullptr);
+  if (dtype == DT_BF16) return (int)f((__nv_bfloat16*)nullptr);
+  if (dtype == DT_F32) return (int)f((float*)nullptr);
+  return (int)cudaErrorInvalidValue;
+}
+
+// 16 bytes (VN elements) or a single element
+template <typename T, bool VEC> struct Pack {
+  static constexpr int n = VEC ? 16 / (int)sizeof(T) : 1;
+};
+
+template <typename T, bool VEC>
+__device__ __forceinline__ void load_pack(const T* p, float (&f)[Pack<T, VEC>::n]) {
+  if constexpr (!VEC) {
+    f[0] = DT<T>::to_f(*p);
+  } else {
+    const uint4 v = *reinterpret_cast<const uint4*>(p);
+    const T* e = reinterpret_cast<const T*>(&v);
+#pragma unroll
+    for (int i = 0; i < Pack<T, VEC>::n; ++i) f[i] = DT<T>::to_f(e[i]);
+  }
+}
+
+__device__ __forceinline__ float mixed(float v, float first, float lambda) { return (1.0f - lambda) * v + lambda * first; }
+
+// ---------------------------------------------------------------------------------------------- append
+struct AppendArgs {
+  const void* k;        // T [tokens, ld] at head * dim
+  const void* v;        // T [tokens, ld] at head * vdim
+  const void* vfirst;   // T [tokens, ld_vf] or null
+  void* kc;             // cache rows: slot * k_slot + head * k_head + position * dim
+  void* vc;
+  void* vt;             // T [heads * vdim, ld_vt] or null
+  const int* slot;
+  const int* pos;
+  int64_t ld, ld_vf, k_slot, k_head, v_slot, v_head, ld_vt;
+  float lambda;
+  int tokens, dim, vdim;
+};
+
+// CTA = 64 tokens of one head.
+template <typename T>
+__global__ void __launch_bounds__(kThreads) kv_append_kernel(AppendArgs a) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  T* sv = reinterpret_cast<T*>(smem);              // [64][vdim + pad] when vt is wanted
+  const int t0 = blockIdx.x * 64, g = blockIdx.y, nt = min(64, a.tokens - t0);
+  const int ldsv = (a.vdim + 1) | 1;               // odd: columns fall into different banks
+  pdl_launch_dependents();
+  pdl_wait();
+  const T* k = reinterpret_cast<const T*>(a.k);
+  const T* v = reinterpret_cast<const T*>(a.v);
+  const T* vf = reinterpret_cast<const T*>(a.vfirst);
+  T* kc = reinterpret_cast<T*>(a.kc);
+  T* vc = reinterpret_cast<T*>(a.vc);
+  constexpr int VN = 16 / (int)sizeof(T);
+  const bool kvec = a.dim % VN == 0 && a.ld % VN == 0 && (((uintptr_t)k | (uintptr_t)kc) & 15) == 0;
+  if (kvec) {
+    const int nv = a.dim / VN;
+    for (int i = threadIdx.x; i < nt * nv; i += kThreads) {
+      const int t = i / nv, c = i % nv;
+      const uint4 x = *reinterpret_cast<const uint4*>(k + (int64_t)(t0 + t) * a.ld + (int64_t)g * a.dim + c * VN);
+      T* row = kc + (int64_t)a.slot[t0 + t] * a.k_slot + (int64_t)g * a.k_head + (int64_t)a.pos[t0 + t] * a.dim;
+      *reinterpret_cast<uint4*>(row + c * VN) = x;
+    }
+  } else {
+    for (int i = threadIdx.x; i < nt * a.dim; i += kThreads) {
+      const int t = i / a.dim, c = i % a.dim;
+      kc[(int64_t)a.slot[t0 + t] * a.k_slot + (int64_t)g * a.k_head + (int64_t)a.pos[t0 + t] * a.dim + c] =
+          k[(int64_t)(t0 + t) * a.ld + (int64_t)g * a.dim + c];
+    }
+  }
+  const bool vvec = a.vdim % VN == 0 && a.ld % VN == 0 && (((uintptr_t)v | (uintptr_t)vc) & 15) == 0 &&
+                    (vf == nullptr || (a.ld_vf % VN == 0 && ((uintptr_t)vf & 15) == 0));
+  auto values = [&](auto tag) {
+    constexpr bool VEC = decltype(tag)::value;
+    constexpr int N = Pack<T, VEC>::n;
+    const int nv = a.vdim / N;
+    for (int i = threadIdx.x; i < nt * nv; i += kThreads) {
+      const int t = i / nv, c = (i % nv) * N;
+      float x[N];
+      load_pack<T, VEC>(v + (int64_t)(t0 + t) * a.ld + (int64_t)g * a.vdim + c, x);
+      if (vf != nullptr) {
+        float y[N];
+        load_pack<T, VEC>(vf + (int64_t)(t0 + t) * a.ld_vf + (int64_t)g * a.vdim + c, y);
+#pragma unroll
+        for (int j = 0; j < N; ++j) x[j] = mixed(x[j], y[j], a.lambda);
+      }
+      __align__(16) T o[N];
+#pragma unroll
+      for (int j = 0; j < N; ++j) o[j] = DT<T>::from_f(x[j]);
+      T* row = vc + (int64_t)a.slot[t0 + t] * a.v_slot + (int64_t)g * a.v_head + (int64_t)a.pos[t0 + t] * a.vdim + c;
+      if constexpr (VEC) *reinterpret_cast<uint4*>(row) = *reinterpret_cast<const uint4*>(o);
+      else row[0] = o[0];
+      if (a.vt != nullptr) {
+#pragma unroll
+        for (int j = 0; j < N; ++j) sv[t * ldsv + c + j] = o[j];
+      }
+    }
+  };
+  if (vvec) values(std::true_type{});
+  else values(std::false_type{});
+  if (a.vt == nullptr) return;
+  __syncthreads();
+  // ld_vt is a multiple of VN, so whole vectors of tokens always fit; tokens past the end are zero
+  T* vt = reinterpret_cast<T*>(a.vt);
+  constexpr int TV = 64 / VN;
+  for (int i = threadIdx.x; i < a.vdim * TV; i += kThreads) {
+    const int c = i / TV, t = (i % TV) * VN;
+    if (t >= nt) continue;
+    __align__(16) T o[VN];
+#pragma unroll
+    for (int j = 0; j < VN; ++j) o[j] = t + j < nt ? sv[(t + j) * ldsv + c] : DT<T>::from_f(0.f);
+    *reinterpret_cast<uint4*>(vt + (int64_t)(g * a.vdim + c) * a.ld_vt + t0 + t) = *reinterpret_cast<const uint4*>(o);
+  }
+}
+
+// ---------------------------------------------------------------------------------------------- attention
+struct AttnArgs {
+  const void* q;        // T [tokens, ldq], head h at h * dim
+  const void* k;        // append: this launch's own keys and values, T [tokens, ldq] at kv head * dim / vdim
+  const void* v;
+  const void* vfirst;   // T [tokens, ld_vf] or null
+  void* kc;
+  void* vc;
+  void* out;            // T [tokens, ldo], head h at h * vdim
+  const int* slot;
+  const int* pos;
+  const int* start;     // [slots] position of the sequence's first token
+  int64_t ldq, ld_vf, ldo, k_slot, k_head, v_slot, v_head;
+  float lambda, scale;
+  int heads, kv_heads, dim, vdim, window, sink, append;
+};
+
+// N values on each of 8 lanes (a power of two) -> sums over the 8 lanes, spread so that a lane keeps max(1, N / 8) of
+// them: value i ends on the lanes whose id matches, in the order of the folds
+template <int N, int OFF>
+__device__ __forceinline__ void fold(float* v, int lane) {
+  if constexpr (N > 1) {
+    const bool up = lane & OFF;
+#pragma unroll
+    for (int i = 0; i < N / 2; ++i) {
+      const float keep = up ? v[i + N / 2] : v[i], give = up ? v[i] : v[i + N / 2];
+      v[i] = keep + __shfl_xor_sync(0xffffffffu, give, OFF);
+    }
+    if constexpr (OFF > 1) fold<N / 2, OFF / 2>(v, lane);
+  } else {
+    v[0] += __shfl_xor_sync(0xffffffffu, v[0], OFF);
+    if constexpr (OFF > 1) fold<1, OFF / 2>(v, lane);
+  }
+}
+
+template <typename T, int RT, bool VEC>
+__global__ void __launch_bounds__(kThreads) kv_attn_kernel(AttnArgs a, int nrb) {
+  constexpr int VN = Pack<T, VEC>::n;
+  extern __shared__ __align__(16) float sm[];
+  cg::cluster_group cluster = cg::this_cluster();
+  const int nsplit = gridDim.x, split = blockIdx.x;
+  const int g = blockIdx.y / nrb, rb = blockIdx.y % nrb, tok = blockIdx.z;
+  const int R = a.heads / a.kv_heads, r0 = rb * RT, rows = min(RT, R - r0);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int dimp = (a.dim + 3) & ~3;
+  float* sq = sm;                                // [RT][dimp] scaled queries
+  float* ss = sq + RT * dimp;                    // [RT][kTile] scores, then weights
+  float* sc = ss + RT * kTile;                   // [RT] factor of what was gathered before this tile
+  float* sml = sc + RT;                          // [RT][2] maximum and sum
+  float* so = sml + 2 * RT;                      // [RT][vdim] this CTA's part of the output
+  float* sred = so + RT * ((a.vdim + 3) & ~3);   // [subsets][RT][vdim]
+  pdl_launch_dependents();
+  pdl_wait();
+  const int slot = a.slot[tok], pos = a.pos[tok], start = a.start[slot];
+  const int lo = max(start, a.window > 0 ? pos - a.window + 1 : 0), n = pos + 1 - lo;
+  const int chunk = (n + nsplit - 1) / nsplit;
+  const int j0 = lo + min(n, split * chunk), j1 = lo + min(n, (split + 1) * chunk);
+  T* kc = reinterpret_cast<T*>(a.kc) + (int64_t)slot * a.k_slot + (int64_t)g * a.k_head;
+  T* vc = reinterpret_cast<T*>(a.vc) + (int64_t)slot * a.v_slot + (int64_t)g * a.v_head;
+  if (a.append && j1 == pos + 1 && j0 < j1) {
+    // this CTA owns the newest key: it files the row and reads it back like the others (every row block of the head
+    // does, with the same values)
+    const T* k = reinterpret_cast<const T*>(a.k) + (int64_t)tok * a.ldq + (int64_t)g * a.dim;
+    const T* v = reinterpret_cast<const T*>(a.v) + (int64_t)tok * a.ldq + (int64_t)g * a.vdim;
+    const T* vf = reinterpret_cast<const T*>(a.vfirst) + (int64_t)tok * a.ld_vf + (int64_t)g * a.vdim;
+    for (int i = tid; i < a.dim; i += kThreads) kc[(int64_t)pos * a.dim + i] = k[i];
+    for (int i = tid; i < a.vdim; i += kThreads) {
+      const float own = DT<T>::to_f(v[i]);
+      vc[(int64_t)pos * a.vdim + i] =
+          a.vfirst != nullptr ? DT<T>::from_f(mixed(own, DT<T>::to_f(vf[i]), a.lambda)) : v[i];
+    }
+  }
+  {
+    const T* q = reinterpret_cast<const T*>(a.q) + (int64_t)tok * a.ldq + (int64_t)(g * R + r0) * a.dim;
+    for (int i = tid; i < RT * a.dim; i += kThreads) {
+      const int r = i / a.dim, c = i % a.dim;
+      sq[r * dimp + c] = r < rows ? DT<T>::to_f(q[(int64_t)r * a.dim + c]) * a.scale : 0.f;
+    }
+  }
+  __syncthreads();
+
+  const int nvk = a.dim / VN, nvv = a.vdim / VN;
+  const int subsets = kThreads / nvv, vv = tid % nvv, sub = tid / nvv;
+  const bool von = sub < subsets;
+  float acc[RT][VN];
+#pragma unroll
+  for (int r = 0; r < RT; ++r)
+#pragma unroll
+    for (int i = 0; i < VN; ++i) acc[r][i] = 0.f;
+  float m_row = -INFINITY, l_row = 0.f;          // of row `warp` (rows <= 8 warps)
+
+  const int kg = lane >> 3, ks = lane & 7;       // a warp: four keys at a time, eight lanes each
+  for (int t0 = j0; t0 < j1; t0 += kTile) {
+    const int tn = min(kTile, j1 - t0);
+    // ---- scores: warp w takes keys w * 16 .. + 15 of the tile
+    if (warp * 16 < tn) {
+      float s[4 * RT];
+#pragma unroll
+      for (int i = 0; i < 4 * RT; ++i) s[i] = 0.f;
+      const T* kp[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) kp[u] = kc + (int64_t)(t0 + min(tn - 1, warp * 16 + u * 4 + kg)) * a.dim;
+      for (int c = ks; c < nvk; c += 8) {
+        float kf[4][VN];
+#pragma unroll
+        for (int u = 0; u < 4; ++u) load_pack<T, VEC>(kp[u] + c * VN, kf[u]);
+#pragma unroll
+        for (int r = 0; r < RT; ++r) {
+          float qf[VN];
+          if constexpr (VN == 1) {
+            qf[0] = sq[r * dimp + c];
+          } else {
+#pragma unroll
+            for (int i = 0; i < VN / 4; ++i) {
+              const float4 x = *reinterpret_cast<const float4*>(sq + r * dimp + c * VN + 4 * i);
+              qf[4 * i] = x.x; qf[4 * i + 1] = x.y; qf[4 * i + 2] = x.z; qf[4 * i + 3] = x.w;
+            }
+          }
+#pragma unroll
+          for (int u = 0; u < 4; ++u)
+#pragma unroll
+            for (int i = 0; i < VN; ++i) s[u * RT + r] = fmaf(kf[u][i], qf[i], s[u * RT + r]);
+        }
+      }
+      // value index u * RT + r; after the folds a lane holds the block of indices its bits select
+      fold<4 * RT, 4>(s, lane);
+      constexpr int kKeep = 4 * RT >= 8 ? 4 * RT / 8 : 1;
+      int first = 0, width = 4 * RT;
+#pragma unroll
+      for (int off = 4; off > 0; off >>= 1)
+        if (width > 1) {
+          width >>= 1;
+          if (lane & off) first += width;
+        }
+      const bool writer = 4 * RT >= 8 || (lane & 1) == 0;        // four values on eight lanes: two lanes hold each
+      if (writer) {
+#pragma unroll
+        for (int i = 0; i < kKeep; ++i) {
+          const int idx = first + i, key = warp * 16 + idx / RT * 4 + kg;
+          ss[(idx % RT) * kTile + key] = key < tn ? s[i] : -INFINITY;
+        }
+      }
+    }
+    __syncthreads();
+    // ---- weights: a warp per row
+    if (warp < RT) {
+      float* row = ss + warp * kTile;
+      float x[kTile / 32], mx = m_row;
+#pragma unroll
+      for (int i = 0; i < kTile / 32; ++i) {
+        const int j = lane + 32 * i;
+        x[i] = j < tn ? row[j] : -INFINITY;
+        mx = fmaxf(mx, x[i]);
+      }
+      mx = warp_max(mx);
+      const float ref = mx == -INFINITY ? 0.f : mx;
+      float sum = 0.f;
+#pragma unroll
+      for (int i = 0; i < kTile / 32; ++i) {
+        const int j = lane + 32 * i;
+        const float p = x[i] == -INFINITY ? 0.f : expf(x[i] - ref);
+        sum += p;
+        if (j < tn) row[j] = p;
+      }
+      const float corr = m_row == -INFINITY ? 0.f : expf(m_row - ref);
+      l_row = l_row * corr + warp_sum(sum);
+      m_row = mx;
+      if (lane == 0) sc[warp] = corr;
+    }
+    __syncthreads();
+    // ---- values
+    if (von) {
+#pragma unroll
+      for (int r = 0; r < RT; ++r) {
+        const float c = sc[r];
+#pragma unroll
+        for (int i = 0; i < VN; ++i) acc[r][i] *= c;
+      }
+      const T* vp = vc + (int64_t)t0 * a.vdim + vv * VN;
+#pragma unroll 4
+      for (int j = sub; j < tn; j += subsets) {
+        float vf[VN];
+        load_pack<T, VEC>(vp + (int64_t)j * a.vdim, vf);
+#pragma unroll
+        for (int r = 0; r < RT; ++r) {
+          const float p = ss[r * kTile + j];
+#pragma unroll
+          for (int i = 0; i < VN; ++i) acc[r][i] = fmaf(p, vf[i], acc[r][i]);
+        }
+      }
+    }
+    __syncthreads();
+  }
+  // ---- this CTA's part
+  if (von) {
+#pragma unroll
+    for (int r = 0; r < RT; ++r)
+#pragma unroll
+      for (int i = 0; i < VN; ++i) sred[((size_t)sub * RT + r) * a.vdim + vv * VN + i] = acc[r][i];
+  }
+  if (warp < RT && lane == 0) {
+    sml[2 * warp] = m_row;
+    sml[2 * warp + 1] = l_row;
+  }
+  __syncthreads();
+  for (int i = tid; i < rows * a.vdim; i += kThreads) {
+    float s = 0.f;
+    for (int u = 0; u < subsets; ++u) s += sred[(size_t)u * RT * a.vdim + i];
+    so[i] = s;
+  }
+  if (nsplit > 1) cluster.sync();
+  else __syncthreads();
+  // ---- merge: every CTA of the cluster finishes its share of the outputs
+  T* out = reinterpret_cast<T*>(a.out) + (int64_t)tok * a.ldo + (int64_t)(g * R + r0) * a.vdim;
+  for (int i = split * kThreads + tid; i < rows * a.vdim; i += nsplit * kThreads) {
+    const int r = i / a.vdim;
+    float m = a.sink ? 0.f : -INFINITY;
+    for (int s = 0; s < nsplit; ++s) {
+      const float* p = nsplit > 1 ? cluster.map_shared_rank(sml, s) : sml;
+      m = fmaxf(m, p[2 * r]);
+    }
+    float l = a.sink ? expf(-m) : 0.f, o = 0.f;
+    for (int s = 0; s < nsplit; ++s) {
+      const float* p = nsplit > 1 ? cluster.map_shared_rank(sml, s) : sml;
+      const float* po = nsplit > 1 ? cluster.map_shared_rank(so, s) : so;
+      const float c = p[2 * r] == -INFINITY ? 0.f : expf(p[2 * r] - m);
+      l = fmaf(p[2 * r + 1], c, l);
+      o = fmaf(po[i], c, o);
+    }
+    out[i] = DT<T>::from_f(l > 0.f ? o / l : 0.f);
+  }
+  if (nsplit > 1) cluster.sync();      // the others may still read this CTA's part
+}
+
+template <typename T, int RT, bool VEC>
+cudaError_t launch_attn(const AttnArgs& a, int tokens, int nsplit, bool pdl, cudaStream_t st) {
+  constexpr int VN = Pack<T, VEC>::n;
+  const int dimp = (a.dim + 3) & ~3, vp = (a.vdim + 3) & ~3, R = a.heads / a.kv_heads;
+  const int nrb = (R + RT - 1) / RT, subsets = kThreads / (a.vdim / VN);
+  const size_t smem = ((size_t)RT * (dimp + kTile + 3 + vp) + (size_t)subsets * RT * a.vdim + 4) * sizeof(float);
+  if (smem > 220 * 1024 || (int64_t)a.kv_heads * nrb > 65535) return cudaErrorInvalidValue;
+  auto kern = kv_attn_kernel<T, RT, VEC>;
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return e;
+  }
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(nsplit, a.kv_heads * nrb, tokens);
+  cfg.blockDim = dim3(kThreads);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = st;
+  cudaLaunchAttribute attr[2];
+  int na = 0;
+  if (nsplit > 1) {
+    attr[na].id = cudaLaunchAttributeClusterDimension;
+    attr[na].val.clusterDim.x = nsplit;
+    attr[na].val.clusterDim.y = 1;
+    attr[na].val.clusterDim.z = 1;
+    ++na;
+  }
+  if (pdl) {
+    attr[na].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[na].val.programmaticStreamSerializationAllowed = 1;
+    ++na;
+  }
+  cfg.attrs = attr;
+  cfg.numAttrs = na;
+  return cudaLaunchKernelEx(&cfg, kern, a, nrb);
+}
+
+template <typename T, bool VEC>
+cudaError_t pick_rows(const AttnArgs& a, int tokens, int nsplit, bool pdl, cudaStream_t st) {
+  const int R = a.heads / a.kv_heads;
+  if (R <= 1) return launch_attn<T, 1, VEC>(a, tokens, nsplit, pdl, st);
+  if (R <= 2) return launch_attn<T, 2, VEC>(a, tokens, nsplit, pdl, st);
+  if (R <= 4) return launch_attn<T, 4, VEC>(a, tokens, nsplit, pdl, st);
+  return launch_attn<T, 8, VEC>(a, tokens, nsplit, pdl, st);
+}
+
+}  // namespace
+
+// Keys and values of `tokens` new tokens (k / v: rows of `ld` elements, heads behind one another) into the cache rows
+// of their slots and positions; v is mixed with vfirst (may be null) by lambda.  vt (may be null): the mixed values
+// transposed, [heads * vdim, ld_vt], ld_vt a multiple of 16 bytes and at least `tokens`.
+IPEX_API int ipex_kv_append(const void* k, const void* v, int64_t ld, const void* vfirst, int64_t ld_vf, float lambda,
+                            void* kc, int64_t k_slot, int64_t k_head, void* vc, int64_t v_slot, int64_t v_head, void* vt,
+                            int64_t ld_vt, const int* slot, const int* pos, int tokens, int kv_heads, int dim, int vdim,
+                            int dtype, int pdl, void* stream) {
+  if (tokens < 1 || kv_heads < 1 || kv_heads > 65535 || dim < 1 || vdim < 1) return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    constexpr int VN = 16 / (int)sizeof(T);
+    if (vt != nullptr && (ld_vt % VN || ld_vt < tokens || ((uintptr_t)vt & 15))) return cudaErrorInvalidValue;
+    AppendArgs a = {k, v, vfirst, kc, vc, vt, slot, pos, ld, ld_vf, k_slot, k_head, v_slot, v_head, ld_vt, lambda,
+                    tokens, dim, vdim};
+    const size_t smem = vt != nullptr ? (size_t)64 * (vdim + 2) * sizeof(T) : 0;
+    if (smem > 220 * 1024) return cudaErrorInvalidValue;
+    auto kern = kv_append_kernel<T>;
+    if (smem > 48 * 1024) {
+      cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      if (e != cudaSuccess) return e;
+    }
+    return launch_kernel(kern, dim3((tokens + 63) / 64, kv_heads), dim3(kThreads), smem, (cudaStream_t)stream, pdl != 0, a);
+  });
+}
+
+// Attention of `tokens` query tokens (q: rows of ldq elements, `heads` of `dim`) over positions
+// [max(start, pos - window + 1), pos] of their slots; window 0: unlimited.  append: file the tokens' own rows k / v
+// (same row stride as q, v mixed with vfirst) first - then no two tokens may share a slot; otherwise the cache holds
+// them.  nsplit: CTAs (1, 2, 4 or 8) the keys of a token are shared by.  sink: a score of 0 without a value in every
+// softmax.
+IPEX_API int ipex_kv_attn(const void* q, const void* k, const void* v, int64_t ldq, const void* vfirst, int64_t ld_vf,
+                          float lambda, void* kc, int64_t k_slot, int64_t k_head, void* vc, int64_t v_slot,
+                          int64_t v_head, void* out, int64_t ldo, const int* slot, const int* pos, const int* start,
+                          int tokens, int heads, int kv_heads, int dim, int vdim, int window, int sink, int append,
+                          int nsplit, float scale, int dtype, int pdl, void* stream) {
+  if (tokens < 1 || tokens > 65535 || kv_heads < 1 || heads % kv_heads != 0 || dim < 1 || vdim < 1 || window < 0 ||
+      nsplit < 1 || nsplit > 8 || (nsplit & (nsplit - 1)))
+    return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    constexpr int VN = 16 / (int)sizeof(T);
+    AttnArgs a = {q, k, v, vfirst, kc, vc, out, slot, pos, start, ldq, ld_vf, ldo, k_slot, k_head, v_slot, v_head,
+                  lambda, scale, heads, kv_heads, dim, vdim, window, sink, append};
+    const bool vec = dim % VN == 0 && vdim % VN == 0 && vdim / VN <= kThreads && (((uintptr_t)kc | (uintptr_t)vc) & 15) == 0;
+    cudaStream_t st = (cudaStream_t)stream;
+    if (vec) return pick_rows<T, true>(a, tokens, nsplit, pdl != 0, st);
+    if (vdim > kThreads) return cudaErrorInvalidValue;
+    return pick_rows<T, false>(a, tokens, nsplit, pdl != 0, st);
+  });
+}

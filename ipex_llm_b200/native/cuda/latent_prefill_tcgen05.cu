@@ -1,4 +1,5 @@
-// Prompt attention of multi-head latent attention on the 5th-generation tensor cores, sm_100a.
+// Prompt attention over packed sequences on the 5th-generation tensor cores, sm_100a: multi-head latent attention, and
+// attention with plain key / value heads (shared by groups of query heads), with or without a window and a sink.
 //
 // Keys and values are expanded from the latents by two GEMMs before this kernel; a head's key is then made of two
 // parts that live in different tensors: `dim` values of its own and `rd` rotated values shared by all heads.  Neither
@@ -51,6 +52,8 @@ struct Args {
   int dim, rd, vd, window;
   int nbn, nbr;           // k-blocks of the own and of the shared part
   int kst, vst;           // stages of the K and V^T rings (1 or 2)
+  int group;              // query heads per key / value head
+  int sink;               // one more score of 0, without a value, in every softmax
   float scale_log2;
 };
 
@@ -61,7 +64,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
                       const __grid_constant__ CUtensorMap tm_vt, Args a) {
   constexpr int kVBytes = DV * kBKV * 2;
   constexpr uint32_t kTmemCols = 512;
-  const int h = blockIdx.x, b = blockIdx.z;
+  const int h = blockIdx.x, b = blockIdx.z, hk = h / a.group;
   const int len = a.seq_len[b], row0 = a.seq_row[b];
   const int nqb = (len + kBQ - 1) / kBQ;
   const int qb = (int)gridDim.y - 1 - (int)blockIdx.y;      // longest rows of the longest sequence first
@@ -133,7 +136,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
         if (!mbar_wait(&k_empty[ks], kp ^ 1, abort_flag)) { ok = false; report(a.err, 34); break; }
         uint8_t* dk = sK + ks * nb * kBlkBytes;
         mbar_expect_tx(&k_full[ks], nb * kBlkBytes);
-        for (int i = 0; i < a.nbn; ++i) tma_load_3d(dk + i * kBlkBytes, &tm_kn, i * 64, h, krow, &k_full[ks]);
+        for (int i = 0; i < a.nbn; ++i) tma_load_3d(dk + i * kBlkBytes, &tm_kn, i * 64, hk, krow, &k_full[ks]);
         for (int i = 0; i < a.nbr; ++i) tma_load_2d(dk + (a.nbn + i) * kBlkBytes, &tm_kr, i * 64, krow, &k_full[ks]);
         if (++ks == a.kst) { ks = 0; kp ^= 1; }
         if (!mbar_wait(&v_empty[vs], vp ^ 1, abort_flag)) { ok = false; report(a.err, 34); break; }
@@ -141,7 +144,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
         mbar_expect_tx(&v_full[vs], kVBytes);
 #pragma unroll
         for (int i = 0; i < kBKV / 64; ++i)
-          tma_load_2d(dv + i * (DV * 128), &tm_vt, krow + i * 64, h * a.vd, &v_full[vs]);
+          tma_load_2d(dv + i * (DV * 128), &tm_vt, krow + i * 64, hk * a.vd, &v_full[vs]);
         if (++vs == a.vst) { vs = 0; vp ^= 1; }
       }
       if (!ok) {
@@ -294,6 +297,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
       mbar_arrive(x_full);
       ok = mbar_wait(x_full, nblk & 1, abort_flag);
       l += xch[(hf ^ 1) * 128 + r];
+      if (a.sink) l += ex2(-m);      // both halves hold the row's maximum
     }
     if (!ok && lane == 0) report(a.err, 36);
     if (ok && qpos < len) {
@@ -335,8 +339,8 @@ size_t smem_need(int nb, int dv, int kst, int vst) {
 }
 
 template <typename T, int DV>
-int launch(const void* q, int64_t ldq, const void* k, const void* kr, int64_t ld_kr, const void* vt, int64_t ld_vt,
-           Args& a, int B, int H, int tokens, int max_len, cudaStream_t stream) {
+int launch(const void* q, int64_t ldq, const void* k, int64_t ldk, const void* kr, int64_t ld_kr, const void* vt,
+           int64_t ld_vt, Args& a, int B, int H, int tokens, int max_len, cudaStream_t stream) {
   const CUtensorMapDataType dt =
       std::is_same<T, __half>::value ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   const int nb = a.nbn + a.nbr;
@@ -347,9 +351,10 @@ int launch(const void* q, int64_t ldq, const void* k, const void* kr, int64_t ld
   if (smem > kSmemMax) return (int)cudaErrorInvalidValue;
   CUtensorMap qn, qr, kn, krm, vm;
   const T* qp = reinterpret_cast<const T*>(q);
+  const int G = H / a.group;
   if (!encode_heads(&qn, dt, qp, a.dim, H, tokens, a.dim + a.rd, ldq) ||
-      !encode_heads(&kn, dt, k, a.dim, H, tokens, a.dim, (int64_t)H * a.dim) ||
-      !encode_2d_sw128(&vm, dt, vt, (uint64_t)tokens, (uint64_t)H * a.vd, (uint64_t)ld_vt * 2, 64, DV))
+      !encode_heads(&kn, dt, k, a.dim, G, tokens, a.dim, ldk) ||
+      !encode_2d_sw128(&vm, dt, vt, (uint64_t)tokens, (uint64_t)G * a.vd, (uint64_t)ld_vt * 2, 64, DV))
     return -1;
   qr = qn;
   krm = qn;
@@ -374,18 +379,20 @@ IPEX_API int ipex_latent_prefill_ok(int dim, int rd, int vd, int R, int dtype) {
   return (dim + 63) / 64 + (rd + 63) / 64 <= 4 && vd <= 128;
 }
 
-// Causal (windowed) attention of packed sequences: q [tokens, ldq] holds per head [dim | rd (rotated)], k [tokens,
-// H * dim], kr [tokens, ld_kr] (rotated, shared), vt [H * vd, ld_vt] (V transposed).  seq_row / seq_len: device, [B];
-// max_len: the largest length.  window 0: unlimited.  Strides multiples of 8 elements, bases 16-byte aligned.
-// Returns a cudaError_t, or -1 when the tensor-map encoder rejects the operands.
-IPEX_API int ipex_latent_prefill(const void* q, int64_t ldq, const void* k, const void* kr, int64_t ld_kr,
+// Causal (windowed) attention of packed sequences: q [tokens, ldq] holds per head [dim | rd (rotated)], k [tokens, ldk]
+// the G key heads of `dim`, kr [tokens, ld_kr] the rotated part shared by all heads (rd = 0: none), vt [G * vd, ld_vt]
+// the values transposed.  Query head h uses key / value head h / (H / G).  seq_row / seq_len: device, [B]; max_len: the
+// largest length.  window 0: unlimited.  sink: every softmax has one more score of 0 whose value is nothing.  Strides
+// multiples of 8 elements, bases 16-byte aligned.  Returns a cudaError_t, or -1 when the tensor-map encoder rejects
+// the operands.
+IPEX_API int ipex_packed_prefill(const void* q, int64_t ldq, const void* k, int64_t ldk, const void* kr, int64_t ld_kr,
                                  const void* vt, int64_t ld_vt, void* out, int64_t ldo, const int* seq_row,
-                                 const int* seq_len, int B, int H, int tokens, int max_len, int dim, int rd, int vd,
-                                 int window, float scale, int dtype, int* err, void* stream) {
+                                 const int* seq_len, int B, int H, int G, int tokens, int max_len, int dim, int rd,
+                                 int vd, int window, int sink, float scale, int dtype, int* err, void* stream) {
   if (!ipex_latent_prefill_ok(dim, rd, vd, 8, dtype) || B < 1 || B > 65535 || H < 1 || tokens < 1 || max_len < 1 ||
-      window < 0 || (max_len + kBQ - 1) / kBQ > 65535)
+      window < 0 || (max_len + kBQ - 1) / kBQ > 65535 || G < 1 || H % G != 0)
     return (int)cudaErrorInvalidValue;
-  if ((ldq % 8) || (ld_vt % 8) || (ldo % 8) || (rd > 0 && (ld_kr % 8)) || ld_vt < tokens)
+  if ((ldq % 8) || (ldk % 8) || (ld_vt % 8) || (ldo % 8) || (rd > 0 && (ld_kr % 8)) || ld_vt < tokens)
     return (int)cudaErrorInvalidValue;
   if (((uintptr_t)q | (uintptr_t)k | (uintptr_t)kr | (uintptr_t)vt | (uintptr_t)out) & 15)
     return (int)cudaErrorInvalidValue;
@@ -394,11 +401,13 @@ IPEX_API int ipex_latent_prefill(const void* q, int64_t ldq, const void* k, cons
   a.dim = dim; a.rd = rd; a.vd = vd; a.window = window;
   a.nbn = (dim + 63) / 64;
   a.nbr = (rd + 63) / 64;
+  a.group = H / G;
+  a.sink = sink;
   a.scale_log2 = scale * 1.4426950408889634f;
   cudaStream_t st = (cudaStream_t)stream;
   if (dtype == DT_F16)
-    return vd <= 64 ? launch<__half, 64>(q, ldq, k, kr, ld_kr, vt, ld_vt, a, B, H, tokens, max_len, st)
-                    : launch<__half, 128>(q, ldq, k, kr, ld_kr, vt, ld_vt, a, B, H, tokens, max_len, st);
-  return vd <= 64 ? launch<__nv_bfloat16, 64>(q, ldq, k, kr, ld_kr, vt, ld_vt, a, B, H, tokens, max_len, st)
-                  : launch<__nv_bfloat16, 128>(q, ldq, k, kr, ld_kr, vt, ld_vt, a, B, H, tokens, max_len, st);
+    return vd <= 64 ? launch<__half, 64>(q, ldq, k, ldk, kr, ld_kr, vt, ld_vt, a, B, H, tokens, max_len, st)
+                    : launch<__half, 128>(q, ldq, k, ldk, kr, ld_kr, vt, ld_vt, a, B, H, tokens, max_len, st);
+  return vd <= 64 ? launch<__nv_bfloat16, 64>(q, ldq, k, ldk, kr, ld_kr, vt, ld_vt, a, B, H, tokens, max_len, st)
+                  : launch<__nv_bfloat16, 128>(q, ldq, k, ldk, kr, ld_kr, vt, ld_vt, a, B, H, tokens, max_len, st);
 }

@@ -1,6 +1,7 @@
 // Element-wise and routing kernels of decoders with a 32-bit residual stream, sm_100a: embedding (scaled, with an
-// optional bigram table), RMS norm of the stream into the activation dtype, tanh soft-cap of fp32 logits, and the
-// data movement around a dense expert bank for prompts (slots grouped by expert on the device, row gather, clamped
+// optional bigram table), RMS norm of the stream into the activation dtype, the joint of a block that norms a
+// sublayer's output before it is added, tanh soft-cap of fp32 logits, biases and gelu-gated units behind library or
+// packed products, and the data movement around a dense expert bank for prompts (slots grouped by expert on the device, row gather, clamped
 // gated unit, combination into the stream), plus a plain tiled product for sizes the tensor-core kernels do not take
 // and for 32-bit models.
 #include "common/utils.cuh"
@@ -61,8 +62,8 @@ __global__ void embed_stream_kernel(const int64_t* __restrict__ tokens, const in
   }
 }
 
-template <typename T>
-__global__ void norm_stream_kernel(const float* __restrict__ x, int64_t ldx, const T* __restrict__ w,
+template <typename T, typename TW>
+__global__ void norm_stream_kernel(const float* __restrict__ x, int64_t ldx, const TW* __restrict__ w,
                                    T* __restrict__ out, int64_t ldo, const int* __restrict__ rows, int K, float eps) {
   __shared__ float red[32];
   pdl_launch_dependents();
@@ -86,15 +87,120 @@ __global__ void norm_stream_kernel(const float* __restrict__ x, int64_t ldx, con
     for (int k = threadIdx.x; k < K / 4; k += blockDim.x) {
       const float4 f = reinterpret_cast<const float4*>(src)[k];
       __align__(16) T o[4];
-      o[0] = DT<T>::from_f(f.x * inv * DT<T>::to_f(w[4 * k]));
-      o[1] = DT<T>::from_f(f.y * inv * DT<T>::to_f(w[4 * k + 1]));
-      o[2] = DT<T>::from_f(f.z * inv * DT<T>::to_f(w[4 * k + 2]));
-      o[3] = DT<T>::from_f(f.w * inv * DT<T>::to_f(w[4 * k + 3]));
+      o[0] = DT<T>::from_f(f.x * inv * DT<TW>::to_f(w[4 * k]));
+      o[1] = DT<T>::from_f(f.y * inv * DT<TW>::to_f(w[4 * k + 1]));
+      o[2] = DT<T>::from_f(f.z * inv * DT<TW>::to_f(w[4 * k + 2]));
+      o[3] = DT<T>::from_f(f.w * inv * DT<TW>::to_f(w[4 * k + 3]));
       if constexpr (sizeof(T) == 2) reinterpret_cast<uint2*>(dst)[k] = *reinterpret_cast<const uint2*>(o);
       else reinterpret_cast<uint4*>(dst)[k] = *reinterpret_cast<const uint4*>(o);
     }
   } else {
-    for (int k = threadIdx.x; k < K; k += blockDim.x) dst[k] = DT<T>::from_f(src[k] * inv * DT<T>::to_f(w[k]));
+    for (int k = threadIdx.x; k < K; k += blockDim.x) dst[k] = DT<T>::from_f(src[k] * inv * DT<TW>::to_f(w[k]));
+  }
+}
+
+// x += norm(y) * w_out, and h = norm(x) * w_in in the activation dtype: what stands between two sublayers when the
+// first one's output is normed before it is added.  One CTA per row; a thread keeps its part of the row in registers.
+constexpr int kJointVec = 4;
+template <typename T>
+__global__ void add_norm_stream_kernel(float* __restrict__ x, int64_t ldx, const float* __restrict__ y, int64_t ldy,
+                                       const float* __restrict__ w_out, const float* __restrict__ w_in,
+                                       T* __restrict__ out, int64_t ldo, int K, float eps) {
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  float* xr = x + (int64_t)blockIdx.x * ldx;
+  const float* yr = y + (int64_t)blockIdx.x * ldy;
+  T* dst = out + (int64_t)blockIdx.x * ldo;
+  const int nt = blockDim.x, tid = threadIdx.x;
+  if (K % 4 == 0 && ldx % 4 == 0 && ldy % 4 == 0 && K <= nt * kJointVec * 4) {
+    float4 xv[kJointVec], yv[kJointVec];
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < kJointVec; ++i) {
+      const int k = tid + i * nt;
+      yv[i] = xv[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (k < K / 4) {
+        yv[i] = reinterpret_cast<const float4*>(yr)[k];
+        xv[i] = reinterpret_cast<const float4*>(xr)[k];
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < kJointVec; ++i)
+      s += yv[i].x * yv[i].x + yv[i].y * yv[i].y + yv[i].z * yv[i].z + yv[i].w * yv[i].w;
+    s = block_sum(s, red);
+    float inv = 1.0f / sqrtf(s / (float)K + eps);
+    s = 0.f;
+#pragma unroll
+    for (int i = 0; i < kJointVec; ++i) {
+      const int k = tid + i * nt;
+      if (k < K / 4) {
+        const float4 w = reinterpret_cast<const float4*>(w_out)[k];
+        xv[i].x += yv[i].x * inv * w.x;
+        xv[i].y += yv[i].y * inv * w.y;
+        xv[i].z += yv[i].z * inv * w.z;
+        xv[i].w += yv[i].w * inv * w.w;
+        reinterpret_cast<float4*>(xr)[k] = xv[i];
+        s += xv[i].x * xv[i].x + xv[i].y * xv[i].y + xv[i].z * xv[i].z + xv[i].w * xv[i].w;
+      }
+    }
+    if (out == nullptr) return;
+    s = block_sum(s, red);
+    inv = 1.0f / sqrtf(s / (float)K + eps);
+#pragma unroll
+    for (int i = 0; i < kJointVec; ++i) {
+      const int k = tid + i * nt;
+      if (k < K / 4) {
+        const float4 w = reinterpret_cast<const float4*>(w_in)[k];
+        const float o[4] = {xv[i].x * inv * w.x, xv[i].y * inv * w.y, xv[i].z * inv * w.z, xv[i].w * inv * w.w};
+        if (ldo % 4 == 0) {
+          __align__(16) T t[4];
+#pragma unroll
+          for (int j = 0; j < 4; ++j) t[j] = DT<T>::from_f(o[j]);
+          if constexpr (sizeof(T) == 2) reinterpret_cast<uint2*>(dst)[k] = *reinterpret_cast<const uint2*>(t);
+          else reinterpret_cast<uint4*>(dst)[k] = *reinterpret_cast<const uint4*>(t);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 4; ++j) dst[4 * k + j] = DT<T>::from_f(o[j]);
+        }
+      }
+    }
+    return;
+  }
+  float s = 0.f;
+  for (int k = tid; k < K; k += nt) s = fmaf(yr[k], yr[k], s);
+  s = block_sum(s, red);
+  float inv = 1.0f / sqrtf(s / (float)K + eps);
+  s = 0.f;
+  for (int k = tid; k < K; k += nt) {
+    const float v = xr[k] + yr[k] * inv * w_out[k];
+    xr[k] = v;
+    s = fmaf(v, v, s);
+  }
+  if (out == nullptr) return;
+  s = block_sum(s, red);
+  inv = 1.0f / sqrtf(s / (float)K + eps);
+  for (int k = tid; k < K; k += nt) dst[k] = DT<T>::from_f(xr[k] * inv * w_in[k]);
+}
+
+// y += bias, row by row
+template <typename TY, typename T>
+__global__ void bias_rows_kernel(TY* __restrict__ y, int64_t ldy, const T* __restrict__ bias, int N) {
+  TY* r = y + (int64_t)blockIdx.x * ldy;
+  for (int n = threadIdx.x; n < N; n += blockDim.x) r[n] = DT<TY>::from_f(DT<TY>::to_f(r[n]) + DT<T>::to_f(bias[n]));
+}
+
+// out[r, i] = gelu_tanh(gate + bias) * (up + bias) from a row of 2 I products; interleaved: gate and up alternate in
+// blocks of eight
+template <typename TY, typename T>
+__global__ void gelu_glu_rows_kernel(const TY* __restrict__ gu, int64_t ld, const T* __restrict__ bias,
+                                     T* __restrict__ out, int64_t ldo, int I, int interleaved) {
+  const TY* r = gu + (int64_t)blockIdx.x * ld;
+  for (int i = threadIdx.x; i < I; i += blockDim.x) {
+    const int g = interleaved ? (i >> 3) * 16 + (i & 7) : i, u = interleaved ? g + 8 : I + i;
+    const float bg = bias != nullptr ? DT<T>::to_f(bias[g]) : 0.f, bu = bias != nullptr ? DT<T>::to_f(bias[u]) : 0.f;
+    out[(int64_t)blockIdx.x * ldo + i] =
+        DT<T>::from_f(gelu_tanh(DT<TY>::to_f(r[g]) + bg) * (DT<TY>::to_f(r[u]) + bu));
   }
 }
 
@@ -298,14 +404,61 @@ IPEX_API int ipex_embed_stream(const int64_t* tokens, const int* slot, const int
   });
 }
 
-// out[i] = RMS norm of row rows[i] (or i) of the fp32 stream, in the activation dtype.
-IPEX_API int ipex_norm_stream(const float* x, int64_t ldx, const void* w, void* out, int64_t ldo, const int* rows, int n,
-                              int K, float eps, int dtype, int pdl, void* stream) {
+// out[i] = RMS norm of row rows[i] (or i) of the fp32 stream, in the activation dtype; the weight has that dtype too, or
+// is fp32 (w_f32).
+IPEX_API int ipex_norm_stream(const float* x, int64_t ldx, const void* w, int w_f32, void* out, int64_t ldo,
+                              const int* rows, int n, int K, float eps, int dtype, int pdl, void* stream) {
   if (n < 1 || K < 1) return (int)cudaErrorInvalidValue;
   return by_dtype(dtype, [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
-    return launch_kernel(norm_stream_kernel<T>, dim3(n), dim3(256), 0, (cudaStream_t)stream, pdl != 0, x, ldx,
+    if (w_f32)
+      return launch_kernel(norm_stream_kernel<T, float>, dim3(n), dim3(256), 0, (cudaStream_t)stream, pdl != 0, x, ldx,
+                           (const float*)w, (T*)out, ldo, rows, K, eps);
+    return launch_kernel(norm_stream_kernel<T, T>, dim3(n), dim3(256), 0, (cudaStream_t)stream, pdl != 0, x, ldx,
                          (const T*)w, (T*)out, ldo, rows, K, eps);
+  });
+}
+
+// x [n, K] += RMS norm of y times w_out; out (may be null) = RMS norm of the new x times w_in.  Weights fp32, 16-byte
+// aligned like x and y.
+IPEX_API int ipex_add_norm_stream(float* x, int64_t ldx, const float* y, int64_t ldy, const float* w_out,
+                                  const float* w_in, void* out, int64_t ldo, int n, int K, float eps, int dtype, int pdl,
+                                  void* stream) {
+  if (n < 1 || K < 1 || (out != nullptr && w_in == nullptr)) return (int)cudaErrorInvalidValue;
+  if (((uintptr_t)x | (uintptr_t)y | (uintptr_t)w_out | (uintptr_t)w_in | (uintptr_t)out) & 15)
+    return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    const int threads = K <= 2048 ? 256 : K <= 4096 ? 512 : 1024;
+    return launch_kernel(add_norm_stream_kernel<T>, dim3(n), dim3(threads), 0, (cudaStream_t)stream, pdl != 0, x, ldx, y,
+                         ldy, w_out, w_in, (T*)out, ldo, K, eps);
+  });
+}
+
+// y [n, N] (the bias's dtype, or fp32) += bias
+IPEX_API int ipex_bias_rows(void* y, int64_t ldy, int y_f32, const void* bias, int n, int N, int dtype, void* stream) {
+  if (n < 1 || N < 1) return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    if (y_f32) bias_rows_kernel<float, T><<<n, 256, 0, (cudaStream_t)stream>>>((float*)y, ldy, (const T*)bias, N);
+    else bias_rows_kernel<T, T><<<n, 256, 0, (cudaStream_t)stream>>>((T*)y, ldy, (const T*)bias, N);
+    return cudaGetLastError();
+  });
+}
+
+// out [n, I] = gelu_tanh(gate + bias) * (up + bias) of gu [n, 2 I] (the activation dtype, or fp32)
+IPEX_API int ipex_gelu_glu_rows(const void* gu, int64_t ld, int gu_f32, const void* bias, void* out, int64_t ldo, int n,
+                                int I, int interleaved, int dtype, void* stream) {
+  if (n < 1 || I < 1 || (interleaved && I % 8 != 0)) return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    if (gu_f32)
+      gelu_glu_rows_kernel<float, T><<<n, 256, 0, (cudaStream_t)stream>>>((const float*)gu, ld, (const T*)bias, (T*)out,
+                                                                          ldo, I, interleaved);
+    else
+      gelu_glu_rows_kernel<T, T><<<n, 256, 0, (cudaStream_t)stream>>>((const T*)gu, ld, (const T*)bias, (T*)out, ldo, I,
+                                                                      interleaved);
+    return cudaGetLastError();
   });
 }
 

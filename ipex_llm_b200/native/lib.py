@@ -103,7 +103,7 @@ def stream_lib() -> ctypes.CDLL:
             lib = cuda_lib()
         else:
             lib = None
-        if lib is None or not hasattr(lib, "ipex_gemm_stream"):
+        if lib is None or not hasattr(lib, "ipex_delta_step"):
             with _lock:
                 lib = ctypes.CDLL(_build.build_component("stream"))
         from . import cuda_api

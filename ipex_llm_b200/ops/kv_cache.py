@@ -14,6 +14,7 @@ each cache is a ``Cache`` whose layers are ``CacheLayerMixin`` objects with
 from __future__ import annotations
 
 import os
+from dataclasses import dataclass
 
 import torch
 from transformers.cache_utils import Cache, DynamicLayer
@@ -329,11 +330,99 @@ class LatentLayer(NormalLayer):
         return (torch.zeros(bsz, heads, cap, dk, dtype=dtype, device=device),
                 torch.zeros(bsz, heads, cap, 0, dtype=dtype, device=device))
 
+    def open(self, slots, capacity, shape, dtype, device):
+        """Storage of ``shape`` (the row width) for that many slots and tokens; what is held already is kept."""
+        self._grow(slots, capacity, 1, int(shape), 0, dtype, device)
 
-class LatentCache(_BlockCache):
-    """Cache of a decoder with latent attention, plus what else a sequence carries along: the history of its token
+    def _grow(self, slots, capacity, heads, dk, dv, dtype, device):
+        k, v, n = self._k, self._v, self.length
+        self.preallocate(slots, heads, capacity, dk, dv, dtype, device)
+        if k is not None:
+            self._k[:k.shape[0], :, :k.shape[2]] = k
+            self._v[:v.shape[0], :, :v.shape[2]] = v
+            self.set_length(n)
+
+
+class KeyValueLayer(LatentLayer):
+    """Keys and values of different sizes, a row per token and key head: ``_k [slots, heads, capacity, dim]``,
+    ``_v [slots, heads, capacity, vdim]``."""
+
+    def open(self, slots, capacity, shape, dtype, device):
+        self._grow(slots, capacity, shape.heads, shape.dim, shape.vdim, dtype, device)
+
+    def _alloc(self, bsz, heads, cap, dk, dv, dtype, device):
+        return NormalLayer._alloc(self, bsz, heads, cap, dk, dv, dtype, device)
+
+
+class DeltaStateLayer(NormalLayer):
+    """State of a recurrent layer, of one size however long the sequence is: ``_k [slots, heads, dim, vdim]`` in fp32,
+    and the last inputs of its short convolutions, ``_v [slots, 1, taps, channels]`` (row = position mod taps).  A slot
+    that starts a new sequence is not cleared: the kernels take everything before a sequence's first token as zero."""
+
+    def open(self, slots, capacity, shape, dtype, device):
+        k, v, n = self._k, self._v, self.length
+        if k is None or k.shape[0] < slots:
+            self.dtype, self.device, self.is_initialized = dtype, device, True
+            self._k = torch.zeros(slots, shape.heads, shape.dim, shape.vdim, dtype=torch.float32, device=device)
+            self._v = torch.zeros(slots, 1, shape.taps, shape.channels, dtype=dtype, device=device)
+            if k is not None:
+                self._k[:k.shape[0]], self._v[:v.shape[0]] = k, v
+        self.set_length(n)
+
+    def set_length(self, n: int):
+        self.length, self.keys, self.values = n, self._k, self._v
+
+    def reserve(self, extra_tokens: int):
+        pass
+
+    def crop(self, max_length: int) -> None:
+        if max_length < 0:
+            max_length = self.length - abs(max_length)
+        if max_length < self.length:
+            raise NotImplementedError("a recurrent state cannot be taken back to an earlier token")
+
+    def reset(self):
+        self.length = 0
+
+    def update(self, key_states, value_states, *args, **kwargs):
+        raise NotImplementedError("a recurrent state is not a sequence of keys and values")
+
+    def batch_repeat_interleave(self, repeats: int):
+        super().batch_repeat_interleave(repeats)
+        self.set_length(self.length)
+
+    def batch_select_indices(self, indices):
+        super().batch_select_indices(indices)
+        self.set_length(self.length)
+
+    def reorder_cache(self, beam_idx):
+        super().reorder_cache(beam_idx)
+        self.set_length(self.length)
+
+
+@dataclass(frozen=True)
+class KeyValueShape:
+    heads: int
+    dim: int
+    vdim: int
+    layer_cls = KeyValueLayer
+
+
+@dataclass(frozen=True)
+class DeltaStateShape:
+    heads: int
+    dim: int
+    vdim: int
+    taps: int
+    channels: int
+    layer_cls = DeltaStateLayer
+
+
+class SlotCache(_BlockCache):
+    """Cache of a decoder that runs packed batches, plus what else a sequence carries along: the history of its token
     ids (``history [slots, capacity]``, the previous token of an embedding over token pairs) and the row of its first
-    token (``start [slots]``; later rows of a left-padded batch are not the first).
+    token (``start [slots]``; later rows of a left-padded batch are not the first).  Layers may differ in kind: a
+    layer's shape (``LatentLayer``: an int) names its class.
 
     Rows of the batch dimension are slots: a sequence takes one (``acquire``), keeps it however the batch around it
     changes, and gives it back (``release``); ``lengths`` counts the tokens each slot holds."""
@@ -344,6 +433,8 @@ class LatentCache(_BlockCache):
         self.history = None
         self.start = None
         self.lengths = []
+        self.shapes = []
+        self.dtype = None
         self._free = []
         self._first = []         # host copy of ``start``
 
@@ -356,21 +447,18 @@ class LatentCache(_BlockCache):
     def capacity(self) -> int:
         return 0 if self.history is None else self.history.shape[1]
 
-    def allocate(self, slots: int, capacity: int, row_widths, dtype, device) -> bool:
-        """Room for ``slots`` sequences of ``capacity`` tokens; ``row_widths``: one cache row width per layer.  What the
-        cache holds already is kept.  True when the storage moved."""
+    def allocate(self, slots: int, capacity: int, shapes, dtype, device) -> bool:
+        """Room for ``slots`` sequences of ``capacity`` tokens; ``shapes``: one per layer.  What the cache holds already
+        is kept.  True when the storage moved."""
         if slots <= self.slots and capacity <= self.capacity:
             return False
         old_slots = self.slots
         slots, capacity = max(slots, old_slots), max(capacity, self.capacity)
-        while len(self.layers) < len(row_widths):
-            self.layers.append(self.layer_class_to_replicate())
-        for layer, row in zip(self.layers, row_widths):
-            prev, n = layer._k, layer.length
-            layer.preallocate(slots, 1, capacity, row, 0, dtype, device)
-            if prev is not None:
-                layer._k[:prev.shape[0], :, :prev.shape[2]] = prev
-                layer.set_length(n)
+        self.shapes, self.dtype = list(shapes), dtype
+        while len(self.layers) < len(shapes):
+            self.layers.append(getattr(shapes[len(self.layers)], "layer_cls", self.layer_cls)())
+        for layer, shape in zip(self.layers, shapes):
+            layer.open(slots, capacity, shape, dtype, device)
         history = torch.zeros(slots, capacity, dtype=torch.int32, device=device)
         start = torch.zeros(slots, dtype=torch.int32, device=device)
         if self.history is not None:
@@ -385,9 +473,11 @@ class LatentCache(_BlockCache):
         """Room for ``extra_tokens`` behind what a padded batch holds."""
         need = self.get_seq_length() + extra_tokens
         if self.layers and need > self.capacity:
-            k = self.layers[0]._k
-            self.allocate(self.slots, need + KV_CACHE_ALLOC_BLOCK_LENGTH, [layer._k.shape[-1] for layer in self.layers],
-                          k.dtype, k.device)
+            self.allocate(self.slots, need + KV_CACHE_ALLOC_BLOCK_LENGTH, self.shapes, self.dtype, self.history.device)
+
+    def step_state(self):
+        """Tensors a decode step changes in a way that running it again would not repeat."""
+        return [t for layer in self.layers if isinstance(layer, DeltaStateLayer) for t in (layer._k, layer._v)]
 
     # -- slots ------------------------------------------------------------------------------------------------
     def acquire(self) -> int:
@@ -452,6 +542,10 @@ class LatentCache(_BlockCache):
         super().crop(max_length)
         n = self.get_seq_length()
         self.lengths = [min(x, n) for x in self.lengths]
+
+
+class LatentCache(SlotCache):
+    """``SlotCache`` of a decoder with multi-head latent attention: every shape is a row width."""
 
 
 def is_fp8_cache(cache) -> bool:

@@ -1,136 +1,23 @@
-"""Python front of the kernels for decoders with a 32-bit residual stream: row products and GEMMs that read or add to
-the stream, a dense expert bank, and multi-head latent attention (see the ``.cu`` files of the "stream" component).
+"""Python front of the kernels of latent-attention decoders: a dense expert bank and multi-head latent attention (see
+``moe_*`` in ``gemv_dense.cu`` / ``stream_ops.cu`` and the ``latent_*.cu`` files), beside what they share with the other
+decoders on a 32-bit residual stream (``ops/stream.py``).
 
-Every function launches on the current stream; there is no eager substitute.  The stream is ``x [tokens, width]`` fp32;
-``dtype`` below is the weight and activation dtype (fp16, bf16 or fp32).
+Every function launches on the current stream; there is no eager substitute.
 """
 from __future__ import annotations
-
-from contextlib import contextmanager
 
 import torch
 
 from ..native import cuda_api as api
 from ..native.lib import current_stream, ptr, stream_lib
 from .cuda_ops import error_flag
+from .stream import (ACT_GELU_GLU, ACT_GLU, ACT_NONE, ACT_RELU2, OUT_ACT, OUT_ADD, OUT_F32, _dt, _tile, add_stream_,
+                     argmax_rows, embed_stream, gemm, gemm_ok, gemv_rows, norm_stream, relu2_, rows_max, softcap_)
 
-OUT_ACT, OUT_ADD, OUT_F32 = 0, 1, 2        # activation dtype / added to the stream / fp32
-ACT_NONE, ACT_RELU2, ACT_GLU = 0, 1, 2
-
-
-def _dt(t) -> int:
-    return api.dtype_code(t if isinstance(t, torch.dtype) else t.dtype)
-
-
-@contextmanager
-def _true_fp32():
-    """Library products of 32-bit models in full precision, whatever the process has allowed."""
-    m = torch.backends.cuda.matmul
-    old = m.allow_tf32
-    m.allow_tf32 = False
-    try:
-        yield
-    finally:
-        m.allow_tf32 = old
-
-
-# ------------------------------------------------------------------------------------------------
-# products
-# ------------------------------------------------------------------------------------------------
-def rows_max(K: int, dtype) -> int:
-    return int(stream_lib().ipex_gemv_rows_max(K, _dt(dtype)))
-
-
-def gemv_rows(w, x, out, mode: int, norm=None, eps: float = 0.0, act: int = 0, softcap: float = 0.0, pdl=False):
-    """``act(x @ w.T)`` for a few rows.  ``norm``: ``x`` is the stream and is RMS-normed with this weight on the way
-    (inside the product for one or two rows; a CTA would spend longer on the norms of more rows than on its weights)."""
-    M, N, K = x.shape[0], w.shape[0], w.shape[1]
-    if norm is not None and M > 2 and w.dtype != torch.float32:
-        x, norm = norm_stream(x, norm, eps, pdl=pdl), None
-    rc = stream_lib().ipex_gemv_rows(ptr(w), w.stride(0), ptr(x), x.stride(0), ptr(norm), eps, ptr(out), out.stride(0),
-                                     M, N, K, mode, act, softcap, _dt(w), int(pdl), current_stream())
-    api.check(rc, "gemv_rows")
-    return out
-
-
-def gemm_ok(x, w) -> bool:
-    return w.dtype in (torch.float16, torch.bfloat16) and x.dtype == w.dtype and w.shape[-1] % 8 == 0 and \
-        x.stride(-1) == 1 and x.stride(0) % 8 == 0 and w.stride(-2) % 8 == 0 and \
-        x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0
-
-
-def _tile(rows: float) -> int:
-    return 32 if rows <= 32 else 64 if rows <= 64 else 128 if rows <= 128 else 256
-
-
-def gemm(x, w, out, mode: int, act: int = 0):
-    """``x [M, K] @ w[N, K].T`` into ``out`` (see ``OUT_*``): the tcgen05 kernel, or the library product for 32-bit
-    weights and rows that are no multiple of 16 bytes."""
-    M, (N, K) = x.shape[0], w.shape
-    if gemm_ok(x, w):
-        rc = stream_lib().ipex_gemm_stream(ptr(x), x.stride(0), ptr(w), w.stride(0), ptr(out), out.stride(0), None, None,
-                                           1, M, N, K, mode, act, 0.0, 0.0, _tile(M), _dt(w), ptr(error_flag(x.device)),
-                                           current_stream())
-        if rc == -1:
-            raise RuntimeError("ipex_llm_b200: the driver's tensor-map encoder rejected the GEMM operands")
-        api.check(rc, "gemm_stream")
-        return out
-    with _true_fp32():
-        if mode == OUT_ACT:
-            torch.matmul(x, w.t(), out=out) if out.is_contiguous() else out.copy_(torch.matmul(x, w.t()))
-            if act == ACT_RELU2:
-                relu2_(out)
-        elif x.dtype == torch.float32:
-            out.addmm_(x, w.t(), beta=1.0 if mode == OUT_ADD else 0.0)
-        else:
-            y = torch.matmul(x.float(), w.float().t())
-            out.add_(y) if mode == OUT_ADD else out.copy_(y)
-    return out
-
-
-def relu2_(x):
-    if not x.is_contiguous():
-        raise ValueError("relu2_ wants a contiguous tensor")
-    api.check(stream_lib().ipex_relu2_inplace(ptr(x), x.numel(), _dt(x), current_stream()), "relu2")
-    return x
-
-
-def add_stream_(x, y):
-    """``x += y`` for the fp32 stream and a contiguous activation."""
-    api.check(stream_lib().ipex_add_stream(ptr(x), ptr(y), x.numel(), _dt(y), current_stream()), "add_stream")
-    return x
-
-
-def softcap_(logits, cap: float):
-    api.check(stream_lib().ipex_softcap_f32(ptr(logits), logits.numel(), cap, current_stream()), "softcap")
-    return logits
-
-
-# ------------------------------------------------------------------------------------------------
-# stream
-# ------------------------------------------------------------------------------------------------
-def embed_stream(tokens, slot, pos, cache, table, scale: float, bigram=None, buckets=0, mul_prev=0, mul_cur=0, out=None,
-                 pdl=False):
-    """``table[token] * scale (+ bigram row)`` for every entry, and the ids filed in ``cache.history``."""
-    n, (V, W) = tokens.shape[0], table.shape
-    if out is None:
-        out = torch.empty(n, W, dtype=torch.float32, device=tokens.device)
-    rc = stream_lib().ipex_embed_stream(ptr(tokens), ptr(slot), ptr(pos), ptr(cache.start), ptr(cache.history),
-                                        cache.capacity, ptr(table), ptr(bigram), ptr(out), n, W, V, scale, buckets,
-                                        mul_prev, mul_cur, _dt(table), int(pdl), current_stream())
-    api.check(rc, "embed_stream")
-    return out
-
-
-def norm_stream(x, weight, eps: float, rows=None, out=None, pdl=False):
-    """RMS norm of the stream (or of its rows ``rows``, int32) in the weight's dtype."""
-    n, K = (x.shape[0] if rows is None else rows.shape[0]), x.shape[1]
-    if out is None:
-        out = torch.empty(n, K, dtype=weight.dtype, device=x.device)
-    rc = stream_lib().ipex_norm_stream(ptr(x), x.stride(0), ptr(weight), ptr(out), out.stride(0), ptr(rows), n, K, eps,
-                                       _dt(weight), int(pdl), current_stream())
-    api.check(rc, "norm_stream")
-    return out
+__all__ = ["ACT_GELU_GLU", "ACT_GLU", "ACT_NONE", "ACT_RELU2", "OUT_ACT", "OUT_ADD", "OUT_F32", "ExpertBank", "LatentSpec",
+           "add_stream_", "argmax_rows", "embed_stream", "gemm", "gemm_ok", "gemv_rows", "latent_prompt", "latent_step",
+           "moe_grouped", "moe_rows", "norm_stream", "pick_latent_splits", "relu2_", "rotary_table", "rows_max",
+           "sigmoid_topk", "softcap_"]
 
 
 # ------------------------------------------------------------------------------------------------
@@ -198,9 +85,9 @@ def moe_grouped(bank: ExpertBank, x, h):
     y = torch.empty(S, W, dtype=dtype, device=dev)
     if bank.interleaved and gemm_ok(hs, bank.gate_up) and gemm_ok(a, bank.down):
         err, bt = ptr(error_flag(dev)), _tile(S / E * 1.25)
-        api.check(lib.ipex_gemm_stream(ptr(hs), W, ptr(bank.gate_up), W, ptr(a), I, ptr(ws), ptr(ranges), E, S, 2 * I, W,
+        api.check(lib.ipex_gemm_stream(ptr(hs), W, ptr(bank.gate_up), W, ptr(a), I, None, ptr(ws), ptr(ranges), E, S, 2 * I, W,
                                        OUT_ACT, ACT_GLU, bank.limit, bank.alpha, bt, dt, err, st), "gemm_stream(glu)")
-        api.check(lib.ipex_gemm_stream(ptr(a), I, ptr(bank.down), I, ptr(y), W, None, ptr(ranges), E, S, W, I, OUT_ACT,
+        api.check(lib.ipex_gemm_stream(ptr(a), I, ptr(bank.down), I, ptr(y), W, None, None, ptr(ranges), E, S, W, I, OUT_ACT,
                                        0, 0.0, 0.0, bt, dt, err, st), "gemm_stream(down)")
     else:
         gu = torch.empty(S, 2 * I, dtype=torch.float32, device=dev)
@@ -295,17 +182,11 @@ def latent_prompt(spec: LatentSpec, qkv, w_uk, w_uv, kv_norm, cos, sin, slot, po
     ld = (T + 7) // 8 * 8
     vt = torch.empty(H * spec.v_dim, ld, dtype=dtype, device=dev)
     gemm(w_uv, c, vt, OUT_ACT)                    # V transposed: rows are value dimensions, columns tokens
-    rc = lib.ipex_latent_prefill(ptr(qkv), qkv.stride(0), ptr(k), ptr(kr), kr.stride(0), ptr(vt), ld, ptr(out),
-                                 out.stride(0), ptr(seq_row), ptr(seq_len), seq_row.shape[0], H, T, max_len, spec.dim,
-                                 spec.rot_dim, spec.v_dim, spec.window, spec.scale, dt, ptr(error_flag(dev)), st)
+    rc = lib.ipex_packed_prefill(ptr(qkv), qkv.stride(0), ptr(k), k.stride(0), ptr(kr), kr.stride(0), ptr(vt), ld,
+                                 ptr(out), out.stride(0), ptr(seq_row), ptr(seq_len), seq_row.shape[0], H, H, T, max_len,
+                                 spec.dim, spec.rot_dim, spec.v_dim, spec.window, 0, spec.scale, dt, ptr(error_flag(dev)),
+                                 st)
     if rc == -1:
         raise RuntimeError("ipex_llm_b200: the driver's tensor-map encoder rejected the attention operands")
-    api.check(rc, "latent_prefill")
-    return out
-
-
-def argmax_rows(logits, out, pdl=False):
-    rc = stream_lib().ipex_argmax(ptr(logits), ptr(out), logits.shape[0], logits.shape[1], logits.stride(0), _dt(logits),
-                                  int(pdl), current_stream())
-    api.check(rc, "argmax")
+    api.check(rc, "packed_prefill")
     return out

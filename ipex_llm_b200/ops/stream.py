@@ -1,0 +1,180 @@
+"""Python front of the kernels that decoders with a 32-bit residual stream share: row products and GEMMs that read or
+add to the stream, embedding, norms, arg-max (see the ``.cu`` files of the "stream" component).
+
+Every function launches on the current stream; there is no eager substitute.  The stream is ``x [tokens, width]`` fp32;
+``dtype`` below is the weight and activation dtype (fp16, bf16 or fp32).
+"""
+from __future__ import annotations
+
+from contextlib import contextmanager
+
+import torch
+
+from ..native import cuda_api as api
+from ..native.lib import current_stream, ptr, stream_lib
+from .cuda_ops import error_flag
+
+OUT_ACT, OUT_ADD, OUT_F32 = 0, 1, 2        # activation dtype / added to the stream / fp32
+ACT_NONE, ACT_RELU2 = 0, 1
+ACT_GLU, ACT_GELU_GLU = 2, 3                # grouped GEMM only / gate and up rows in blocks of eight
+
+
+def _dt(t) -> int:
+    return api.dtype_code(t if isinstance(t, torch.dtype) else t.dtype)
+
+
+@contextmanager
+def _true_fp32():
+    """Library products of 32-bit models in full precision, whatever the process has allowed."""
+    m = torch.backends.cuda.matmul
+    old = m.allow_tf32
+    m.allow_tf32 = False
+    try:
+        yield
+    finally:
+        m.allow_tf32 = old
+
+
+# ------------------------------------------------------------------------------------------------
+# products
+# ------------------------------------------------------------------------------------------------
+def rows_max(K: int, dtype) -> int:
+    return int(stream_lib().ipex_gemv_rows_max(K, _dt(dtype)))
+
+
+def gemv_rows(w, x, out, mode: int, norm=None, eps: float = 0.0, act: int = 0, softcap: float = 0.0, pdl=False, bias=None,
+              w2=None, out2=None, interleaved=True):
+    """``act(x @ w.T + bias)`` for a few rows.  ``norm``: ``x`` is the stream and is RMS-normed with this weight on the way
+    (inside the product for one or two rows; a CTA would spend longer on the norms of more rows than on its weights).
+    ``w2`` / ``out2``: more rows for the same ``x``, with fp32 results.  ``ACT_GELU_GLU``: ``w`` holds gate and up rows (in
+    blocks of eight, or not ``interleaved``), half as many columns come out."""
+    M, N, K = x.shape[0], w.shape[0], w.shape[1]
+    if norm is not None and M > 2 and w.dtype != torch.float32:
+        x, norm = norm_stream(x, norm, eps, pdl=pdl), None
+    rc = stream_lib().ipex_gemv_rows(ptr(w), w.stride(0), ptr(x), x.stride(0), ptr(norm), eps, ptr(bias), ptr(out),
+                                     out.stride(0), ptr(w2), 0 if w2 is None else w2.shape[0], ptr(out2),
+                                     0 if out2 is None else out2.stride(0), M, N, K, mode, act, int(interleaved),
+                                     softcap, _dt(w), int(pdl), current_stream())
+    api.check(rc, "gemv_rows")
+    return out
+
+
+def gemm_ok(x, w) -> bool:
+    return w.dtype in (torch.float16, torch.bfloat16) and x.dtype == w.dtype and w.shape[-1] % 8 == 0 and \
+        x.stride(-1) == 1 and x.stride(0) % 8 == 0 and w.stride(-2) % 8 == 0 and \
+        x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0
+
+
+def _tile(rows: float) -> int:
+    return 32 if rows <= 32 else 64 if rows <= 64 else 128 if rows <= 128 else 256
+
+
+def gemm(x, w, out, mode: int, act: int = 0, bias=None, interleaved=True):
+    """``x [M, K] @ w[N, K].T (+ bias)`` into ``out`` (see ``OUT_*``): the tcgen05 kernel, or the library product for
+    32-bit weights and rows that are no multiple of 16 bytes.  ``ACT_GELU_GLU``: see ``gemv_rows``."""
+    M, (N, K) = x.shape[0], w.shape
+    if gemm_ok(x, w) and not (act == ACT_GELU_GLU and not interleaved):
+        rc = stream_lib().ipex_gemm_stream(ptr(x), x.stride(0), ptr(w), w.stride(0), ptr(out), out.stride(0), ptr(bias),
+                                           None, None, 1, M, N, K, mode, act, 0.0, 0.0, _tile(M), _dt(w),
+                                           ptr(error_flag(x.device)), current_stream())
+        if rc == -1:
+            raise RuntimeError("ipex_llm_b200: the driver's tensor-map encoder rejected the GEMM operands")
+        api.check(rc, "gemm_stream")
+        return out
+    with _true_fp32():
+        if act == ACT_GELU_GLU:
+            return gelu_glu_rows(torch.matmul(x.float(), w.float().t()), bias, out, interleaved)
+        if mode == OUT_ACT:
+            torch.matmul(x, w.t(), out=out) if out.is_contiguous() else out.copy_(torch.matmul(x, w.t()))
+            if bias is not None:
+                bias_rows_(out, bias)
+            if act == ACT_RELU2:
+                relu2_(out)
+            return out
+        if x.dtype == torch.float32:
+            out.addmm_(x, w.t(), beta=1.0 if mode == OUT_ADD else 0.0)
+        else:
+            y = torch.matmul(x.float(), w.float().t())
+            out.add_(y) if mode == OUT_ADD else out.copy_(y)
+    return out if bias is None else bias_rows_(out, bias)
+
+
+def bias_rows_(y, bias):
+    """``y [n, N] += bias`` for rows in the bias's dtype or fp32."""
+    rc = stream_lib().ipex_bias_rows(ptr(y), y.stride(0), int(y.dtype == torch.float32), ptr(bias), y.shape[0], y.shape[1],
+                                     _dt(bias), current_stream())
+    api.check(rc, "bias_rows")
+    return y
+
+
+def gelu_glu_rows(gu, bias, out, interleaved=True):
+    """``gelu_tanh(gate + bias) * (up + bias)`` of finished products ``gu [n, 2 I]`` (the dtype of ``out``, or fp32)."""
+    rc = stream_lib().ipex_gelu_glu_rows(ptr(gu), gu.stride(0), int(gu.dtype == torch.float32), ptr(bias), ptr(out),
+                                         out.stride(0), gu.shape[0], gu.shape[1] // 2, int(interleaved), _dt(out),
+                                         current_stream())
+    api.check(rc, "gelu_glu_rows")
+    return out
+
+
+def relu2_(x):
+    if not x.is_contiguous():
+        raise ValueError("relu2_ wants a contiguous tensor")
+    api.check(stream_lib().ipex_relu2_inplace(ptr(x), x.numel(), _dt(x), current_stream()), "relu2")
+    return x
+
+
+def add_stream_(x, y):
+    """``x += y`` for the fp32 stream and a contiguous activation."""
+    api.check(stream_lib().ipex_add_stream(ptr(x), ptr(y), x.numel(), _dt(y), current_stream()), "add_stream")
+    return x
+
+
+def softcap_(logits, cap: float):
+    api.check(stream_lib().ipex_softcap_f32(ptr(logits), logits.numel(), cap, current_stream()), "softcap")
+    return logits
+
+
+# ------------------------------------------------------------------------------------------------
+# stream
+# ------------------------------------------------------------------------------------------------
+def embed_stream(tokens, slot, pos, cache, table, scale: float, bigram=None, buckets=0, mul_prev=0, mul_cur=0, out=None,
+                 pdl=False):
+    """``table[token] * scale (+ bigram row)`` for every entry, and the ids filed in ``cache.history``."""
+    n, (V, W) = tokens.shape[0], table.shape
+    if out is None:
+        out = torch.empty(n, W, dtype=torch.float32, device=tokens.device)
+    rc = stream_lib().ipex_embed_stream(ptr(tokens), ptr(slot), ptr(pos), ptr(cache.start), ptr(cache.history),
+                                        cache.capacity, ptr(table), ptr(bigram), ptr(out), n, W, V, scale, buckets,
+                                        mul_prev, mul_cur, _dt(table), int(pdl), current_stream())
+    api.check(rc, "embed_stream")
+    return out
+
+
+def norm_stream(x, weight, eps: float, rows=None, out=None, pdl=False, dtype=None):
+    """RMS norm of the stream (or of its rows ``rows``, int32) in ``dtype``: the weight's own, unless that is fp32 and a
+    16-bit one is asked for."""
+    n, K = (x.shape[0] if rows is None else rows.shape[0]), x.shape[1]
+    dtype = dtype or weight.dtype
+    if out is None:
+        out = torch.empty(n, K, dtype=dtype, device=x.device)
+    rc = stream_lib().ipex_norm_stream(ptr(x), x.stride(0), ptr(weight), int(weight.dtype == torch.float32), ptr(out),
+                                       out.stride(0), ptr(rows), n, K, eps, _dt(dtype), int(pdl), current_stream())
+    api.check(rc, "norm_stream")
+    return out
+
+
+def add_norm_stream(x, y, w_out, w_in, eps: float, dtype, pdl=False):
+    """``x += norm(y) * w_out`` and, unless ``w_in`` is None, ``norm(x) * w_in`` in ``dtype``: the joint between two
+    sublayers when a sublayer's output is normed before it joins the stream.  ``y`` and the weights are fp32."""
+    h = None if w_in is None else torch.empty(x.shape, dtype=dtype, device=x.device)
+    rc = stream_lib().ipex_add_norm_stream(ptr(x), x.stride(0), ptr(y), y.stride(0), ptr(w_out), ptr(w_in), ptr(h),
+                                           x.shape[1], x.shape[0], x.shape[1], eps, _dt(dtype), int(pdl), current_stream())
+    api.check(rc, "add_norm_stream")
+    return h
+
+
+def argmax_rows(logits, out, pdl=False):
+    rc = stream_lib().ipex_argmax(ptr(logits), ptr(out), logits.shape[0], logits.shape[1], logits.stride(0), _dt(logits),
+                                  int(pdl), current_stream())
+    api.check(rc, "argmax")
+    return out

@@ -1,0 +1,117 @@
+"""Python front of the attention over cached keys and values of different sizes (``kv_attn.cu``, and the packed tcgen05
+prompt kernel of ``latent_prefill_tcgen05.cu``): grouped query heads, sliding window, optional sink in the soft-max, values
+mixed with those of an earlier layer.
+
+Every function launches on the current stream; there is no eager substitute.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+
+from ..native import cuda_api as api
+from ..native.lib import current_stream, ptr, stream_lib
+from .cuda_ops import error_flag
+from .stream import _dt
+
+
+@dataclass(frozen=True)
+class AttnSpec:
+    """Sizes and constants of one layer.  ``window`` 0: every earlier key.  ``sink``: one more score of 0 without a value."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    window: int = 0
+    sink: bool = False
+
+    @property
+    def k_at(self) -> int:
+        """Column of the keys in the fused projection (queries come first)."""
+        return self.heads * self.dim
+
+    @property
+    def v_at(self) -> int:
+        return (self.heads + self.kv_heads) * self.dim
+
+    @property
+    def rows(self) -> int:
+        return self.v_at + self.kv_heads * self.vdim
+
+    def prefill_ok(self, dtype) -> bool:
+        """Does the tcgen05 prompt kernel take these sizes?"""
+        return bool(stream_lib().ipex_latent_prefill_ok(self.dim, 0, self.vdim, 8, _dt(dtype)))
+
+
+@dataclass
+class ValueMix:
+    """Values of an earlier layer (a ``[tokens, kv_heads * vdim]`` view) and their share."""
+    first: torch.Tensor
+    share: float
+
+
+def pick_splits(tokens: int, spec: AttnSpec, visible: int, n_sm: int = 148) -> int:
+    """CTAs that share the keys of a query token: up to a cluster of eight, at least 64 keys each, about two waves."""
+    group = spec.heads // spec.kv_heads
+    ctas = tokens * spec.kv_heads * -(-group // 8)
+    n = 1
+    while n < 8 and visible >= 128 * n and ctas * n < n_sm:
+        n *= 2
+    return n
+
+
+def _mix_args(mix: Optional[ValueMix], at: int = 0):
+    return (None, 0, 0.0) if mix is None else (mix.first[at:], mix.first.stride(0), mix.share)
+
+
+def attend_step(spec: AttnSpec, qkv, mix: Optional[ValueMix], slot, pos, cache, layer_idx: int, out, visible: int,
+                single: bool, pdl=False, nsplit: Optional[int] = None):
+    """Attention of query tokens against the cache, which gets their own rows first.  ``single``: every token is another
+    sequence's next one (the append is then part of the attention kernel).  ``visible`` bounds the number of keys a
+    token can see (it sizes the split, nothing else)."""
+    lib, layer = stream_lib(), cache.layers[layer_idx]
+    k, v = layer._k, layer._v
+    M, dt, st = qkv.shape[0], _dt(qkv), current_stream()
+    cols = (qkv[:, spec.k_at:], qkv[:, spec.v_at:])
+    if not single:
+        first, ld_vf, share = _mix_args(mix)
+        api.check(lib.ipex_kv_append(ptr(cols[0]), ptr(cols[1]), qkv.stride(0), ptr(first), ld_vf, share, ptr(k), k.stride(0),
+                                     k.stride(1), ptr(v), v.stride(0), v.stride(1), None, 0, ptr(slot), ptr(pos), M,
+                                     spec.kv_heads, spec.dim, spec.vdim, dt, int(pdl), st), "kv_append")
+    step = 65535
+    for s in range(0, M, step):
+        m = min(step, M - s)
+        first, ld_vf, share = _mix_args(mix, s)
+        api.check(lib.ipex_kv_attn(ptr(qkv[s:]), ptr(cols[0][s:]), ptr(cols[1][s:]), qkv.stride(0), ptr(first), ld_vf, share,
+                                   ptr(k), k.stride(0), k.stride(1), ptr(v), v.stride(0), v.stride(1), ptr(out[s:]),
+                                   out.stride(0), ptr(slot[s:]), ptr(pos[s:]), ptr(cache.start), m, spec.heads,
+                                   spec.kv_heads, spec.dim, spec.vdim, spec.window, int(spec.sink), int(single),
+                                   nsplit or pick_splits(m, spec, visible), spec.scale, dt, int(pdl), st), "kv_attn")
+    return out
+
+
+def attend_prompt(spec: AttnSpec, qkv, mix: Optional[ValueMix], slot, pos, seq_row, seq_len, max_len: int, cache,
+                  layer_idx: int, out):
+    """Attention of whole prompts, packed one behind the other (``seq_row`` / ``seq_len``: int32, first row and length of
+    each), on the tensor cores; the cache gets keys and mixed values."""
+    lib, layer = stream_lib(), cache.layers[layer_idx]
+    k, v = layer._k, layer._v
+    T, dt, st, dev = qkv.shape[0], _dt(qkv), current_stream(), qkv.device
+    ld = (T + 7) // 8 * 8
+    vt = torch.empty(spec.kv_heads * spec.vdim, ld, dtype=qkv.dtype, device=dev)
+    first, ld_vf, share = _mix_args(mix)
+    keys = qkv[:, spec.k_at:]
+    api.check(lib.ipex_kv_append(ptr(keys), ptr(qkv[:, spec.v_at:]), qkv.stride(0), ptr(first), ld_vf, share, ptr(k),
+                                 k.stride(0), k.stride(1), ptr(v), v.stride(0), v.stride(1), ptr(vt), ld, ptr(slot),
+                                 ptr(pos), T, spec.kv_heads, spec.dim, spec.vdim, dt, 0, st), "kv_append")
+    rc = lib.ipex_packed_prefill(ptr(qkv), qkv.stride(0), ptr(keys), qkv.stride(0), None, 0, ptr(vt), ld, ptr(out),
+                                 out.stride(0), ptr(seq_row), ptr(seq_len), seq_row.shape[0], spec.heads, spec.kv_heads, T,
+                                 max_len, spec.dim, 0, spec.vdim, spec.window, int(spec.sink), spec.scale, dt,
+                                 ptr(error_flag(dev)), st)
+    if rc == -1:
+        raise RuntimeError("ipex_llm_b200: the driver's tensor-map encoder rejected the attention operands")
+    api.check(rc, "packed_prefill")
+    return out

@@ -225,6 +225,8 @@ def _replace_with_low_bit_linear(model, qtype, modules_to_not_convert=None, conv
             # routers stay in full precision: their modeling code multiplies by ``.weight`` directly or carries the
             # top-k selection in a Linear subclass (the reference keeps them out per family, convert.py:1100-1135)
             continue
+        if is_linear and name in getattr(model, "_ipex_keep_dense", ()):
+            continue                    # small projections whose results steer a recurrence
         if is_fused_experts(module) and qtype not in qt.FLOAT_QTYPES:
             new_mod = convert_fused_experts(module, qtype, device=device, convert_shape_only=convert_shape_only,
                                             enable_scale_search=enable_scale_search)

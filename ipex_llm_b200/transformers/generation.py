@@ -38,6 +38,12 @@ def ipex_generate(self, inputs=None, generation_config=None, logits_processor=No
                                           **kwargs)
     lookahead = kwargs.pop("lookahead", None)
     perf_mode = cfg.performance_mode()
+    if not getattr(self, "_ipex_rolls_back", True):
+        # drafted tokens that are rejected would have to leave the cache again
+        if lookahead or getattr(self, "draft_model", None) is not None or assistant_model is not None:
+            raise NotImplementedError(f"{type(self).__name__} keeps a recurrent state, which cannot be taken back to an "
+                                      "earlier token: no drafting strategies")
+        perf_mode = False
     if lookahead is None and perf_mode and inputs is not None and inputs.shape[0] == 1 and inputs.shape[1] >= 100 \
             and getattr(self, "draft_model", None) is None:
         lookahead = 2

@@ -252,9 +252,10 @@ def kernels(z, prompt: int, peaks):
     i32 = dict(device=dev, dtype=torch.int32)
     row, ln, err = torch.zeros(1, **i32), torch.full((1,), T, **i32), cuda_ops.error_flag(torch.device("cuda", 0))
     for win in (z["window"], 0):
-        us = _graph_us(lambda i: lib.ipex_latent_prefill(
-            L.ptr(qs[i]), ldq, L.ptr(ks[i]), L.ptr(kr), z["rd"], L.ptr(vt), T, L.ptr(out), H * z["vd"], L.ptr(row),
-            L.ptr(ln), 1, H, T, T, z["dim"], z["rd"], z["vd"], win, 0.05, 1, L.ptr(err), L.current_stream()), n)
+        us = _graph_us(lambda i: lib.ipex_packed_prefill(
+            L.ptr(qs[i]), ldq, L.ptr(ks[i]), H * z["dim"], L.ptr(kr), z["rd"], L.ptr(vt), T, L.ptr(out), H * z["vd"],
+            L.ptr(row), L.ptr(ln), 1, H, H, T, T, z["dim"], z["rd"], z["vd"], win, 0, 0.05, 1, L.ptr(err),
+            L.current_stream()), n)
         w = win or T
         pairs = T * min(w, T) - min(w, T) * (min(w, T) - 1) / 2
         fl = 2.0 * H * pairs * (z["dim"] + z["rd"] + z["vd"])
