@@ -292,8 +292,9 @@ __global__ void __launch_bounds__(kThreads) delta_prep_kernel(ChunkArgs s) {
   float* sv = sk + kC * ldk;             // [32][Vp + 8]
   float* sA = sv + kC * ldv;             // [32][36]
   float* sT = sA + kC * 36;              // [32][36]
-  float* sL = sT + kC * 36;              // [32] running sum of log g
-  float* sB = sL + kC;                   // [32] beta
+  // [32] running sum of log g, in 64-bit: its differences must keep 32-bit accuracy when single tokens decay to nothing
+  double* sL = reinterpret_cast<double*>(sT + kC * 36);
+  float* sB = reinterpret_cast<float*>(sL + kC);      // [32] beta
   const int seq = s.chunk_seq[chunk], hk = h / (a.heads / a.kv_heads);
   const int row0 = a.seq_row[seq], off = (chunk - s.seq_chunk[seq]) * kC, n = min(kC, a.seq_len[seq] - off);
   const int slot = a.slot[row0], start = a.start[slot], p0 = a.pos[row0] + off, t0 = row0 + off;
@@ -316,7 +317,8 @@ __global__ void __launch_bounds__(kThreads) delta_prep_kernel(ChunkArgs s) {
     }
   }
   if (warp == 0) {
-    float lg = 0.f, beta = 0.f;
+    double lg = 0.0;
+    float beta = 0.f;
     if (lane < n) {
       const float* gt = a.gates + (int64_t)(t0 + lane) * 2 * a.heads;
       beta = sigmoidf(gt[h]);
@@ -324,7 +326,7 @@ __global__ void __launch_bounds__(kThreads) delta_prep_kernel(ChunkArgs s) {
     }
 #pragma unroll
     for (int o = 1; o < 32; o <<= 1) {
-      const float x = __shfl_up_sync(0xffffffffu, lg, o);
+      const double x = __shfl_up_sync(0xffffffffu, lg, o);
       if (lane >= o) lg += x;
     }
     sL[lane] = lg;
@@ -332,7 +334,7 @@ __global__ void __launch_bounds__(kThreads) delta_prep_kernel(ChunkArgs s) {
   }
   __syncthreads();
   // ---- unit vectors; the decayed copies go out right away
-  const float lend = sL[kC - 1];
+  const double lend = sL[kC - 1];
   for (int t = warp; t < kC; t += kThreads / 32) {
     float qq = 0.f, kk = 0.f;
     for (int d = lane; d < Dp; d += 32) {
@@ -341,7 +343,7 @@ __global__ void __launch_bounds__(kThreads) delta_prep_kernel(ChunkArgs s) {
       kk = fmaf(y, y, kk);
     }
     const float iq = a.qscale / sqrtf(warp_sum(qq) + kUnitEps), ik = 1.0f / sqrtf(warp_sum(kk) + kUnitEps);
-    const float gq = expf(sL[t]), gk = expf(lend - sL[t]);
+    const float gq = expf((float)sL[t]), gk = expf((float)(lend - sL[t]));
     for (int d = lane; d < Dp; d += 32) {
       const float x = sq[t * ldk + d] * iq, y = sk[t * ldk + d] * ik;
       sq[t * ldk + d] = x;
@@ -350,7 +352,7 @@ __global__ void __launch_bounds__(kThreads) delta_prep_kernel(ChunkArgs s) {
       out[L.k() + t * Dp + d] = y * gk;
     }
   }
-  if (tid == 0) out[L.g()] = expf(lend);
+  if (tid == 0) out[L.g()] = expf((float)lend);
   __syncthreads();
   // ---- A (strictly below the diagonal) and P (with it): warp = one 16 x 8 tile of each
   {
@@ -368,7 +370,7 @@ __global__ void __launch_bounds__(kThreads) delta_prep_kernel(ChunkArgs s) {
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int t = m0 + g + 8 * (i >> 1), j = n0 + 2 * t4 + (i & 1);
-      const float dec = j <= t ? expf(sL[t] - sL[j]) : 0.f;
+      const float dec = j <= t ? expf((float)(sL[t] - sL[j])) : 0.f;
       sA[t * 36 + j] = j < t ? sB[t] * dec * aa.get(i) : 0.f;
       out[L.p() + t * kC + j] = j <= t ? dec * pp.get(i) : 0.f;
     }
@@ -407,7 +409,7 @@ __global__ void __launch_bounds__(kThreads) delta_prep_kernel(ChunkArgs s) {
     for (int k0 = 0; k0 < kC; k0 += 8) {
       const FragB b = frag_b([&](int k, int j) {
         const float y = src[(k0 + k) * lds + n0 + j];
-        return isw ? y * expf(sL[k0 + k]) : y;
+        return isw ? y * expf((float)sL[k0 + k]) : y;
       }, g, t4);
 #pragma unroll
       for (int m = 0; m < 2; ++m)
@@ -656,7 +658,7 @@ cudaError_t launch_step(const StepArgs& s, int seqs, bool fused, bool pdl, cudaS
 }
 
 size_t prep_smem(const Scratch& L) {
-  return (size_t)(2 * kC * (L.Dp + 4) + kC * (L.Vp + 8) + 2 * kC * 36 + 2 * kC) * sizeof(float);
+  return (size_t)(2 * kC * (L.Dp + 4) + kC * (L.Vp + 8) + 2 * kC * 36 + 3 * kC) * sizeof(float);
 }
 size_t chunk_smem(const Scratch& L, int D, int stages) {
   const int Dm = (D + 15) / 16 * 16;

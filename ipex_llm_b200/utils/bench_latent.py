@@ -12,6 +12,7 @@ model on the same shape, with its distance from the roofline (measured copy band
 from __future__ import annotations
 
 import argparse
+import gc
 import json
 
 import torch
@@ -81,6 +82,7 @@ def run_model(cfg, prompt: int, batches, iters: int):
     from ..ops.cuda_ops import check_error_flag
     check_error_flag(torch.device("cuda", torch.cuda.current_device()))
     del eng, model
+    gc.collect()            # model and engine refer to each other: their graphs must not be freed during a later capture
     torch.cuda.empty_cache()
     return out
 
