@@ -26,14 +26,16 @@
 #include <cooperative_groups.h>
 
 #include "common/utils.cuh"
+#include "tcgen05_common.cuh"
 
 namespace {
 
 namespace cg = cooperative_groups;
 
 constexpr int kThreads = 256;
+constexpr int kChunkThreads = 512;    // of the sequential half
 constexpr int kC = 32;                // tokens per chunk
-constexpr int kVS = 32;               // state columns per CTA
+constexpr int kVS = 32;               // state columns per CTA of the chunked form
 
 template <typename F>
 int by_dtype(int dtype, F&& f) {
@@ -63,19 +65,34 @@ struct Common {
 
 constexpr float kUnitEps = 1e-6f;
 
-// Channel c of the convolution at packed token t (position p), after silu.
-template <typename T>
-__device__ __forceinline__ float conv_silu(const Common& a, int c, int t, int row0, int p, int start, int slot) {
-  const T* proj = reinterpret_cast<const T*>(a.proj);
-  const T* w = reinterpret_cast<const T*>(a.conv) + (int64_t)c * a.taps;
+// silu of a 16-bit model's convolution
+__device__ __forceinline__ float fast_silu(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
+
+// Channel c of the convolution after silu, at packed token t: token j of its portion, position p of its sequence.  w: the
+// channel's last tap.
+template <typename T, typename TW>
+__device__ __forceinline__ float conv_silu(const Common& a, int c, int t, int j, int p, int start, int slot,
+                                           const TW* w) {
+  const T* proj = reinterpret_cast<const T*>(a.proj) + (int64_t)t * a.ldp + c;
   const T* ring = reinterpret_cast<const T*>(a.ring) + (int64_t)slot * a.taps * a.channels + c;
+  const int pm = p % a.taps, seen = min(a.taps, p - start + 1);
   float s = 0.f;
-  for (int i = 0; i < a.taps; ++i) {
-    const int back = a.taps - 1 - i;
-    if (p - back < start) continue;
-    const float x = t - back >= row0 ? DT<T>::to_f(proj[(int64_t)(t - back) * a.ldp + c])
-                                     : DT<T>::to_f(ring[(int64_t)((p - back) % a.taps) * a.channels]);
-    s = fmaf(x, DT<T>::to_f(w[i]), s);
+  for (int b0 = 0; b0 < seen; b0 += 4) {
+    T x[4];
+    float wv[4];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      const int back = b0 + u;
+      x[u] = DT<T>::from_f(0.f);
+      wv[u] = 0.f;
+      if (back < seen) {
+        const int r = pm - back;
+        x[u] = back <= j ? proj[-(int64_t)back * a.ldp] : ring[(int64_t)(r < 0 ? r + a.taps : r) * a.channels];
+        wv[u] = DT<TW>::to_f(w[-back]);
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < 4; ++u) s = fmaf(DT<T>::to_f(x[u]), wv[u], s);
   }
   return silu(s);
 }
@@ -98,45 +115,93 @@ struct StepArgs {
   float eps;
   int gate_off;           // column of the output gates in proj
   int ring_write;         // one token per sequence: file its convolution inputs
+  int prefetch;           // slots are final before the kernels in front of this one end: fetch states early
 };
 
-// A warp owns the state rows warp, warp + 8, ...; a lane one of 32 columns.
-template <typename T, int NR>
-__global__ void __launch_bounds__(kThreads) delta_step_kernel(StepArgs s) {
+template <int N>
+__device__ __forceinline__ void load_cols(const float* p, float (&v)[N]) {
+  if constexpr (N == 4) {
+    const float4 x = *reinterpret_cast<const float4*>(p);
+    v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+  } else if constexpr (N == 2) {
+    const float2 x = *reinterpret_cast<const float2*>(p);
+    v[0] = x.x; v[1] = x.y;
+  } else {
+    v[0] = *p;
+  }
+}
+template <int N>
+__device__ __forceinline__ void store_cols(float* p, const float (&v)[N]) {
+  if constexpr (N == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  else if constexpr (N == 2) *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
+  else *p = v[0];
+}
+
+// A warp owns the state rows warp, warp + 8, ...; a lane CV neighbouring columns of the CTA's 32 CV.
+template <typename T, int NR, int CV>
+__global__ void __launch_bounds__(kThreads, NR * CV <= 64 ? 2 : 1) delta_step_kernel(StepArgs s) {
+  constexpr int VS = 32 * CV;
   extern __shared__ __align__(16) float sm[];
   const Common& a = s.c;
   const int D = a.dim, V = a.vdim, h = blockIdx.y, sq_id = blockIdx.z, slice = blockIdx.x;
-  const int hk = h / (a.heads / a.kv_heads), v0 = slice * kVS, nv = min(kVS, V - v0);
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  float* buf = sm;                      // [2][2 D + 32]: q, k, v of a token
-  float* red = buf + 2 * (2 * D + kVS); // [2][2][8][32]
+  const int hk = h / (a.heads / a.kv_heads), v0 = slice * VS, nv = min(VS, V - v0);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, c0 = lane * CV;
+  float* red = sm;                      // [2][2][8][VS]
+  float* buf = red + 2 * 2 * 8 * VS;    // [2][2 D + VS]: q, k, v of a token
+  float* wt = buf + 2 * (2 * D + VS);   // [2 D + VS][taps]: convolution weights
   __shared__ float s_ss;
   const int row0 = a.seq_row != nullptr ? a.seq_row[sq_id] : sq_id, len = a.seq_len != nullptr ? a.seq_len[sq_id] : 1;
+  const int qc = hk * D, kc = a.kv_heads * D + hk * D, vc = 2 * a.kv_heads * D + h * V + v0;
+  const bool col = c0 < nv;             // CV divides V: a lane's columns exist together
   pdl_launch_dependents();
+  if (s.prefetch) {
+    // slots do not change while a step is in flight; the state's rows come to L2 while the projections finish
+    const float* st = a.state + (((int64_t)a.slot[row0] * a.heads + h) * D) * V + v0;
+    if (nv == V) {
+      if (tid == 0) prefetch_l2_bulk(st, (uint32_t)(D * V * sizeof(float)));
+    } else {
+      for (int d = tid; d < D; d += kThreads) prefetch_l2_bulk(st + (int64_t)d * V, (uint32_t)(nv * sizeof(float)));
+    }
+  }
+  for (int i = tid; i < 2 * D + nv; i += kThreads) {
+    const int c = i < D ? qc + i : i < 2 * D ? kc + i - D : vc + i - 2 * D;
+    for (int j = 0; j < a.taps; ++j) wt[i * a.taps + j] = DT<T>::to_f(reinterpret_cast<const T*>(a.conv)[(int64_t)c * a.taps + j]);
+  }
+  const float alog = a.a_log[h], dtb = a.dt_bias[h];
+  float nw[CV];
+#pragma unroll
+  for (int c = 0; c < CV; ++c)
+    nw[c] = s.raw == nullptr && col ? DT<T>::to_f(reinterpret_cast<const T*>(s.norm_w)[v0 + c0 + c]) : 0.f;
   pdl_wait();
   const int slot = a.slot[row0], start = a.start[slot], p0 = a.pos[row0];
-  float* st = a.state + (((int64_t)slot * a.heads + h) * D) * V + v0 + lane;
-  float S[NR];
-  const bool fresh = p0 <= start, col = lane < nv;
+  float* st = a.state + (((int64_t)slot * a.heads + h) * D) * V + v0 + c0;
+  float S[NR][CV];
+  const bool fresh = p0 <= start;
 #pragma unroll
   for (int i = 0; i < NR; ++i) {
     const int d = warp + 8 * i;
-    S[i] = !fresh && col && d < D ? st[(int64_t)d * V] : 0.f;
+#pragma unroll
+    for (int c = 0; c < CV; ++c) S[i][c] = 0.f;
+    if (!fresh && col && d < D) load_cols<CV>(st + (int64_t)d * V, S[i]);
   }
-  const int qc = hk * D, kc = a.kv_heads * D + hk * D, vc = 2 * a.kv_heads * D + h * V + v0;
-  const float alog = a.a_log[h], dtb = a.dt_bias[h];
   for (int j = 0; j < len; ++j) {
     const int t = row0 + j, p = p0 + j;
-    float* q = buf + (j & 1) * (2 * D + kVS);
+    float* q = buf + (j & 1) * (2 * D + VS);
     float* k = q + D;
     float* v = k + D;
-    float* rd = red + (j & 1) * (2 * 8 * 32);
+    float* rd = red + (j & 1) * (2 * 8 * VS);
+    const float bg = a.gates[(int64_t)t * 2 * a.heads + h], ag = a.gates[(int64_t)t * 2 * a.heads + a.heads + h];
+    float gate[CV];
+    if (s.raw == nullptr && warp == 0 && col) {
+#pragma unroll
+      for (int c = 0; c < CV; ++c)
+        gate[c] = DT<T>::to_f(reinterpret_cast<const T*>(a.proj)[(int64_t)t * a.ldp + s.gate_off + h * V + v0 + c0 + c]);
+    }
     for (int i = tid; i < 2 * D + nv; i += kThreads) {
       const int c = i < D ? qc + i : i < 2 * D ? kc + i - D : vc + i - 2 * D;
-      q[i] = conv_silu<T>(a, c, t, row0, p, start, slot);
+      q[i] = conv_silu<T>(a, c, t, j, p, start, slot, wt + i * a.taps + a.taps - 1);
     }
-    const float beta = sigmoidf(a.gates[(int64_t)t * 2 * a.heads + h]);
-    const float g = expf(log_decay(a.gates[(int64_t)t * 2 * a.heads + a.heads + h], dtb, alog));
+    const float beta = sigmoidf(bg), g = expf(log_decay(ag, dtb, alog));
     __syncthreads();
     float qq = 0.f, kk = 0.f, qk = 0.f;
     for (int d = lane; d < D; d += 32) {
@@ -144,42 +209,68 @@ __global__ void __launch_bounds__(kThreads) delta_step_kernel(StepArgs s) {
       kk = fmaf(k[d], k[d], kk);
       qk = fmaf(q[d], k[d], qk);
     }
-    const float iq = a.qscale / sqrtf(warp_sum(qq) + kUnitEps), ik = 1.0f / sqrtf(warp_sum(kk) + kUnitEps);
-    qk = warp_sum(qk) * iq * ik;
-    float sk = 0.f, sq = 0.f;
+    float sk[CV], sq[CV];
+#pragma unroll
+    for (int c = 0; c < CV; ++c) sk[c] = sq[c] = 0.f;
 #pragma unroll
     for (int i = 0; i < NR; ++i) {
       const int d = warp + 8 * i;
       if (d < D) {
-        sk = fmaf(S[i], k[d], sk);
-        sq = fmaf(S[i], q[d], sq);
+        const float kd = k[d], qd = q[d];
+#pragma unroll
+        for (int c = 0; c < CV; ++c) {
+          sk[c] = fmaf(S[i][c], kd, sk[c]);
+          sq[c] = fmaf(S[i][c], qd, sq[c]);
+        }
       }
     }
-    rd[warp * 32 + lane] = sk;
-    rd[(8 + warp) * 32 + lane] = sq;
+    store_cols<CV>(rd + warp * VS + c0, sk);
+    store_cols<CV>(rd + (8 + warp) * VS + c0, sq);
+    const float iq = a.qscale / sqrtf(warp_sum(qq) + kUnitEps), ik = 1.0f / sqrtf(warp_sum(kk) + kUnitEps);
+    qk = warp_sum(qk) * iq * ik;
     __syncthreads();
-    sk = sq = 0.f;
+#pragma unroll
+    for (int c = 0; c < CV; ++c) sk[c] = sq[c] = 0.f;
 #pragma unroll
     for (int w = 0; w < 8; ++w) {
-      sk += rd[w * 32 + lane];
-      sq += rd[(8 + w) * 32 + lane];
+      float x[CV], y[CV];
+      load_cols<CV>(rd + w * VS + c0, x);
+      load_cols<CV>(rd + (8 + w) * VS + c0, y);
+#pragma unroll
+      for (int c = 0; c < CV; ++c) {
+        sk[c] += x[c];
+        sq[c] += y[c];
+      }
     }
-    const float u = col ? beta * (v[lane] - g * ik * sk) : 0.f;
-    const float o = g * iq * sq + qk * u;            // S^T q after the write
-    const float ku = ik * u;
+    float u[CV], o[CV];
+#pragma unroll
+    for (int c = 0; c < CV; ++c) {
+      const float uc = col ? beta * (v[c0 + c] - g * ik * sk[c]) : 0.f;
+      o[c] = g * iq * sq[c] + qk * uc;               // S^T q after the write
+      u[c] = ik * uc;
+    }
 #pragma unroll
     for (int i = 0; i < NR; ++i) {
       const int d = warp + 8 * i;
-      if (d < D) S[i] = fmaf(k[d], ku, g * S[i]);
+      if (d < D) {
+        const float kd = k[d];
+#pragma unroll
+        for (int c = 0; c < CV; ++c) S[i][c] = fmaf(kd, u[c], g * S[i][c]);
+      }
     }
     if (s.raw != nullptr) {
-      if (warp == 0 && col) s.raw[((int64_t)t * a.heads + h) * V + v0 + lane] = o;
+      if (warp == 0 && col) {
+#pragma unroll
+        for (int c = 0; c < CV; ++c) s.raw[((int64_t)t * a.heads + h) * V + v0 + c0 + c] = o[c];
+      }
     } else {
       // one token: norm over all columns of the head, which the CTAs of the cluster hold slice by slice
-      const float ss = warp_sum(o * o);
-      if (tid == 0) s_ss = ss;
-      float total = ss;
+      float ss = 0.f;
+#pragma unroll
+      for (int c = 0; c < CV; ++c) ss = fmaf(o[c], o[c], ss);
+      float total = ss = warp_sum(ss);
       if (gridDim.x > 1) {
+        if (tid == 0) s_ss = ss;
         cg::cluster_group cluster = cg::this_cluster();
         cluster.sync();
         total = 0.f;
@@ -188,17 +279,16 @@ __global__ void __launch_bounds__(kThreads) delta_step_kernel(StepArgs s) {
       }
       if (warp == 0 && col) {
         const float inv = 1.0f / sqrtf(total / (float)V + s.eps);
-        const int c = h * V + v0 + lane;
-        const float gate = DT<T>::to_f(reinterpret_cast<const T*>(a.proj)[(int64_t)t * a.ldp + s.gate_off + c]);
-        const float w = DT<T>::to_f(reinterpret_cast<const T*>(s.norm_w)[v0 + lane]);
-        reinterpret_cast<T*>(s.out)[(int64_t)t * s.ldo + c] = DT<T>::from_f(o * inv * w * silu(gate));
+        T* out = reinterpret_cast<T*>(s.out) + (int64_t)t * s.ldo + h * V + v0 + c0;
+#pragma unroll
+        for (int c = 0; c < CV; ++c) out[c] = DT<T>::from_f(o[c] * inv * nw[c] * silu(gate[c]));
       }
     }
   }
 #pragma unroll
   for (int i = 0; i < NR; ++i) {
     const int d = warp + 8 * i;
-    if (col && d < D) st[(int64_t)d * V] = S[i];
+    if (col && d < D) store_cols<CV>(st + (int64_t)d * V, S[i]);
   }
   if (s.ring_write) {
     // nobody reads this row in this launch; the first head of a group files the shared q / k channels
@@ -209,14 +299,14 @@ __global__ void __launch_bounds__(kThreads) delta_step_kernel(StepArgs s) {
         const int c = i < D ? qc + i : kc + i - D;
         ring[c] = proj[c];
       }
-    if (tid < nv) ring[vc + tid] = proj[vc + tid];
+    for (int i = tid; i < nv; i += kThreads) ring[vc + i] = proj[vc + i];
   }
 }
 
 // ---------------------------------------------------------------------------------------------- tf32 pairs
 __device__ __forceinline__ void split_tf32(float x, uint32_t& hi, uint32_t& lo) {
   hi = __float_as_uint(x) & 0xFFFFE000u;
-  lo = __float_as_uint(x - __uint_as_float(hi)) & 0xFFFFE000u;
+  lo = __float_as_uint(x - __uint_as_float(hi));       // exact; the instruction reads its upper 19 bits
 }
 __device__ __forceinline__ void mma_tf32(float (&c)[4], const uint32_t (&a)[4], const uint32_t (&b)[2]) {
   asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -257,17 +347,21 @@ struct Acc {
   __device__ __forceinline__ float get(int i) const { return m[i] + (x[i] + y[i]); }
 };
 
-// Scratch of one (chunk, head): W, Q and K parts [32][Dp] each, P [32][32], Ub [32][Vp], decay of the whole chunk
+// Scratch of one (chunk, head), laid out like the shared memory that reads it (row strides keep the fragments' banks
+// apart): W, Q and K parts of 32 rows, P [32][36], decay of the whole chunk; then Ub [32][40] per slice of 32 columns.
 struct Scratch {
-  int Dp, Vp;
-  __host__ __device__ Scratch(int D, int V) : Dp((D + 7) / 8 * 8), Vp((V + kVS - 1) / kVS * kVS) {}
-  __host__ __device__ int64_t floats() const { return (int64_t)kC * (3 * Dp + kC + Vp) + 4; }
-  __host__ __device__ int64_t w() const { return 0; }
-  __host__ __device__ int64_t q() const { return (int64_t)kC * Dp; }
-  __host__ __device__ int64_t k() const { return (int64_t)kC * 2 * Dp; }
-  __host__ __device__ int64_t p() const { return (int64_t)kC * 3 * Dp; }
-  __host__ __device__ int64_t ub() const { return p() + kC * kC; }
-  __host__ __device__ int64_t g() const { return ub() + (int64_t)kC * Vp; }
+  static constexpr int ldp = 36, ldu = 40;
+  int Dp, slices, ldw, ldk;
+  __host__ __device__ Scratch(int D, int V)
+      : Dp((D + 7) / 8 * 8), slices((V + kVS - 1) / kVS), ldw(Dp + 4), ldk(Dp + 8) {}
+  __host__ __device__ int q() const { return kC * ldw; }
+  __host__ __device__ int k() const { return kC * 2 * ldw; }
+  __host__ __device__ int p() const { return k() + kC * ldk; }
+  __host__ __device__ int g() const { return p() + kC * ldp; }
+  __host__ __device__ int shared_part() const { return g() + 4; }
+  __host__ __device__ int ub(int slice) const { return shared_part() + slice * kC * ldu; }
+  __host__ __device__ int floats() const { return ub(slices); }
+  __host__ __device__ int stage() const { return shared_part() + kC * ldu; }
 };
 
 struct ChunkArgs {
@@ -276,16 +370,63 @@ struct ChunkArgs {
   const int* seq_chunk;     // [sequences + 1] first chunk of a sequence
   float* scratch;           // of the chunks [c0, c1), [chunk - c0][head]
   float* raw;               // o [tokens, heads, vdim]
+  int* err;
   int c0, c1;
+  int vec;                  // rows of proj and ring can be read 16 bytes at a time
 };
 
-template <typename T>
-__global__ void __launch_bounds__(kThreads) delta_prep_kernel(ChunkArgs s) {
+// Eight neighbouring channels of the convolution for four tokens: every input row is read once.  TP: taps, 0 if only
+// known at run time.  first: token (of the chunk) of the first output; ws [taps][ldws]: weights of these channels.
+template <typename T, int TP>
+__device__ __forceinline__ void conv_block(const Common& a, int c, int t0, int row0, int p0, int start, int slot, int n,
+                                           int first, const float* ws, int ldws, float (&acc)[4][8]) {
+  const int taps = TP > 0 ? TP : a.taps;
+  const T* proj = reinterpret_cast<const T*>(a.proj) + c;
+  const T* ring = reinterpret_cast<const T*>(a.ring) + (int64_t)slot * taps * a.channels + c;
+#pragma unroll
+  for (int j = 0; j < 4; ++j)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) acc[j][e] = 0.f;
+  auto row = [&](int rr) {
+    const int rel = first - (taps - 1) + rr, p = p0 + rel, t = t0 + rel;
+    uint4 raw = make_uint4(0, 0, 0, 0);
+    if (p >= start && rel < n)
+      raw = *reinterpret_cast<const uint4*>(t >= row0 ? proj + (int64_t)t * a.ldp
+                                                      : ring + (int64_t)(p % taps) * a.channels);
+    return raw;
+  };
+  auto use = [&](int rr, const uint4& raw) {
+    const T* e8 = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int i = rr - j;
+      if (i >= 0 && i < taps) {
+        const float4 w0 = *reinterpret_cast<const float4*>(ws + i * ldws);
+        const float4 w1 = *reinterpret_cast<const float4*>(ws + i * ldws + 4);
+        const float w[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[j][e] = fmaf(DT<T>::to_f(e8[e]), w[e], acc[j][e]);
+      }
+    }
+  };
+  if constexpr (TP > 0) {
+    uint4 raw[TP + 3];
+#pragma unroll
+    for (int rr = 0; rr < TP + 3; ++rr) raw[rr] = row(rr);
+#pragma unroll
+    for (int rr = 0; rr < TP + 3; ++rr) use(rr, raw[rr]);
+  } else {
+    for (int rr = 0; rr < taps + 3; ++rr) use(rr, row(rr));
+  }
+}
+
+template <typename T, int TP>
+__global__ void __launch_bounds__(kThreads, 2) delta_prep_kernel(ChunkArgs s) {
   extern __shared__ __align__(16) float sm[];
   const Common& a = s.c;
   const int D = a.dim, V = a.vdim, h = blockIdx.y, chunk = s.c0 + blockIdx.x;
   const Scratch L(D, V);
-  const int Dp = L.Dp, Vp = L.Vp, ldk = Dp + 4, ldv = Vp + 8;
+  const int Dp = L.Dp, Vp = L.slices * kVS, ldk = Dp + 4, ldv = Vp + 8;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
   float* sq = sm;                        // [32][Dp + 4]
   float* sk = sq + kC * ldk;             // [32][Dp + 4]
@@ -295,6 +436,7 @@ __global__ void __launch_bounds__(kThreads) delta_prep_kernel(ChunkArgs s) {
   // [32] running sum of log g, in 64-bit: its differences must keep 32-bit accuracy when single tokens decay to nothing
   double* sL = reinterpret_cast<double*>(sT + kC * 36);
   float* sB = reinterpret_cast<float*>(sL + kC);      // [32] beta
+  float* sE = sB + kC;                                // [32] e^L
   const int seq = s.chunk_seq[chunk], hk = h / (a.heads / a.kv_heads);
   const int row0 = a.seq_row[seq], off = (chunk - s.seq_chunk[seq]) * kC, n = min(kC, a.seq_len[seq] - off);
   const int slot = a.slot[row0], start = a.start[slot], p0 = a.pos[row0] + off, t0 = row0 + off;
@@ -302,18 +444,53 @@ __global__ void __launch_bounds__(kThreads) delta_prep_kernel(ChunkArgs s) {
   const int qc = hk * D, kcol = a.kv_heads * D + hk * D, vcol = 2 * a.kv_heads * D + h * V;
 
   // ---- convolutions (zeros behind the sequence's end and past the sizes)
-  const int per = 2 * Dp + Vp;
-  for (int i = tid; i < kC * per; i += kThreads) {
-    const int t = i / per, c = i % per;
-    float x = 0.f;
-    if (c < 2 * Dp) {
-      const int d = c < Dp ? c : c - Dp;
-      if (t < n && d < D) x = conv_silu<T>(a, (c < Dp ? qc : kcol) + d, t0 + t, row0, p0 + t, start, slot);
-      (c < Dp ? sq : sk)[t * ldk + d] = x;
-    } else {
-      const int d = c - 2 * Dp;
-      if (t < n && d < V) x = conv_silu<T>(a, vcol + d, t0 + t, row0, p0 + t, start, slot);
-      sv[t * ldv + d] = x;
+  const T* taps_end = reinterpret_cast<const T*>(a.conv) + a.taps - 1;
+  if (s.vec) {
+    const int per = 2 * D + V, nvec = per / 8;
+    float* ws = sA;                      // [taps][per], over what comes later (the launch checks that it fits)
+    auto channel = [&](int c) { return c < D ? qc + c : c < 2 * D ? kcol + c - D : vcol + c - 2 * D; };
+    for (int c = tid; c < per; c += kThreads) {
+      const T* w = reinterpret_cast<const T*>(a.conv) + (int64_t)channel(c) * a.taps;
+      for (int i = 0; i < a.taps; ++i) ws[i * per + c] = DT<T>::to_f(w[i]);
+    }
+    for (int i = tid; i < kC * (Vp - V); i += kThreads) sv[i / (Vp - V) * ldv + V + i % (Vp - V)] = 0.f;
+    __syncthreads();
+    for (int i = tid; i < nvec * (kC / 4); i += kThreads) {
+      const int c = (i % nvec) * 8, first = (i / nvec) * 4;
+      float acc[4][8];
+      conv_block<T, TP>(a, channel(c), t0, row0, p0, start, slot, n, first, ws + c, per, acc);
+      float* dst = c < D ? sq + c : c < 2 * D ? sk + c - D : sv + c - 2 * D;
+      const int ld = c < 2 * D ? ldk : ldv;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const bool on = first + j < n;
+#pragma unroll
+        for (int e = 0; e < 8; e += 4)
+          *reinterpret_cast<float4*>(dst + (first + j) * ld + e) =
+              on ? make_float4(fast_silu(acc[j][e]), fast_silu(acc[j][e + 1]), fast_silu(acc[j][e + 2]),
+                               fast_silu(acc[j][e + 3]))
+                 : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+    }
+    __syncthreads();                     // the weights' place is free
+  } else {
+    const int per = 2 * Dp + Vp;
+    for (int i = tid; i < kC * per; i += kThreads) {
+      const int t = i / per, c = i % per;
+      float x = 0.f;
+      if (c < 2 * Dp) {
+        const int d = c < Dp ? c : c - Dp;
+        if (t < n && d < D) {
+          const int ch = (c < Dp ? qc : kcol) + d;
+          x = conv_silu<T>(a, ch, t0 + t, off + t, p0 + t, start, slot, taps_end + (int64_t)ch * a.taps);
+        }
+        (c < Dp ? sq : sk)[t * ldk + d] = x;
+      } else {
+        const int d = c - 2 * Dp;
+        if (t < n && d < V) 
+          x = conv_silu<T>(a, vcol + d, t0 + t, off + t, p0 + t, start, slot, taps_end + (int64_t)(vcol + d) * a.taps);
+        sv[t * ldv + d] = x;
+      }
     }
   }
   if (warp == 0) {
@@ -331,6 +508,7 @@ __global__ void __launch_bounds__(kThreads) delta_prep_kernel(ChunkArgs s) {
     }
     sL[lane] = lg;
     sB[lane] = beta;
+    sE[lane] = expf((float)lg);
   }
   __syncthreads();
   // ---- unit vectors; the decayed copies go out right away
@@ -343,13 +521,13 @@ __global__ void __launch_bounds__(kThreads) delta_prep_kernel(ChunkArgs s) {
       kk = fmaf(y, y, kk);
     }
     const float iq = a.qscale / sqrtf(warp_sum(qq) + kUnitEps), ik = 1.0f / sqrtf(warp_sum(kk) + kUnitEps);
-    const float gq = expf((float)sL[t]), gk = expf((float)(lend - sL[t]));
+    const float gq = sE[t], gk = expf((float)(lend - sL[t]));
     for (int d = lane; d < Dp; d += 32) {
       const float x = sq[t * ldk + d] * iq, y = sk[t * ldk + d] * ik;
       sq[t * ldk + d] = x;
       sk[t * ldk + d] = y;
-      out[L.q() + t * Dp + d] = x * gq;
-      out[L.k() + t * Dp + d] = y * gk;
+      out[L.q() + t * L.ldw + d] = x * gq;
+      out[L.k() + t * L.ldk + d] = y * gk;
     }
   }
   if (tid == 0) out[L.g()] = expf((float)lend);
@@ -372,30 +550,59 @@ __global__ void __launch_bounds__(kThreads) delta_prep_kernel(ChunkArgs s) {
       const int t = m0 + g + 8 * (i >> 1), j = n0 + 2 * t4 + (i & 1);
       const float dec = j <= t ? expf((float)(sL[t] - sL[j])) : 0.f;
       sA[t * 36 + j] = j < t ? sB[t] * dec * aa.get(i) : 0.f;
-      out[L.p() + t * kC + j] = j <= t ? dec * pp.get(i) : 0.f;
+      out[L.p() + t * L.ldp + j] = j <= t ? dec * pp.get(i) : 0.f;
     }
   }
   __syncthreads();
-  // ---- inverse of I + A: lane j solves for column j
-  if (warp == 0) {
-    float x[kC];
+  // ---- inverse of I + A by halves: two warps solve the 16 x 16 blocks on the diagonal, a lane per column ...
+  if (warp < 2) {
+    const int b = warp * 16;
+    float x[16];
 #pragma unroll
-    for (int t = 0; t < kC; ++t) {
+    for (int t = 0; t < 16; ++t) {
       float r0 = t == lane ? 1.f : 0.f, r1 = 0.f, r2 = 0.f, r3 = 0.f;
 #pragma unroll
       for (int i = 0; i < t; i += 4) {
-        const float4 w = *reinterpret_cast<const float4*>(sA + t * 36 + i);
+        const float4 w = *reinterpret_cast<const float4*>(sA + (b + t) * 36 + b + i);
         r0 = fmaf(-w.x, x[i], r0);
         if (i + 1 < t) r1 = fmaf(-w.y, x[i + 1], r1);
         if (i + 2 < t) r2 = fmaf(-w.z, x[i + 2], r2);
         if (i + 3 < t) r3 = fmaf(-w.w, x[i + 3], r3);
       }
       x[t] = (r0 + r1) + (r2 + r3);
-      sT[t * 36 + lane] = x[t] * sB[lane];      // column j times beta_j: the right-hand sides carry it
+      if (lane < 16) sT[(b + t) * 36 + b + lane] = x[t];
     }
   }
   __syncthreads();
-  // ---- W = T (beta e^L) K and Ub = T beta V: warps take 8-wide column tiles, both row tiles
+  // ... and the block below is -T22 (A21 T11), eight columns per warp (A11's place holds the product in between)
+  if (warp < 2) {
+    const int n0 = warp * 8;
+    Acc acc;
+    acc.zero();
+#pragma unroll
+    for (int k0 = 0; k0 < 16; k0 += 8)
+      acc.mac(frag_a([&](int r, int k) { return sA[(16 + r) * 36 + k0 + k]; }, g, t4),
+              frag_b([&](int k, int j) { return sT[(k0 + k) * 36 + n0 + j]; }, g, t4));
+#pragma unroll
+    for (int i = 0; i < 4; ++i) sA[(g + 8 * (i >> 1)) * 36 + n0 + 2 * t4 + (i & 1)] = acc.get(i);
+    __syncwarp();
+    acc.zero();
+#pragma unroll
+    for (int k0 = 0; k0 < 16; k0 += 8)
+      acc.mac(frag_a([&](int r, int k) { return sT[(16 + r) * 36 + 16 + k0 + k]; }, g, t4),
+              frag_b([&](int k, int j) { return sA[(k0 + k) * 36 + n0 + j]; }, g, t4));
+#pragma unroll
+    for (int i = 0; i < 4; ++i) sT[(16 + g + 8 * (i >> 1)) * 36 + n0 + 2 * t4 + (i & 1)] = -acc.get(i);
+  }
+  __syncthreads();
+  // ---- W = T (beta e^L) K and Ub = T beta V: T's fragments stay in registers (its upper right block is zero), warps
+  // take 8-wide column tiles
+  FragA ft[6];                           // row tile 0: k 0, 8; row tile 1: k 0, 8, 16, 24
+#pragma unroll
+  for (int f = 0; f < 6; ++f) {
+    const int m = f < 2 ? 0 : 16, k0 = (f < 2 ? f : f - 2) * 8;
+    ft[f] = frag_a([&](int r, int k) { return sT[(m + r) * 36 + k0 + k] * sB[k0 + k]; }, g, t4);
+  }
   const int nw = Dp / 8, ntile = nw + Vp / 8;
   for (int tile = warp; tile < ntile; tile += kThreads / 32) {
     const bool isw = tile < nw;
@@ -406,184 +613,174 @@ __global__ void __launch_bounds__(kThreads) delta_prep_kernel(ChunkArgs s) {
     acc[0].zero();
     acc[1].zero();
 #pragma unroll
-    for (int k0 = 0; k0 < kC; k0 += 8) {
+    for (int f = 0; f < 4; ++f) {
       const FragB b = frag_b([&](int k, int j) {
-        const float y = src[(k0 + k) * lds + n0 + j];
-        return isw ? y * expf((float)sL[k0 + k]) : y;
+        const float y = src[(f * 8 + k) * lds + n0 + j];
+        return isw ? y * sE[f * 8 + k] : y;
       }, g, t4);
-#pragma unroll
-      for (int m = 0; m < 2; ++m)
-        acc[m].mac(frag_a([&](int r, int k) { return sT[(m * 16 + r) * 36 + k0 + k]; }, g, t4), b);
+      if (f < 2) acc[0].mac(ft[f], b);
+      acc[1].mac(ft[2 + f], b);
     }
-    float* dst = isw ? out + L.w() : out + L.ub();
-    const int ldd = isw ? Dp : Vp;
+    float* dst = isw ? out + n0 : out + L.ub(n0 / kVS) + n0 % kVS;
+    const int ldd = isw ? L.ldw : L.ldu;
 #pragma unroll
     for (int m = 0; m < 2; ++m)
 #pragma unroll
       for (int i = 0; i < 4; i += 2)
-        *reinterpret_cast<float2*>(dst + (m * 16 + g + 4 * i) * ldd + n0 + 2 * t4) =
+        *reinterpret_cast<float2*>(dst + (m * 16 + g + 4 * i) * ldd + 2 * t4) =
             make_float2(acc[m].get(i), acc[m].get(i + 1));
   }
 }
 
-__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+__device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
+                   tc5::smem_u32(dst)), "l"(src), "r"(bytes), "r"(tc5::smem_u32(bar))
+               : "memory");
 }
 
 template <int MT>
-__global__ void __launch_bounds__(kThreads, 1) delta_chunks_kernel(ChunkArgs s, int stages) {
+__global__ void __launch_bounds__(kChunkThreads, 1) delta_chunks_kernel(ChunkArgs s, int stages) {
   extern __shared__ __align__(16) float sm[];
+  __shared__ __align__(8) uint64_t full[2];
+  __shared__ int abort_word;
+  volatile int* abort_flag = &abort_word;
   const Common& a = s.c;
   const int D = a.dim, V = a.vdim, h = blockIdx.y, seq = blockIdx.z, v0 = blockIdx.x * kVS, nv = min(kVS, V - v0);
   const Scratch L(D, V);
-  const int Dp = L.Dp, Dm = (D + 15) / 16 * 16, ldw = Dp + 4, ldk = Dp + 8, ldu = 40;
+  const int Dp = L.Dp, Dm = (D + 15) / 16 * 16, ldw = L.ldw, ldk = L.ldk, ldu = L.ldu;
   const int first = s.seq_chunk[seq], last = s.seq_chunk[seq + 1];
   const int ca = max(first, s.c0), cb = min(last, s.c1);
   if (ca >= cb) return;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
-  const int stage_floats = kC * (2 * ldw + 36 + 40) + kC * ldk + 8;
-  float* sS = sm;                              // [Dm][40]
+  float* stage0 = sm;
+  float* sS = stage0 + stages * L.stage();     // [Dm][40]
   float* sU = sS + Dm * ldu;                   // [32][40]
-  float* stage0 = sU + kC * ldu;
   const int row0 = a.seq_row[seq], len = a.seq_len[seq];
   const int slot = a.slot[row0], start = a.start[slot], p0 = a.pos[row0];
   float* st = a.state + (((int64_t)slot * a.heads + h) * D) * V + v0;
 
-  struct View { float *w, *q, *p, *ub, *k, *gc; };
+  struct View { const float *w, *q, *p, *ub, *k, *gc; };
   auto view = [&](int i) {
-    float* b = stage0 + (i % stages) * stage_floats;
-    View v;
-    v.w = b;
-    v.q = v.w + kC * ldw;
-    v.p = v.q + kC * ldw;
-    v.ub = v.p + kC * 36;
-    v.k = v.ub + kC * 40;
-    v.gc = v.k + kC * ldk;
-    return v;
+    const float* b = stage0 + (i % stages) * L.stage();
+    return View{b, b + L.q(), b + L.p(), b + L.shared_part(), b + L.k(), b + L.g()};
   };
-  auto fetch = [&](int c) {
-    if (c < cb) {
-      const float* src = s.scratch + ((int64_t)(c - s.c0) * a.heads + h) * L.floats();
-      const View v = view(c - ca);
-      const int nd = Dp / 4;
-      for (int i = tid; i < kC * nd; i += kThreads) {
-        const int t = i / nd, d = (i % nd) * 4;
-        cp_async16(v.w + t * ldw + d, src + L.w() + t * Dp + d);
-        cp_async16(v.q + t * ldw + d, src + L.q() + t * Dp + d);
-        cp_async16(v.k + t * ldk + d, src + L.k() + t * Dp + d);
-      }
-      for (int i = tid; i < kC * 8; i += kThreads) {
-        const int t = i / 8, d = (i % 8) * 4;
-        cp_async16(v.p + t * 36 + d, src + L.p() + t * kC + d);
-        cp_async16(v.ub + t * 40 + d, src + L.ub() + t * L.Vp + v0 + d);
-      }
-      if (tid == 0) cp_async16(v.gc, src + L.g());
-    }
-    asm volatile("cp.async.commit_group;" ::: "memory");
+  auto fetch = [&](int c) {                    // one thread
+    if (c >= cb) return;
+    const float* src = s.scratch + ((int64_t)(c - s.c0) * a.heads + h) * L.floats();
+    float* dst = stage0 + ((c - ca) % stages) * L.stage();
+    uint64_t* bar = &full[(c - ca) % stages];
+    tc5::mbar_expect_tx(bar, (uint32_t)(L.stage() * sizeof(float)));
+    bulk_load(dst, src, (uint32_t)(L.shared_part() * sizeof(float)), bar);
+    bulk_load(dst + L.shared_part(), src + L.ub(blockIdx.x), (uint32_t)(kC * ldu * sizeof(float)), bar);
   };
 
-  fetch(ca);
-  // ---- state: accumulator fragments of the row tiles warp, warp + 8, ... (MT of them)
-  float S[MT][4][4];
+  if (tid == 0) {
+    tc5::mbar_init(&full[0], 1);
+    tc5::mbar_init(&full[1], 1);
+    abort_word = 0;
+    tc5::fence_barrier_init();
+    for (int i = 0; i < stages; ++i) fetch(ca + i);
+  }
+  // ---- state: accumulator fragments of the row tiles warp / 2, warp / 2 + 8, ... (MT of them), two column tiles each
+  const int wm = warp >> 1, wn = (warp & 1) * 2;
+  float S[MT][2][4];
   const bool fresh = ca == first && p0 <= start;
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
-    for (int n = 0; n < 4; ++n)
+    for (int n = 0; n < 2; ++n)
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const int d = (warp + 8 * m) * 16 + g + 8 * (i >> 1), c = n * 8 + 2 * t4 + (i & 1);
+        const int d = (wm + 8 * m) * 16 + g + 8 * (i >> 1), c = (wn + n) * 8 + 2 * t4 + (i & 1);
         S[m][n][i] = !fresh && d < D && c < nv ? st[(int64_t)d * V + c] : 0.f;
         if (d < Dm) sS[d * ldu + c] = S[m][n][i];
       }
 
-  const int mt = warp >> 1, nt0 = (warp & 1) * 2;      // row tile of [W; Q], first of two column tiles
+  const int mt = warp >> 2, nt = (warp & 3) * 8;       // row tile of [W; Q], first column
+  bool ok = true;
   for (int c = ca; c < cb; ++c) {
-    if (stages > 1) {
-      fetch(c + 1);
-      asm volatile("cp.async.wait_group 1;" ::: "memory");
-    } else {
-      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                                   // the state is in place (and, first, the barriers)
+    if (!tc5::mbar_wait(&full[(c - ca) % stages], ((c - ca) / stages) & 1, abort_flag)) {
+      if (lane == 0) tc5::report(s.err, 40);
+      ok = false;
+      break;
     }
-    __syncthreads();                                   // this chunk's parts and the state are in place
     const View v = view(c - ca);
-    Acc acc[2];
-    acc[0].zero();
-    acc[1].zero();
+    Acc acc;
+    acc.zero();
     {
       const float* left = mt < 2 ? v.w + mt * 16 * ldw : v.q + (mt - 2) * 16 * ldw;
 #pragma unroll 4
       for (int k0 = 0; k0 < Dp; k0 += 8) {
-        const FragA fa = frag_a([&](int r, int k) { return left[r * ldw + k0 + k]; }, g, t4);
-#pragma unroll
-        for (int n = 0; n < 2; ++n)
-          acc[n].mac(fa, frag_b([&](int k, int j) { return sS[(k0 + k) * ldu + (nt0 + n) * 8 + j]; }, g, t4));
+        acc.mac(frag_a([&](int r, int k) { return left[r * ldw + k0 + k]; }, g, t4),
+                frag_b([&](int k, int j) { return sS[(k0 + k) * ldu + nt + j]; }, g, t4));
       }
     }
     if (mt < 2) {
 #pragma unroll
-      for (int n = 0; n < 2; ++n)
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const int t = mt * 16 + g + 8 * (i >> 1), col = (nt0 + n) * 8 + 2 * t4 + (i & 1);
-          sU[t * ldu + col] = v.ub[t * 40 + col] - acc[n].get(i);
-        }
+      for (int i = 0; i < 4; ++i) {
+        const int t = mt * 16 + g + 8 * (i >> 1), col = nt + 2 * t4 + (i & 1);
+        sU[t * ldu + col] = v.ub[t * ldu + col] - acc.get(i);
+      }
     }
     __syncthreads();                                   // U is complete, the old state is read
     if (mt >= 2) {
 #pragma unroll
       for (int k0 = 0; k0 < kC; k0 += 8) {
-        const FragA fa = frag_a([&](int r, int k) { return v.p[((mt - 2) * 16 + r) * 36 + k0 + k]; }, g, t4);
-#pragma unroll
-        for (int n = 0; n < 2; ++n)
-          acc[n].mac(fa, frag_b([&](int k, int j) { return sU[(k0 + k) * ldu + (nt0 + n) * 8 + j]; }, g, t4));
+        acc.mac(frag_a([&](int r, int k) { return v.p[((mt - 2) * 16 + r) * L.ldp + k0 + k]; }, g, t4),
+                frag_b([&](int k, int j) { return sU[(k0 + k) * ldu + nt + j]; }, g, t4));
       }
       const int off = (c - first) * kC;
 #pragma unroll
-      for (int n = 0; n < 2; ++n)
-#pragma unroll
-        for (int i = 0; i < 4; ++i) {
-          const int t = off + (mt - 2) * 16 + g + 8 * (i >> 1), col = (nt0 + n) * 8 + 2 * t4 + (i & 1);
-          if (t < len && col < nv) s.raw[((int64_t)(row0 + t) * a.heads + h) * V + v0 + col] = acc[n].get(i);
-        }
+      for (int i = 0; i < 4; ++i) {
+        const int t = off + (mt - 2) * 16 + g + 8 * (i >> 1), col = nt + 2 * t4 + (i & 1);
+        if (t < len && col < nv) s.raw[((int64_t)(row0 + t) * a.heads + h) * V + v0 + col] = acc.get(i);
+      }
     }
     const float gc = *v.gc;
 #pragma unroll
     for (int m = 0; m < MT; ++m) {
-      const int d0 = (warp + 8 * m) * 16;
+      const int d0 = (wm + 8 * m) * 16;
       if (d0 < Dm) {
-        Acc up[4];
-#pragma unroll
-        for (int n = 0; n < 4; ++n) up[n].zero();
+        Acc up[2];
+        up[0].zero();
+        up[1].zero();
 #pragma unroll
         for (int k0 = 0; k0 < kC; k0 += 8) {
           const FragA fa = frag_a([&](int r, int k) { return d0 + r < Dp ? v.k[(k0 + k) * ldk + d0 + r] : 0.f; }, g, t4);
 #pragma unroll
-          for (int n = 0; n < 4; ++n)
-            up[n].mac(fa, frag_b([&](int k, int j) { return sU[(k0 + k) * ldu + n * 8 + j]; }, g, t4));
+          for (int n = 0; n < 2; ++n)
+            up[n].mac(fa, frag_b([&](int k, int j) { return sU[(k0 + k) * ldu + (wn + n) * 8 + j]; }, g, t4));
         }
 #pragma unroll
-        for (int n = 0; n < 4; ++n)
+        for (int n = 0; n < 2; ++n)
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
             S[m][n][i] = fmaf(gc, S[m][n][i], up[n].get(i));
-            sS[(d0 + g + 8 * (i >> 1)) * ldu + n * 8 + 2 * t4 + (i & 1)] = S[m][n][i];
+            sS[(d0 + g + 8 * (i >> 1)) * ldu + (wn + n) * 8 + 2 * t4 + (i & 1)] = S[m][n][i];
           }
       }
     }
     __syncthreads();                                   // the stage and U are free again
-    if (stages == 1) fetch(c + 1);
+    if (tid == 0) fetch(c + stages);
+  }
+  if (!ok) {                                           // copies in flight still write to this CTA's memory
+    if (tid == 0)
+      for (int i = 0; i < stages; ++i) {
+        tc5::mbar_wait_quiet(&full[i], 0, 1 << 12);
+        tc5::mbar_wait_quiet(&full[i], 1, 1 << 12);
+      }
+    return;
   }
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
-    for (int n = 0; n < 4; ++n)
+    for (int n = 0; n < 2; ++n)
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const int d = (warp + 8 * m) * 16 + g + 8 * (i >> 1), c = n * 8 + 2 * t4 + (i & 1);
+        const int d = (wm + 8 * m) * 16 + g + 8 * (i >> 1), c = (wn + n) * 8 + 2 * t4 + (i & 1);
         if (d < D && c < nv) st[(int64_t)d * V + c] = S[m][n][i];
       }
-  asm volatile("cp.async.wait_group 0;" ::: "memory");
 }
 
 template <typename T>
@@ -597,23 +794,51 @@ __global__ void __launch_bounds__(kThreads) delta_tail_kernel(Common a) {
     ring[(int64_t)((p0 + j) % a.taps) * a.channels] = proj[(int64_t)(row0 + j) * a.ldp];
 }
 
-// A warp per (token, head).
-template <typename T>
+// A warp per (token, head); VEC: four neighbouring columns per lane and step.
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(kThreads) gated_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate,
                                                               int64_t ldg, const T* __restrict__ w, T* __restrict__ out,
                                                               int64_t ldo, int64_t rows, int heads, int V, float eps) {
+  constexpr int N = VEC ? 4 : 1;
   const int64_t r = (int64_t)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
   if (r >= rows) return;
   const int64_t t = r / heads;
   const int h = (int)(r % heads);
   const float* src = o + r * V;
-  float ss = 0.f;
-  for (int i = lane; i < V; i += 32) ss = fmaf(src[i], src[i], ss);
+  const T* gt = gate + t * ldg + (int64_t)h * V;
+  T* dst = out + t * ldo + (int64_t)h * V;
+  auto load = [&](const T* p, float (&v)[N]) {
+    if constexpr (VEC && sizeof(T) == 2) {
+      const uint2 raw = *reinterpret_cast<const uint2*>(p);
+#pragma unroll
+      for (int c = 0; c < N; ++c) v[c] = DT<T>::to_f(reinterpret_cast<const T*>(&raw)[c]);
+    } else {
+#pragma unroll
+      for (int c = 0; c < N; ++c) v[c] = DT<T>::to_f(p[c]);
+    }
+  };
+  float x[N], gv[N], wv[N], ss = 0.f;
+  for (int i = lane * N; i < V; i += 32 * N) {
+    load_cols<N>(src + i, x);
+#pragma unroll
+    for (int c = 0; c < N; ++c) ss = fmaf(x[c], x[c], ss);
+  }
   const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)V + eps);
-  for (int i = lane; i < V; i += 32)
-    out[t * ldo + h * V + i] =
-        DT<T>::from_f(src[i] * inv * DT<T>::to_f(w[i]) * silu(DT<T>::to_f(gate[t * ldg + h * V + i])));
+  for (int i = lane * N; i < V; i += 32 * N) {
+    load_cols<N>(src + i, x);
+    load(gt + i, gv);
+    load(w + i, wv);
+    __align__(16) T y[N];
+#pragma unroll
+    for (int c = 0; c < N; ++c) y[c] = DT<T>::from_f(x[c] * inv * wv[c] * silu(gv[c]));
+    if constexpr (VEC && sizeof(T) == 2) {
+      *reinterpret_cast<uint2*>(dst + i) = *reinterpret_cast<const uint2*>(y);
+    } else {
+#pragma unroll
+      for (int c = 0; c < N; ++c) dst[i + c] = y[c];
+    }
+  }
 }
 
 bool sizes_ok(int heads, int kv_heads, int dim, int vdim, int taps) {
@@ -629,10 +854,18 @@ Common common_args(const void* proj, int64_t ldp, const float* gates, const void
   return c;
 }
 
-template <typename T, int NR>
+constexpr size_t kSmemMax = 226 * 1024;
+
+template <typename T, int NR, int CV>
 cudaError_t launch_step(const StepArgs& s, int seqs, bool fused, bool pdl, cudaStream_t st) {
-  const int slices = (s.c.vdim + kVS - 1) / kVS;
-  const size_t smem = (2 * (2 * (size_t)s.c.dim + kVS) + 2 * 2 * 8 * 32) * sizeof(float);
+  const int slices = (s.c.vdim + 32 * CV - 1) / (32 * CV);
+  if (fused && slices > 8) return cudaErrorInvalidValue;
+  const size_t smem = ((2 + s.c.taps) * (2 * (size_t)s.c.dim + 32 * CV) + 2 * 2 * 8 * 32 * CV) * sizeof(float);
+  if (smem > kSmemMax) return cudaErrorInvalidValue;
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(delta_step_kernel<T, NR, CV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return e;
+  }
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(slices, s.c.heads, seqs);
   cfg.blockDim = dim3(kThreads);
@@ -654,19 +887,27 @@ cudaError_t launch_step(const StepArgs& s, int seqs, bool fused, bool pdl, cudaS
   }
   cfg.attrs = attr;
   cfg.numAttrs = na;
-  return cudaLaunchKernelEx(&cfg, delta_step_kernel<T, NR>, s);
+  return cudaLaunchKernelEx(&cfg, delta_step_kernel<T, NR, CV>, s);
+}
+
+// Columns per lane: as many as V divides into and the registers of NR rows leave room for.
+template <typename T, int NR>
+cudaError_t pick_cols(const StepArgs& s, int seqs, bool fused, bool pdl, cudaStream_t st) {
+  const int V = s.c.vdim;
+  if constexpr (NR <= 16)
+    if (V % 4 == 0 && V > 64) return launch_step<T, NR, 4>(s, seqs, fused, pdl, st);
+  if constexpr (NR <= 32)
+    if (V % 2 == 0 && V > 32) return launch_step<T, NR, 2>(s, seqs, fused, pdl, st);
+  return launch_step<T, NR, 1>(s, seqs, fused, pdl, st);
 }
 
 size_t prep_smem(const Scratch& L) {
-  return (size_t)(2 * kC * (L.Dp + 4) + kC * (L.Vp + 8) + 2 * kC * 36 + 3 * kC) * sizeof(float);
+  return (size_t)(2 * kC * (L.Dp + 4) + kC * (L.slices * kVS + 8) + 2 * kC * 36 + 4 * kC) * sizeof(float);
 }
 size_t chunk_smem(const Scratch& L, int D, int stages) {
   const int Dm = (D + 15) / 16 * 16;
-  return ((size_t)(Dm + kC) * 40 +
-          (size_t)stages * (kC * (2 * (L.Dp + 4) + 36 + 40) + kC * (L.Dp + 8) + 8)) * sizeof(float);
+  return ((size_t)(Dm + kC) * L.ldu + (size_t)stages * L.stage()) * sizeof(float);
 }
-constexpr size_t kSmemMax = 226 * 1024;
-
 }  // namespace
 
 // Can the chunked form take these sizes?
@@ -675,8 +916,8 @@ IPEX_API int ipex_delta_chunks_ok(int dim, int vdim) {
   return dim >= 1 && dim <= 256 && vdim >= 1 && prep_smem(L) <= kSmemMax && chunk_smem(L, dim, 1) <= kSmemMax;
 }
 IPEX_API int64_t ipex_delta_scratch_floats(int dim, int vdim) { return Scratch(dim, vdim).floats(); }
-// Column slices of a head: the fused norm of a decode step takes up to eight.
-IPEX_API int ipex_delta_slices(int vdim) { return (vdim + kVS - 1) / kVS; }
+// Can a decode step of these sizes norm its outputs on the way?
+IPEX_API int ipex_delta_fused_ok(int vdim) { return vdim >= 1 && vdim <= 256; }
 
 // Token by token.  seq_row / seq_len null: `seqs` sequences of one token each, whose convolution inputs are filed on
 // the way; norm_w / out [tokens, ldo] then take the gated norm's result (vdim <= 256).  raw (when out is null): the
@@ -689,19 +930,19 @@ IPEX_API int ipex_delta_step(const void* proj, int64_t ldp, int gate_off, const 
   if (!sizes_ok(heads, kv_heads, dim, vdim, taps) || seqs < 1 || seqs > 65535 || (seq_row == nullptr) != (seq_len == nullptr))
     return (int)cudaErrorInvalidValue;
   const bool fused = raw == nullptr;
-  if (fused && (seq_row != nullptr || out == nullptr || norm_w == nullptr || ipex_delta_slices(vdim) > 8))
+  if (fused && (seq_row != nullptr || out == nullptr || norm_w == nullptr || !ipex_delta_fused_ok(vdim)))
     return (int)cudaErrorInvalidValue;
   return by_dtype(dtype, [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
     StepArgs s = {common_args(proj, ldp, gates, conv, a_log, dt_bias, ring, state, slot, pos, start, seq_row, seq_len,
                               heads, kv_heads, dim, vdim, taps),
-                  norm_w, out, raw, ldo, eps, gate_off, seq_row == nullptr};
+                  norm_w, out, raw, ldo, eps, gate_off, seq_row == nullptr, pdl && fused && vdim % 4 == 0};
     cudaStream_t st = (cudaStream_t)stream;
-    if (dim <= 32) return launch_step<T, 4>(s, seqs, fused, pdl != 0, st);
-    if (dim <= 64) return launch_step<T, 8>(s, seqs, fused, pdl != 0, st);
-    if (dim <= 128) return launch_step<T, 16>(s, seqs, fused, pdl != 0, st);
-    if (dim <= 256) return launch_step<T, 32>(s, seqs, fused, pdl != 0, st);
-    return launch_step<T, 64>(s, seqs, fused, pdl != 0, st);
+    if (dim <= 32) return pick_cols<T, 4>(s, seqs, fused, pdl != 0, st);
+    if (dim <= 64) return pick_cols<T, 8>(s, seqs, fused, pdl != 0, st);
+    if (dim <= 128) return pick_cols<T, 16>(s, seqs, fused, pdl != 0, st);
+    if (dim <= 256) return pick_cols<T, 32>(s, seqs, fused, pdl != 0, st);
+    return pick_cols<T, 64>(s, seqs, fused, pdl != 0, st);
   });
 }
 
@@ -711,7 +952,7 @@ IPEX_API int ipex_delta_chunks(const void* proj, int64_t ldp, const float* gates
                                const float* dt_bias, void* ring, float* state, const int* slot, const int* pos,
                                const int* start, const int* seq_row, const int* seq_len, int seqs, const int* chunk_seq,
                                const int* seq_chunk, int c0, int c1, float* scratch, float* raw, int heads, int kv_heads,
-                               int dim, int vdim, int taps, int dtype, void* stream) {
+                               int dim, int vdim, int taps, int dtype, int* err, void* stream) {
   if (!sizes_ok(heads, kv_heads, dim, vdim, taps) || !ipex_delta_chunks_ok(dim, vdim) || seqs < 1 || seqs > 65535 ||
       c0 < 0 || c1 <= c0 || seq_row == nullptr || seq_len == nullptr || (((uintptr_t)scratch) & 15) || dtype == DT_F32)
     return (int)cudaErrorInvalidValue;
@@ -719,13 +960,17 @@ IPEX_API int ipex_delta_chunks(const void* proj, int64_t ldp, const float* gates
     using T = std::remove_pointer_t<decltype(tag)>;
     ChunkArgs s = {common_args(proj, ldp, gates, conv, a_log, dt_bias, ring, state, slot, pos, start, seq_row, seq_len,
                                heads, kv_heads, dim, vdim, taps),
-                   chunk_seq, seq_chunk, scratch, raw, c0, c1};
+                   chunk_seq, seq_chunk, scratch, raw, err, c0, c1, 0};
+    // 16-byte reads, and room for the convolution weights where A and its inverse go later
+    s.vec = dim % 8 == 0 && vdim % 8 == 0 && ldp % 8 == 0 && (((uintptr_t)proj | (uintptr_t)ring) & 15) == 0 &&
+            (2 * dim + vdim) * taps <= 2 * kC * 36;
     cudaStream_t st = (cudaStream_t)stream;
     const Scratch L(dim, vdim);
     const size_t ps = prep_smem(L);
-    cudaError_t e = cudaFuncSetAttribute(delta_prep_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ps);
+    auto prep = taps == 4 ? delta_prep_kernel<T, 4> : delta_prep_kernel<T, 0>;
+    cudaError_t e = cudaFuncSetAttribute(prep, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ps);
     if (e != cudaSuccess) return e;
-    delta_prep_kernel<T><<<dim3(c1 - c0, heads), kThreads, ps, st>>>(s);
+    prep<<<dim3(c1 - c0, heads), kThreads, ps, st>>>(s);
     e = cudaGetLastError();
     if (e != cudaSuccess) return e;
     const int stages = chunk_smem(L, dim, 2) <= kSmemMax ? 2 : 1;
@@ -733,7 +978,7 @@ IPEX_API int ipex_delta_chunks(const void* proj, int64_t ldp, const float* gates
     auto kern = dim <= 128 ? delta_chunks_kernel<1> : delta_chunks_kernel<2>;
     e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)cs);
     if (e != cudaSuccess) return e;
-    kern<<<dim3(ipex_delta_slices(vdim), heads, seqs), kThreads, cs, st>>>(s, stages);
+    kern<<<dim3(L.slices, heads, seqs), kChunkThreads, cs, st>>>(s, stages);
     return cudaGetLastError();
   };
   return (int)(dtype == DT_F16 ? run((__half*)nullptr) : run((__nv_bfloat16*)nullptr));
@@ -761,8 +1006,11 @@ IPEX_API int ipex_gated_norm(const float* o, const void* gate, int64_t ldg, cons
   return by_dtype(dtype, [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
     const int64_t rows = (int64_t)tokens * heads;
-    gated_norm_kernel<T><<<(unsigned)((rows + 7) / 8), kThreads, 0, (cudaStream_t)stream>>>(
-        o, (const T*)gate, ldg, (const T*)w, (T*)out, ldo, rows, heads, vdim, eps);
+    const bool vec = vdim % 4 == 0 && ldg % 4 == 0 && ldo % 4 == 0 && ((uintptr_t)o & 15) == 0 &&
+                     (((uintptr_t)gate | (uintptr_t)w | (uintptr_t)out) & 7) == 0;
+    auto kern = vec ? gated_norm_kernel<T, true> : gated_norm_kernel<T, false>;
+    kern<<<(unsigned)((rows + 7) / 8), kThreads, 0, (cudaStream_t)stream>>>(o, (const T*)gate, ldg, (const T*)w, (T*)out,
+                                                                            ldo, rows, heads, vdim, eps);
     return cudaGetLastError();
   });
 }

@@ -193,16 +193,19 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
         const int64_t r0 = xrow + c * 32;
         const float bn = a.bias != nullptr && n < a.N ? to_float<T>(reinterpret_cast<const T*>(a.bias)[n]) : 0.f;
         if (a.act == 3) {
-          // lanes with bit 3 clear hold gate rows, the lanes eight above them the matching up rows
+          // lanes with bit 3 clear hold gate rows, the lanes eight above them the matching up rows: the former finish
+          // the even tokens of a pair, the latter the odd ones
           const int n_out = (tl.nb * kBM + qd * 32) / 2 + (lane >> 4) * 8 + (lane & 7);
-          T* out = reinterpret_cast<T*>(a.out) + r0 * a.ldo + n_out;
-          const bool writer = (lane & 8) == 0 && n_out < a.N / 2;
+          const bool upper = lane & 8, writer = n_out < a.N / 2;
+          T* out = reinterpret_cast<T*>(a.out) + (r0 + upper) * a.ldo + n_out;
 #pragma unroll
-          for (int j = 0; j < 32; ++j) {
-            const float sv = __uint_as_float(v[j]) + bn;
-            const float u = __shfl_down_sync(0xffffffffu, sv, 8);
-            const float y = 0.7978845608028654f * (sv + 0.044715f * sv * sv * sv);
-            if (writer && j < lim) out[(int64_t)j * a.ldo] = from_float<T>(sv / (1.0f + __expf(-2.0f * y)) * u);
+          for (int j = 0; j < 32; j += 2) {
+            const float s0 = __uint_as_float(v[j]) + bn, s1 = __uint_as_float(v[j + 1]) + bn;
+            const float got = __shfl_xor_sync(0xffffffffu, upper ? s0 : s1, 8);
+            const float gv = upper ? got : s0, uv = upper ? s1 : got;
+            const float y = 0.7978845608028654f * (gv + 0.044715f * gv * gv * gv);
+            if (writer && j + upper < lim)
+              out[(int64_t)j * a.ldo] = from_float<T>(__fdividef(gv, 1.0f + __expf(-2.0f * y)) * uv);
           }
         } else if (a.act == 2) {
           // lanes 0..15 hold gate rows, lanes 16..31 the matching up rows

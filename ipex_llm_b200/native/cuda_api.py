@@ -100,11 +100,11 @@ _STREAM = {
     "ipex_kv_attn": [vp, vp, vp, i64, vp, i64, cf, vp, i64, i64, vp, i64, i64, vp, i64, vp, vp, vp, ci, ci, ci, ci, ci, ci,
                      ci, ci, ci, cf, ci, ci, vp],
     "ipex_delta_chunks_ok": [ci, ci],
-    "ipex_delta_slices": [ci],
+    "ipex_delta_fused_ok": [ci],
     "ipex_delta_step": [vp, i64, ci, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, ci, vp, cf, vp, i64, vp, ci, ci, ci, ci, ci,
                         ci, ci, vp],
     "ipex_delta_chunks": [vp, i64, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, ci, vp, vp, ci, ci, vp, vp, ci, ci, ci, ci,
-                          ci, ci, vp],
+                          ci, ci, vp, vp],
     "ipex_delta_tail": [vp, i64, vp, vp, vp, vp, vp, ci, ci, ci, ci, vp],
     "ipex_gated_norm": [vp, vp, i64, vp, vp, i64, ci, ci, ci, cf, ci, vp],
 }

@@ -11,6 +11,7 @@ import torch
 
 from ..native import cuda_api as api
 from ..native.lib import current_stream, ptr, stream_lib
+from .cuda_ops import error_flag
 from .stream import _dt
 
 SCRATCH_BYTES = 256 << 20        # of the chunked form; longer prompts run in several passes
@@ -60,7 +61,7 @@ def delta_mix(spec: DeltaSpec, w: DeltaWeights, proj, gates, slot, pos, cache, l
     common = (ptr(gates), ptr(w.conv), ptr(w.a_log), ptr(w.dt_bias), ptr(layer._v), ptr(layer._k), ptr(slot), ptr(pos),
               ptr(cache.start))
     gate_at = spec.channels
-    if portions is None and lib.ipex_delta_slices(spec.vdim) <= 8:
+    if portions is None and lib.ipex_delta_fused_ok(spec.vdim):
         api.check(lib.ipex_delta_step(ptr(proj), proj.stride(0), gate_at, *common, None, None, T, ptr(w.norm), w.eps,
                                       ptr(out), out.stride(0), None, *sizes, int(pdl), st), "delta_step")
         return out
@@ -79,7 +80,8 @@ def delta_mix(spec: DeltaSpec, w: DeltaWeights, proj, gates, slot, pos, cache, l
             for c in range(0, portions.chunks, most):
                 api.check(lib.ipex_delta_chunks(ptr(proj), proj.stride(0), *common, ptr(row), ptr(ln), n,
                                                 ptr(portions.chunk_seq), ptr(portions.seq_chunk), c,
-                                                min(portions.chunks, c + most), ptr(scratch), ptr(raw), *sizes, st),
+                                                min(portions.chunks, c + most), ptr(scratch), ptr(raw), *sizes,
+                                                ptr(error_flag(dev)), st),
                           "delta_chunks")
         else:
             api.check(lib.ipex_delta_step(ptr(proj), proj.stride(0), gate_at, *common, ptr(row), ptr(ln), n, None, 0.0, None,

@@ -65,8 +65,12 @@ def gemm_ok(x, w) -> bool:
         x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0
 
 
-def _tile(rows: float) -> int:
-    return 32 if rows <= 32 else 64 if rows <= 64 else 128 if rows <= 128 else 256
+def _tile(rows: float, cols: int = 1 << 20) -> int:
+    """Token tile of the tcgen05 GEMM: no wider than the rows, and narrower where few columns leave most SMs idle."""
+    bt = 32 if rows <= 32 else 64 if rows <= 64 else 128 if rows <= 128 else 256
+    while bt > 32 and -(-rows // bt) * -(-cols // 128) < 48:
+        bt //= 2
+    return bt
 
 
 def gemm(x, w, out, mode: int, act: int = 0, bias=None, interleaved=True):
@@ -75,7 +79,7 @@ def gemm(x, w, out, mode: int, act: int = 0, bias=None, interleaved=True):
     M, (N, K) = x.shape[0], w.shape
     if gemm_ok(x, w) and not (act == ACT_GELU_GLU and not interleaved):
         rc = stream_lib().ipex_gemm_stream(ptr(x), x.stride(0), ptr(w), w.stride(0), ptr(out), out.stride(0), ptr(bias),
-                                           None, None, 1, M, N, K, mode, act, 0.0, 0.0, _tile(M), _dt(w),
+                                           None, None, 1, M, N, K, mode, act, 0.0, 0.0, _tile(M, N), _dt(w),
                                            ptr(error_flag(x.device)), current_stream())
         if rc == -1:
             raise RuntimeError("ipex_llm_b200: the driver's tensor-map encoder rejected the GEMM operands")
