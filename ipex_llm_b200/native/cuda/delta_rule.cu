@@ -33,7 +33,7 @@ namespace {
 namespace cg = cooperative_groups;
 
 constexpr int kThreads = 256;
-constexpr int kChunkThreads = 512;    // of the sequential half
+constexpr int kChunkThreads = 256;    // of the sequential half
 constexpr int kC = 32;                // tokens per chunk
 constexpr int kVS = 32;               // state columns per CTA of the chunked form
 
@@ -421,7 +421,7 @@ __device__ __forceinline__ void conv_block(const Common& a, int c, int t0, int r
 }
 
 template <typename T, int TP>
-__global__ void __launch_bounds__(kThreads, 2) delta_prep_kernel(ChunkArgs s) {
+__global__ void __launch_bounds__(kThreads, 3) delta_prep_kernel(ChunkArgs s) {
   extern __shared__ __align__(16) float sm[];
   const Common& a = s.c;
   const int D = a.dim, V = a.vdim, h = blockIdx.y, chunk = s.c0 + blockIdx.x;
@@ -640,6 +640,7 @@ __device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t b
 
 template <int MT>
 __global__ void __launch_bounds__(kChunkThreads, 1) delta_chunks_kernel(ChunkArgs s, int stages) {
+  constexpr int NW = kChunkThreads / 32, N1 = 16 / NW, N2 = 32 / NW;   // column tiles per warp: of [W; Q] S, of the state
   extern __shared__ __align__(16) float sm[];
   __shared__ __align__(8) uint64_t full[2];
   __shared__ int abort_word;
@@ -681,14 +682,14 @@ __global__ void __launch_bounds__(kChunkThreads, 1) delta_chunks_kernel(ChunkArg
     tc5::fence_barrier_init();
     for (int i = 0; i < stages; ++i) fetch(ca + i);
   }
-  // ---- state: accumulator fragments of the row tiles warp / 2, warp / 2 + 8, ... (MT of them), two column tiles each
-  const int wm = warp >> 1, wn = (warp & 1) * 2;
-  float S[MT][2][4];
+  // ---- state: accumulator fragments of MT row tiles (eight apart), N2 column tiles each
+  const int wm = warp / (4 / N2), wn = warp % (4 / N2) * N2;
+  float S[MT][N2][4];
   const bool fresh = ca == first && p0 <= start;
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
-    for (int n = 0; n < 2; ++n)
+    for (int n = 0; n < N2; ++n)
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int d = (wm + 8 * m) * 16 + g + 8 * (i >> 1), c = (wn + n) * 8 + 2 * t4 + (i & 1);
@@ -696,7 +697,7 @@ __global__ void __launch_bounds__(kChunkThreads, 1) delta_chunks_kernel(ChunkArg
         if (d < Dm) sS[d * ldu + c] = S[m][n][i];
       }
 
-  const int mt = warp >> 2, nt = (warp & 3) * 8;       // row tile of [W; Q], first column
+  const int mt = warp / (4 / N1), nt = warp % (4 / N1) * N1;           // row tile of [W; Q], first column tile
   bool ok = true;
   for (int c = ca; c < cb; ++c) {
     __syncthreads();                                   // the state is in place (and, first, the barriers)
@@ -706,54 +707,63 @@ __global__ void __launch_bounds__(kChunkThreads, 1) delta_chunks_kernel(ChunkArg
       break;
     }
     const View v = view(c - ca);
-    Acc acc;
-    acc.zero();
+    Acc acc[N1];
+#pragma unroll
+    for (int n = 0; n < N1; ++n) acc[n].zero();
     {
       const float* left = mt < 2 ? v.w + mt * 16 * ldw : v.q + (mt - 2) * 16 * ldw;
 #pragma unroll 4
       for (int k0 = 0; k0 < Dp; k0 += 8) {
-        acc.mac(frag_a([&](int r, int k) { return left[r * ldw + k0 + k]; }, g, t4),
-                frag_b([&](int k, int j) { return sS[(k0 + k) * ldu + nt + j]; }, g, t4));
+        const FragA fa = frag_a([&](int r, int k) { return left[r * ldw + k0 + k]; }, g, t4);
+#pragma unroll
+        for (int n = 0; n < N1; ++n)
+          acc[n].mac(fa, frag_b([&](int k, int j) { return sS[(k0 + k) * ldu + (nt + n) * 8 + j]; }, g, t4));
       }
     }
     if (mt < 2) {
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int t = mt * 16 + g + 8 * (i >> 1), col = nt + 2 * t4 + (i & 1);
-        sU[t * ldu + col] = v.ub[t * ldu + col] - acc.get(i);
-      }
+      for (int n = 0; n < N1; ++n)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int t = mt * 16 + g + 8 * (i >> 1), col = (nt + n) * 8 + 2 * t4 + (i & 1);
+          sU[t * ldu + col] = v.ub[t * ldu + col] - acc[n].get(i);
+        }
     }
     __syncthreads();                                   // U is complete, the old state is read
     if (mt >= 2) {
 #pragma unroll
       for (int k0 = 0; k0 < kC; k0 += 8) {
-        acc.mac(frag_a([&](int r, int k) { return v.p[((mt - 2) * 16 + r) * L.ldp + k0 + k]; }, g, t4),
-                frag_b([&](int k, int j) { return sU[(k0 + k) * ldu + nt + j]; }, g, t4));
+        const FragA fa = frag_a([&](int r, int k) { return v.p[((mt - 2) * 16 + r) * L.ldp + k0 + k]; }, g, t4);
+#pragma unroll
+        for (int n = 0; n < N1; ++n)
+          acc[n].mac(fa, frag_b([&](int k, int j) { return sU[(k0 + k) * ldu + (nt + n) * 8 + j]; }, g, t4));
       }
       const int off = (c - first) * kC;
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int t = off + (mt - 2) * 16 + g + 8 * (i >> 1), col = nt + 2 * t4 + (i & 1);
-        if (t < len && col < nv) s.raw[((int64_t)(row0 + t) * a.heads + h) * V + v0 + col] = acc.get(i);
-      }
+      for (int n = 0; n < N1; ++n)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const int t = off + (mt - 2) * 16 + g + 8 * (i >> 1), col = (nt + n) * 8 + 2 * t4 + (i & 1);
+          if (t < len && col < nv) s.raw[((int64_t)(row0 + t) * a.heads + h) * V + v0 + col] = acc[n].get(i);
+        }
     }
     const float gc = *v.gc;
 #pragma unroll
     for (int m = 0; m < MT; ++m) {
       const int d0 = (wm + 8 * m) * 16;
       if (d0 < Dm) {
-        Acc up[2];
-        up[0].zero();
-        up[1].zero();
+        Acc up[N2];
+#pragma unroll
+        for (int n = 0; n < N2; ++n) up[n].zero();
 #pragma unroll
         for (int k0 = 0; k0 < kC; k0 += 8) {
           const FragA fa = frag_a([&](int r, int k) { return d0 + r < Dp ? v.k[(k0 + k) * ldk + d0 + r] : 0.f; }, g, t4);
 #pragma unroll
-          for (int n = 0; n < 2; ++n)
+          for (int n = 0; n < N2; ++n)
             up[n].mac(fa, frag_b([&](int k, int j) { return sU[(k0 + k) * ldu + (wn + n) * 8 + j]; }, g, t4));
         }
 #pragma unroll
-        for (int n = 0; n < 2; ++n)
+        for (int n = 0; n < N2; ++n)
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
             S[m][n][i] = fmaf(gc, S[m][n][i], up[n].get(i));
@@ -775,7 +785,7 @@ __global__ void __launch_bounds__(kChunkThreads, 1) delta_chunks_kernel(ChunkArg
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
-    for (int n = 0; n < 2; ++n)
+    for (int n = 0; n < N2; ++n)
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int d = (wm + 8 * m) * 16 + g + 8 * (i >> 1), c = (wn + n) * 8 + 2 * t4 + (i & 1);
@@ -890,14 +900,17 @@ cudaError_t launch_step(const StepArgs& s, int seqs, bool fused, bool pdl, cudaS
   return cudaLaunchKernelEx(&cfg, delta_step_kernel<T, NR, CV>, s);
 }
 
-// Columns per lane: as many as V divides into and the registers of NR rows leave room for.
+// Columns per lane: as many as V divides into and the registers of NR rows leave room for, fewer while that spreads the
+// states of a few sequences over more SMs.
 template <typename T, int NR>
 cudaError_t pick_cols(const StepArgs& s, int seqs, bool fused, bool pdl, cudaStream_t st) {
   const int V = s.c.vdim;
+  int cv = NR <= 16 && V % 4 == 0 && V > 64 ? 4 : NR <= 32 && V % 2 == 0 && V > 32 ? 2 : 1;
+  while (cv > 1 && (int64_t)s.c.heads * seqs * ((V + 16 * cv - 1) / (16 * cv)) <= 2 * 148) cv /= 2;
   if constexpr (NR <= 16)
-    if (V % 4 == 0 && V > 64) return launch_step<T, NR, 4>(s, seqs, fused, pdl, st);
+    if (cv == 4) return launch_step<T, NR, 4>(s, seqs, fused, pdl, st);
   if constexpr (NR <= 32)
-    if (V % 2 == 0 && V > 32) return launch_step<T, NR, 2>(s, seqs, fused, pdl, st);
+    if (cv == 2) return launch_step<T, NR, 2>(s, seqs, fused, pdl, st);
   return launch_step<T, NR, 1>(s, seqs, fused, pdl, st);
 }
 
