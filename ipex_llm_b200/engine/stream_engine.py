@@ -109,7 +109,8 @@ class StreamStack:
 
     def _linear(self, P: _Proj, h, out, mode, act=0, pdl=False, interleaved=True, w2=None, out2=None):
         """``act(h @ w.T + bias)`` into ``out`` (see ``OUT_*``); ``w2`` / ``out2``: further dense rows with fp32 results."""
-        if self._few(P, h.shape[0]):
+        # (the tensor-core row product, which takes up to sixteen rows, wants gate and up rows in blocks)
+        if self._few(P, h.shape[0]) and (interleaved or h.shape[0] <= 8):
             return K.gemv_rows(P.w, h, out, mode, act=act, pdl=pdl, bias=P.bias, w2=w2, out2=out2, interleaved=interleaved)
         if w2 is not None:
             if h.shape[0] <= K.rows_max(w2.shape[1], self.dtype):

@@ -872,7 +872,7 @@ cudaError_t launch_step(const StepArgs& s, int seqs, bool fused, bool pdl, cudaS
   if (fused && slices > 8) return cudaErrorInvalidValue;
   const size_t smem = ((2 + s.c.taps) * (2 * (size_t)s.c.dim + 32 * CV) + 2 * 2 * 8 * 32 * CV) * sizeof(float);
   if (smem > kSmemMax) return cudaErrorInvalidValue;
-  if (smem > 48 * 1024) {
+  if (smem > 40 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(delta_step_kernel<T, NR, CV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;
   }

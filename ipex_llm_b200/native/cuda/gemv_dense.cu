@@ -427,7 +427,7 @@ template <typename T, int M, int R, bool GLU = false>
 cudaError_t launch_gemv(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
   auto kern = gemv_rows_kernel<T, M, R, GLU>;
   const size_t smem = (size_t)M * a.kp * sizeof(T);      // rows past a.M are read (and dropped), never used
-  if (smem > 48 * 1024) {
+  if (smem > 40 * 1024) {                 // (static shared memory counts against the default limit too)
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;
   }
@@ -452,7 +452,7 @@ cudaError_t launch_gemv_mma(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
   a.kp = (a.K + 31) / 32 * 32 + 32;        // 64 bytes of skew between rows: neighbouring tokens in different banks
   const size_t smem = (size_t)2 * kWarps * NT * 128 * sizeof(float) + (a.norm_w != nullptr ? (size_t)a.M * a.kp * sizeof(T) : 0);
   if (smem > 226 * 1024) return cudaErrorInvalidValue;
-  if (smem > 48 * 1024) {
+  if (smem > 40 * 1024) {                 // (static shared memory counts against the default limit too)
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;
   }
@@ -640,7 +640,7 @@ int vec_ok(const void* p, int64_t ld, int K) {
 
 template <typename K>
 cudaError_t allow_smem(K kern, size_t smem) {
-  if (smem <= 48 * 1024) return cudaSuccess;
+  if (smem <= 40 * 1024) return cudaSuccess;      // static shared memory counts against the default limit too
   if (smem > 226 * 1024) return cudaErrorInvalidValue;
   return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
 }

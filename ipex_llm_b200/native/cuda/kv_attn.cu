@@ -381,7 +381,7 @@ cudaError_t launch_attn(const AttnArgs& a, int tokens, int nsplit, bool pdl, cud
   const size_t smem = ((size_t)RT * (dimp + kTile + 3 + vp) + (size_t)subsets * RT * a.vdim + 4) * sizeof(float);
   if (smem > 220 * 1024 || (int64_t)a.kv_heads * nrb > 65535) return cudaErrorInvalidValue;
   auto kern = kv_attn_kernel<T, RT, VEC>;
-  if (smem > 48 * 1024) {
+  if (smem > 40 * 1024) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;
   }
@@ -437,7 +437,7 @@ IPEX_API int ipex_kv_append(const void* k, const void* v, int64_t ld, const void
     const size_t smem = vt != nullptr ? (size_t)64 * (vdim + 2) * sizeof(T) : 0;
     if (smem > 220 * 1024) return cudaErrorInvalidValue;
     auto kern = kv_append_kernel<T>;
-    if (smem > 48 * 1024) {
+    if (smem > 40 * 1024) {
       cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
       if (e != cudaSuccess) return e;
     }

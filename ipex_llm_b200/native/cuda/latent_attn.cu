@@ -599,7 +599,7 @@ __global__ void __launch_bounds__(kUvThreads) latent_uv_kernel(UvArgs a) {
 
 template <typename K>
 cudaError_t allow_smem(K kern, size_t smem) {
-  if (smem <= 48 * 1024) return cudaSuccess;
+  if (smem <= 40 * 1024) return cudaSuccess;      // static shared memory counts against the default limit too
   if (smem > 226 * 1024) return cudaErrorInvalidValue;
   return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
 }

@@ -66,7 +66,7 @@ def test_gated_unit_with_biases(dtype, M, ff, K):
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
-@pytest.mark.parametrize("M,N,K,N2", [(1, 97, 136, 5), (3, 40, 60, 12), (11, 2500, 520, 64), (2, 33, 7, 1), (40, 120, 64, 6),
+@pytest.mark.parametrize("M,N,K,N2", [(1, 97, 136, 5), (3, 40, 60, 12), (11, 2500, 520, 64), (2, 33, 7, 1), (7, 136, 1536, 4), (40, 120, 64, 6),
                                       (9, 64, 30, 10)])
 def test_bias_and_second_matrix(dtype, M, N, K, N2):
     from ipex_llm_b200.ops import stream as S
@@ -479,7 +479,13 @@ def cfg_delta():
             "layers": [O.delta_layer(2, 2, 32, 32, conv=4, ff=128), O.delta_layer(4, 2, 16, 32, conv=4)]}
 
 
-CFGS = {"a": cfg_a, "odd": cfg_odd, "attention": cfg_attention, "delta": cfg_delta}
+def cfg_ff20():
+    """A hidden size that is no multiple of eight in a model whose other sizes are."""
+    return {"architecture": "Letarax", "vocab": 90, "width": 64, "norm": {"eps": 1e-6},
+            "layers": [O.attention_layer(2, 1, 16, 32, window=30, ff=20), O.delta_layer(2, 1, 16, 32, conv=4, ff=20)]}
+
+
+CFGS = {"a": cfg_a, "odd": cfg_odd, "attention": cfg_attention, "delta": cfg_delta, "ff 20": cfg_ff20}
 _models, _want = {}, {}
 
 
@@ -601,12 +607,13 @@ def test_mixed_portions_in_one_batch(dtype):
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
-def test_many_sequences_decode_through_the_gemms(dtype):
-    """More rows than the row products take: GEMMs in the decode graph."""
-    model, cfg, _ = make("a", dtype)
-    seqs = [tokens(20 + 3 * i, cfg["vocab"], 80 + i) for i in range(19)]
-    want = [oracle("a", s) for s in seqs]
-    eng = engine(model, 19)
+@pytest.mark.parametrize("name,count", [("a", 19), ("a", 12), ("odd", 11), ("ff 20", 12)])
+def test_many_sequences_decode_together(name, count, dtype):
+    """More rows than the small row products take, then more than any of them does: GEMMs in the decode graph."""
+    model, cfg, _ = make(name, dtype)
+    seqs = [tokens(20 + 3 * i, cfg["vocab"], 80 + i) for i in range(count)]
+    want = [oracle(name, s) for s in seqs]
+    eng = engine(model, count)
     slots = [eng.cache.acquire() for _ in seqs]
     eng.step_rows([(sl, s[:-4], []) for sl, s in zip(slots, seqs)])
     for k in range(4, 0, -1):
