@@ -26,6 +26,8 @@ def _one_plus(norm):
 
 
 class HybridStack(StreamStack):
+    components = ("stream", "hybrid")
+
     def __init__(self, model):
         base = model.model
         super().__init__(model, [blk.mixer.in_proj for blk in base.layers])

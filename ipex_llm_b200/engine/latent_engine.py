@@ -23,6 +23,7 @@ from .stream_engine import Portions, StreamEngine, StreamStack, _Layer, _Proj
 
 class LatentStack(StreamStack):
     cache_cls = LatentCache
+    components = ("stream", "latent")
 
     def __init__(self, model):
         cfg, base = model.config, model.model

@@ -13,6 +13,7 @@ from typing import List, Optional, Sequence, Tuple
 
 import torch
 
+from ..native.lib import prepare_components
 from ..ops import cuda_ops, stream as K
 from ..ops.kv_cache import SlotCache
 from ..ops.linear import LowBitLinear
@@ -60,6 +61,7 @@ def stack_for(model, cls) -> "StreamStack":
 
 class StreamStack:
     cache_cls = SlotCache
+    components = ("stream",)         # parts of the kernel library the family needs (native/build.py)
     softcap = 0.0
     kernel_launches_per_step = 0
 
@@ -69,6 +71,7 @@ class StreamStack:
         self.device = next(model.parameters()).device
         if self.device.type != "cuda":
             raise RuntimeError(f"{type(model).__name__} runs on CUDA only: call model.to('cuda')")
+        prepare_components(*self.components)
         self.config = cfg
         self.dtype = dt = self._dtype([*linears, model.lm_head])
         self.eps = float(cfg.norm["eps"])
@@ -112,6 +115,8 @@ class StreamStack:
         # (the tensor-core row product, which takes up to sixteen rows, wants gate and up rows in blocks)
         if self._few(P, h.shape[0]) and (interleaved or h.shape[0] <= 8):
             return K.gemv_rows(P.w, h, out, mode, act=act, pdl=pdl, bias=P.bias, w2=w2, out2=out2, interleaved=interleaved)
+        if w2 is not None and P.packed is None:
+            return K.gemm(h, P.w, out, mode, act, P.bias, interleaved, w2, out2)
         if w2 is not None:
             if h.shape[0] <= K.rows_max(w2.shape[1], self.dtype):
                 K.gemv_rows(w2, h, out2, K.OUT_F32)

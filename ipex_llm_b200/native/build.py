@@ -36,8 +36,10 @@ CUDA_LIB = os.path.join(HERE, "libipex_llm_cuda.so")
 # Parts of the kernel library that stand on their own.  A process that needs one of them and finds no complete library
 # compiles just these sources (seconds instead of minutes); ``build_cuda`` always builds everything.
 COMPONENTS = {
-    "stream": ("delta_rule.cu", "elementwise.cu", "gemm_stream_tcgen05.cu", "gemv_dense.cu", "kv_attn.cu",
-               "latent_attn.cu", "latent_prefill_tcgen05.cu", "stream_ops.cu"),
+    # what decoders with a 32-bit residual stream share, and what only some of them need
+    "stream": ("elementwise.cu", "gemm_stream_tcgen05.cu", "gemv_dense.cu", "packed_prefill_tcgen05.cu", "stream_ops.cu"),
+    "latent": ("latent_attn.cu",),
+    "hybrid": ("delta_rule.cu", "kv_attn.cu"),
 }
 
 NVCC_ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]
@@ -126,6 +128,12 @@ def component_lib(name: str) -> str:
 def build_component(name: str, force=False, verbose=False):
     """The library of one entry of ``COMPONENTS``."""
     return _build_cuda([os.path.join(CUDA_DIR, f) for f in COMPONENTS[name]], component_lib(name), force, verbose)
+
+
+def build_components(names):
+    """Several of them at once (their sources compile side by side)."""
+    with ThreadPoolExecutor(max_workers=len(names)) as ex:
+        return list(ex.map(build_component, names))
 
 
 def build_cuda(force=False, verbose=False):

@@ -5,6 +5,8 @@
 //     y = glu(row_scale * (x . W_gu^T))                    gate / up rows interleaved in 16-row tiles, N / 2 columns
 //     y = gelu_tanh(gate) * up, with biases                gate / up rows interleaved in 8-row tiles, N / 2 columns
 //
+// A second matrix (w2) may ride along: its rows multiply the same x and leave as fp32 in an output of their own.
+//
 // With `ranges` the launch covers a whole bank of weight matrices: group e multiplies its rows
 // [ranges[e][0], + ranges[e][1]) of x, read from DEVICE memory, so one launch serves all experts of a prompt and the
 // host never learns the routing.  The tile list is laid out over the groups at kernel start.
@@ -31,6 +33,9 @@ struct Args {
   int out_mode, act;        // act 1: squared relu (out_mode 0); 2: clamped gated unit; 3: gelu-gated unit
   float limit, alpha;
   const void* bias;         // T [N] or null
+  float* out2;              // fp32 [M, ldo2], results of the second matrix's N2 rows (0: there is none)
+  int64_t ldo2;
+  int N2;
 };
 
 template <int BT>
@@ -52,13 +57,15 @@ template <int BT>
 struct Walker {
   const Args& a;
   const int* first;     // shared: first tile of every group, [groups + 1]
-  int n_tiles;
+  int n_tiles;          // of the first matrix, then of both
+  int all_tiles;
   int e = 0;
-  __device__ Walker(const Args& args, const int* f) : a(args), first(f), n_tiles((args.N + kBM - 1) / kBM) {}
+  __device__ Walker(const Args& args, const int* f)
+      : a(args), first(f), n_tiles((args.N + kBM - 1) / kBM), all_tiles(n_tiles + (args.N2 + kBM - 1) / kBM) {}
   __device__ __forceinline__ bool get(int t, Tile& o) {
     if (a.ranges == nullptr) {
       const int mt = (a.M + BT - 1) / BT;
-      if (t >= mt * n_tiles) return false;
+      if (t >= mt * all_tiles) return false;
       o = {0, t / mt, t % mt, 0, a.M};
       return true;
     }
@@ -72,7 +79,8 @@ struct Walker {
 
 template <typename T, int BT>
 __global__ void __launch_bounds__(kThreads, 1)
-gemm_stream_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ CUtensorMap tm_x, Args a) {
+gemm_stream_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ CUtensorMap tm_w2,
+                   const __grid_constant__ CUtensorMap tm_x, Args a) {
   using C = Cfg<BT>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -129,16 +137,19 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
   if (warp == 0) {
     if (lane == 0) {
       prefetch_tmap(&tm_w);
+      if (a.N2 > 0) prefetch_tmap(&tm_w2);
       prefetch_tmap(&tm_x);
       int s = 0;
       uint32_t ph = 0;
       bool ok = true;
       for (int t = blockIdx.x; ok && walk.get(t, tl); t += gridDim.x) {
-        const int wrow = tl.e * a.N + tl.nb * kBM, xrow = tl.row0 + tl.mb * BT;
+        const bool second = tl.nb >= walk.n_tiles;
+        const CUtensorMap* tm = second ? &tm_w2 : &tm_w;
+        const int wrow = second ? (tl.nb - walk.n_tiles) * kBM : tl.e * a.N + tl.nb * kBM, xrow = tl.row0 + tl.mb * BT;
         for (int kb = 0; kb < kblocks; ++kb) {
           if (!mbar_wait(&empty[s], ph ^ 1, abort_flag)) { ok = false; report(a.err, 37); break; }
           mbar_expect_tx(&full[s], C::kStageBytes);
-          tma_load_2d(sA + s * C::kABytes, &tm_w, kb * kBK, wrow, &full[s]);
+          tma_load_2d(sA + s * C::kABytes, tm, kb * kBK, wrow, &full[s]);
           tma_load_2d(sB + s * C::kBBytes, &tm_x, kb * kBK, xrow, &full[s]);
           if (++s == C::kStages) { s = 0; ph ^= 1; }
         }
@@ -182,7 +193,8 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
         break;
       }
       tcgen05_fence_after();
-      const int n = tl.nb * kBM + qd * 32 + lane;
+      const bool second = tl.nb >= walk.n_tiles;
+      const int n = (second ? tl.nb - walk.n_tiles : tl.nb) * kBM + qd * 32 + lane;
       const int rows = tl.rows - tl.mb * BT;                  // rows of this tile that exist
       const int64_t xrow = tl.row0 + tl.mb * BT;
 #pragma unroll 1
@@ -191,6 +203,15 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
         tmem_ld_32x32(tmem_base + (uint32_t(qd * 32) << 16) + acc * BT + c * 32, v);
         const int lim = min(32, rows - c * 32);
         const int64_t r0 = xrow + c * 32;
+        if (second) {
+          if (n < a.N2) {
+            float* out = a.out2 + r0 * a.ldo2 + n;
+#pragma unroll
+            for (int j = 0; j < 32; ++j)
+              if (j < lim) out[(int64_t)j * a.ldo2] = __uint_as_float(v[j]);
+          }
+          continue;
+        }
         const float bn = a.bias != nullptr && n < a.N ? to_float<T>(reinterpret_cast<const T*>(a.bias)[n]) : 0.f;
         if (a.act == 3) {
           // lanes with bit 3 clear hold gate rows, the lanes eight above them the matching up rows: the former finish
@@ -268,32 +289,35 @@ int sm_count() {
 }
 
 template <typename T, int BT>
-int launch(const void* x, int64_t ldx, int x_rows, const void* w, int64_t ldw, const Args& a, cudaStream_t st) {
+int launch(const void* x, int64_t ldx, int x_rows, const void* w, int64_t ldw, const void* w2, const Args& a,
+           cudaStream_t st) {
   const CUtensorMapDataType dt =
       std::is_same<T, __half>::value ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
-  CUtensorMap tw, tx;
+  CUtensorMap tw, tw2, tx;
   if (!encode_2d_sw128(&tw, dt, w, (uint64_t)a.K, (uint64_t)a.N * a.groups, (uint64_t)ldw * 2, kBK, kBM)) return -1;
   if (!encode_2d_sw128(&tx, dt, x, (uint64_t)a.K, (uint64_t)x_rows, (uint64_t)ldx * 2, kBK, BT)) return -1;
+  tw2 = tw;
+  if (a.N2 > 0 && !encode_2d_sw128(&tw2, dt, w2, (uint64_t)a.K, (uint64_t)a.N2, (uint64_t)ldw * 2, kBK, kBM)) return -1;
   auto kern = gemm_stream_kernel<T, BT>;
   const int smem = Cfg<BT>::kSmemBytes + (a.ranges != nullptr ? (a.groups + 1) * 4 : 0);
   if (smem > 227 * 1024) return (int)cudaErrorInvalidValue;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
   if (e != cudaSuccess) return (int)e;
   const int64_t mt = (a.M + BT - 1) / BT + (a.ranges != nullptr ? a.groups : 0);    // upper bound of the tile count
-  const int64_t tiles = mt * ((a.N + kBM - 1) / kBM);
+  const int64_t tiles = mt * ((a.N + kBM - 1) / kBM + (a.N2 + kBM - 1) / kBM);
   const int sms = sm_count();
-  kern<<<tiles < sms ? (int)tiles : sms, kThreads, smem, st>>>(tw, tx, a);
+  kern<<<tiles < sms ? (int)tiles : sms, kThreads, smem, st>>>(tw, tw2, tx, a);
   return (int)cudaGetLastError();
 }
 
 template <typename T>
-int dispatch(int bt, const void* x, int64_t ldx, int x_rows, const void* w, int64_t ldw, const Args& a,
+int dispatch(int bt, const void* x, int64_t ldx, int x_rows, const void* w, int64_t ldw, const void* w2, const Args& a,
              cudaStream_t st) {
   switch (bt) {
-    case 32: return launch<T, 32>(x, ldx, x_rows, w, ldw, a, st);
-    case 64: return launch<T, 64>(x, ldx, x_rows, w, ldw, a, st);
-    case 128: return launch<T, 128>(x, ldx, x_rows, w, ldw, a, st);
-    case 256: return launch<T, 256>(x, ldx, x_rows, w, ldw, a, st);
+    case 32: return launch<T, 32>(x, ldx, x_rows, w, ldw, w2, a, st);
+    case 64: return launch<T, 64>(x, ldx, x_rows, w, ldw, w2, a, st);
+    case 128: return launch<T, 128>(x, ldx, x_rows, w, ldw, w2, a, st);
+    case 256: return launch<T, 256>(x, ldx, x_rows, w, ldw, w2, a, st);
     default: return (int)cudaErrorInvalidValue;
   }
 }
@@ -303,10 +327,11 @@ int dispatch(int bt, const void* x, int64_t ldx, int x_rows, const void* w, int6
 // See the head of this file.  M: rows of x; with `ranges` the groups' rows partition them.  w: [groups * N, K].  bt:
 // token tile (32 / 64 / 128 / 256).  row_scale only with act 2 (then out_mode 0 and N a multiple of 32).  act 3: out_mode
 // 0, N a multiple of 16.  bias (may be null) has N entries of the operands' type; not with act 2 or ranges.
+// w2 / out2 (N2 = 0: none): N2 more rows of the same row stride, results in fp32; not with ranges or act 2.
 // Strides of x and w multiples of 8 elements, bases 16-byte aligned.  Returns a cudaError_t, or -1 when the
 // tensor-map encoder rejects the operands.
 IPEX_API int ipex_gemm_stream(const void* x, int64_t ldx, const void* w, int64_t ldw, void* out, int64_t ldo,
-                              const void* bias, const float* row_scale, const int* ranges, int groups, int M, int N, int K, int out_mode,
+                              const void* bias, const void* w2, int N2, float* out2, int64_t ldo2, const float* row_scale, const int* ranges, int groups, int M, int N, int K, int out_mode,
                               int act, float limit, float alpha, int bt, int dtype, int* err, void* stream) {
   if (M < 1 || N < 1 || K < 1 || groups < 1 || (ldx % 8) != 0 || (ldw % 8) != 0 || out_mode < 0 || out_mode > 2)
     return (int)cudaErrorInvalidValue;
@@ -317,9 +342,13 @@ IPEX_API int ipex_gemm_stream(const void* x, int64_t ldx, const void* w, int64_t
     return (int)cudaErrorInvalidValue;
   if ((reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15)) return (int)cudaErrorInvalidValue;
   if ((int64_t)groups * N > 0x7fffffff) return (int)cudaErrorInvalidValue;
-  Args a = {out, row_scale, ranges, err, ldo, M, N, K, groups, out_mode, act, limit, alpha, bias};
+  if (N2 < 0 || (N2 > 0 && (w2 == nullptr || out2 == nullptr || ranges != nullptr || act == 2 ||
+                            (reinterpret_cast<uintptr_t>(w2) & 15))))
+    return (int)cudaErrorInvalidValue;
+  Args a = {out, row_scale, ranges, err, ldo, M, N, K, groups, out_mode, act, limit, alpha, bias,
+            out2, ldo2, N2};
   cudaStream_t st = (cudaStream_t)stream;
-  if (dtype == DT_F16) return dispatch<__half>(bt, x, ldx, M, w, ldw, a, st);
-  if (dtype == DT_BF16) return dispatch<__nv_bfloat16>(bt, x, ldx, M, w, ldw, a, st);
+  if (dtype == DT_F16) return dispatch<__half>(bt, x, ldx, M, w, ldw, w2, a, st);
+  if (dtype == DT_BF16) return dispatch<__nv_bfloat16>(bt, x, ldx, M, w, ldw, w2, a, st);
   return (int)cudaErrorInvalidValue;
 }

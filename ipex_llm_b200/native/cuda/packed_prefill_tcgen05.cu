@@ -59,7 +59,7 @@ struct Args {
 
 template <typename T, int DV>
 __global__ void __launch_bounds__(kThreads, 1)
-latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_constant__ CUtensorMap tm_qr,
+packed_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_constant__ CUtensorMap tm_qr,
                       const __grid_constant__ CUtensorMap tm_kn, const __grid_constant__ CUtensorMap tm_kr,
                       const __grid_constant__ CUtensorMap tm_vt, Args a) {
   constexpr int kVBytes = DV * kBKV * 2;
@@ -361,7 +361,7 @@ int launch(const void* q, int64_t ldq, const void* k, int64_t ldk, const void* k
   if (a.nbr > 0 && (!encode_heads(&qr, dt, qp + a.dim, a.rd, H, tokens, a.dim + a.rd, ldq) ||
                     !encode_2d_sw128(&krm, dt, kr, (uint64_t)a.rd, (uint64_t)tokens, (uint64_t)ld_kr * 2, 64, kBKV)))
     return -1;
-  auto kern = latent_prefill_kernel<T, DV>;
+  auto kern = packed_prefill_kernel<T, DV>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   dim3 grid(H, (max_len + kBQ - 1) / kBQ, B);
@@ -373,7 +373,7 @@ int launch(const void* q, int64_t ldq, const void* k, int64_t ldk, const void* k
 
 // Sizes the kernel takes: parts that keep every TMA stride a multiple of 16 bytes, at most 256 score columns in
 // 64-wide blocks, values up to 128.
-IPEX_API int ipex_latent_prefill_ok(int dim, int rd, int vd, int R, int dtype) {
+IPEX_API int ipex_packed_prefill_ok(int dim, int rd, int vd, int R, int dtype) {
   if (dtype != DT_F16 && dtype != DT_BF16) return 0;
   if (dim < 8 || rd < 0 || vd < 8 || (dim % 8) || (rd % 8) || (vd % 8) || (R % 8)) return 0;
   return (dim + 63) / 64 + (rd + 63) / 64 <= 4 && vd <= 128;
@@ -389,7 +389,7 @@ IPEX_API int ipex_packed_prefill(const void* q, int64_t ldq, const void* k, int6
                                  const void* vt, int64_t ld_vt, void* out, int64_t ldo, const int* seq_row,
                                  const int* seq_len, int B, int H, int G, int tokens, int max_len, int dim, int rd,
                                  int vd, int window, int sink, float scale, int dtype, int* err, void* stream) {
-  if (!ipex_latent_prefill_ok(dim, rd, vd, 8, dtype) || B < 1 || B > 65535 || H < 1 || tokens < 1 || max_len < 1 ||
+  if (!ipex_packed_prefill_ok(dim, rd, vd, 8, dtype) || B < 1 || B > 65535 || H < 1 || tokens < 1 || max_len < 1 ||
       window < 0 || (max_len + kBQ - 1) / kBQ > 65535 || G < 1 || H % G != 0)
     return (int)cudaErrorInvalidValue;
   if ((ldq % 8) || (ldk % 8) || (ld_vt % 8) || (ldo % 8) || (rd > 0 && (ld_kr % 8)) || ld_vt < tokens)

@@ -63,59 +63,72 @@ _OPTIONAL = {
 }
 
 
-# the "stream" component (see native/build.py): decoders with a 32-bit residual stream
-_STREAM = {
-    "ipex_argmax": _SIGS["ipex_argmax"],
-    "ipex_gemv_rows_max": [ci, ci],
-    "ipex_gemv_rows": [vp, i64, vp, i64, vp, cf, vp, vp, i64, vp, ci, vp, i64, ci, ci, ci, ci, ci, ci, cf, ci, ci, vp],
-    "ipex_moe_router_sigmoid": [vp, i64, vp, cf, vp, vp, vp, ci, ci, ci, ci, ci, ci, vp],
-    "ipex_moe_glu_rows": [vp, i64, vp, cf, vp, vp, vp, vp, ci, ci, ci, ci, ci, cf, cf, ci, ci, ci, vp],
-    "ipex_moe_down_rows": [vp, vp, vp, i64, vp, ci, ci, ci, ci, ci, ci, ci, vp],
-    "ipex_embed_stream": [vp, vp, vp, vp, vp, i64, vp, vp, vp, ci, ci, i64, cf, i64, i64, i64, ci, ci, vp],
-    "ipex_norm_stream": [vp, i64, vp, ci, vp, i64, vp, ci, ci, cf, ci, ci, vp],
-    "ipex_add_norm_stream": [vp, i64, vp, i64, vp, vp, vp, i64, ci, ci, cf, ci, ci, vp],
-    "ipex_bias_rows": [vp, i64, ci, vp, ci, ci, ci, vp],
-    "ipex_gelu_glu_rows": [vp, i64, ci, vp, vp, i64, ci, ci, ci, ci, vp],
-    "ipex_softcap_f32": [vp, i64, cf, vp],
-    "ipex_add_stream": [vp, vp, i64, ci, vp],
-    "ipex_relu2_inplace": [vp, i64, ci, vp],
-    "ipex_moe_sigmoid_topk": [vp, i64, vp, vp, ci, ci, ci, vp],
-    "ipex_moe_group_slots": [vp, ci, ci, vp, vp, vp, vp],
-    "ipex_moe_gather_slots": [vp, vp, vp, vp, vp, ci, ci, ci, ci, vp],
-    "ipex_moe_glu_from_gu": [vp, vp, vp, ci, ci, cf, cf, ci, ci, vp],
-    "ipex_moe_combine_slots": [vp, vp, vp, ci, ci, ci, ci, vp],
-    "ipex_gemm_plain": [vp, vp, vp, vp, ci, ci, ci, ci, ci, ci, vp],
-    "ipex_gemm_stream": [vp, i64, vp, i64, vp, i64, vp, vp, vp, ci, ci, ci, ci, ci, ci, cf, cf, ci, ci, vp, vp],
-    "ipex_latent_prep": [vp, i64, vp, cf, vp, vp, vp, vp, vp, vp, vp, i64, i64, vp, ci, ci, ci, ci, ci, ci, ci, ci, vp],
-    "ipex_latent_prompt_prep": [vp, i64, vp, cf, vp, vp, vp, vp, vp, vp, i64, i64, vp, i64, vp, i64, ci, ci, ci, ci,
-                                ci, ci, ci, ci, vp],
-    "ipex_latent_row": [ci, ci, ci],
-    "ipex_latent_attn_fast": [ci, ci, ci],
-    "ipex_latent_attn": [vp, vp, i64, vp, i64, i64, vp, vp, vp, vp, vp, ci, ci, ci, ci, ci, ci, ci, cf, ci, ci, ci, vp],
-    "ipex_latent_uv": [vp, vp, vp, vp, i64, ci, ci, ci, ci, ci, ci, ci, vp],
-    "ipex_latent_prefill_ok": [ci, ci, ci, ci, ci],
-    "ipex_packed_prefill": [vp, i64, vp, i64, vp, i64, vp, i64, vp, i64, vp, vp, ci, ci, ci, ci, ci, ci, ci, ci, ci, ci, cf,
-                            ci, vp, vp],
-    "ipex_kv_append": [vp, vp, i64, vp, i64, cf, vp, i64, i64, vp, i64, i64, vp, i64, vp, vp, ci, ci, ci, ci, ci, ci, vp],
-    "ipex_kv_attn": [vp, vp, vp, i64, vp, i64, cf, vp, i64, i64, vp, i64, i64, vp, i64, vp, vp, vp, ci, ci, ci, ci, ci, ci,
-                     ci, ci, ci, cf, ci, ci, vp],
-    "ipex_delta_chunks_ok": [ci, ci],
-    "ipex_delta_fused_ok": [ci],
-    "ipex_delta_step": [vp, i64, ci, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, ci, vp, cf, vp, i64, vp, ci, ci, ci, ci, ci,
-                        ci, ci, vp],
-    "ipex_delta_chunks": [vp, i64, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, ci, vp, vp, ci, ci, vp, vp, ci, ci, ci, ci,
-                          ci, ci, vp, vp],
-    "ipex_delta_tail": [vp, i64, vp, vp, vp, vp, vp, ci, ci, ci, ci, vp],
-    "ipex_gated_norm": [vp, vp, i64, vp, vp, i64, ci, ci, ci, cf, ci, vp],
+# the components of the decoders with a 32-bit residual stream (see native/build.py)
+COMPONENT_SIGS = {
+    "stream": {
+        "ipex_argmax": _SIGS["ipex_argmax"],
+        "ipex_gemv_rows_max": [ci, ci],
+        "ipex_gemv_rows": [vp, i64, vp, i64, vp, cf, vp, vp, i64, vp, ci, vp, i64, ci, ci, ci, ci, ci, ci, cf, ci, ci,
+                           vp],
+        "ipex_moe_router_sigmoid": [vp, i64, vp, cf, vp, vp, vp, ci, ci, ci, ci, ci, ci, vp],
+        "ipex_moe_glu_rows": [vp, i64, vp, cf, vp, vp, vp, vp, ci, ci, ci, ci, ci, cf, cf, ci, ci, ci, vp],
+        "ipex_moe_down_rows": [vp, vp, vp, i64, vp, ci, ci, ci, ci, ci, ci, ci, vp],
+        "ipex_embed_stream": [vp, vp, vp, vp, vp, i64, vp, vp, vp, ci, ci, i64, cf, i64, i64, i64, ci, ci, vp],
+        "ipex_norm_stream": [vp, i64, vp, ci, vp, i64, vp, ci, ci, cf, ci, ci, vp],
+        "ipex_add_norm_stream": [vp, i64, vp, i64, vp, vp, vp, i64, ci, ci, cf, ci, ci, vp],
+        "ipex_bias_rows": [vp, i64, ci, vp, ci, ci, ci, vp],
+        "ipex_gelu_glu_rows": [vp, i64, ci, vp, vp, i64, ci, ci, ci, ci, vp],
+        "ipex_softcap_f32": [vp, i64, cf, vp],
+        "ipex_add_stream": [vp, vp, i64, ci, vp],
+        "ipex_relu2_inplace": [vp, i64, ci, vp],
+        "ipex_moe_sigmoid_topk": [vp, i64, vp, vp, ci, ci, ci, vp],
+        "ipex_moe_group_slots": [vp, ci, ci, vp, vp, vp, vp],
+        "ipex_moe_gather_slots": [vp, vp, vp, vp, vp, ci, ci, ci, ci, vp],
+        "ipex_moe_glu_from_gu": [vp, vp, vp, ci, ci, cf, cf, ci, ci, vp],
+        "ipex_moe_combine_slots": [vp, vp, vp, ci, ci, ci, ci, vp],
+        "ipex_gemm_plain": [vp, vp, vp, vp, ci, ci, ci, ci, ci, ci, vp],
+        "ipex_gemm_stream": [vp, i64, vp, i64, vp, i64, vp, vp, ci, vp, i64, vp, vp, ci, ci, ci, ci, ci, ci, cf, cf,
+                             ci, ci, vp, vp],
+        "ipex_packed_prefill_ok": [ci, ci, ci, ci, ci],
+        "ipex_packed_prefill": [vp, i64, vp, i64, vp, i64, vp, i64, vp, i64, vp, vp, ci, ci, ci, ci, ci, ci, ci, ci,
+                                ci, ci, cf, ci, vp, vp],
+    },
+    "latent": {
+        "ipex_latent_prep": [vp, i64, vp, cf, vp, vp, vp, vp, vp, vp, vp, i64, i64, vp, ci, ci, ci, ci, ci, ci, ci, ci,
+                             vp],
+        "ipex_latent_prompt_prep": [vp, i64, vp, cf, vp, vp, vp, vp, vp, vp, i64, i64, vp, i64, vp, i64, ci, ci, ci,
+                                    ci, ci, ci, ci, ci, vp],
+        "ipex_latent_row": [ci, ci, ci],
+        "ipex_latent_attn_fast": [ci, ci, ci],
+        "ipex_latent_attn": [vp, vp, i64, vp, i64, i64, vp, vp, vp, vp, vp, ci, ci, ci, ci, ci, ci, ci, cf, ci, ci, ci,
+                             vp],
+        "ipex_latent_uv": [vp, vp, vp, vp, i64, ci, ci, ci, ci, ci, ci, ci, vp],
+    },
+    "hybrid": {
+        "ipex_kv_append": [vp, vp, i64, vp, i64, cf, vp, i64, i64, vp, i64, i64, vp, i64, vp, vp, ci, ci, ci, ci, ci,
+                           ci, vp],
+        "ipex_kv_attn": [vp, vp, vp, i64, vp, i64, cf, vp, i64, i64, vp, i64, i64, vp, i64, vp, vp, vp, ci, ci, ci, ci,
+                         ci, ci, ci, ci, ci, cf, ci, ci, vp],
+        "ipex_delta_chunks_ok": [ci, ci],
+        "ipex_delta_fused_ok": [ci],
+        "ipex_delta_step": [vp, i64, ci, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, ci, vp, cf, vp, i64, vp, ci, ci,
+                            ci, ci, ci, ci, ci, vp],
+        "ipex_delta_chunks": [vp, i64, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, ci, vp, vp, ci, ci, vp, vp, ci, ci,
+                              ci, ci, ci, ci, vp, vp],
+        "ipex_delta_tail": [vp, i64, vp, vp, vp, vp, vp, ci, ci, ci, ci, vp],
+        "ipex_gated_norm": [vp, vp, i64, vp, vp, i64, ci, ci, ci, cf, ci, vp],
+    },
 }
 
 
-def declare_stream(lib: ctypes.CDLL):
-    lib.ipex_gemv_rows_tune.argtypes, lib.ipex_gemv_rows_tune.restype = [ci], None
-    lib.ipex_delta_scratch_floats.argtypes, lib.ipex_delta_scratch_floats.restype = [ci, ci], i64
-    for name, args in _STREAM.items():
-        fn = getattr(lib, name)
+def declare_component(lib: ctypes.CDLL, name: str):
+    for fn_name, args in COMPONENT_SIGS[name].items():
+        fn = getattr(lib, fn_name)
         fn.argtypes, fn.restype = args, ci
+    if name == "stream":
+        lib.ipex_gemv_rows_tune.argtypes, lib.ipex_gemv_rows_tune.restype = [ci], None
+    if name == "hybrid":
+        lib.ipex_delta_scratch_floats.argtypes, lib.ipex_delta_scratch_floats.restype = [ci, ci], i64
 
 
 def declare(lib: ctypes.CDLL):

@@ -19,7 +19,7 @@ from . import build as _build
 _lock = threading.Lock()
 _host = None
 _cuda = None
-_stream = None
+_components = {}
 
 c_void_p = ctypes.c_void_p
 c_int = ctypes.c_int
@@ -94,22 +94,28 @@ def cuda_lib() -> ctypes.CDLL:
     return _cuda
 
 
-def stream_lib() -> ctypes.CDLL:
-    """The kernels of the "stream" component: the complete library when it is there and has them, else the component's
-    own library, built on first use."""
-    global _stream
-    if _stream is None:
+def stream_lib(name: str = "stream") -> ctypes.CDLL:
+    """The kernels of a component (``native/build.py``) of the decoders with a 32-bit residual stream: the complete library
+    when it is there and has them, else the component's own library, built on first use."""
+    lib = _components.get(name)
+    if lib is None:
+        from . import cuda_api
+        sigs = cuda_api.COMPONENT_SIGS[name]
         if os.path.exists(os.environ.get("IPEX_LLM_CUDA_LIB") or _build.CUDA_LIB):
             lib = cuda_lib()
-        else:
-            lib = None
-        if lib is None or not hasattr(lib, "ipex_delta_step"):
+        if lib is None or not all(hasattr(lib, fn) for fn in sigs):
             with _lock:
-                lib = ctypes.CDLL(_build.build_component("stream"))
-        from . import cuda_api
-        cuda_api.declare_stream(lib)
-        _stream = lib
-    return _stream
+                lib = ctypes.CDLL(_build.build_component(name))
+        cuda_api.declare_component(lib, name)
+        _components[name] = lib
+    return lib
+
+
+def prepare_components(*names: str):
+    """Build what is missing of several components side by side, before the first of them is used."""
+    if not os.path.exists(os.environ.get("IPEX_LLM_CUDA_LIB") or _build.CUDA_LIB):
+        with _lock:
+            _build.build_components(names)
 
 
 def ptr(t) -> ctypes.c_void_p:

@@ -37,7 +37,7 @@ class DeltaSpec:
         return self.channels + self.heads * self.vdim
 
     def chunks_ok(self, dtype) -> bool:
-        return dtype != torch.float32 and bool(stream_lib().ipex_delta_chunks_ok(self.dim, self.vdim))
+        return dtype != torch.float32 and bool(stream_lib("hybrid").ipex_delta_chunks_ok(self.dim, self.vdim))
 
 
 class DeltaWeights:
@@ -55,7 +55,7 @@ def delta_mix(spec: DeltaSpec, w: DeltaWeights, proj, gates, slot, pos, cache, l
     output gates before their convolutions and activations) and ``gates [tokens, 2 heads]`` (write strengths, decays;
     fp32); the slots' states and convolution inputs move on.  ``portions``: how the tokens belong together, None when
     every token is another sequence's next one.  ``chunked`` overrides the choice of the form."""
-    lib, layer = stream_lib(), cache.layers[layer_idx]
+    lib, layer = stream_lib("hybrid"), cache.layers[layer_idx]
     T, dt, st, dev = proj.shape[0], _dt(proj), current_stream(), proj.device
     sizes = (spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.taps, dt)
     common = (ptr(gates), ptr(w.conv), ptr(w.a_log), ptr(w.dt_bias), ptr(layer._v), ptr(layer._k), ptr(slot), ptr(pos),

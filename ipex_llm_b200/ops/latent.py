@@ -85,9 +85,9 @@ def moe_grouped(bank: ExpertBank, x, h):
     y = torch.empty(S, W, dtype=dtype, device=dev)
     if bank.interleaved and gemm_ok(hs, bank.gate_up) and gemm_ok(a, bank.down):
         err, bt = ptr(error_flag(dev)), _tile(S / E * 1.25)
-        api.check(lib.ipex_gemm_stream(ptr(hs), W, ptr(bank.gate_up), W, ptr(a), I, None, ptr(ws), ptr(ranges), E, S, 2 * I, W,
+        api.check(lib.ipex_gemm_stream(ptr(hs), W, ptr(bank.gate_up), W, ptr(a), I, None, None, 0, None, 0, ptr(ws), ptr(ranges), E, S, 2 * I, W,
                                        OUT_ACT, ACT_GLU, bank.limit, bank.alpha, bt, dt, err, st), "gemm_stream(glu)")
-        api.check(lib.ipex_gemm_stream(ptr(a), I, ptr(bank.down), I, ptr(y), W, None, None, ptr(ranges), E, S, W, I, OUT_ACT,
+        api.check(lib.ipex_gemm_stream(ptr(a), I, ptr(bank.down), I, ptr(y), W, None, None, 0, None, 0, None, ptr(ranges), E, S, W, I, OUT_ACT,
                                        0, 0.0, 0.0, bt, dt, err, st), "gemm_stream(down)")
     else:
         gu = torch.empty(S, 2 * I, dtype=torch.float32, device=dev)
@@ -118,10 +118,10 @@ class LatentSpec:
         self.scale, self.window, self.pairs, self.eps = scale, window, pairs, eps
 
     def row(self, dtype) -> int:
-        return int(stream_lib().ipex_latent_row(self.rank, self.rot_dim, _dt(dtype)))
+        return int(stream_lib("latent").ipex_latent_row(self.rank, self.rot_dim, _dt(dtype)))
 
     def prefill_ok(self, dtype) -> bool:
-        return bool(stream_lib().ipex_latent_prefill_ok(self.dim, self.rot_dim, self.v_dim, self.rank, _dt(dtype)))
+        return bool(stream_lib().ipex_packed_prefill_ok(self.dim, self.rot_dim, self.v_dim, self.rank, _dt(dtype)))
 
 
 def pick_latent_splits(tokens: int, heads: int, visible: int, n_sm: int = 148) -> int:
@@ -136,7 +136,7 @@ def latent_step(spec: LatentSpec, qkv, w_uk, w_uv, kv_norm, cos, sin, slot, pos,
     """Absorbed attention of query tokens against the cache, which gets their own rows first.  ``qkv [M, ...]`` is
     the fused projection (its query parts are rotated in place), ``out [M, H * vd]``; ``visible`` bounds the number of
     keys a token can see (it sizes the split, nothing else)."""
-    lib = stream_lib()
+    lib = stream_lib("latent")
     rows = cache.layers[layer_idx]._k
     M, H, R = qkv.shape[0], spec.heads, spec.rank
     dt, st = _dt(qkv), current_stream()
@@ -167,7 +167,7 @@ def latent_prompt(spec: LatentSpec, qkv, w_uk, w_uv, kv_norm, cos, sin, slot, po
                   cache, layer_idx: int, out):
     """Attention of whole prompts, packed one behind the other (``seq_row`` / ``seq_len``: int32, first row and length
     of each): keys and values are expanded from the latents, then the tcgen05 kernel; the cache gets the latents."""
-    lib = stream_lib()
+    lib = stream_lib("latent")
     rows = cache.layers[layer_idx]._k
     T, H, R, dev, dtype = qkv.shape[0], spec.heads, spec.rank, qkv.device, qkv.dtype
     dt, st = _dt(qkv), current_stream()
@@ -182,10 +182,10 @@ def latent_prompt(spec: LatentSpec, qkv, w_uk, w_uv, kv_norm, cos, sin, slot, po
     ld = (T + 7) // 8 * 8
     vt = torch.empty(H * spec.v_dim, ld, dtype=dtype, device=dev)
     gemm(w_uv, c, vt, OUT_ACT)                    # V transposed: rows are value dimensions, columns tokens
-    rc = lib.ipex_packed_prefill(ptr(qkv), qkv.stride(0), ptr(k), k.stride(0), ptr(kr), kr.stride(0), ptr(vt), ld,
-                                 ptr(out), out.stride(0), ptr(seq_row), ptr(seq_len), seq_row.shape[0], H, H, T, max_len,
-                                 spec.dim, spec.rot_dim, spec.v_dim, spec.window, 0, spec.scale, dt, ptr(error_flag(dev)),
-                                 st)
+    rc = stream_lib().ipex_packed_prefill(ptr(qkv), qkv.stride(0), ptr(k), k.stride(0), ptr(kr), kr.stride(0), ptr(vt), ld,
+                                          ptr(out), out.stride(0), ptr(seq_row), ptr(seq_len), seq_row.shape[0], H, H, T,
+                                          max_len, spec.dim, spec.rot_dim, spec.v_dim, spec.window, 0, spec.scale, dt,
+                                          ptr(error_flag(dev)), st)
     if rc == -1:
         raise RuntimeError("ipex_llm_b200: the driver's tensor-map encoder rejected the attention operands")
     api.check(rc, "packed_prefill")

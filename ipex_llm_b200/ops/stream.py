@@ -73,18 +73,25 @@ def _tile(rows: float, cols: int = 1 << 20) -> int:
     return bt
 
 
-def gemm(x, w, out, mode: int, act: int = 0, bias=None, interleaved=True):
+def gemm(x, w, out, mode: int, act: int = 0, bias=None, interleaved=True, w2=None, out2=None):
     """``x [M, K] @ w[N, K].T (+ bias)`` into ``out`` (see ``OUT_*``): the tcgen05 kernel, or the library product for
-    32-bit weights and rows that are no multiple of 16 bytes.  ``ACT_GELU_GLU``: see ``gemv_rows``."""
+    32-bit weights and rows that are no multiple of 16 bytes.  ``ACT_GELU_GLU``, ``w2`` / ``out2``: see ``gemv_rows``."""
     M, (N, K) = x.shape[0], w.shape
     if gemm_ok(x, w) and not (act == ACT_GELU_GLU and not interleaved):
+        both = w2 is not None and gemm_ok(x, w2) and w2.stride(0) == w.stride(0)
+        if w2 is not None and not both:
+            gemm(x, w2, out2, OUT_F32)
         rc = stream_lib().ipex_gemm_stream(ptr(x), x.stride(0), ptr(w), w.stride(0), ptr(out), out.stride(0), ptr(bias),
-                                           None, None, 1, M, N, K, mode, act, 0.0, 0.0, _tile(M, N), _dt(w),
-                                           ptr(error_flag(x.device)), current_stream())
+                                           ptr(w2 if both else None), w2.shape[0] if both else 0,
+                                           ptr(out2 if both else None), out2.stride(0) if both else 0, None, None, 1, M, N,
+                                           K, mode, act, 0.0, 0.0, _tile(M, N), _dt(w), ptr(error_flag(x.device)),
+                                           current_stream())
         if rc == -1:
             raise RuntimeError("ipex_llm_b200: the driver's tensor-map encoder rejected the GEMM operands")
         api.check(rc, "gemm_stream")
         return out
+    if w2 is not None:
+        gemm(x, w2, out2, OUT_F32)
     with _true_fp32():
         if act == ACT_GELU_GLU:
             return gelu_glu_rows(torch.matmul(x.float(), w.float().t()), bias, out, interleaved)

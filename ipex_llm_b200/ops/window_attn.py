@@ -1,5 +1,5 @@
 """Python front of the attention over cached keys and values of different sizes (``kv_attn.cu``, and the packed tcgen05
-prompt kernel of ``latent_prefill_tcgen05.cu``): grouped query heads, sliding window, optional sink in the soft-max, values
+prompt kernel of ``packed_prefill_tcgen05.cu``): grouped query heads, sliding window, optional sink in the soft-max, values
 mixed with those of an earlier layer.
 
 Every function launches on the current stream; there is no eager substitute.
@@ -43,7 +43,7 @@ class AttnSpec:
 
     def prefill_ok(self, dtype) -> bool:
         """Does the tcgen05 prompt kernel take these sizes?"""
-        return bool(stream_lib().ipex_latent_prefill_ok(self.dim, 0, self.vdim, 8, _dt(dtype)))
+        return bool(stream_lib().ipex_packed_prefill_ok(self.dim, 0, self.vdim, 8, _dt(dtype)))
 
 
 @dataclass
@@ -72,7 +72,7 @@ def attend_step(spec: AttnSpec, qkv, mix: Optional[ValueMix], slot, pos, cache, 
     """Attention of query tokens against the cache, which gets their own rows first.  ``single``: every token is another
     sequence's next one (the append is then part of the attention kernel).  ``visible`` bounds the number of keys a
     token can see (it sizes the split, nothing else)."""
-    lib, layer = stream_lib(), cache.layers[layer_idx]
+    lib, layer = stream_lib("hybrid"), cache.layers[layer_idx]
     k, v = layer._k, layer._v
     M, dt, st = qkv.shape[0], _dt(qkv), current_stream()
     cols = (qkv[:, spec.k_at:], qkv[:, spec.v_at:])
@@ -97,7 +97,7 @@ def attend_prompt(spec: AttnSpec, qkv, mix: Optional[ValueMix], slot, pos, seq_r
                   layer_idx: int, out):
     """Attention of whole prompts, packed one behind the other (``seq_row`` / ``seq_len``: int32, first row and length of
     each), on the tensor cores; the cache gets keys and mixed values."""
-    lib, layer = stream_lib(), cache.layers[layer_idx]
+    lib, layer = stream_lib("hybrid"), cache.layers[layer_idx]
     k, v = layer._k, layer._v
     T, dt, st, dev = qkv.shape[0], _dt(qkv), current_stream(), qkv.device
     ld = (T + 7) // 8 * 8
@@ -107,10 +107,10 @@ def attend_prompt(spec: AttnSpec, qkv, mix: Optional[ValueMix], slot, pos, seq_r
     api.check(lib.ipex_kv_append(ptr(keys), ptr(qkv[:, spec.v_at:]), qkv.stride(0), ptr(first), ld_vf, share, ptr(k),
                                  k.stride(0), k.stride(1), ptr(v), v.stride(0), v.stride(1), ptr(vt), ld, ptr(slot),
                                  ptr(pos), T, spec.kv_heads, spec.dim, spec.vdim, dt, 0, st), "kv_append")
-    rc = lib.ipex_packed_prefill(ptr(qkv), qkv.stride(0), ptr(keys), qkv.stride(0), None, 0, ptr(vt), ld, ptr(out),
-                                 out.stride(0), ptr(seq_row), ptr(seq_len), seq_row.shape[0], spec.heads, spec.kv_heads, T,
-                                 max_len, spec.dim, 0, spec.vdim, spec.window, int(spec.sink), spec.scale, dt,
-                                 ptr(error_flag(dev)), st)
+    rc = stream_lib().ipex_packed_prefill(ptr(qkv), qkv.stride(0), ptr(keys), qkv.stride(0), None, 0, ptr(vt), ld, ptr(out),
+                                          out.stride(0), ptr(seq_row), ptr(seq_len), seq_row.shape[0], spec.heads,
+                                          spec.kv_heads, T, max_len, spec.dim, 0, spec.vdim, spec.window, int(spec.sink),
+                                          spec.scale, dt, ptr(error_flag(dev)), st)
     if rc == -1:
         raise RuntimeError("ipex_llm_b200: the driver's tensor-map encoder rejected the attention operands")
     api.check(rc, "packed_prefill")

@@ -147,15 +147,16 @@ def kernels(z, prompt: int, peaks):
         del cache, st
     # --- prompt GEMMs
     T = prompt
-    for name, N, K, mode, act in (("gemm q/k/v + bias", att.rows, W, 0, 0), ("gemm recurrent projections", dl.rows, W, 0, 0),
-                                  ("gemm gates, fp32", 2 * dH, W, 2, 0), ("gemm o_proj, fp32", W, H * D, 2, 0),
+    for name, N, K, mode, act in (("gemm q/k/v + bias", att.rows, W, 0, 0), ("gemm recurrent projections + gates", dl.rows, W, 0, 0),
+                                  ("gemm o_proj, fp32", W, H * D, 2, 0),
                                   ("gemm gate / up, gelu", 2 * ff, W, 0, S.ACT_GELU_GLU),
                                   ("gemm down + bias, fp32", W, ff, 2, 0)):
         n = _sets(2.0 * (N * K + T * K))
         ws, xk, bias = [mat(N, K) for _ in range(n)], [mat(T, K, s=1.0) for _ in range(n)], mat(N)
         No = N // 2 if act else N
         out = torch.zeros(T, No, device=dev, dtype=bf if mode == 0 else torch.float32)
-        us = _graph_us(lambda i: S.gemm(xk[i], ws[i], out, mode, act, bias), n)
+        two = (gate_rows, torch.empty(T, 2 * dH, device=dev)) if "gates" in name else (None, None)
+        us = _graph_us(lambda i: S.gemm(xk[i], ws[i], out, mode, act, bias, True, *two), n)
         ob, res = torch.empty(T, No, device=dev, dtype=bf), mat(T, N) if mode == 2 else None
         like = _graph_us(lambda i: tcgen05_gemm.gemm_dense(xk[i], ws[i], residual=res, out=ob, act=2 if act else 0), n)
         fl, nb = 2.0 * T * N * K, 2.0 * (T * K + N * K)
@@ -195,14 +196,13 @@ def kernels(z, prompt: int, peaks):
     add(f"delta_chunks (4 kernels) T={T}", us, nb, fl, f"rwkv5 {like:.1f} us",
         max(16.0 * T * dH * dV / hbm, 4.0 * T * dH * dV * dV / tf) / like)
     from ..native.lib import ptr, stream_lib
-    lib, layer = stream_lib(), cache.layers[0]
+    lib = stream_lib("hybrid")
     per = dH * lib.ipex_delta_scratch_floats(dD, dV)
     rows.append({"kernel": f"delta scratch, MB for T={T}", "us": round(nc * per * 4 / 1e6, 1)})
     raw = torch.empty(T, dH, dV, device=dev)
     us = _graph_us(lambda i: lib.ipex_gated_norm(ptr(raw), ptr(projs[i][:, dl.channels:]), dl.rows, ptr(w.norm), ptr(out),
                                                  out.stride(0), T, dH, dV, 1e-6, 1, S.current_stream()), 4)
     add(f"gated_norm T={T}", us, 8.0 * T * dH * dV)
-    del layer
     cuda_ops.check_error_flag(torch.device("cuda", 0))
     return rows
 

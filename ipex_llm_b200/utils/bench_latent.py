@@ -153,7 +153,7 @@ def kernels(z, prompt: int, peaks):
     spec = L.LatentSpec(H, z["dim"], z["rd"], z["vd"], R, 0.1, z["window"], z["rd"] // 2, 1e-6)
     cos, sin = L.rotary_table(4096, 1e4, z["rd"] // 2, dev)
     uk, uv, kn = mat(H * z["dim"], R), mat(H * z["vd"], R), torch.ones(R, device=dev, dtype=bf)
-    lib, st = L.stream_lib(), L.current_stream
+    lib, st = L.stream_lib("latent"), L.current_stream
     for B in (1, 8, 32):
         ctx = z["window"]
         n = _sets(B * ctx * (R + z["rd"]) * 2)
@@ -254,7 +254,7 @@ def kernels(z, prompt: int, peaks):
     i32 = dict(device=dev, dtype=torch.int32)
     row, ln, err = torch.zeros(1, **i32), torch.full((1,), T, **i32), cuda_ops.error_flag(torch.device("cuda", 0))
     for win in (z["window"], 0):
-        us = _graph_us(lambda i: lib.ipex_packed_prefill(
+        us = _graph_us(lambda i: L.stream_lib().ipex_packed_prefill(
             L.ptr(qs[i]), ldq, L.ptr(ks[i]), H * z["dim"], L.ptr(kr), z["rd"], L.ptr(vt), T, L.ptr(out), H * z["vd"],
             L.ptr(row), L.ptr(ln), 1, H, H, T, T, z["dim"], z["rd"], z["vd"], win, 0, 0.05, 1, L.ptr(err),
             L.current_stream()), n)

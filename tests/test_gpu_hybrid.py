@@ -66,7 +66,7 @@ def test_gated_unit_with_biases(dtype, M, ff, K):
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
-@pytest.mark.parametrize("M,N,K,N2", [(1, 97, 136, 5), (3, 40, 60, 12), (11, 2500, 520, 64), (2, 33, 7, 1), (7, 136, 1536, 4), (40, 120, 64, 6),
+@pytest.mark.parametrize("M,N,K,N2", [(1, 97, 136, 5), (3, 40, 60, 12), (11, 2500, 520, 64), (2, 33, 7, 1), (7, 136, 1536, 4), (40, 120, 64, 6), (300, 257, 136, 150),
                                       (9, 64, 30, 10)])
 def test_bias_and_second_matrix(dtype, M, N, K, N2):
     from ipex_llm_b200.ops import stream as S
@@ -83,6 +83,10 @@ def test_bias_and_second_matrix(dtype, M, N, K, N2):
         close(S.gemv_rows(W, X, f, S.OUT_F32, bias=B), want, F32, "fp32", 5)
         close(S.gemv_rows(W, X, R, S.OUT_ADD, bias=B), res + want, F32, "stream", 5)
         R.copy_(res)
+    g2 = torch.full((M, N2 + 3), 7.0, dtype=F32, device="cuda")
+    close(S.gemm(X, W, torch.empty_like(out), S.OUT_ACT, bias=B, w2=W2, out2=g2[:, :N2]), want, dtype, "gemm")
+    close(g2[:, :N2], x @ w2.T, F32, "gemm, second matrix", 5)
+    assert bool((g2[:, N2:] == 7.0).all())
     close(S.gemm(X, W, torch.empty_like(out), S.OUT_ACT, bias=B), want, dtype, "gemm")
     close(S.gemm(X, W, torch.empty_like(f), S.OUT_F32, bias=B), want, F32, "gemm fp32", 5)
     close(S.gemm(X, W, R, S.OUT_ADD, bias=B), res + want, F32, "gemm stream", 5)
