@@ -77,7 +77,7 @@ __device__ __forceinline__ float conv_silu(const Common& a, int c, int t, int j,
   const T* ring = reinterpret_cast<const T*>(a.ring) + (int64_t)slot * a.taps * a.channels + c;
   const int pm = p % a.taps, seen = min(a.taps, p - start + 1);
   float s = 0.f;
-  for (int b0 = 0; b0 < seen; b0 += 4) {
+  for (int b0 = 0; b0 < a.taps; b0 += 4) {
     T x[4];
     float wv[4];
 #pragma unroll
@@ -85,14 +85,15 @@ __device__ __forceinline__ float conv_silu(const Common& a, int c, int t, int j,
       const int back = b0 + u;
       x[u] = DT<T>::from_f(0.f);
       wv[u] = 0.f;
-      if (back < seen) {
+      if (back < a.taps) {                       // (rows from before the start are read and not used: `start` comes late)
         const int r = pm - back;
         x[u] = back <= j ? proj[-(int64_t)back * a.ldp] : ring[(int64_t)(r < 0 ? r + a.taps : r) * a.channels];
         wv[u] = DT<TW>::to_f(w[-back]);
       }
     }
 #pragma unroll
-    for (int u = 0; u < 4; ++u) s = fmaf(DT<T>::to_f(x[u]), wv[u], s);
+    for (int u = 0; u < 4; ++u)
+      if (b0 + u < seen) s = fmaf(DT<T>::to_f(x[u]), wv[u], s);
   }
   return silu(s);
 }
@@ -182,7 +183,13 @@ __global__ void __launch_bounds__(kThreads, NR * CV <= 64 ? 2 : 1) delta_step_ke
     const int d = warp + 8 * i;
 #pragma unroll
     for (int c = 0; c < CV; ++c) S[i][c] = 0.f;
-    if (!fresh && col && d < D) load_cols<CV>(st + (int64_t)d * V, S[i]);
+    if (col && d < D) load_cols<CV>(st + (int64_t)d * V, S[i]);
+  }
+  if (fresh) {
+#pragma unroll
+    for (int i = 0; i < NR; ++i)
+#pragma unroll
+      for (int c = 0; c < CV; ++c) S[i][c] = 0.f;
   }
   for (int j = 0; j < len; ++j) {
     const int t = row0 + j, p = p0 + j;
@@ -901,12 +908,12 @@ cudaError_t launch_step(const StepArgs& s, int seqs, bool fused, bool pdl, cudaS
 }
 
 // Columns per lane: as many as V divides into and the registers of NR rows leave room for, fewer while that spreads the
-// states of a few sequences over more SMs.
+// large states of a few sequences over more SMs.
 template <typename T, int NR>
 cudaError_t pick_cols(const StepArgs& s, int seqs, bool fused, bool pdl, cudaStream_t st) {
   const int V = s.c.vdim;
   int cv = NR <= 16 && V % 4 == 0 && V > 64 ? 4 : NR <= 32 && V % 2 == 0 && V > 32 ? 2 : 1;
-  while (cv > 1 && (int64_t)s.c.heads * seqs * ((V + 16 * cv - 1) / (16 * cv)) <= 2 * 148) cv /= 2;
+  while (cv > 1 && s.c.dim * 32 * cv > 4096 && (int64_t)s.c.heads * seqs * ((V + 16 * cv - 1) / (16 * cv)) <= 2 * 148) cv /= 2;
   if constexpr (NR <= 16)
     if (cv == 4) return launch_step<T, NR, 4>(s, seqs, fused, pdl, st);
   if constexpr (NR <= 32)
