@@ -128,7 +128,7 @@ class StreamStack:
         if P.packed is None:
             return K.gemm(h, P.w, out, mode, act, P.bias, interleaved)
         w, M = P.packed, h.shape[0]
-        glu = act == K.ACT_GELU_GLU
+        glu = act in (K.ACT_GELU_GLU, K.ACT_SILU_GLU)
         y = out if mode == K.OUT_ACT and not glu else torch.empty(M, w.N, dtype=h.dtype, device=h.device)
         if M <= cuda_ops.GEMV_MAX_M:
             per = cuda_ops._gemv_rows_per_call(w.K)
@@ -137,7 +137,7 @@ class StreamStack:
         else:
             cuda_ops.gemm_lowbit(h, w.data, w.qtype, w.N, w.K, out=y)
         if glu:
-            return K.gelu_glu_rows(y, P.bias, out, interleaved)
+            return K.glu_rows(y, P.bias, out, act, interleaved)
         if P.bias is not None:
             K.bias_rows_(y, P.bias)
         if mode == K.OUT_ACT:

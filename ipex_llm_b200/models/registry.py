@@ -150,6 +150,8 @@ FAMILIES = {
     "dobetar": Family(engine="latent"),
     # windowed attention and gated-delta-rule layers on a 32-bit residual stream: likewise
     "letarax": Family(engine="hybrid"),
+    # several 32-bit residual streams, latent attention, attention and linear attention side by side: likewise
+    "dodilix": Family(engine="multistream"),
     # LayerNorm families without a dedicated forward file: low-bit linears + the fused LayerNorm kernel
     "gpt_neox": Family(post=[("LayerNorm", C.layer_norm_forward)]),
     "bloom": Family(post=[("LayerNorm", C.layer_norm_forward)]),

@@ -40,6 +40,7 @@ COMPONENTS = {
     "stream": ("elementwise.cu", "gemm_stream_tcgen05.cu", "gemv_dense.cu", "packed_prefill_tcgen05.cu", "stream_ops.cu"),
     "latent": ("latent_attn.cu",),
     "hybrid": ("delta_rule.cu", "kv_attn.cu"),
+    "linear": ("linear_attn.cu",),
 }
 
 NVCC_ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]

@@ -50,6 +50,24 @@ __device__ __forceinline__ float warp_max(float v) {
   return v;
 }
 
+// N values on each of 8 lanes (a power of two) -> sums over the 8 lanes, spread so that a lane keeps max(1, N / 8) of
+// them: value i ends on the lanes whose id matches, in the order of the folds
+template <int N, int OFF>
+__device__ __forceinline__ void fold(float* v, int lane) {
+  if constexpr (N > 1) {
+    const bool up = lane & OFF;
+#pragma unroll
+    for (int i = 0; i < N / 2; ++i) {
+      const float keep = up ? v[i + N / 2] : v[i], give = up ? v[i] : v[i + N / 2];
+      v[i] = keep + __shfl_xor_sync(0xffffffffu, give, OFF);
+    }
+    if constexpr (OFF > 1) fold<N / 2, OFF / 2>(v, lane);
+  } else {
+    v[0] += __shfl_xor_sync(0xffffffffu, v[0], OFF);
+    if constexpr (OFF > 1) fold<1, OFF / 2>(v, lane);
+  }
+}
+
 // Tanh form of gelu, 0.5 z (1 + tanh(c (z + 0.044715 z^3))), through 0.5 (1 + tanh y) = 1 / (1 + e^(-2y)).
 __device__ __forceinline__ float gelu_tanh(float z) {
   const float y = 0.7978845608028654f * (z + 0.044715f * z * z * z);

@@ -25,6 +25,7 @@
 // state there, so a slot needs no clearing when it changes hands.
 #include <cooperative_groups.h>
 
+#include "common/tf32_pairs.cuh"
 #include "common/utils.cuh"
 #include "tcgen05_common.cuh"
 
@@ -309,50 +310,6 @@ __global__ void __launch_bounds__(kThreads, NR * CV <= 64 ? 2 : 1) delta_step_ke
     for (int i = tid; i < nv; i += kThreads) ring[vc + i] = proj[vc + i];
   }
 }
-
-// ---------------------------------------------------------------------------------------------- tf32 pairs
-__device__ __forceinline__ void split_tf32(float x, uint32_t& hi, uint32_t& lo) {
-  hi = __float_as_uint(x) & 0xFFFFE000u;
-  lo = __float_as_uint(x - __uint_as_float(hi));       // exact; the instruction reads its upper 19 bits
-}
-__device__ __forceinline__ void mma_tf32(float (&c)[4], const uint32_t (&a)[4], const uint32_t (&b)[2]) {
-  asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
-}
-struct FragA { uint32_t hi[4], lo[4]; };
-struct FragB { uint32_t hi[2], lo[2]; };
-// lane (g, t): A rows g, g + 8 and columns t, t + 4; B row (k) t, t + 4 of column g; C rows g, g + 8, columns 2t, 2t + 1
-template <typename F>
-__device__ __forceinline__ FragA frag_a(F&& at, int g, int t) {
-  FragA f;
-  split_tf32(at(g, t), f.hi[0], f.lo[0]);
-  split_tf32(at(g + 8, t), f.hi[1], f.lo[1]);
-  split_tf32(at(g, t + 4), f.hi[2], f.lo[2]);
-  split_tf32(at(g + 8, t + 4), f.hi[3], f.lo[3]);
-  return f;
-}
-template <typename F>
-__device__ __forceinline__ FragB frag_b(F&& at, int g, int t) {
-  FragB f;
-  split_tf32(at(t, g), f.hi[0], f.lo[0]);
-  split_tf32(at(t + 4, g), f.hi[1], f.lo[1]);
-  return f;
-}
-// independent accumulators for the main and the two correction products: three short chains instead of a long one
-struct Acc {
-  float m[4], x[4], y[4];
-  __device__ __forceinline__ void zero() {
-#pragma unroll
-    for (int i = 0; i < 4; ++i) m[i] = x[i] = y[i] = 0.f;
-  }
-  __device__ __forceinline__ void mac(const FragA& a, const FragB& b) {
-    mma_tf32(m, a.hi, b.hi);
-    mma_tf32(x, a.hi, b.lo);
-    mma_tf32(y, a.lo, b.hi);
-  }
-  __device__ __forceinline__ float get(int i) const { return m[i] + (x[i] + y[i]); }
-};
 
 // Scratch of one (chunk, head), laid out like the shared memory that reads it (row strides keep the fragments' banks
 // apart): W, Q and K parts of 32 rows, P [32][36], decay of the whole chunk; then Ub [32][40] per slice of 32 columns.
@@ -639,12 +596,6 @@ __global__ void __launch_bounds__(kThreads, 3) delta_prep_kernel(ChunkArgs s) {
   }
 }
 
-__device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
-  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
-                   tc5::smem_u32(dst)), "l"(src), "r"(bytes), "r"(tc5::smem_u32(bar))
-               : "memory");
-}
-
 template <int MT>
 __global__ void __launch_bounds__(kChunkThreads, 1) delta_chunks_kernel(ChunkArgs s, int stages) {
   constexpr int NW = kChunkThreads / 32, N1 = 16 / NW, N2 = 32 / NW;   // column tiles per warp: of [W; Q] S, of the state
@@ -815,7 +766,8 @@ __global__ void __launch_bounds__(kThreads) delta_tail_kernel(Common a) {
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(kThreads) gated_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate,
                                                               int64_t ldg, const T* __restrict__ w, T* __restrict__ out,
-                                                              int64_t ldo, int64_t rows, int heads, int V, float eps) {
+                                                              int64_t ldo, int64_t rows, int heads, int V, float eps,
+                                                              float scale) {
   constexpr int N = VEC ? 4 : 1;
   const int64_t r = (int64_t)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
@@ -841,7 +793,7 @@ __global__ void __launch_bounds__(kThreads) gated_norm_kernel(const float* __res
 #pragma unroll
     for (int c = 0; c < N; ++c) ss = fmaf(x[c], x[c], ss);
   }
-  const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)V + eps);
+  const float inv = scale / sqrtf(warp_sum(ss) / (float)V + eps);
   for (int i = lane * N; i < V; i += 32 * N) {
     load_cols<N>(src + i, x);
     load(gt + i, gv);
@@ -1019,9 +971,9 @@ IPEX_API int ipex_delta_tail(const void* proj, int64_t ldp, void* ring, const in
   });
 }
 
-// out[t, h, :] = o / sqrt(mean(o^2) + eps) * w * silu(gate), o [tokens, heads, vdim] fp32
+// out[t, h, :] = scale * o / sqrt(mean(o^2) + eps) * w * silu(gate), o [tokens, heads, vdim] fp32
 IPEX_API int ipex_gated_norm(const float* o, const void* gate, int64_t ldg, const void* w, void* out, int64_t ldo,
-                             int tokens, int heads, int vdim, float eps, int dtype, void* stream) {
+                             int tokens, int heads, int vdim, float eps, float scale, int dtype, void* stream) {
   if (tokens < 1 || heads < 1 || vdim < 1) return (int)cudaErrorInvalidValue;
   return by_dtype(dtype, [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
@@ -1030,7 +982,7 @@ IPEX_API int ipex_gated_norm(const float* o, const void* gate, int64_t ldg, cons
                      (((uintptr_t)gate | (uintptr_t)w | (uintptr_t)out) & 7) == 0;
     auto kern = vec ? gated_norm_kernel<T, true> : gated_norm_kernel<T, false>;
     kern<<<(unsigned)((rows + 7) / 8), kThreads, 0, (cudaStream_t)stream>>>(o, (const T*)gate, ldg, (const T*)w, (T*)out,
-                                                                            ldo, rows, heads, vdim, eps);
+                                                                            ldo, rows, heads, vdim, eps, scale);
     return cudaGetLastError();
   });
 }

@@ -3,7 +3,7 @@
 //     out = x[M, K] . W[N, K]^T (+ bias)  out_mode 0: 16-bit, optionally squared relu      1: added to an fp32 stream
 //                                         2: fp32 (router scores, logits)
 //     y = glu(row_scale * (x . W_gu^T))                    gate / up rows interleaved in 16-row tiles, N / 2 columns
-//     y = gelu_tanh(gate) * up, with biases                gate / up rows interleaved in 8-row tiles, N / 2 columns
+//     y = gelu_tanh(gate) * up or silu(gate) * up          gate / up rows interleaved in 8-row tiles, N / 2 columns
 //
 // A second matrix (w2) may ride along: its rows multiply the same x and leave as fp32 in an output of their own.
 //
@@ -30,7 +30,7 @@ struct Args {
   int* err;
   int64_t ldo;
   int M, N, K, groups;
-  int out_mode, act;        // act 1: squared relu (out_mode 0); 2: clamped gated unit; 3: gelu-gated unit
+  int out_mode, act;        // act 1: squared relu (out_mode 0); 2: clamped gated unit; 3 / 4: gelu- / silu-gated unit
   float limit, alpha;
   const void* bias;         // T [N] or null
   float* out2;              // fp32 [M, ldo2], results of the second matrix's N2 rows (0: there is none)
@@ -213,7 +213,7 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
           continue;
         }
         const float bn = a.bias != nullptr && n < a.N ? to_float<T>(reinterpret_cast<const T*>(a.bias)[n]) : 0.f;
-        if (a.act == 3) {
+        if (a.act >= 3) {
           // lanes with bit 3 clear hold gate rows, the lanes eight above them the matching up rows: the former finish
           // the even tokens of a pair, the latter the odd ones
           const int n_out = (tl.nb * kBM + qd * 32) / 2 + (lane >> 4) * 8 + (lane & 7);
@@ -224,9 +224,9 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
             const float s0 = __uint_as_float(v[j]) + bn, s1 = __uint_as_float(v[j + 1]) + bn;
             const float got = __shfl_xor_sync(0xffffffffu, upper ? s0 : s1, 8);
             const float gv = upper ? got : s0, uv = upper ? s1 : got;
-            const float y = 0.7978845608028654f * (gv + 0.044715f * gv * gv * gv);
+            const float e = a.act == 4 ? gv : 1.5957691216057308f * (gv + 0.044715f * gv * gv * gv);
             if (writer && j + upper < lim)
-              out[(int64_t)j * a.ldo] = from_float<T>(__fdividef(gv, 1.0f + __expf(-2.0f * y)) * uv);
+              out[(int64_t)j * a.ldo] = from_float<T>(__fdividef(gv, 1.0f + __expf(-e)) * uv);
           }
         } else if (a.act == 2) {
           // lanes 0..15 hold gate rows, lanes 16..31 the matching up rows
@@ -325,7 +325,7 @@ int dispatch(int bt, const void* x, int64_t ldx, int x_rows, const void* w, int6
 }  // namespace
 
 // See the head of this file.  M: rows of x; with `ranges` the groups' rows partition them.  w: [groups * N, K].  bt:
-// token tile (32 / 64 / 128 / 256).  row_scale only with act 2 (then out_mode 0 and N a multiple of 32).  act 3: out_mode
+// token tile (32 / 64 / 128 / 256).  row_scale only with act 2 (then out_mode 0 and N a multiple of 32).  act 3, 4: out_mode
 // 0, N a multiple of 16.  bias (may be null) has N entries of the operands' type; not with act 2 or ranges.
 // w2 / out2 (N2 = 0: none): N2 more rows of the same row stride, results in fp32; not with ranges or act 2.
 // Strides of x and w multiples of 8 elements, bases 16-byte aligned.  Returns a cudaError_t, or -1 when the
@@ -337,7 +337,7 @@ IPEX_API int ipex_gemm_stream(const void* x, int64_t ldx, const void* w, int64_t
     return (int)cudaErrorInvalidValue;
   if ((groups > 1) != (ranges != nullptr) && ranges == nullptr) return (int)cudaErrorInvalidValue;
   if (act == 2 && (row_scale == nullptr || out_mode != 0 || (N % 32) != 0)) return (int)cudaErrorInvalidValue;
-  if (act < 0 || act > 3 || (act == 1 && out_mode != 0) || (act == 3 && (out_mode != 0 || (N % 16) != 0)) ||
+  if (act < 0 || act > 4 || (act == 1 && out_mode != 0) || (act >= 3 && (out_mode != 0 || (N % 16) != 0)) ||
       (bias != nullptr && (act == 2 || ranges != nullptr)))
     return (int)cudaErrorInvalidValue;
   if ((reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15)) return (int)cudaErrorInvalidValue;

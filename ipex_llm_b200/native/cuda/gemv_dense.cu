@@ -3,17 +3,19 @@
 //   gemv_rows    y[M <= 8, N] = act( x . W[N, K]^T )   with x either activations in the weight dtype or the fp32
 //                residual stream, RMS-normed while it is staged in shared memory; the result (plus a bias) goes out in
 //                the weight dtype, is added to an fp32 residual, or leaves as fp32 with an optional tanh soft-cap
-//                (logits); gate and up rows may be joined to gelu_tanh(gate) * up, and the rows of a second matrix
-//                may ride along with fp32 results (gates of a recurrence beside its projections)
-//   moe_router   norm + router scores in fp32 + sigmoid + top-k of one token per CTA
-//   moe_glu      per (token, choice) slot: clamped gated unit of the chosen expert, the routing weight applied to the
-//                expert's input
-//   moe_down     residual[t] += sum over the token's choices of down_e(y)
+//                (logits); gate and up rows may be joined to gelu_tanh(gate) * up or silu(gate) * up, and the rows of a
+//                second matrix may ride along with fp32 results (gates of a recurrence beside its projections)
+//   moe_router   norm + router scores in fp32 + sigmoid + top-k of one token per CTA; or, from finished rows, soft-max
+//                scores, group-limited top-k with renormalised weights, and the gate of a shared expert
+//   moe_glu      per (token, choice) slot: gated unit of the chosen expert - clamped, the routing weight applied to the
+//                expert's input, or silu; a shared expert of another size is one more choice
+//   moe_down     residual[t] += sum over the token's choices of down_e(y), or fp32 rows of the weighted sum
 //
 // All products are fp32 FMAs over 16-byte weight loads: with up to eight rows the weights are the traffic, and eight
 // rows of FMAs still fit under the memory time.  A warp owns R weight rows and walks K in steps of 32 vectors with
 // several loads in flight per lane.  With programmatic dependent launch the rows a warp touches first are pulled
 // into L2 while the previous kernel drains.
+#include "common/routing.cuh"
 #include "common/utils.cuh"
 
 namespace {
@@ -187,14 +189,14 @@ struct GemvRowsArgs {
   int64_t ldw, ldx, ldo;
   float eps, softcap;
   int M, N, K, kp;
-  int out_mode, act;     // act 1: square of relu; 3: gelu_tanh(gate) * up, N / 2 columns come out
+  int out_mode, act;     // act 1: square of relu; 3 / 4: gelu_tanh / silu(gate) * up, N / 2 columns come out
   int vec;
   const void* bias;      // T [N] or null
   const void* w2;        // rows N1 .. N (row stride ldw), or null (then N1 = N)
   float* out2;           // ... and their results, fp32
   int64_t ldo2;
   int N1;
-  int interleaved;       // act 3: gate and up rows alternate in blocks of eight, else gate rows before up rows
+  int interleaved;       // act 3, 4: gate and up rows alternate in blocks of eight, else gate rows before up rows
 };
 
 __device__ __forceinline__ float finish(float v, int act) { return act == 1 ? (v > 0.f ? v * v : 0.f) : v; }
@@ -213,7 +215,8 @@ __device__ __forceinline__ float bias_of(const GemvRowsArgs& a, int n) {
 // hidden unit i of token m from its two products (weight rows ng and nu)
 template <typename T>
 __device__ __forceinline__ void store_gated(const GemvRowsArgs& a, int m, int i, int ng, int nu, float g, float u) {
-  const float v = gelu_tanh(g + bias_of<T>(a, ng)) * (u + bias_of<T>(a, nu));
+  const float z = g + bias_of<T>(a, ng);
+  const float v = (a.act == 4 ? silu(z) : gelu_tanh(z)) * (u + bias_of<T>(a, nu));
   reinterpret_cast<T*>(a.out)[(int64_t)m * a.ldo + i] = DT<T>::from_f(v);
 }
 
@@ -366,7 +369,7 @@ __global__ void __launch_bounds__(kThreads) gemv_mma_kernel(GemvRowsArgs a, int 
       __syncthreads();
       // the group's warps share the sums: value (n, i) goes to warp (n * 4 + i) % split
       const float* grp = part + ((size_t)par * kWarps + warp / split * split) * (NT * 128);
-      if (a.act == 3) {
+      if (a.act >= 3) {
 #pragma unroll
         for (int n = 0; n < NT; ++n)
 #pragma unroll
@@ -392,7 +395,7 @@ __global__ void __launch_bounds__(kThreads) gemv_mma_kernel(GemvRowsArgs a, int 
             const int row = tile * 16 + g + 8 * (i >> 1), m = n * 8 + 2 * t + (i & 1);
             if (tile < ntile && row < a.N && m < a.M) store_row<T>(a, m, row, v);
           }
-    } else if (a.act == 3) {
+    } else if (a.act >= 3) {
 #pragma unroll
       for (int n = 0; n < NT; ++n)
 #pragma unroll
@@ -440,7 +443,7 @@ cudaError_t launch_gemv(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
 template <typename T, int M>
 cudaError_t pick_rows(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
   const int warps = sm_count() * kWarps;
-  if (a.act == 3) return launch_gemv<T, M, 2, true>(a, pdl, st);
+  if (a.act >= 3) return launch_gemv<T, M, 2, true>(a, pdl, st);
   if (a.N >= 4 * warps) return launch_gemv<T, M, 4>(a, pdl, st);
   if (a.N >= warps) return launch_gemv<T, M, 2>(a, pdl, st);
   return launch_gemv<T, M, 1>(a, pdl, st);
@@ -471,7 +474,7 @@ template <typename T>
 cudaError_t pick_m(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
   if constexpr (sizeof(T) == 2) {
     const bool direct = a.norm_w != nullptr || ((reinterpret_cast<uintptr_t>(a.x) & 15) == 0 && a.ldx % 8 == 0);
-    if (a.vec && direct && mma_from(a) && (a.act != 3 || a.interleaved)) {
+    if (a.vec && direct && mma_from(a) && (a.act < 3 || a.interleaved)) {
       if (a.M <= 8) return launch_gemv_mma<T, 1>(a, pdl, st);
       return launch_gemv_mma<T, 2>(a, pdl, st);
     }
@@ -558,19 +561,63 @@ __global__ void __launch_bounds__(kThreads) moe_router_kernel(RouterArgs a) {
   }
 }
 
+struct SoftRouterArgs {
+  const void* h;         // T [tokens, ldh], normed
+  const void* w;         // T [E (+ 1), K]: the last row gates a shared expert
+  float* weights;        // [tokens, k (+ 1)]
+  int64_t* idx;          // [tokens, k (+ 1)]; the shared expert is number E
+  int64_t ldh;
+  float scale;
+  int K, E, k, groups, keep, shared, vec, kp;
+};
+
+template <typename T>
+__global__ void __launch_bounds__(kThreads) moe_soft_router_kernel(SoftRouterArgs a) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  __shared__ float red[kWarps];
+  T* sx = reinterpret_cast<T*>(smem);
+  float* sc = reinterpret_cast<float*>(smem + (size_t)a.kp * sizeof(T));     // [E + 1] scores, [groups]
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, rows = a.E + a.shared;
+  pdl_launch_dependents();
+  if (a.vec && warp < rows && lane == 0)
+    prefetch_l2_bulk(reinterpret_cast<const T*>(a.w) + (int64_t)warp * a.K, (uint32_t)(a.K * sizeof(T)));
+  pdl_wait();
+  stage_rows<T>(sx, a.kp, reinterpret_cast<const T*>(a.h) + (int64_t)t * a.ldh, 0, (const T*)nullptr, 0.f, 1, a.K, red);
+  for (int e = warp; e < rows; e += kWarps) {
+    const T* w[1] = {reinterpret_cast<const T*>(a.w) + (int64_t)e * a.K};
+    float acc[1][1] = {};
+    dot_rows<T, 1, 1>(w, sx, a.kp, a.K, a.vec != 0, lane, acc);
+    if (lane == 0) sc[e] = acc[0][0];
+  }
+  __syncthreads();
+  if (warp != 0) return;
+  const int kt = a.k + a.shared;
+  if (a.shared && lane == 0) {
+    a.weights[(int64_t)t * kt + a.k] = 1.0f / (1.0f + expf(-sc[a.E]));
+    a.idx[(int64_t)t * kt + a.k] = a.E;
+  }
+  softmax_grouped_topk(sc, sc + rows, a.E, a.groups, a.keep, a.k, a.scale, a.weights + (int64_t)t * kt,
+                       a.idx + (int64_t)t * kt, lane);
+}
+
 struct MoeArgs {
-  const float* x;          // glu: residual stream [tokens, K]
+  const void* x;           // glu: residual stream [tokens, K] (normed on the way), or finished rows of T (norm_w null)
   const void* norm_w;
   const void* w;           // glu: [E, 2I, K]; down: [E, N, I]
-  const void* y_in;        // down: [tokens * k, I]
-  void* out;               // glu: T [tokens * k, I]; down: fp32 residual [tokens, N], accumulated into
+  const void* y_in;        // down: [tokens * k, ldy]
+  void* out;               // glu: T [tokens * k, ldy]; down: fp32 [tokens, N], accumulated into or written
   const float* weights;    // [tokens, k]
   const int64_t* idx;      // [tokens, k]
   int64_t ldx, ldo;
   float eps, limit, alpha;
   int K, I, E, k, kp;
-  int interleaved;         // gate / up rows in alternating 16-row tiles, else gate rows then up rows
+  int tile;                // gate / up rows in alternating tiles of this many rows; 0: gate rows then up rows
   int vec;
+  int act;                 // glu: 2 clamped, on weighted inputs; 4 silu(gate) * up
+  const void* ws;          // the shared expert, number E of idx: glu [2 Is, K], down [N, Is]
+  int Is, vec_s, tile_s;
+  int64_t ldy;             // row stride of the hidden units (at least I and Is)
+  int weighted;            // down: weights applied here, results written instead of added
 };
 
 template <typename T>
@@ -583,20 +630,28 @@ __global__ void __launch_bounds__(kThreads) moe_glu_kernel(MoeArgs a) {
   pdl_launch_dependents();
   pdl_wait();
   const int e = (int)a.idx[slot];
-  stage_rows<T>(sx, a.kp, a.x + (int64_t)t * a.ldx, 0, reinterpret_cast<const T*>(a.norm_w), a.eps, 1, a.K, red);
-  const T* W = reinterpret_cast<const T*>(a.w) + (int64_t)e * 2 * a.I * a.K;
+  const bool shared = e == a.E;
+  const int64_t row = (int64_t)t * a.ldx;
+  stage_rows<T>(sx, a.kp, a.norm_w != nullptr ? (const void*)(reinterpret_cast<const float*>(a.x) + row)
+                                              : (const void*)(reinterpret_cast<const T*>(a.x) + row),
+                0, reinterpret_cast<const T*>(a.norm_w), a.eps, 1, a.K, red);
+  const T* W = shared ? reinterpret_cast<const T*>(a.ws) : reinterpret_cast<const T*>(a.w) + (int64_t)e * 2 * a.I * a.K;
+  const int I = shared ? a.Is : a.I, tile = shared ? a.tile_s : a.tile;
+  const bool vec = shared ? a.vec_s != 0 : a.vec != 0;
   const float rw = a.weights[slot];
-  for (int i = blockIdx.x * kWarps + warp; i < a.I; i += gridDim.x * kWarps) {
-    const int g = a.interleaved ? (i >> 4) * 32 + (i & 15) : i;
-    const int u = a.interleaved ? g + 16 : a.I + i;
+  for (int i = blockIdx.x * kWarps + warp; i < I; i += gridDim.x * kWarps) {
+    const int g = tile > 0 ? i / tile * 2 * tile + i % tile : i;
+    const int u = tile > 0 ? g + tile : I + i;
     const T* w[2] = {W + (int64_t)g * a.K, W + (int64_t)u * a.K};
     float acc[1][2] = {};
-    dot_rows<T, 1, 2>(w, sx, a.kp, a.K, a.vec != 0, lane, acc);
-    if (lane == 0) {
+    dot_rows<T, 1, 2>(w, sx, a.kp, a.K, vec, lane, acc);
+    if (lane == 0 && a.act == 4) {
+      reinterpret_cast<T*>(a.out)[(int64_t)slot * a.ldy + i] = DT<T>::from_f(silu(acc[0][0]) * acc[0][1]);
+    } else if (lane == 0) {
       const float gv = fminf(acc[0][0] * rw, a.limit);
       const float uv = fminf(fmaxf(acc[0][1] * rw, -a.limit), a.limit);
       const float y = gv / (1.0f + expf(-a.alpha * gv)) * (uv + 1.0f);
-      reinterpret_cast<T*>(a.out)[(int64_t)slot * a.I + i] = DT<T>::from_f(y);
+      reinterpret_cast<T*>(a.out)[(int64_t)slot * a.ldy + i] = DT<T>::from_f(y);
     }
   }
 }
@@ -609,24 +664,30 @@ __global__ void __launch_bounds__(kThreads) moe_down_kernel(MoeArgs a) {
   const int t = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   pdl_launch_dependents();
   pdl_wait();
-  stage_rows<T>(sx, a.kp, reinterpret_cast<const T*>(a.y_in) + (int64_t)t * a.k * a.I, a.I, (const T*)nullptr, 0.f,
-                a.k, a.I, red);
+  const T* y = reinterpret_cast<const T*>(a.y_in) + (int64_t)t * a.k * a.ldy;
+  const int own = a.Is > 0 ? a.k - 1 : a.k;            // a shared expert is the last choice
+  stage_rows<T>(sx, a.kp, y, a.ldy, (const T*)nullptr, 0.f, own, a.I, red);
+  if (own < a.k)
+    stage_rows<T>(sx + (size_t)own * a.kp, a.kp, y + own * a.ldy, 0, (const T*)nullptr, 0.f, 1, a.Is, red);
   const int N = a.K;
   for (int n2 = blockIdx.x * kWarps + warp; n2 * 2 < N; n2 += gridDim.x * kWarps) {
     const int n = n2 * 2;
     float s0 = 0.f, s1 = 0.f;
     for (int j = 0; j < a.k; ++j) {
-      const int64_t e = a.idx[(int64_t)t * a.k + j];
-      const T* We = reinterpret_cast<const T*>(a.w) + e * (int64_t)N * a.I;
-      const T* w[2] = {We + (int64_t)n * a.I, We + (int64_t)min(n + 1, N - 1) * a.I};
+      const bool shared = j >= own;
+      const int I = shared ? a.Is : a.I;
+      const T* We = shared ? reinterpret_cast<const T*>(a.ws)
+                           : reinterpret_cast<const T*>(a.w) + a.idx[(int64_t)t * a.k + j] * (int64_t)N * I;
+      const T* w[2] = {We + (int64_t)n * I, We + (int64_t)min(n + 1, N - 1) * I};
       float acc[1][2] = {};
-      dot_rows<T, 1, 2>(w, sx + (size_t)j * a.kp, a.kp, a.I, a.vec != 0, lane, acc);
-      s0 += acc[0][0];
-      s1 += acc[0][1];
+      dot_rows<T, 1, 2>(w, sx + (size_t)j * a.kp, a.kp, I, shared ? a.vec_s != 0 : a.vec != 0, lane, acc);
+      const float f = a.weighted ? a.weights[(int64_t)t * a.k + j] : 1.0f;
+      s0 = fmaf(f, acc[0][0], s0);
+      s1 = fmaf(f, acc[0][1], s1);
     }
     float* o = reinterpret_cast<float*>(a.out) + (int64_t)t * a.ldo + n;
-    if (lane == 0) o[0] += s0;
-    if (lane == 1 && n + 1 < N) o[1] += s1;
+    if (lane == 0) o[0] = a.weighted ? s0 : o[0] + s0;
+    if (lane == 1 && n + 1 < N) o[1] = a.weighted ? s1 : o[1] + s1;
   }
 }
 
@@ -667,7 +728,7 @@ IPEX_API int ipex_gemv_rows_max(int K, int dtype) {
 IPEX_API void ipex_gemv_rows_tune(int mma_from_rows) { g_mma_from = mma_from_rows; }
 
 // y = act(x . W^T + bias): see GemvRowsArgs.  M <= ipex_gemv_rows_max(K, dtype).  w2 / out2 (may be null): N2 more
-// rows with the same row stride whose results go to out2 [M, ldo2] in fp32.  act 3: out_mode 0, N even (a multiple of
+// rows with the same row stride whose results go to out2 [M, ldo2] in fp32.  act 3, 4: out_mode 0, N even (a multiple of
 // 16 when interleaved), no second matrix.
 IPEX_API int ipex_gemv_rows(const void* w, int64_t ldw, const void* x, int64_t ldx, const void* norm_w, float eps,
                             const void* bias, void* out, int64_t ldo, const void* w2, int N2, float* out2, int64_t ldo2,
@@ -675,7 +736,7 @@ IPEX_API int ipex_gemv_rows(const void* w, int64_t ldw, const void* x, int64_t l
                             int pdl, void* stream) {
   if (M < 1 || N < 1 || K < 1 || out_mode < 0 || out_mode > 2 || M > ipex_gemv_rows_max(K, dtype))
     return (int)cudaErrorInvalidValue;
-  if (act < 0 || act == 2 || act > 3 || (act == 3 && (out_mode != 0 || (N % 2) || (interleaved && (N % 16)) || w2 != nullptr)) ||
+  if (act < 0 || act == 2 || act > 4 || (act >= 3 && (out_mode != 0 || (N % 2) || (interleaved && (N % 16)) || w2 != nullptr)) ||
       (w2 != nullptr && (N2 < 1 || out2 == nullptr)))
     return (int)cudaErrorInvalidValue;
   return by_dtype(dtype, [&](auto* tag) {
@@ -711,40 +772,68 @@ IPEX_API int ipex_moe_router_sigmoid(const float* x, int64_t ldx, const void* no
   });
 }
 
-// First half of the experts for `tokens` rows: y[token * k + j] = g * sigmoid(alpha g) * (u + 1), g = min(gate, limit),
-// u = clamp(up, +-limit), gate / up of expert idx[token, j] on weight * norm(x).
-IPEX_API int ipex_moe_glu_rows(const float* x, int64_t ldx, const void* norm_w, float eps, const void* w, void* y,
-                               const float* weights, const int64_t* idx, int tokens, int K, int I, int E, int k,
-                               float limit, float alpha, int interleaved, int dtype, int pdl, void* stream) {
-  if (tokens < 1 || K < 1 || I < 1 || k < 1 || (int64_t)tokens * k > 65535 || (interleaved && I % 16 != 0))
+// Router from finished rows h: soft-max over E experts, choice among the `keep` best of `groups` equal groups, weights
+// divided by their sum and times scale; shared: row E of w gates a shared expert, which becomes choice k (number E).
+IPEX_API int ipex_moe_router_softmax(const void* h, int64_t ldh, const void* w, float* weights, int64_t* idx, int tokens,
+                                     int K, int E, int groups, int keep, int k, int shared, float scale, int dtype, int pdl,
+                                     void* stream) {
+  if (tokens < 1 || K < 1 || E < 1 || k < 1 || groups < 1 || E % groups || keep < 1 || keep > groups || k > E / groups * keep)
+    return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    SoftRouterArgs a = {h, w, weights, idx, ldh, scale, K, E, k, groups, keep, shared != 0, vec_ok<T>(w, K, K), padded<T>(K)};
+    const size_t smem = (size_t)a.kp * sizeof(T) + ((size_t)E + 1 + groups) * sizeof(float);
+    cudaError_t e = allow_smem(moe_soft_router_kernel<T>, smem);
+    if (e != cudaSuccess) return e;
+    return launch_kernel(moe_soft_router_kernel<T>, dim3(tokens), dim3(kThreads), smem, (cudaStream_t)stream, pdl != 0, a);
+  });
+}
+
+// First half of the experts for `tokens` rows.  act 2: y[token * k + j] = g * sigmoid(alpha g) * (u + 1), g = min(gate,
+// limit), u = clamp(up, +-limit), gate / up of expert idx[token, j] on weight * norm(x).  act 4: silu(gate) * up of
+// finished rows x (norm_w null).  ws (may be null): the shared expert's rows, [2 Is, K]; tile / tile_s: see MoeArgs.
+IPEX_API int ipex_moe_glu_rows(const void* x, int64_t ldx, const void* norm_w, float eps, const void* w, const void* ws,
+                               void* y, int64_t ldy, const float* weights, const int64_t* idx, int tokens, int K, int I,
+                               int Is, int E, int k, int act, float limit, float alpha, int tile, int tile_s, int dtype,
+                               int pdl, void* stream) {
+  if (tokens < 1 || K < 1 || I < 1 || k < 1 || (int64_t)tokens * k > 65535 || tile < 0 || (tile > 0 && I % tile != 0) ||
+      Is < 0 || (Is > 0 && (ws == nullptr || act != 4)) || tile_s < 0 || (tile_s > 0 && Is % tile_s != 0) || ldy < I ||
+      ldy < Is || (act != 2 && act != 4) || (act == 2) != (norm_w != nullptr))
     return (int)cudaErrorInvalidValue;
   return by_dtype(dtype, [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
     MoeArgs a = {};
     a.x = x; a.norm_w = norm_w; a.w = w; a.out = y; a.weights = weights; a.idx = idx; a.ldx = ldx; a.eps = eps;
-    a.limit = limit; a.alpha = alpha; a.K = K; a.I = I; a.E = E; a.k = k; a.kp = padded<T>(K);
-    a.interleaved = interleaved;
+    a.limit = limit; a.alpha = alpha; a.K = K; a.I = I; a.E = E; a.k = k; a.kp = padded<T>(K); a.act = act;
+    a.ws = ws; a.Is = Is; a.ldy = ldy; a.tile = tile; a.tile_s = tile_s;
     a.vec = vec_ok<T>(w, K, K);
+    a.vec_s = ws != nullptr && vec_ok<T>(ws, K, K);
     const size_t smem = (size_t)a.kp * sizeof(T);
     cudaError_t e = allow_smem(moe_glu_kernel<T>, smem);
     if (e != cudaSuccess) return e;
-    const int slots = tokens * k, want = (I + kWarps - 1) / kWarps;
+    const int slots = tokens * k, want = ((I > Is ? I : Is) + kWarps - 1) / kWarps;
     const int cap = (sm_count() * 4 + slots - 1) / slots;
     return launch_kernel(moe_glu_kernel<T>, dim3(want < cap ? want : cap, slots), dim3(kThreads), smem,
                          (cudaStream_t)stream, pdl != 0, a);
   });
 }
 
-// Second half: residual[token] += sum_j down_{idx[token, j]}(y[token * k + j]).
-IPEX_API int ipex_moe_down_rows(const void* y, const void* w, float* residual, int64_t ldr, const int64_t* idx,
-                                int tokens, int N, int I, int E, int k, int dtype, int pdl, void* stream) {
-  if (tokens < 1 || tokens > 65535 || N < 1 || I < 1 || k < 1) return (int)cudaErrorInvalidValue;
+// Second half: out[token] += sum_j down_{idx[token, j]}(y[token * k + j]); with weights: out[token] = the weighted sum.
+// ws (may be null): the shared expert's rows, [N, Is]; it is then the last of the k choices.
+IPEX_API int ipex_moe_down_rows(const void* y, int64_t ldy, const void* w, const void* ws, const float* weights, float* out,
+                                int64_t ldo, const int64_t* idx, int tokens, int N, int I, int Is, int E, int k, int dtype,
+                                int pdl, void* stream) {
+  if (tokens < 1 || tokens > 65535 || N < 1 || I < 1 || k < 1 || Is < 0 || (Is > 0 && (ws == nullptr || k < 2)) ||
+      ldy < I || ldy < Is)
+    return (int)cudaErrorInvalidValue;
   return by_dtype(dtype, [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
     MoeArgs a = {};
-    a.y_in = y; a.w = w; a.out = residual; a.idx = idx; a.ldo = ldr; a.K = N; a.I = I; a.E = E; a.k = k;
-    a.kp = padded<T>(I);
+    a.y_in = y; a.w = w; a.out = out; a.idx = idx; a.ldo = ldo; a.K = N; a.I = I; a.E = E; a.k = k;
+    a.kp = padded<T>(I > Is ? I : Is);
+    a.weights = weights; a.weighted = weights != nullptr; a.ws = ws; a.Is = Is; a.ldy = ldy;
     a.vec = vec_ok<T>(w, I, I);
+    a.vec_s = ws != nullptr && vec_ok<T>(ws, Is, Is);
     const size_t smem = (size_t)a.kp * k * sizeof(T);
     cudaError_t e = allow_smem(moe_down_kernel<T>, smem);
     if (e != cudaSuccess) return e;

@@ -1,9 +1,12 @@
-// Windowed attention over cached keys and values of different sizes, with an optional sink and mixed values, sm_100a.
+// Attention over cached keys and values of different sizes, sm_100a: everything earlier, a sliding window or the query's
+// own chunk of positions, with an optional sink (a score of 0 or one learned number per head), mixed values, rotated and
+// unit-normed queries and keys, and gated outputs.
 //
+//   qk_prepare  rotation and unit norm of the query and key heads of many tokens in place (prompts, portions)
 //   kv_append   keys and values of the new tokens into the cache, the values mixed with those of an earlier layer;
 //               for prompts also the transposed values that the tcgen05 prompt attention reads
-//   kv_attn     attention of query tokens against what their slots hold: decoding (which appends its own row on the
-//               way), portions of prompts, and whole prompts of sizes or formats the tensor-core kernel does not take
+//   kv_attn     attention of query tokens against what their slots hold: decoding (which prepares and appends its own
+//               row on the way), portions of prompts, and whole prompts of sizes or formats the tensor-core kernel does not take
 //
 // kv_attn: a cluster of up to eight CTAs shares the visible keys of one query token for up to RT query heads of one key
 // head.  A CTA walks its keys in tiles: eight lanes share a key for the scores (every lane has four keys in flight), the
@@ -47,6 +50,53 @@ __device__ __forceinline__ void load_pack(const T* p, float (&f)[Pack<T, VEC>::n
 }
 
 __device__ __forceinline__ float mixed(float v, float first, float lambda) { return (1.0f - lambda) * v + lambda * first; }
+
+// ---------------------------------------------------------------------------------------------- rotation and unit norm
+struct Prepare {
+  const float* cosp;    // [positions, half], row = position in the sequence
+  const float* sinp;
+  int half;             // pairs (i, i + half) of a head turn
+  int unit;             // divide by the root mean square
+  float eps;
+};
+
+// One vector by one warp; load(i) / store(i, value) for its elements.  The norm does not change under the rotation, so
+// it is taken first and every lane finishes its own pairs.
+template <typename L, typename S>
+__device__ __forceinline__ void prepare_vector(const Prepare& p, int dim, int rel, float scale, int lane, L&& load, S&& store) {
+  float f = scale;
+  if (p.unit) {
+    float ss = 0.f;
+    for (int i = lane; i < dim; i += 32) {
+      const float x = load(i);
+      ss = fmaf(x, x, ss);
+    }
+    f = scale / sqrtf(warp_sum(ss) / (float)dim + p.eps);
+  }
+  const float* cp = p.cosp + (int64_t)rel * p.half;
+  const float* sp = p.sinp + (int64_t)rel * p.half;
+  for (int i = lane; i < p.half; i += 32) {
+    const float u = load(i), v = load(i + p.half), c = cp[i], s = sp[i];
+    store(i, (u * c - v * s) * f);
+    store(i + p.half, (v * c + u * s) * f);
+  }
+  for (int i = 2 * p.half + lane; i < dim; i += 32) store(i, load(i) * f);
+}
+
+// A warp per (token, head) of x: rows of `ld`, heads behind one another.
+template <typename T>
+__global__ void __launch_bounds__(kThreads) qk_prepare_kernel(T* __restrict__ x, int64_t ld, const int* __restrict__ slot,
+                                                              const int* __restrict__ pos, const int* __restrict__ start,
+                                                              Prepare p, int64_t rows, int heads, int dim) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t r = (int64_t)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
+  if (r >= rows) return;
+  const int t = (int)(r / heads), h = (int)(r % heads);
+  T* v = x + (int64_t)t * ld + (int64_t)h * dim;
+  prepare_vector(p, dim, pos[t] - start[slot[t]], 1.0f, threadIdx.x & 31, [&](int i) { return DT<T>::to_f(v[i]); },
+                 [&](int i, float y) { v[i] = DT<T>::from_f(y); });
+}
 
 // ---------------------------------------------------------------------------------------------- append
 struct AppendArgs {
@@ -154,25 +204,14 @@ struct AttnArgs {
   int64_t ldq, ld_vf, ldo, k_slot, k_head, v_slot, v_head;
   float lambda, scale;
   int heads, kv_heads, dim, vdim, window, sink, append;
+  int chunk;            // keys of the query's own chunk of this many positions only; 0: all
+  const float* sinks;   // [heads] scores of the sink; null: 0
+  const void* gate;     // T [tokens, ldg], head h at h * vdim, or null: outputs times gate_scale * sigmoid(gate)
+  int64_t ldg;
+  float gate_scale;
+  Prepare prep;
+  int prepare;          // with append: queries and the new key are rotated / normed here
 };
-
-// N values on each of 8 lanes (a power of two) -> sums over the 8 lanes, spread so that a lane keeps max(1, N / 8) of
-// them: value i ends on the lanes whose id matches, in the order of the folds
-template <int N, int OFF>
-__device__ __forceinline__ void fold(float* v, int lane) {
-  if constexpr (N > 1) {
-    const bool up = lane & OFF;
-#pragma unroll
-    for (int i = 0; i < N / 2; ++i) {
-      const float keep = up ? v[i + N / 2] : v[i], give = up ? v[i] : v[i + N / 2];
-      v[i] = keep + __shfl_xor_sync(0xffffffffu, give, OFF);
-    }
-    if constexpr (OFF > 1) fold<N / 2, OFF / 2>(v, lane);
-  } else {
-    v[0] += __shfl_xor_sync(0xffffffffu, v[0], OFF);
-    if constexpr (OFF > 1) fold<1, OFF / 2>(v, lane);
-  }
-}
 
 template <typename T, int RT, bool VEC>
 __global__ void __launch_bounds__(kThreads) kv_attn_kernel(AttnArgs a, int nrb) {
@@ -184,8 +223,8 @@ __global__ void __launch_bounds__(kThreads) kv_attn_kernel(AttnArgs a, int nrb) 
   const int R = a.heads / a.kv_heads, r0 = rb * RT, rows = min(RT, R - r0);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int dimp = (a.dim + 3) & ~3;
-  float* sq = sm;                                // [RT][dimp] scaled queries
-  float* ss = sq + RT * dimp;                    // [RT][kTile] scores, then weights
+  float* sq = sm;                                // [RT + 1][dimp] scaled queries, the new key
+  float* ss = sq + (RT + 1) * dimp;              // [RT][kTile] scores, then weights
   float* sc = ss + RT * kTile;                   // [RT] factor of what was gathered before this tile
   float* sml = sc + RT;                          // [RT][2] maximum and sum
   float* so = sml + 2 * RT;                      // [RT][vdim] this CTA's part of the output
@@ -193,7 +232,9 @@ __global__ void __launch_bounds__(kThreads) kv_attn_kernel(AttnArgs a, int nrb) 
   pdl_launch_dependents();
   pdl_wait();
   const int slot = a.slot[tok], pos = a.pos[tok], start = a.start[slot];
-  const int lo = max(start, a.window > 0 ? pos - a.window + 1 : 0), n = pos + 1 - lo;
+  int lo = max(start, a.window > 0 ? pos - a.window + 1 : 0);
+  if (a.chunk > 0) lo = max(lo, pos - (pos - start) % a.chunk);
+  const int n = pos + 1 - lo;
   const int chunk = (n + nsplit - 1) / nsplit;
   const int j0 = lo + min(n, split * chunk), j1 = lo + min(n, (split + 1) * chunk);
   T* kc = reinterpret_cast<T*>(a.kc) + (int64_t)slot * a.k_slot + (int64_t)g * a.k_head;
@@ -204,7 +245,18 @@ __global__ void __launch_bounds__(kThreads) kv_attn_kernel(AttnArgs a, int nrb) 
     const T* k = reinterpret_cast<const T*>(a.k) + (int64_t)tok * a.ldq + (int64_t)g * a.dim;
     const T* v = reinterpret_cast<const T*>(a.v) + (int64_t)tok * a.ldq + (int64_t)g * a.vdim;
     const T* vf = reinterpret_cast<const T*>(a.vfirst) + (int64_t)tok * a.ld_vf + (int64_t)g * a.vdim;
-    for (int i = tid; i < a.dim; i += kThreads) kc[(int64_t)pos * a.dim + i] = k[i];
+    if (a.prepare) {
+      if (warp == RT % (kThreads / 32)) {
+        float* sk = sq + RT * dimp;
+        for (int i = lane; i < a.dim; i += 32) sk[i] = DT<T>::to_f(k[i]);
+        __syncwarp();
+        T* dst = kc + (int64_t)pos * a.dim;
+        prepare_vector(a.prep, a.dim, pos - start, 1.0f, lane, [&](int i) { return sk[i]; },
+                       [&](int i, float y) { dst[i] = DT<T>::from_f(y); });
+      }
+    } else {
+      for (int i = tid; i < a.dim; i += kThreads) kc[(int64_t)pos * a.dim + i] = k[i];
+    }
     for (int i = tid; i < a.vdim; i += kThreads) {
       const float own = DT<T>::to_f(v[i]);
       vc[(int64_t)pos * a.vdim + i] =
@@ -213,9 +265,20 @@ __global__ void __launch_bounds__(kThreads) kv_attn_kernel(AttnArgs a, int nrb) 
   }
   {
     const T* q = reinterpret_cast<const T*>(a.q) + (int64_t)tok * a.ldq + (int64_t)(g * R + r0) * a.dim;
-    for (int i = tid; i < RT * a.dim; i += kThreads) {
-      const int r = i / a.dim, c = i % a.dim;
-      sq[r * dimp + c] = r < rows ? DT<T>::to_f(q[(int64_t)r * a.dim + c]) * a.scale : 0.f;
+    if (a.prepare) {
+      if (warp < RT) {
+        float* dst = sq + warp * dimp;
+        for (int i = lane; i < a.dim; i += 32) dst[i] = warp < rows ? DT<T>::to_f(q[(int64_t)warp * a.dim + i]) : 0.f;
+        __syncwarp();
+        if (warp < rows)
+          prepare_vector(a.prep, a.dim, pos - start, a.scale, lane, [&](int i) { return dst[i]; },
+                         [&](int i, float y) { dst[i] = y; });
+      }
+    } else {
+      for (int i = tid; i < RT * a.dim; i += kThreads) {
+        const int r = i / a.dim, c = i % a.dim;
+        sq[r * dimp + c] = r < rows ? DT<T>::to_f(q[(int64_t)r * a.dim + c]) * a.scale : 0.f;
+      }
     }
   }
   __syncthreads();
@@ -355,12 +418,13 @@ __global__ void __launch_bounds__(kThreads) kv_attn_kernel(AttnArgs a, int nrb) 
   T* out = reinterpret_cast<T*>(a.out) + (int64_t)tok * a.ldo + (int64_t)(g * R + r0) * a.vdim;
   for (int i = split * kThreads + tid; i < rows * a.vdim; i += nsplit * kThreads) {
     const int r = i / a.vdim;
-    float m = a.sink ? 0.f : -INFINITY;
+    const float zs = a.sinks != nullptr ? a.sinks[g * R + r0 + r] : 0.f;
+    float m = a.sink ? zs : -INFINITY;
     for (int s = 0; s < nsplit; ++s) {
       const float* p = nsplit > 1 ? cluster.map_shared_rank(sml, s) : sml;
       m = fmaxf(m, p[2 * r]);
     }
-    float l = a.sink ? expf(-m) : 0.f, o = 0.f;
+    float l = a.sink ? expf(zs - m) : 0.f, o = 0.f;
     for (int s = 0; s < nsplit; ++s) {
       const float* p = nsplit > 1 ? cluster.map_shared_rank(sml, s) : sml;
       const float* po = nsplit > 1 ? cluster.map_shared_rank(so, s) : so;
@@ -368,7 +432,12 @@ __global__ void __launch_bounds__(kThreads) kv_attn_kernel(AttnArgs a, int nrb) 
       l = fmaf(p[2 * r + 1], c, l);
       o = fmaf(po[i], c, o);
     }
-    out[i] = DT<T>::from_f(l > 0.f ? o / l : 0.f);
+    o = l > 0.f ? o / l : 0.f;
+    if (a.gate != nullptr) {
+      const float z = DT<T>::to_f(reinterpret_cast<const T*>(a.gate)[(int64_t)tok * a.ldg + (int64_t)(g * R + r0) * a.vdim + i]);
+      o *= a.gate_scale / (1.0f + expf(-z));
+    }
+    out[i] = DT<T>::from_f(o);
   }
   if (nsplit > 1) cluster.sync();      // the others may still read this CTA's part
 }
@@ -378,7 +447,7 @@ cudaError_t launch_attn(const AttnArgs& a, int tokens, int nsplit, bool pdl, cud
   constexpr int VN = Pack<T, VEC>::n;
   const int dimp = (a.dim + 3) & ~3, vp = (a.vdim + 3) & ~3, R = a.heads / a.kv_heads;
   const int nrb = (R + RT - 1) / RT, subsets = kThreads / (a.vdim / VN);
-  const size_t smem = ((size_t)RT * (dimp + kTile + 3 + vp) + (size_t)subsets * RT * a.vdim + 4) * sizeof(float);
+  const size_t smem = ((size_t)RT * (dimp + kTile + 3 + vp) + dimp + (size_t)subsets * RT * a.vdim + 4) * sizeof(float);
   if (smem > 220 * 1024 || (int64_t)a.kv_heads * nrb > 65535) return cudaErrorInvalidValue;
   auto kern = kv_attn_kernel<T, RT, VEC>;
   if (smem > 40 * 1024) {
@@ -445,24 +514,47 @@ IPEX_API int ipex_kv_append(const void* k, const void* v, int64_t ld, const void
   });
 }
 
+// Queries and keys of many tokens in place, x [tokens, ld] with `heads` of `dim`: pairs (i, i + half) turn by the tables'
+// angles for the token's place in its sequence; unit: divided by sqrt(mean square + eps).
+IPEX_API int ipex_qk_prepare(void* x, int64_t ld, const int* slot, const int* pos, const int* start, const float* cosp,
+                             const float* sinp, int half, int unit, float eps, int tokens, int heads, int dim, int dtype,
+                             int pdl, void* stream) {
+  if (tokens < 1 || heads < 1 || dim < 1 || half < 0 || 2 * half > dim || (half > 0 && (cosp == nullptr || sinp == nullptr)))
+    return (int)cudaErrorInvalidValue;
+  const int64_t rows = (int64_t)tokens * heads, blocks = (rows + kThreads / 32 - 1) / (kThreads / 32);
+  if (blocks > 0x7fffffff) return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    const Prepare p = {cosp, sinp, half, unit, eps};
+    return launch_kernel(qk_prepare_kernel<T>, dim3((unsigned)blocks), dim3(kThreads), 0, (cudaStream_t)stream, pdl != 0,
+                         (T*)x, ld, slot, pos, start, p, rows, heads, dim);
+  });
+}
+
 // Attention of `tokens` query tokens (q: rows of ldq elements, `heads` of `dim`) over positions
-// [max(start, pos - window + 1), pos] of their slots; window 0: unlimited.  append: file the tokens' own rows k / v
-// (same row stride as q, v mixed with vfirst) first - then no two tokens may share a slot; otherwise the cache holds
-// them.  nsplit: CTAs (1, 2, 4 or 8) the keys of a token are shared by.  sink: a score of 0 without a value in every
-// softmax.
+// [max(start, pos - window + 1), pos] of their slots (window 0: unlimited; chunk > 0: those of the query's own chunk, counted
+// from start).  append: file the tokens' own rows k / v (same row stride as q, v mixed with vfirst) first - then no two
+// tokens may share a slot; otherwise the cache holds them.  prepare (with append): queries and new keys are rotated and
+// normed on the way (see ipex_qk_prepare).  nsplit: CTAs (1, 2, 4 or 8) the keys of a token are shared by.  sink: one more
+// score without a value in every softmax, 0 or sinks[head].  gate (may be null): outputs times gate_scale * sigmoid.
 IPEX_API int ipex_kv_attn(const void* q, const void* k, const void* v, int64_t ldq, const void* vfirst, int64_t ld_vf,
                           float lambda, void* kc, int64_t k_slot, int64_t k_head, void* vc, int64_t v_slot,
                           int64_t v_head, void* out, int64_t ldo, const int* slot, const int* pos, const int* start,
-                          int tokens, int heads, int kv_heads, int dim, int vdim, int window, int sink, int append,
-                          int nsplit, float scale, int dtype, int pdl, void* stream) {
-  if (tokens < 1 || tokens > 65535 || kv_heads < 1 || heads % kv_heads != 0 || dim < 1 || vdim < 1 || window < 0 ||
+                          int tokens, int heads, int kv_heads, int dim, int vdim, int window, int chunk, int sink,
+                          const float* sinks, const void* gate, int64_t ldg, float gate_scale, int append, int prepare,
+                          const float* cosp, const float* sinp, int half, int unit, float eps, int nsplit, float scale,
+                          int dtype, int pdl, void* stream) {
+  if (tokens < 1 || tokens > 65535 || kv_heads < 1 || heads % kv_heads != 0 || dim < 1 || vdim < 1 || window < 0 || chunk < 0 ||
       nsplit < 1 || nsplit > 8 || (nsplit & (nsplit - 1)))
+    return (int)cudaErrorInvalidValue;
+  if (prepare && (!append || half < 0 || 2 * half > dim || (half > 0 && (cosp == nullptr || sinp == nullptr))))
     return (int)cudaErrorInvalidValue;
   return by_dtype(dtype, [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
     constexpr int VN = 16 / (int)sizeof(T);
     AttnArgs a = {q, k, v, vfirst, kc, vc, out, slot, pos, start, ldq, ld_vf, ldo, k_slot, k_head, v_slot, v_head,
-                  lambda, scale, heads, kv_heads, dim, vdim, window, sink, append};
+                  lambda, scale, heads, kv_heads, dim, vdim, window, sink, append, chunk, sinks, gate, ldg, gate_scale,
+                  {cosp, sinp, half, unit, eps}, prepare};
     const bool vec = dim % VN == 0 && vdim % VN == 0 && vdim / VN <= kThreads && (((uintptr_t)kc | (uintptr_t)vc) & 15) == 0;
     cudaStream_t st = (cudaStream_t)stream;
     if (vec) return pick_rows<T, true>(a, tokens, nsplit, pdl != 0, st);

@@ -51,7 +51,8 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 }
 
 struct PrepArgs {
-  void* qkv;            // T [M, ldq]: per head [dim | rd] queries, then R latents, then rd key values
+  void* q;              // T [M, ldq]: per head [dim | rd]
+  const void* kv;       // T [M, ldkv]: R latents, then rd key values; null: the cache holds the tokens' rows already
   const void* norm_w;   // T [R]
   const void* w_uk;     // T [H * dim, R]
   const float* cosp;    // [positions, half]
@@ -63,7 +64,7 @@ struct PrepArgs {
   void* qabs;           // T [M, H, R]
   void* c_out;          // prompt path: T [M, ld_c]
   void* kr_out;         // prompt path: T [M, ld_kr]
-  int64_t ldq, slot_stride, ldc, ld_c, ld_kr;
+  int64_t ldq, ldkv, slot_stride, ldc, ld_c, ld_kr;
   float eps;
   int M, H, dim, rd, R, half;
 };
@@ -79,7 +80,7 @@ __device__ __forceinline__ void rotate_pair(T* v, int i, int half, float c, floa
 // norm of the latent part, rotation of the key part, append to the cache (whole block, one token)
 template <typename T>
 __device__ void append_token(const PrepArgs& a, int m, float* red) {
-  const T* row = reinterpret_cast<const T*>(a.qkv) + (int64_t)m * a.ldq + (int64_t)a.H * (a.dim + a.rd);
+  const T* row = reinterpret_cast<const T*>(a.kv) + (int64_t)m * a.ldkv;
   const T* nw = reinterpret_cast<const T*>(a.norm_w);
   const int s = a.slot[m], p = a.pos[m], rel = p - a.start[s];
   T* dst = reinterpret_cast<T*>(a.cache) + (int64_t)s * a.slot_stride + (int64_t)p * a.ldc;
@@ -110,7 +111,8 @@ __device__ void append_token(const PrepArgs& a, int m, float* red) {
 constexpr int kPrepThreads = 256;
 constexpr int kPrepCols = 128;     // latent columns per block
 
-// grid (H * column blocks + 1, token groups of MT): the last x block appends the group's tokens to the cache.
+// grid (H * column blocks + 1, token groups of MT): the last x block appends the group's tokens to the cache (and is not
+// launched when there is nothing to append).
 template <typename T, int V, int MT>
 __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(PrepArgs a) {
   __shared__ float red[kPrepThreads / 32];
@@ -127,7 +129,7 @@ __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(PrepArgs a) {
     return;
   }
   const int h = blockIdx.x / cb, c0 = (blockIdx.x % cb) * kPrepCols;
-  T* q0 = reinterpret_cast<T*>(a.qkv) + (int64_t)m0 * a.ldq + (int64_t)h * (a.dim + a.rd);
+  T* q0 = reinterpret_cast<T*>(a.q) + (int64_t)m0 * a.ldq + (int64_t)h * (a.dim + a.rd);
   if (c0 == 0) {
     for (int i = threadIdx.x; i < mn * a.half; i += kPrepThreads) {
       const int m = i / a.half, j = i % a.half;
@@ -189,14 +191,14 @@ __global__ void __launch_bounds__(256) latent_prompt_prep_kernel(PrepArgs a) {
   const int m = blockIdx.x;
   pdl_launch_dependents();
   pdl_wait();
-  T* q = reinterpret_cast<T*>(a.qkv) + (int64_t)m * a.ldq;
+  T* q = reinterpret_cast<T*>(a.q) + (int64_t)m * a.ldq;
   const int64_t rel = a.pos[m] - a.start[a.slot[m]];
   for (int i = threadIdx.x; i < a.H * a.half; i += blockDim.x) {
     const int h = i / a.half, j = i % a.half;
     rotate_pair<T>(q + (int64_t)h * (a.dim + a.rd) + a.dim, j, a.half, a.cosp[rel * a.half + j],
                    a.sinp[rel * a.half + j]);
   }
-  append_token<T>(a, m, red);
+  if (a.kv != nullptr) append_token<T>(a, m, red);
 }
 
 struct LatentAttnArgs {
@@ -485,6 +487,8 @@ struct UvArgs {
   void* out;            // T [M, ldo], head h at h * vd
   int64_t ldo;
   int M, H, R, vd, nsplit, rows_per_block;
+  const void* gate;     // T [M, ldg], head h at h * vd, or null: outputs times sigmoid(gate)
+  int64_t ldg;
 };
 
 constexpr int kUvThreads = 256;
@@ -590,9 +594,12 @@ __global__ void __launch_bounds__(kUvThreads) latent_uv_kernel(UvArgs a) {
     for (int q = 0; q < RW; ++q)
 #pragma unroll
       for (int mm = 0; mm < MT; ++mm) {
-        const float s = warp_sum(acc[q][mm]);
-        if (lane == q * MT + mm && mm < mn && v + q < v1)
+        float s = warp_sum(acc[q][mm]);
+        if (lane == q * MT + mm && mm < mn && v + q < v1) {
+          if (a.gate != nullptr)
+            s /= 1.0f + expf(-DT<T>::to_f(reinterpret_cast<const T*>(a.gate)[(int64_t)(m0 + mm) * a.ldg + (int64_t)h * a.vd + v + q]));
           reinterpret_cast<T*>(a.out)[(int64_t)(m0 + mm) * a.ldo + (int64_t)h * a.vd + v + q] = DT<T>::from_f(s);
+        }
       }
   }
 }
@@ -611,7 +618,7 @@ cudaError_t launch_prep(const PrepArgs& a, bool pdl, cudaStream_t st) {
   cudaError_t e = allow_smem(kern, smem);
   if (e != cudaSuccess) return e;
   const int cb = (a.R + kPrepCols - 1) / kPrepCols;
-  return launch_kernel(kern, dim3(a.H * cb + 1, (a.M + MT - 1) / MT), dim3(kPrepThreads), smem, st, pdl, a);
+  return launch_kernel(kern, dim3(a.H * cb + (a.kv != nullptr), (a.M + MT - 1) / MT), dim3(kPrepThreads), smem, st, pdl, a);
 }
 
 template <typename T, int V, int MT>
@@ -625,8 +632,8 @@ cudaError_t launch_uv(UvArgs& a, int blocks_y, bool pdl, cudaStream_t st) {
 
 }  // namespace
 
-// Before the absorbed attention of M query tokens; see PrepArgs.  half: rotated pairs (2 * half <= rd).
-IPEX_API int ipex_latent_prep(void* qkv, int64_t ldq, const void* norm_w, float eps, const void* w_uk, const float* cosp,
+// Before the absorbed attention of M query tokens; see PrepArgs (kv null: queries only).  half: rotated pairs (2 * half <= rd).
+IPEX_API int ipex_latent_prep(void* q, int64_t ldq, const void* kv, int64_t ldkv, const void* norm_w, float eps, const void* w_uk, const float* cosp,
                               const float* sinp, const int* slot, const int* pos, const int* start, void* cache,
                               int64_t slot_stride, int64_t ldc, void* qabs, int M, int H, int dim, int rd, int R,
                               int half, int dtype, int pdl, void* stream) {
@@ -634,7 +641,7 @@ IPEX_API int ipex_latent_prep(void* qkv, int64_t ldq, const void* norm_w, float 
     return (int)cudaErrorInvalidValue;
   return by_dtype(dtype, [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
-    PrepArgs a = {qkv, norm_w, w_uk, cosp, sinp, slot, pos, start, cache, qabs, nullptr, nullptr, ldq, slot_stride, ldc,
+    PrepArgs a = {q, kv, norm_w, w_uk, cosp, sinp, slot, pos, start, cache, qabs, nullptr, nullptr, ldq, ldkv, slot_stride, ldc,
                   0, 0, eps, M, H, dim, rd, R, half};
     cudaStream_t st = (cudaStream_t)stream;
     const bool vec = R % Vec<T>::n == 0 && (reinterpret_cast<uintptr_t>(w_uk) & 15) == 0;
@@ -644,17 +651,18 @@ IPEX_API int ipex_latent_prep(void* qkv, int64_t ldq, const void* norm_w, float 
 }
 
 // Before the prompt attention: rotates the queries in place, appends to the cache, writes contiguous latents
-// c_out [M, ld_c] and rotated key parts kr_out [M, ld_kr].
-IPEX_API int ipex_latent_prompt_prep(void* qkv, int64_t ldq, const void* norm_w, float eps, const float* cosp,
+// c_out [M, ld_c] and rotated key parts kr_out [M, ld_kr] (kv null: the queries only).
+IPEX_API int ipex_latent_prompt_prep(void* q, int64_t ldq, const void* kv, int64_t ldkv, const void* norm_w, float eps, const float* cosp,
                                      const float* sinp, const int* slot, const int* pos, const int* start, void* cache,
                                      int64_t slot_stride, int64_t ldc, void* c_out, int64_t ld_c, void* kr_out,
                                      int64_t ld_kr, int M, int H, int dim, int rd, int R, int half, int dtype, int pdl,
                                      void* stream) {
-  if (M < 1 || H < 1 || dim < 1 || rd < 0 || R < 1 || half < 0 || 2 * half > rd || ldc < R + rd || ld_c < R || ld_kr < rd)
+  if (M < 1 || H < 1 || dim < 1 || rd < 0 || R < 1 || half < 0 || 2 * half > rd || ldc < R + rd ||
+      (kv != nullptr && (ld_c < R || ld_kr < rd)))
     return (int)cudaErrorInvalidValue;
   return by_dtype(dtype, [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
-    PrepArgs a = {qkv, norm_w, nullptr, cosp, sinp, slot, pos, start, cache, nullptr, c_out, kr_out, ldq, slot_stride,
+    PrepArgs a = {q, kv, norm_w, nullptr, cosp, sinp, slot, pos, start, cache, nullptr, c_out, kr_out, ldq, ldkv, slot_stride,
                   ldc, ld_c, ld_kr, eps, M, H, dim, rd, R, half};
     return launch_kernel(latent_prompt_prep_kernel<T>, dim3(M), dim3(256), 0, (cudaStream_t)stream, pdl != 0, a);
   });
@@ -697,8 +705,9 @@ IPEX_API int ipex_latent_attn(const void* qabs, const void* qkv, int64_t ldq, co
   });
 }
 
-// out[m, h * vd + v] = W_uv[h * vd + v] . (merged latent output of head h)
-IPEX_API int ipex_latent_uv(const float* o, const float* ml, const void* w_uv, void* out, int64_t ldo, int M, int H,
+// out[m, h * vd + v] = W_uv[h * vd + v] . (merged latent output of head h), times sigmoid(gate [M, ldg]) unless gate is null
+IPEX_API int ipex_latent_uv(const float* o, const float* ml, const void* w_uv, const void* gate, int64_t ldg, void* out,
+                            int64_t ldo, int M, int H,
                             int R, int vd, int nsplit, int dtype, int pdl, void* stream) {
   if (M < 1 || H < 1 || R < 1 || vd < 1 || nsplit < 1) return (int)cudaErrorInvalidValue;
   return by_dtype(dtype, [&](auto* tag) {
@@ -710,7 +719,7 @@ IPEX_API int ipex_latent_uv(const float* o, const float* ml, const void* w_uv, v
     int by = (296 + have - 1) / have;
     const int most = (vd + 31) / 32;
     by = by < 1 ? 1 : (by > most ? most : by);
-    UvArgs a = {o, ml, w_uv, out, ldo, M, H, R, vd, nsplit, (vd + by - 1) / by};
+    UvArgs a = {o, ml, w_uv, out, ldo, M, H, R, vd, nsplit, (vd + by - 1) / by, gate, ldg};
     cudaStream_t st = (cudaStream_t)stream;
     const bool vec = R % Vec<T>::n == 0 && (reinterpret_cast<uintptr_t>(w_uv) & 15) == 0;
     if (mt == 1) return vec ? launch_uv<T, Vec<T>::n, 1>(a, by, pdl, st) : launch_uv<T, 1, 1>(a, by, pdl, st);

@@ -1,5 +1,6 @@
 // Prompt attention over packed sequences on the 5th-generation tensor cores, sm_100a: multi-head latent attention, and
-// attention with plain key / value heads (shared by groups of query heads), with or without a window and a sink.
+// attention with plain key / value heads (shared by groups of query heads), over everything earlier, a window or the
+// query's own chunk, with or without a sink and an output gate.
 //
 // Keys and values are expanded from the latents by two GEMMs before this kernel; a head's key is then made of two
 // parts that live in different tensors: `dim` values of its own and `rd` rotated values shared by all heads.  Neither
@@ -53,8 +54,13 @@ struct Args {
   int nbn, nbr;           // k-blocks of the own and of the shared part
   int kst, vst;           // stages of the K and V^T rings (1 or 2)
   int group;              // query heads per key / value head
-  int sink;               // one more score of 0, without a value, in every softmax
+  int sink;               // one more score, without a value, in every softmax: 0, or sinks[head]
   float scale_log2;
+  int chunk;              // keys of the query's own chunk of this many positions only; 0: all
+  const float* sinks;
+  const void* gate;       // T [tokens, ldg], head h at h * vd, or null: outputs times gate_scale * sigmoid(gate)
+  int64_t ldg;
+  float gate_scale;
 };
 
 template <typename T, int DV>
@@ -97,6 +103,7 @@ packed_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
   const int nkv = (qmax + koff) / kBKV + 1;
   int j0 = 0;
   if (a.window > 0) j0 = max(0, qb * kBQ - a.window + 1 + koff) / kBKV;
+  if (a.chunk > 0) j0 = max(j0, (qb * kBQ / a.chunk * a.chunk + koff) / kBKV);
   const int nblk = nkv - j0;
 
   if (threadIdx.x == 0) {
@@ -216,7 +223,8 @@ packed_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
     for (int d = 0; d < kOH; ++d) o[d] = 0.f;
     float m = -INFINITY, l = 0.f;
     bool ok = true;
-    const int first = a.window > 0 ? max(0, qpos - a.window + 1) : 0;
+    int first = a.window > 0 ? max(0, qpos - a.window + 1) : 0;
+    if (a.chunk > 0) first = max(first, qpos / a.chunk * a.chunk);
     for (int jj = 0; jj < nblk; ++jj) {
       const uint32_t jp = jj & 1;
       if (!mbar_wait(&s_full[jj & 1], (jj >> 1) & 1, abort_flag)) { ok = false; break; }
@@ -297,18 +305,33 @@ packed_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
       mbar_arrive(x_full);
       ok = mbar_wait(x_full, nblk & 1, abort_flag);
       l += xch[(hf ^ 1) * 128 + r];
-      if (a.sink) l += ex2(-m);      // both halves hold the row's maximum
+      if (a.sink) {                  // both halves hold the row's maximum, in the log2 domain
+        const float z = a.sinks != nullptr ? a.sinks[h] * 1.4426950408889634f : 0.f;
+        const float top = fmaxf(m, z), f = ex2(m - top);
+        l = l * f + ex2(z - top);
+#pragma unroll
+        for (int d = 0; d < kOH; ++d) o[d] *= f;
+      }
     }
     if (!ok && lane == 0) report(a.err, 36);
     if (ok && qpos < len) {
       const float inv = l > 0.f ? 1.f / l : 0.f;
       T* op = reinterpret_cast<T*>(a.out) + (int64_t)(row0 + qpos) * a.ldo + (int64_t)h * a.vd + hf * kOH;
+      const T* gp = reinterpret_cast<const T*>(a.gate) + (int64_t)(row0 + qpos) * a.ldg + (int64_t)h * a.vd + hf * kOH;
 #pragma unroll
       for (int c = 0; c < kOH / 8; ++c) {
         if (hf * kOH + c * 8 < a.vd) {
           __align__(16) T ov[8];
 #pragma unroll
-          for (int i = 0; i < 8; ++i) ov[i] = from_float<T>(o[c * 8 + i] * inv);
+          for (int i = 0; i < 8; ++i) o[c * 8 + i] *= inv;
+          if (a.gate != nullptr) {
+            const uint4 raw = *reinterpret_cast<const uint4*>(gp + c * 8);
+            const T* gv = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) o[c * 8 + i] *= __fdividef(a.gate_scale, 1.0f + __expf(-to_float<T>(gv[i])));
+          }
+#pragma unroll
+          for (int i = 0; i < 8; ++i) ov[i] = from_float<T>(o[c * 8 + i]);
           *reinterpret_cast<uint4*>(op + c * 8) = *reinterpret_cast<const uint4*>(ov);
         }
       }
@@ -382,19 +405,22 @@ IPEX_API int ipex_packed_prefill_ok(int dim, int rd, int vd, int R, int dtype) {
 // Causal (windowed) attention of packed sequences: q [tokens, ldq] holds per head [dim | rd (rotated)], k [tokens, ldk]
 // the G key heads of `dim`, kr [tokens, ld_kr] the rotated part shared by all heads (rd = 0: none), vt [G * vd, ld_vt]
 // the values transposed.  Query head h uses key / value head h / (H / G).  seq_row / seq_len: device, [B]; max_len: the
-// largest length.  window 0: unlimited.  sink: every softmax has one more score of 0 whose value is nothing.  Strides
-// multiples of 8 elements, bases 16-byte aligned.  Returns a cudaError_t, or -1 when the tensor-map encoder rejects
+// largest length.  window 0: unlimited.  chunk > 0: keys of the query's own chunk only.  sink: every softmax has one more
+// score, 0 or sinks[head], whose value is nothing.  gate (may be null): [tokens, ldg], outputs times gate_scale *
+// sigmoid(gate).  Strides multiples of 8 elements, bases 16-byte aligned.  Returns a cudaError_t, or -1 when the tensor-map encoder rejects
 // the operands.
 IPEX_API int ipex_packed_prefill(const void* q, int64_t ldq, const void* k, int64_t ldk, const void* kr, int64_t ld_kr,
                                  const void* vt, int64_t ld_vt, void* out, int64_t ldo, const int* seq_row,
                                  const int* seq_len, int B, int H, int G, int tokens, int max_len, int dim, int rd,
-                                 int vd, int window, int sink, float scale, int dtype, int* err, void* stream) {
+                                 int vd, int window, int chunk, int sink, const float* sinks, const void* gate,
+                                 int64_t ldg, float gate_scale, float scale, int dtype, int* err, void* stream) {
   if (!ipex_packed_prefill_ok(dim, rd, vd, 8, dtype) || B < 1 || B > 65535 || H < 1 || tokens < 1 || max_len < 1 ||
-      window < 0 || (max_len + kBQ - 1) / kBQ > 65535 || G < 1 || H % G != 0)
+      window < 0 || chunk < 0 || (max_len + kBQ - 1) / kBQ > 65535 || G < 1 || H % G != 0)
     return (int)cudaErrorInvalidValue;
-  if ((ldq % 8) || (ldk % 8) || (ld_vt % 8) || (ldo % 8) || (rd > 0 && (ld_kr % 8)) || ld_vt < tokens)
+  if ((ldq % 8) || (ldk % 8) || (ld_vt % 8) || (ldo % 8) || (rd > 0 && (ld_kr % 8)) || ld_vt < tokens ||
+      (gate != nullptr && (ldg % 8)))
     return (int)cudaErrorInvalidValue;
-  if (((uintptr_t)q | (uintptr_t)k | (uintptr_t)kr | (uintptr_t)vt | (uintptr_t)out) & 15)
+  if (((uintptr_t)q | (uintptr_t)k | (uintptr_t)kr | (uintptr_t)vt | (uintptr_t)out | (uintptr_t)gate) & 15)
     return (int)cudaErrorInvalidValue;
   Args a = {};
   a.out = out; a.seq_row = seq_row; a.seq_len = seq_len; a.err = err; a.ldo = ldo;
@@ -403,6 +429,7 @@ IPEX_API int ipex_packed_prefill(const void* q, int64_t ldq, const void* k, int6
   a.nbr = (rd + 63) / 64;
   a.group = H / G;
   a.sink = sink;
+  a.chunk = chunk; a.sinks = sinks; a.gate = gate; a.ldg = ldg; a.gate_scale = gate_scale;
   a.scale_log2 = scale * 1.4426950408889634f;
   cudaStream_t st = (cudaStream_t)stream;
   if (dtype == DT_F16)

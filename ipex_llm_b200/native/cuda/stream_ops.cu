@@ -1,9 +1,11 @@
 // Element-wise and routing kernels of decoders with a 32-bit residual stream, sm_100a: embedding (scaled, with an
-// optional bigram table), RMS norm of the stream into the activation dtype, the joint of a block that norms a
-// sublayer's output before it is added, tanh soft-cap of fp32 logits, biases and gelu-gated units behind library or
-// packed products, and the data movement around a dense expert bank for prompts (slots grouped by expert on the device, row gather, clamped
-// gated unit, combination into the stream), plus a plain tiled product for sizes the tensor-core kernels do not take
-// and for 32-bit models.
+// optional bigram table, into one or several streams), RMS norm of the stream into the activation dtype, the joint of a
+// block that norms a sublayer's output before it is added, the joint of blocks between which several streams are mixed
+// (hyper-connections), tanh soft-cap of fp32 logits, biases and gated units behind library or packed products, and
+// the data movement around a dense expert bank for prompts (choice of experts, slots grouped by expert on the device,
+// row gather, gated unit, combination), plus a plain tiled product for sizes the tensor-core kernels do not take and for
+// 32-bit models.
+#include "common/routing.cuh"
 #include "common/utils.cuh"
 
 namespace {
@@ -33,7 +35,7 @@ __global__ void embed_stream_kernel(const int64_t* __restrict__ tokens, const in
                                     const int* __restrict__ pos, const int* __restrict__ start, int* history,
                                     int64_t cap, const T* __restrict__ table, const T* __restrict__ bigram,
                                     float* __restrict__ out, int W, int64_t vocab, float scale, int64_t buckets,
-                                    int64_t mul_prev, int64_t mul_cur) {
+                                    int64_t mul_prev, int64_t mul_cur, int copies) {
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
@@ -54,11 +56,11 @@ __global__ void embed_stream_kernel(const int64_t* __restrict__ tokens, const in
   if (threadIdx.x == 0) history[(int64_t)s * cap + p] = (int)tok;
   const T* e = table + tok * W;
   const T* b = bigram + (row < 0 ? 0 : row) * W;
-  float* o = out + (int64_t)t * W;
+  float* o = out + (int64_t)t * copies * W;
   for (int i = threadIdx.x; i < W; i += blockDim.x) {
     float v = DT<T>::to_f(e[i]) * scale;
     if (row >= 0) v += DT<T>::to_f(b[i]);
-    o[i] = v;
+    for (int c = 0; c < copies; ++c) o[(int64_t)c * W + i] = v;
   }
 }
 
@@ -183,6 +185,131 @@ __global__ void add_norm_stream_kernel(float* __restrict__ x, int64_t ldx, const
   for (int k = tid; k < K; k += nt) dst[k] = DT<T>::from_f(xr[k] * inv * w_in[k]);
 }
 
+// Several residual streams x [S, K] per token.  Behind a sublayer with output y all streams are mixed,
+// x_t <- sum_s mix[s, t] x_s + w_out[t] y  (y null: they stay), and the next sublayer's input is the norm of
+// sum_s w_in[s] x_s.  One CTA per token; with NV > 0 a thread keeps its part of all streams in registers.
+struct HyperArgs {
+  float* x;             // [n, S, K]
+  const float* y;       // [n, ldy] or null
+  const float* mix;     // [S, S], from row to column
+  const float* w_out;   // [S]
+  const float* w_in;    // [S]
+  const float* norm;    // [K]
+  void* out;            // T [n, ldo]
+  int64_t ldy, ldo;
+  int S, K;
+  float eps;
+};
+constexpr int kMaxStreams = 16;
+
+template <typename T, int S, int NV>
+__global__ void __launch_bounds__(NV == 1 ? 256 : 1024) hyper_joint_kernel(HyperArgs a) {
+  __shared__ float red[32];
+  __shared__ float s_mix[S * S], s_out[S], s_in[S];
+  pdl_launch_dependents();
+  const int tid = threadIdx.x, nt = blockDim.x, K4 = a.K / 4;
+  if (tid < S) {
+    s_in[tid] = a.w_in[tid];
+    if (a.y != nullptr) s_out[tid] = a.w_out[tid];
+  }
+  if (a.y != nullptr && tid < S * S) s_mix[tid] = a.mix[tid];
+  pdl_wait();
+  __syncthreads();
+  float4* x = reinterpret_cast<float4*>(a.x + (int64_t)blockIdx.x * S * a.K);
+  float4 u[NV];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int k = tid + i * nt;
+    u[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (k >= K4) continue;
+    float4 v[S], n[S];
+#pragma unroll
+    for (int s = 0; s < S; ++s) n[s] = v[s] = x[(int64_t)s * K4 + k];
+    if (a.y != nullptr) {
+      const float4 y = reinterpret_cast<const float4*>(a.y + (int64_t)blockIdx.x * a.ldy)[k];
+#pragma unroll
+      for (int t = 0; t < S; ++t) {
+        const float o = s_out[t];
+        n[t] = make_float4(o * y.x, o * y.y, o * y.z, o * y.w);
+#pragma unroll
+        for (int s = 0; s < S; ++s) {
+          const float m = s_mix[s * S + t];
+          n[t].x = fmaf(m, v[s].x, n[t].x);
+          n[t].y = fmaf(m, v[s].y, n[t].y);
+          n[t].z = fmaf(m, v[s].z, n[t].z);
+          n[t].w = fmaf(m, v[s].w, n[t].w);
+        }
+        x[(int64_t)t * K4 + k] = n[t];
+      }
+    }
+#pragma unroll
+    for (int s = 0; s < S; ++s) {
+      const float m = s_in[s];
+      u[i].x = fmaf(m, n[s].x, u[i].x);
+      u[i].y = fmaf(m, n[s].y, u[i].y);
+      u[i].z = fmaf(m, n[s].z, u[i].z);
+      u[i].w = fmaf(m, n[s].w, u[i].w);
+    }
+    ss += u[i].x * u[i].x + u[i].y * u[i].y + u[i].z * u[i].z + u[i].w * u[i].w;
+  }
+  ss = block_sum(ss, red);
+  const float inv = 1.0f / sqrtf(ss / (float)a.K + a.eps);
+  T* dst = reinterpret_cast<T*>(a.out) + (int64_t)blockIdx.x * a.ldo;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int k = tid + i * nt;
+    if (k >= K4) continue;
+    const float4 w = reinterpret_cast<const float4*>(a.norm)[k];
+    __align__(16) T o[4] = {DT<T>::from_f(u[i].x * inv * w.x), DT<T>::from_f(u[i].y * inv * w.y),
+                            DT<T>::from_f(u[i].z * inv * w.z), DT<T>::from_f(u[i].w * inv * w.w)};
+    if constexpr (sizeof(T) == 2) reinterpret_cast<uint2*>(dst)[k] = *reinterpret_cast<const uint2*>(o);
+    else reinterpret_cast<uint4*>(dst)[k] = *reinterpret_cast<const uint4*>(o);
+  }
+}
+
+template <typename T>
+__global__ void hyper_joint_any_kernel(HyperArgs a) {
+  __shared__ float red[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int tid = threadIdx.x, nt = blockDim.x, S = a.S;
+  float* x = a.x + (int64_t)blockIdx.x * S * a.K;
+  float ss = 0.f;
+  for (int k = tid; k < a.K; k += nt) {
+    float v[kMaxStreams], u = 0.f;
+    for (int s = 0; s < S; ++s) v[s] = x[(int64_t)s * a.K + k];
+    if (a.y != nullptr) {
+      const float y = a.y[(int64_t)blockIdx.x * a.ldy + k];
+      for (int t = 0; t < S; ++t) {
+        float n = a.w_out[t] * y;
+        for (int s = 0; s < S; ++s) n = fmaf(a.mix[s * S + t], v[s], n);
+        x[(int64_t)t * a.K + k] = n;
+        u = fmaf(a.w_in[t], n, u);
+      }
+    } else {
+      for (int s = 0; s < S; ++s) u = fmaf(a.w_in[s], v[s], u);
+    }
+    ss = fmaf(u, u, ss);
+  }
+  ss = block_sum(ss, red);
+  const float inv = 1.0f / sqrtf(ss / (float)a.K + a.eps);
+  T* dst = reinterpret_cast<T*>(a.out) + (int64_t)blockIdx.x * a.ldo;
+  for (int k = tid; k < a.K; k += nt) {
+    float u = 0.f;                                  // a thread reads what it wrote itself
+    for (int s = 0; s < S; ++s) u = fmaf(a.w_in[s], x[(int64_t)s * a.K + k], u);
+    dst[k] = DT<T>::from_f(u * inv * a.norm[k]);
+  }
+}
+
+template <typename T, int S>
+cudaError_t launch_hyper(const HyperArgs& a, int n, bool pdl, cudaStream_t st) {
+  const int k4 = a.K / 4;
+  if (k4 <= 256) return launch_kernel(hyper_joint_kernel<T, S, 1>, dim3(n), dim3((k4 + 31) / 32 * 32), 0, st, pdl, a);
+  const int half = (k4 + 1) / 2, threads = (half + 31) / 32 * 32;
+  return launch_kernel(hyper_joint_kernel<T, S, 2>, dim3(n), dim3(threads < 256 ? 256 : threads), 0, st, pdl, a);
+}
+
 // y += bias, row by row
 template <typename TY, typename T>
 __global__ void bias_rows_kernel(TY* __restrict__ y, int64_t ldy, const T* __restrict__ bias, int N) {
@@ -190,17 +317,17 @@ __global__ void bias_rows_kernel(TY* __restrict__ y, int64_t ldy, const T* __res
   for (int n = threadIdx.x; n < N; n += blockDim.x) r[n] = DT<TY>::from_f(DT<TY>::to_f(r[n]) + DT<T>::to_f(bias[n]));
 }
 
-// out[r, i] = gelu_tanh(gate + bias) * (up + bias) from a row of 2 I products; interleaved: gate and up alternate in
-// blocks of eight
-template <typename TY, typename T>
-__global__ void gelu_glu_rows_kernel(const TY* __restrict__ gu, int64_t ld, const T* __restrict__ bias,
+// out[r, i] = act(gate + bias) * (up + bias) from a row of 2 I products, act gelu_tanh or silu; interleaved: gate and up
+// alternate in blocks of eight
+template <typename TY, typename T, bool SILU>
+__global__ void glu_products_kernel(const TY* __restrict__ gu, int64_t ld, const T* __restrict__ bias,
                                      T* __restrict__ out, int64_t ldo, int I, int interleaved) {
   const TY* r = gu + (int64_t)blockIdx.x * ld;
   for (int i = threadIdx.x; i < I; i += blockDim.x) {
     const int g = interleaved ? (i >> 3) * 16 + (i & 7) : i, u = interleaved ? g + 8 : I + i;
     const float bg = bias != nullptr ? DT<T>::to_f(bias[g]) : 0.f, bu = bias != nullptr ? DT<T>::to_f(bias[u]) : 0.f;
-    out[(int64_t)blockIdx.x * ldo + i] =
-        DT<T>::from_f(gelu_tanh(DT<TY>::to_f(r[g]) + bg) * (DT<TY>::to_f(r[u]) + bu));
+    const float z = DT<TY>::to_f(r[g]) + bg;
+    out[(int64_t)blockIdx.x * ldo + i] = DT<T>::from_f((SILU ? silu(z) : gelu_tanh(z)) * (DT<TY>::to_f(r[u]) + bu));
   }
 }
 
@@ -255,6 +382,23 @@ __global__ void sigmoid_topk_kernel(const float* __restrict__ logits, int64_t ld
     }
     __syncwarp();
   }
+}
+
+// fp32 router logits [tokens, E (+ 1)] -> weights and experts (softmax_grouped_topk); a warp per token.  gate: the logit
+// behind the experts' becomes gate[t] = sigmoid.
+__global__ void softmax_topk_kernel(const float* __restrict__ logits, int64_t ld, float* __restrict__ w,
+                                    int64_t* __restrict__ idx, float* __restrict__ gate, int tokens, int E, int groups,
+                                    int keep, int k, float scale) {
+  extern __shared__ float sh[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, wpb = blockDim.x >> 5;
+  const int t = blockIdx.x * wpb + warp;
+  if (t >= tokens) return;
+  float* sc = sh + (size_t)warp * (E + groups);
+  const float* row = logits + (int64_t)t * ld;
+  for (int e = lane; e < E; e += 32) sc[e] = row[e];
+  if (gate != nullptr && lane == 0) gate[t] = 1.0f / (1.0f + expf(-row[E]));
+  __syncwarp();
+  softmax_grouped_topk(sc, sc + E, E, groups, keep, k, scale, w + (int64_t)t * k, idx + (int64_t)t * k, lane);
 }
 
 // (token, choice) slots grouped by expert, one CTA: order[pos] = slot, inverse[slot] = pos, ranges[e] = (first, count).
@@ -340,6 +484,43 @@ __global__ void combine_slots_kernel(const T* __restrict__ y, const int* __restr
   }
 }
 
+// out[t] = gate[t] * out[t] (gate null: 0) + sum_j w[t, j] y[inverse[t * k + j]]
+template <typename T>
+__global__ void combine_weighted_kernel(const T* __restrict__ y, const int* __restrict__ inverse,
+                                        const float* __restrict__ w, const float* __restrict__ gate,
+                                        float* __restrict__ out, int N, int k) {
+  const int t = blockIdx.x;
+  float* o = out + (int64_t)t * N;
+  const float g = gate != nullptr ? gate[t] : 0.f;
+  constexpr int VN = 16 / (int)sizeof(T);
+  if (N % VN == 0) {
+    for (int n = threadIdx.x * VN; n < N; n += blockDim.x * VN) {
+      float s[VN];
+#pragma unroll
+      for (int i = 0; i < VN; i += 4) {
+        const float4 f = gate != nullptr ? *reinterpret_cast<const float4*>(o + n + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        s[i] = g * f.x; s[i + 1] = g * f.y; s[i + 2] = g * f.z; s[i + 3] = g * f.w;
+      }
+      for (int j = 0; j < k; ++j) {
+        const float wj = w[(int64_t)t * k + j];
+        const uint4 raw = *reinterpret_cast<const uint4*>(y + (int64_t)inverse[(int64_t)t * k + j] * N + n);
+        const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+        for (int i = 0; i < VN; ++i) s[i] = fmaf(wj, DT<T>::to_f(e[i]), s[i]);
+      }
+#pragma unroll
+      for (int i = 0; i < VN; i += 4) *reinterpret_cast<float4*>(o + n + i) = make_float4(s[i], s[i + 1], s[i + 2], s[i + 3]);
+    }
+    return;
+  }
+  for (int n = threadIdx.x; n < N; n += blockDim.x) {
+    float s = gate != nullptr ? g * o[n] : 0.f;
+    for (int j = 0; j < k; ++j)
+      s = fmaf(w[(int64_t)t * k + j], DT<T>::to_f(y[(int64_t)inverse[(int64_t)t * k + j] * N + n]), s);
+    o[n] = s;
+  }
+}
+
 // ------------------------------------------------------------------------------------------- plain tiled product
 // out[m, n] (fp32 or T) = sum_k x[m, k] w[n, k], 64 x 64 tiles, fp32 FMAs; with ranges, group g multiplies its rows
 // [ranges[g][0], + ranges[g][1]) of x by weight matrix g.
@@ -389,18 +570,18 @@ __global__ void __launch_bounds__(256) gemm_plain_kernel(const T* __restrict__ x
 
 }  // namespace
 
-// out[t] = table[token] * scale (+ bigram row), fp32.  history: int32 [slots, cap]; start: int32 [slots], the position
+// out[t] = table[token] * scale (+ bigram row), fp32, `copies` times behind one another.  history: int32 [slots, cap]; start: int32 [slots], the position
 // of each sequence's first token.  bigram may be null (buckets etc. are ignored then).
 IPEX_API int ipex_embed_stream(const int64_t* tokens, const int* slot, const int* pos, const int* start, int* history,
                                int64_t cap, const void* table, const void* bigram, float* out, int n, int W,
-                               int64_t vocab, float scale, int64_t buckets, int64_t mul_prev, int64_t mul_cur, int dtype,
-                               int pdl, void* stream) {
-  if (n < 1 || W < 1 || (bigram != nullptr && buckets < 1)) return (int)cudaErrorInvalidValue;
+                               int64_t vocab, float scale, int64_t buckets, int64_t mul_prev, int64_t mul_cur, int copies,
+                               int dtype, int pdl, void* stream) {
+  if (n < 1 || W < 1 || copies < 1 || (bigram != nullptr && buckets < 1)) return (int)cudaErrorInvalidValue;
   return by_dtype(dtype, [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
     return launch_kernel(embed_stream_kernel<T>, dim3(n), dim3(256), 0, (cudaStream_t)stream, pdl != 0, tokens, slot,
                          pos, start, history, cap, (const T*)table, (const T*)bigram, out, W, vocab, scale, buckets,
-                         mul_prev, mul_cur);
+                         mul_prev, mul_cur, copies);
   });
 }
 
@@ -446,19 +627,42 @@ IPEX_API int ipex_bias_rows(void* y, int64_t ldy, int y_f32, const void* bias, i
   });
 }
 
-// out [n, I] = gelu_tanh(gate + bias) * (up + bias) of gu [n, 2 I] (the activation dtype, or fp32)
-IPEX_API int ipex_gelu_glu_rows(const void* gu, int64_t ld, int gu_f32, const void* bias, void* out, int64_t ldo, int n,
-                                int I, int interleaved, int dtype, void* stream) {
+// out [n, I] = act(gate + bias) * (up + bias) of gu [n, 2 I] (the activation dtype, or fp32); use_silu: silu, else gelu_tanh
+IPEX_API int ipex_glu_rows(const void* gu, int64_t ld, int gu_f32, const void* bias, void* out, int64_t ldo, int n, int I,
+                           int interleaved, int use_silu, int dtype, void* stream) {
   if (n < 1 || I < 1 || (interleaved && I % 8 != 0)) return (int)cudaErrorInvalidValue;
+  cudaStream_t st = (cudaStream_t)stream;
   return by_dtype(dtype, [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
-    if (gu_f32)
-      gelu_glu_rows_kernel<float, T><<<n, 256, 0, (cudaStream_t)stream>>>((const float*)gu, ld, (const T*)bias, (T*)out,
-                                                                          ldo, I, interleaved);
-    else
-      gelu_glu_rows_kernel<T, T><<<n, 256, 0, (cudaStream_t)stream>>>((const T*)gu, ld, (const T*)bias, (T*)out, ldo, I,
-                                                                      interleaved);
+    if (gu_f32) {
+      auto kern = use_silu ? glu_products_kernel<float, T, true> : glu_products_kernel<float, T, false>;
+      kern<<<n, 256, 0, st>>>((const float*)gu, ld, (const T*)bias, (T*)out, ldo, I, interleaved);
+    } else {
+      auto kern = use_silu ? glu_products_kernel<T, T, true> : glu_products_kernel<T, T, false>;
+      kern<<<n, 256, 0, st>>>((const T*)gu, ld, (const T*)bias, (T*)out, ldo, I, interleaved);
+    }
     return cudaGetLastError();
+  });
+}
+
+// Behind a sublayer of a decoder with S residual streams: see HyperArgs.  y null: the streams stay as they are.
+IPEX_API int ipex_hyper_joint(float* x, const float* y, int64_t ldy, const float* mix, const float* w_out,
+                              const float* w_in, const float* norm, void* out, int64_t ldo, int n, int S, int K, float eps,
+                              int dtype, int pdl, void* stream) {
+  if (n < 1 || S < 1 || S > kMaxStreams || K < 1 || x == nullptr || w_in == nullptr || norm == nullptr || out == nullptr ||
+      (y != nullptr && (mix == nullptr || w_out == nullptr)))
+    return (int)cudaErrorInvalidValue;
+  HyperArgs a = {x, y, mix, w_out, w_in, norm, out, ldy, ldo, S, K, eps};
+  const bool vec = K % 4 == 0 && K <= 8192 && ldo % 4 == 0 && ldy % 4 == 0 &&
+                   (((uintptr_t)x | (uintptr_t)y | (uintptr_t)norm | (uintptr_t)out) & 15) == 0;
+  cudaStream_t st = (cudaStream_t)stream;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    if (vec && S == 1) return launch_hyper<T, 1>(a, n, pdl != 0, st);
+    if (vec && S == 2) return launch_hyper<T, 2>(a, n, pdl != 0, st);
+    if (vec && S == 3) return launch_hyper<T, 3>(a, n, pdl != 0, st);
+    if (vec && S == 4) return launch_hyper<T, 4>(a, n, pdl != 0, st);
+    return launch_kernel(hyper_joint_any_kernel<T>, dim3(n), dim3(256), 0, st, pdl != 0, a);
   });
 }
 
@@ -491,6 +695,18 @@ IPEX_API int ipex_moe_sigmoid_topk(const float* logits, int64_t ld, float* w, in
   if (tokens < 1 || E < 1 || E > 3000 || k < 1 || k > E) return (int)cudaErrorInvalidValue;
   sigmoid_topk_kernel<<<(tokens + 3) / 4, 128, (size_t)4 * E * sizeof(float), (cudaStream_t)stream>>>(
       logits, ld, w, idx, tokens, E, k);
+  return (int)cudaGetLastError();
+}
+
+// logits [tokens, E] (with `gate`, E + 1) -> weights and experts [tokens, k]: soft-max, the `keep` best of `groups` equal
+// groups, the k largest, divided by their sum and times scale; gate [tokens] (may be null): sigmoid of the last logit.
+IPEX_API int ipex_moe_softmax_grouped_topk(const float* logits, int64_t ld, float* w, int64_t* idx, float* gate, int tokens,
+                                           int E, int groups, int keep, int k, float scale, void* stream) {
+  if (tokens < 1 || E < 1 || E > 2500 || k < 1 || k > E || groups < 1 || E % groups || keep < 1 || keep > groups ||
+      k > E / groups * keep)
+    return (int)cudaErrorInvalidValue;
+  softmax_topk_kernel<<<(tokens + 3) / 4, 128, (size_t)4 * (E + groups) * sizeof(float), (cudaStream_t)stream>>>(
+      logits, ld, w, idx, gate, tokens, E, groups, keep, k, scale);
   return (int)cudaGetLastError();
 }
 
@@ -528,6 +744,17 @@ IPEX_API int ipex_moe_combine_slots(const void* y, const int* inverse, float* re
   return by_dtype(dtype, [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
     combine_slots_kernel<T><<<tokens, 256, 0, (cudaStream_t)stream>>>((const T*)y, inverse, residual, N, k);
+    return cudaGetLastError();
+  });
+}
+
+// out [tokens, N] fp32 = gate * out (gate null: 0) + sum_j w[t, j] y[inverse[t k + j]]
+IPEX_API int ipex_moe_combine_weighted(const void* y, const int* inverse, const float* w, const float* gate, float* out,
+                                       int tokens, int N, int k, int dtype, void* stream) {
+  if (tokens < 1 || N < 1 || k < 1 || (((uintptr_t)y | (uintptr_t)out) & 15)) return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    combine_weighted_kernel<T><<<tokens, 256, 0, (cudaStream_t)stream>>>((const T*)y, inverse, w, gate, out, N, k);
     return cudaGetLastError();
   });
 }

@@ -71,44 +71,49 @@ COMPONENT_SIGS = {
         "ipex_gemv_rows": [vp, i64, vp, i64, vp, cf, vp, vp, i64, vp, ci, vp, i64, ci, ci, ci, ci, ci, ci, cf, ci, ci,
                            vp],
         "ipex_moe_router_sigmoid": [vp, i64, vp, cf, vp, vp, vp, ci, ci, ci, ci, ci, ci, vp],
-        "ipex_moe_glu_rows": [vp, i64, vp, cf, vp, vp, vp, vp, ci, ci, ci, ci, ci, cf, cf, ci, ci, ci, vp],
-        "ipex_moe_down_rows": [vp, vp, vp, i64, vp, ci, ci, ci, ci, ci, ci, ci, vp],
-        "ipex_embed_stream": [vp, vp, vp, vp, vp, i64, vp, vp, vp, ci, ci, i64, cf, i64, i64, i64, ci, ci, vp],
+        "ipex_moe_router_softmax": [vp, i64, vp, vp, vp, ci, ci, ci, ci, ci, ci, ci, cf, ci, ci, vp],
+        "ipex_moe_glu_rows": [vp, i64, vp, cf, vp, vp, vp, i64, vp, vp, ci, ci, ci, ci, ci, ci, ci, cf, cf, ci, ci, ci, ci, vp],
+        "ipex_moe_down_rows": [vp, i64, vp, vp, vp, vp, i64, vp, ci, ci, ci, ci, ci, ci, ci, ci, vp],
+        "ipex_embed_stream": [vp, vp, vp, vp, vp, i64, vp, vp, vp, ci, ci, i64, cf, i64, i64, i64, ci, ci, ci, vp],
         "ipex_norm_stream": [vp, i64, vp, ci, vp, i64, vp, ci, ci, cf, ci, ci, vp],
         "ipex_add_norm_stream": [vp, i64, vp, i64, vp, vp, vp, i64, ci, ci, cf, ci, ci, vp],
         "ipex_bias_rows": [vp, i64, ci, vp, ci, ci, ci, vp],
-        "ipex_gelu_glu_rows": [vp, i64, ci, vp, vp, i64, ci, ci, ci, ci, vp],
+        "ipex_hyper_joint": [vp, vp, i64, vp, vp, vp, vp, vp, i64, ci, ci, ci, cf, ci, ci, vp],
+        "ipex_glu_rows": [vp, i64, ci, vp, vp, i64, ci, ci, ci, ci, ci, vp],
         "ipex_softcap_f32": [vp, i64, cf, vp],
         "ipex_add_stream": [vp, vp, i64, ci, vp],
         "ipex_relu2_inplace": [vp, i64, ci, vp],
         "ipex_moe_sigmoid_topk": [vp, i64, vp, vp, ci, ci, ci, vp],
+        "ipex_moe_softmax_grouped_topk": [vp, i64, vp, vp, vp, ci, ci, ci, ci, ci, cf, vp],
         "ipex_moe_group_slots": [vp, ci, ci, vp, vp, vp, vp],
         "ipex_moe_gather_slots": [vp, vp, vp, vp, vp, ci, ci, ci, ci, vp],
         "ipex_moe_glu_from_gu": [vp, vp, vp, ci, ci, cf, cf, ci, ci, vp],
         "ipex_moe_combine_slots": [vp, vp, vp, ci, ci, ci, ci, vp],
+        "ipex_moe_combine_weighted": [vp, vp, vp, vp, vp, ci, ci, ci, ci, vp],
         "ipex_gemm_plain": [vp, vp, vp, vp, ci, ci, ci, ci, ci, ci, vp],
         "ipex_gemm_stream": [vp, i64, vp, i64, vp, i64, vp, vp, ci, vp, i64, vp, vp, ci, ci, ci, ci, ci, ci, cf, cf,
                              ci, ci, vp, vp],
         "ipex_packed_prefill_ok": [ci, ci, ci, ci, ci],
         "ipex_packed_prefill": [vp, i64, vp, i64, vp, i64, vp, i64, vp, i64, vp, vp, ci, ci, ci, ci, ci, ci, ci, ci,
-                                ci, ci, cf, ci, vp, vp],
+                                ci, ci, ci, vp, vp, i64, cf, cf, ci, vp, vp],
     },
     "latent": {
-        "ipex_latent_prep": [vp, i64, vp, cf, vp, vp, vp, vp, vp, vp, vp, i64, i64, vp, ci, ci, ci, ci, ci, ci, ci, ci,
-                             vp],
-        "ipex_latent_prompt_prep": [vp, i64, vp, cf, vp, vp, vp, vp, vp, vp, i64, i64, vp, i64, vp, i64, ci, ci, ci,
-                                    ci, ci, ci, ci, ci, vp],
+        "ipex_latent_prep": [vp, i64, vp, i64, vp, cf, vp, vp, vp, vp, vp, vp, vp, i64, i64, vp, ci, ci, ci, ci, ci, ci,
+                             ci, ci, vp],
+        "ipex_latent_prompt_prep": [vp, i64, vp, i64, vp, cf, vp, vp, vp, vp, vp, vp, i64, i64, vp, i64, vp, i64, ci,
+                                    ci, ci, ci, ci, ci, ci, ci, vp],
         "ipex_latent_row": [ci, ci, ci],
         "ipex_latent_attn_fast": [ci, ci, ci],
         "ipex_latent_attn": [vp, vp, i64, vp, i64, i64, vp, vp, vp, vp, vp, ci, ci, ci, ci, ci, ci, ci, cf, ci, ci, ci,
                              vp],
-        "ipex_latent_uv": [vp, vp, vp, vp, i64, ci, ci, ci, ci, ci, ci, ci, vp],
+        "ipex_latent_uv": [vp, vp, vp, vp, i64, vp, i64, ci, ci, ci, ci, ci, ci, ci, vp],
     },
     "hybrid": {
         "ipex_kv_append": [vp, vp, i64, vp, i64, cf, vp, i64, i64, vp, i64, i64, vp, i64, vp, vp, ci, ci, ci, ci, ci,
                            ci, vp],
+        "ipex_qk_prepare": [vp, i64, vp, vp, vp, vp, vp, ci, ci, cf, ci, ci, ci, ci, ci, vp],
         "ipex_kv_attn": [vp, vp, vp, i64, vp, i64, cf, vp, i64, i64, vp, i64, i64, vp, i64, vp, vp, vp, ci, ci, ci, ci,
-                         ci, ci, ci, ci, ci, cf, ci, ci, vp],
+                         ci, ci, ci, ci, vp, vp, i64, cf, ci, ci, vp, vp, ci, ci, cf, ci, cf, ci, ci, vp],
         "ipex_delta_chunks_ok": [ci, ci],
         "ipex_delta_fused_ok": [ci],
         "ipex_delta_step": [vp, i64, ci, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, ci, vp, cf, vp, i64, vp, ci, ci,
@@ -116,7 +121,15 @@ COMPONENT_SIGS = {
         "ipex_delta_chunks": [vp, i64, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, ci, vp, vp, ci, ci, vp, vp, ci, ci,
                               ci, ci, ci, ci, vp, vp],
         "ipex_delta_tail": [vp, i64, vp, vp, vp, vp, vp, ci, ci, ci, ci, vp],
-        "ipex_gated_norm": [vp, vp, i64, vp, vp, i64, ci, ci, ci, cf, ci, vp],
+        "ipex_gated_norm": [vp, vp, i64, vp, vp, i64, ci, ci, ci, cf, cf, ci, vp],
+    },
+    "linear": {
+        "ipex_linear_chunks_ok": [ci, ci, ci],
+        "ipex_linear_fused_ok": [ci],
+        "ipex_linear_step": [vp, i64, ci, vp, vp, vp, vp, vp, vp, vp, vp, vp, ci, vp, cf, cf, vp, i64, vp, ci, ci, ci, ci,
+                             cf, ci, ci, vp],
+        "ipex_linear_chunks": [vp, i64, vp, vp, vp, vp, vp, vp, vp, vp, vp, ci, vp, vp, ci, ci, vp, vp, ci, ci, ci, ci,
+                               cf, ci, vp, vp],
     },
 }
 
@@ -129,6 +142,8 @@ def declare_component(lib: ctypes.CDLL, name: str):
         lib.ipex_gemv_rows_tune.argtypes, lib.ipex_gemv_rows_tune.restype = [ci], None
     if name == "hybrid":
         lib.ipex_delta_scratch_floats.argtypes, lib.ipex_delta_scratch_floats.restype = [ci, ci], i64
+    if name == "linear":
+        lib.ipex_linear_scratch_floats.argtypes, lib.ipex_linear_scratch_floats.restype = [ci, ci], i64
 
 
 def declare(lib: ctypes.CDLL):

@@ -89,5 +89,5 @@ def delta_mix(spec: DeltaSpec, w: DeltaWeights, proj, gates, slot, pos, cache, l
         api.check(lib.ipex_delta_tail(ptr(proj), proj.stride(0), ptr(layer._v), ptr(slot), ptr(pos), ptr(row), ptr(ln), n,
                                       spec.channels, spec.taps, dt, st), "delta_tail")
     api.check(lib.ipex_gated_norm(ptr(raw), ptr(proj[:, gate_at:]), proj.stride(0), ptr(w.norm), ptr(out), out.stride(0), T,
-                                  spec.heads, spec.vdim, w.eps, dt, st), "gated_norm")
+                                  spec.heads, spec.vdim, w.eps, 1.0, dt, st), "gated_norm")
     return out

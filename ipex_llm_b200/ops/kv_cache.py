@@ -356,8 +356,8 @@ class KeyValueLayer(LatentLayer):
 
 class DeltaStateLayer(NormalLayer):
     """State of a recurrent layer, of one size however long the sequence is: ``_k [slots, heads, dim, vdim]`` in fp32,
-    and the last inputs of its short convolutions, ``_v [slots, 1, taps, channels]`` (row = position mod taps).  A slot
-    that starts a new sequence is not cleared: the kernels take everything before a sequence's first token as zero."""
+    and the last inputs of its short convolutions, ``_v [slots, 1, taps, channels]`` (row = position mod taps; empty for
+    a layer without convolutions).  A slot that starts a new sequence is not cleared: the kernels take everything before a sequence's first token as zero."""
 
     def open(self, slots, capacity, shape, dtype, device):
         k, v, n = self._k, self._v, self.length
@@ -422,7 +422,8 @@ class SlotCache(_BlockCache):
     """Cache of a decoder that runs packed batches, plus what else a sequence carries along: the history of its token
     ids (``history [slots, capacity]``, the previous token of an embedding over token pairs) and the row of its first
     token (``start [slots]``; later rows of a left-padded batch are not the first).  Layers may differ in kind: a
-    layer's shape (``LatentLayer``: an int) names its class.
+    layer's shape (``LatentLayer``: an int) names its class.  A decoder layer may own none of them (it reads another's
+    rows) or several.
 
     Rows of the batch dimension are slots: a sequence takes one (``acquire``), keeps it however the batch around it
     changes, and gives it back (``release``); ``lengths`` counts the tokens each slot holds."""

@@ -16,7 +16,7 @@ from .cuda_ops import error_flag
 
 OUT_ACT, OUT_ADD, OUT_F32 = 0, 1, 2        # activation dtype / added to the stream / fp32
 ACT_NONE, ACT_RELU2 = 0, 1
-ACT_GLU, ACT_GELU_GLU = 2, 3                # grouped GEMM only / gate and up rows in blocks of eight
+ACT_GLU, ACT_GELU_GLU, ACT_SILU_GLU = 2, 3, 4     # grouped GEMM only / gate and up rows in blocks of eight
 
 
 def _dt(t) -> int:
@@ -46,8 +46,8 @@ def gemv_rows(w, x, out, mode: int, norm=None, eps: float = 0.0, act: int = 0, s
               w2=None, out2=None, interleaved=True):
     """``act(x @ w.T + bias)`` for a few rows.  ``norm``: ``x`` is the stream and is RMS-normed with this weight on the way
     (inside the product for one or two rows; a CTA would spend longer on the norms of more rows than on its weights).
-    ``w2`` / ``out2``: more rows for the same ``x``, with fp32 results.  ``ACT_GELU_GLU``: ``w`` holds gate and up rows (in
-    blocks of eight, or not ``interleaved``), half as many columns come out."""
+    ``w2`` / ``out2``: more rows for the same ``x``, with fp32 results.  ``ACT_GELU_GLU`` / ``ACT_SILU_GLU``: ``w`` holds gate and up
+    rows (in blocks of eight, or not ``interleaved``), half as many columns come out."""
     M, N, K = x.shape[0], w.shape[0], w.shape[1]
     if norm is not None and M > 2 and w.dtype != torch.float32:
         x, norm = norm_stream(x, norm, eps, pdl=pdl), None
@@ -77,7 +77,8 @@ def gemm(x, w, out, mode: int, act: int = 0, bias=None, interleaved=True, w2=Non
     """``x [M, K] @ w[N, K].T (+ bias)`` into ``out`` (see ``OUT_*``): the tcgen05 kernel, or the library product for
     32-bit weights and rows that are no multiple of 16 bytes.  ``ACT_GELU_GLU``, ``w2`` / ``out2``: see ``gemv_rows``."""
     M, (N, K) = x.shape[0], w.shape
-    if gemm_ok(x, w) and not (act == ACT_GELU_GLU and not interleaved):
+    gated = act in (ACT_GELU_GLU, ACT_SILU_GLU)
+    if gemm_ok(x, w) and not (gated and not interleaved):
         both = w2 is not None and gemm_ok(x, w2) and w2.stride(0) == w.stride(0)
         if w2 is not None and not both:
             gemm(x, w2, out2, OUT_F32)
@@ -93,8 +94,8 @@ def gemm(x, w, out, mode: int, act: int = 0, bias=None, interleaved=True, w2=Non
     if w2 is not None:
         gemm(x, w2, out2, OUT_F32)
     with _true_fp32():
-        if act == ACT_GELU_GLU:
-            return gelu_glu_rows(torch.matmul(x.float(), w.float().t()), bias, out, interleaved)
+        if gated:
+            return glu_rows(torch.matmul(x.float(), w.float().t()), bias, out, act, interleaved)
         if mode == OUT_ACT:
             torch.matmul(x, w.t(), out=out) if out.is_contiguous() else out.copy_(torch.matmul(x, w.t()))
             if bias is not None:
@@ -118,12 +119,12 @@ def bias_rows_(y, bias):
     return y
 
 
-def gelu_glu_rows(gu, bias, out, interleaved=True):
-    """``gelu_tanh(gate + bias) * (up + bias)`` of finished products ``gu [n, 2 I]`` (the dtype of ``out``, or fp32)."""
-    rc = stream_lib().ipex_gelu_glu_rows(ptr(gu), gu.stride(0), int(gu.dtype == torch.float32), ptr(bias), ptr(out),
-                                         out.stride(0), gu.shape[0], gu.shape[1] // 2, int(interleaved), _dt(out),
-                                         current_stream())
-    api.check(rc, "gelu_glu_rows")
+def glu_rows(gu, bias, out, act: int, interleaved=True):
+    """``act(gate + bias) * (up + bias)`` of finished products ``gu [n, 2 I]`` (the dtype of ``out``, or fp32)."""
+    rc = stream_lib().ipex_glu_rows(ptr(gu), gu.stride(0), int(gu.dtype == torch.float32), ptr(bias), ptr(out),
+                                    out.stride(0), gu.shape[0], gu.shape[1] // 2, int(interleaved),
+                                    int(act == ACT_SILU_GLU), _dt(out), current_stream())
+    api.check(rc, "glu_rows")
     return out
 
 
@@ -149,14 +150,15 @@ def softcap_(logits, cap: float):
 # stream
 # ------------------------------------------------------------------------------------------------
 def embed_stream(tokens, slot, pos, cache, table, scale: float, bigram=None, buckets=0, mul_prev=0, mul_cur=0, out=None,
-                 pdl=False):
-    """``table[token] * scale (+ bigram row)`` for every entry, and the ids filed in ``cache.history``."""
+                 pdl=False, streams=1):
+    """``table[token] * scale (+ bigram row)`` for every entry, ``streams`` times, and the ids filed in
+    ``cache.history``."""
     n, (V, W) = tokens.shape[0], table.shape
     if out is None:
-        out = torch.empty(n, W, dtype=torch.float32, device=tokens.device)
+        out = torch.empty(n, streams * W, dtype=torch.float32, device=tokens.device)
     rc = stream_lib().ipex_embed_stream(ptr(tokens), ptr(slot), ptr(pos), ptr(cache.start), ptr(cache.history),
                                         cache.capacity, ptr(table), ptr(bigram), ptr(out), n, W, V, scale, buckets,
-                                        mul_prev, mul_cur, _dt(table), int(pdl), current_stream())
+                                        mul_prev, mul_cur, streams, _dt(table), int(pdl), current_stream())
     api.check(rc, "embed_stream")
     return out
 
@@ -181,6 +183,18 @@ def add_norm_stream(x, y, w_out, w_in, eps: float, dtype, pdl=False):
     rc = stream_lib().ipex_add_norm_stream(ptr(x), x.stride(0), ptr(y), y.stride(0), ptr(w_out), ptr(w_in), ptr(h),
                                            x.shape[1], x.shape[0], x.shape[1], eps, _dt(dtype), int(pdl), current_stream())
     api.check(rc, "add_norm_stream")
+    return h
+
+
+def hyper_joint(x, y, mix, w_out, w_in, norm, eps: float, dtype, pdl=False):
+    """The joint between two sublayers of a decoder with several residual streams ``x [tokens, streams, width]``:
+    ``x_t <- sum_s mix[s, t] x_s + w_out[t] y`` (``y`` None: as they are), and the next input ``norm(sum_s w_in[s] x_s)`` in
+    ``dtype``.  Everything but the result is fp32."""
+    n, S, K = x.shape
+    h = torch.empty(n, (K + 7) // 8 * 8, dtype=dtype, device=x.device)[:, :K]
+    rc = stream_lib().ipex_hyper_joint(ptr(x), ptr(y), 0 if y is None else y.stride(0), ptr(mix), ptr(w_out), ptr(w_in),
+                                       ptr(norm), ptr(h), h.stride(0), n, S, K, eps, _dt(dtype), int(pdl), current_stream())
+    api.check(rc, "hyper_joint")
     return h
 
 

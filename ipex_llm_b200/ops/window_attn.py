@@ -1,6 +1,6 @@
 """Python front of the attention over cached keys and values of different sizes (``kv_attn.cu``, and the packed tcgen05
-prompt kernel of ``packed_prefill_tcgen05.cu``): grouped query heads, sliding window, optional sink in the soft-max, values
-mixed with those of an earlier layer.
+prompt kernel of ``packed_prefill_tcgen05.cu``): grouped query heads, sliding window or chunks, optional sink in the soft-max,
+rotated and unit-normed queries and keys, gated outputs, values mixed with those of an earlier layer.
 
 Every function launches on the current stream; there is no eager substitute.
 """
@@ -19,7 +19,11 @@ from .stream import _dt
 
 @dataclass(frozen=True)
 class AttnSpec:
-    """Sizes and constants of one layer.  ``window`` 0: every earlier key.  ``sink``: one more score of 0 without a value."""
+    """Sizes and constants of one layer.  ``window`` 0: every earlier key; ``chunk``: only those of the query's own chunk of
+    this many positions.  ``sink``: one more score without a value, 0 or a number per head (``AttnTables.sinks``).
+    ``rot_pairs``: pairs (i, i + rot_pairs) of queries and keys turn with the position; ``unit_eps``: they are divided by
+    sqrt(mean square + unit_eps).  ``gated``: the projection ends with gate columns, outputs are multiplied by
+    ``gate_scale`` times their sigmoid."""
     heads: int
     kv_heads: int
     dim: int
@@ -27,6 +31,11 @@ class AttnSpec:
     scale: float
     window: int = 0
     sink: bool = False
+    chunk: int = 0
+    rot_pairs: int = 0
+    unit_eps: Optional[float] = None
+    gated: bool = False
+    gate_scale: float = 1.0
 
     @property
     def k_at(self) -> int:
@@ -38,8 +47,21 @@ class AttnSpec:
         return (self.heads + self.kv_heads) * self.dim
 
     @property
-    def rows(self) -> int:
+    def gate_at(self) -> int:
         return self.v_at + self.kv_heads * self.vdim
+
+    @property
+    def rows(self) -> int:
+        return self.gate_at + (self.heads * self.vdim if self.gated else 0)
+
+    @property
+    def prepared(self) -> bool:
+        """Queries and keys are not used as they are projected."""
+        return self.rot_pairs > 0 or self.unit_eps is not None
+
+    def seen(self, visible: int) -> int:
+        """Upper bound of the keys a token sees when ``visible`` bounds its position."""
+        return min(visible, self.window or visible, self.chunk or visible)
 
     def prefill_ok(self, dtype) -> bool:
         """Does the tcgen05 prompt kernel take these sizes?"""
@@ -51,6 +73,29 @@ class ValueMix:
     """Values of an earlier layer (a ``[tokens, kv_heads * vdim]`` view) and their share."""
     first: torch.Tensor
     share: float
+
+
+@dataclass
+class AttnTables:
+    """What a layer's attention reads beside the projection: sink scores ``[heads]`` and rotation tables ``[positions,
+    rot_pairs]``, fp32."""
+    sinks: Optional[torch.Tensor] = None
+    cos: Optional[torch.Tensor] = None
+    sin: Optional[torch.Tensor] = None
+
+
+NO_TABLES = AttnTables()
+
+
+def _prepare_args(spec: AttnSpec, tables: AttnTables):
+    return (ptr(tables.cos), ptr(tables.sin), spec.rot_pairs, int(spec.unit_eps is not None), spec.unit_eps or 0.0)
+
+
+def prepare_heads(spec: AttnSpec, qkv, slot, pos, cache, tables: AttnTables):
+    """Rotation and unit norm of all query and key heads in place."""
+    api.check(stream_lib("hybrid").ipex_qk_prepare(ptr(qkv), qkv.stride(0), ptr(slot), ptr(pos), ptr(cache.start),
+                                                   *_prepare_args(spec, tables), qkv.shape[0], spec.heads + spec.kv_heads,
+                                                   spec.dim, _dt(qkv), 0, current_stream()), "qk_prepare")
 
 
 def pick_splits(tokens: int, spec: AttnSpec, visible: int, n_sm: int = 148) -> int:
@@ -68,15 +113,17 @@ def _mix_args(mix: Optional[ValueMix], at: int = 0):
 
 
 def attend_step(spec: AttnSpec, qkv, mix: Optional[ValueMix], slot, pos, cache, layer_idx: int, out, visible: int,
-                single: bool, pdl=False, nsplit: Optional[int] = None):
+                single: bool, pdl=False, nsplit: Optional[int] = None, tables: AttnTables = NO_TABLES):
     """Attention of query tokens against the cache, which gets their own rows first.  ``single``: every token is another
-    sequence's next one (the append is then part of the attention kernel).  ``visible`` bounds the number of keys a
+    sequence's next one (preparation and append are then part of the attention kernel).  ``visible`` bounds the number of keys a
     token can see (it sizes the split, nothing else)."""
     lib, layer = stream_lib("hybrid"), cache.layers[layer_idx]
     k, v = layer._k, layer._v
     M, dt, st = qkv.shape[0], _dt(qkv), current_stream()
     cols = (qkv[:, spec.k_at:], qkv[:, spec.v_at:])
     if not single:
+        if spec.prepared:
+            prepare_heads(spec, qkv, slot, pos, cache, tables)
         first, ld_vf, share = _mix_args(mix)
         api.check(lib.ipex_kv_append(ptr(cols[0]), ptr(cols[1]), qkv.stride(0), ptr(first), ld_vf, share, ptr(k), k.stride(0),
                                      k.stride(1), ptr(v), v.stride(0), v.stride(1), None, 0, ptr(slot), ptr(pos), M,
@@ -88,13 +135,16 @@ def attend_step(spec: AttnSpec, qkv, mix: Optional[ValueMix], slot, pos, cache, 
         api.check(lib.ipex_kv_attn(ptr(qkv[s:]), ptr(cols[0][s:]), ptr(cols[1][s:]), qkv.stride(0), ptr(first), ld_vf, share,
                                    ptr(k), k.stride(0), k.stride(1), ptr(v), v.stride(0), v.stride(1), ptr(out[s:]),
                                    out.stride(0), ptr(slot[s:]), ptr(pos[s:]), ptr(cache.start), m, spec.heads,
-                                   spec.kv_heads, spec.dim, spec.vdim, spec.window, int(spec.sink), int(single),
-                                   nsplit or pick_splits(m, spec, visible), spec.scale, dt, int(pdl), st), "kv_attn")
+                                   spec.kv_heads, spec.dim, spec.vdim, spec.window, spec.chunk, int(spec.sink),
+                                   ptr(tables.sinks), ptr(qkv[s:, spec.gate_at:] if spec.gated else None), qkv.stride(0),
+                                   spec.gate_scale, int(single), int(single and spec.prepared),
+                                   *_prepare_args(spec, tables), nsplit or pick_splits(m, spec, visible), spec.scale, dt,
+                                   int(pdl), st), "kv_attn")
     return out
 
 
 def attend_prompt(spec: AttnSpec, qkv, mix: Optional[ValueMix], slot, pos, seq_row, seq_len, max_len: int, cache,
-                  layer_idx: int, out):
+                  layer_idx: int, out, tables: AttnTables = NO_TABLES):
     """Attention of whole prompts, packed one behind the other (``seq_row`` / ``seq_len``: int32, first row and length of
     each), on the tensor cores; the cache gets keys and mixed values."""
     lib, layer = stream_lib("hybrid"), cache.layers[layer_idx]
@@ -104,13 +154,16 @@ def attend_prompt(spec: AttnSpec, qkv, mix: Optional[ValueMix], slot, pos, seq_r
     vt = torch.empty(spec.kv_heads * spec.vdim, ld, dtype=qkv.dtype, device=dev)
     first, ld_vf, share = _mix_args(mix)
     keys = qkv[:, spec.k_at:]
+    if spec.prepared:
+        prepare_heads(spec, qkv, slot, pos, cache, tables)
     api.check(lib.ipex_kv_append(ptr(keys), ptr(qkv[:, spec.v_at:]), qkv.stride(0), ptr(first), ld_vf, share, ptr(k),
                                  k.stride(0), k.stride(1), ptr(v), v.stride(0), v.stride(1), ptr(vt), ld, ptr(slot),
                                  ptr(pos), T, spec.kv_heads, spec.dim, spec.vdim, dt, 0, st), "kv_append")
     rc = stream_lib().ipex_packed_prefill(ptr(qkv), qkv.stride(0), ptr(keys), qkv.stride(0), None, 0, ptr(vt), ld, ptr(out),
                                           out.stride(0), ptr(seq_row), ptr(seq_len), seq_row.shape[0], spec.heads,
-                                          spec.kv_heads, T, max_len, spec.dim, 0, spec.vdim, spec.window, int(spec.sink),
-                                          spec.scale, dt, ptr(error_flag(dev)), st)
+                                          spec.kv_heads, T, max_len, spec.dim, 0, spec.vdim, spec.window, spec.chunk,
+                                          int(spec.sink), ptr(tables.sinks), ptr(qkv[:, spec.gate_at:] if spec.gated else None),
+                                          qkv.stride(0), spec.gate_scale, spec.scale, dt, ptr(error_flag(dev)), st)
     if rc == -1:
         raise RuntimeError("ipex_llm_b200: the driver's tensor-map encoder rejected the attention operands")
     api.check(rc, "packed_prefill")

@@ -201,7 +201,7 @@ def kernels(z, prompt: int, peaks):
     rows.append({"kernel": f"delta scratch, MB for T={T}", "us": round(nc * per * 4 / 1e6, 1)})
     raw = torch.empty(T, dH, dV, device=dev)
     us = _graph_us(lambda i: lib.ipex_gated_norm(ptr(raw), ptr(projs[i][:, dl.channels:]), dl.rows, ptr(w.norm), ptr(out),
-                                                 out.stride(0), T, dH, dV, 1e-6, 1, S.current_stream()), 4)
+                                                 out.stride(0), T, dH, dV, 1e-6, 1.0, 1, S.current_stream()), 4)
     add(f"gated_norm T={T}", us, 8.0 * T * dH * dV)
     cuda_ops.check_error_flag(torch.device("cuda", 0))
     return rows

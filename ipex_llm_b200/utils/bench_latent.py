@@ -174,7 +174,7 @@ def kernels(z, prompt: int, peaks):
 
         def prep(i):
             k = cache.layers[i]._k
-            lib.ipex_latent_prep(p(qkv), qkv.stride(0), p(kn), 1e-6, p(uk), p(cos), p(sin), p(slot), p(pos),
+            lib.ipex_latent_prep(p(qkv), qkv.stride(0), p(qkv[:, -(R + z["rd"]):]), qkv.stride(0), p(kn), 1e-6, p(uk), p(cos), p(sin), p(slot), p(pos),
                                  p(cache.start), p(k), k.stride(0), k.stride(2), p(qabs), B, H, z["dim"], z["rd"], R,
                                  z["rd"] // 2, 1, 1, st())
 
@@ -185,7 +185,7 @@ def kernels(z, prompt: int, peaks):
                                  st())
 
         def up(i):
-            lib.ipex_latent_uv(p(o), p(ml), p(uv), p(out), out.stride(0), B, H, R, z["vd"], ns, 1, 1, st())
+            lib.ipex_latent_uv(p(o), p(ml), p(uv), None, 0, p(out), out.stride(0), B, H, R, z["vd"], ns, 1, 1, st())
         wb = 2.0 * H * z["dim"] * R
         add(f"latent_prep B={B}", _graph_us(prep, n), wb, 2.0 * B * H * z["dim"] * R)
         kvb = 2.0 * B * ctx * (R + z["rd"])
@@ -256,7 +256,8 @@ def kernels(z, prompt: int, peaks):
     for win in (z["window"], 0):
         us = _graph_us(lambda i: L.stream_lib().ipex_packed_prefill(
             L.ptr(qs[i]), ldq, L.ptr(ks[i]), H * z["dim"], L.ptr(kr), z["rd"], L.ptr(vt), T, L.ptr(out), H * z["vd"],
-            L.ptr(row), L.ptr(ln), 1, H, H, T, T, z["dim"], z["rd"], z["vd"], win, 0, 0.05, 1, L.ptr(err),
+            L.ptr(row), L.ptr(ln), 1, H, H, T, T, z["dim"], z["rd"], z["vd"], win, 0, 0, None, None, 0,
+            1.0, 0.05, 1, L.ptr(err),
             L.current_stream()), n)
         w = win or T
         pairs = T * min(w, T) - min(w, T) * (min(w, T) - 1) / 2
