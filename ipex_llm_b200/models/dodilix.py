@@ -109,11 +109,9 @@ class HyperConnection(nn.Module):
         self.mix = nn.Parameter(torch.eye(streams))
 
     def reset(self):
-        s = self.w_in.numel()
-        with torch.no_grad():
-            self.w_in.fill_(1.0 / s)
-            self.w_out.fill_(1.0)
-            self.mix.copy_(torch.eye(s))
+        nn.init.constant_(self.w_in, 1.0 / self.w_in.numel())
+        nn.init.ones_(self.w_out)
+        nn.init.eye_(self.mix)
 
 
 class GatedLatentAttention(nn.Module):

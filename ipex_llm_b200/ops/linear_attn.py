@@ -68,7 +68,7 @@ def linear_mix(spec: LinearSpec, w: LinearWeights, proj, low, slot, pos, cache, 
     row, ln, n = (None, None, T) if portions is None else (portions.row, portions.length, portions.row.shape[0])
     if chunked is None:
         chunked = portions is not None and portions.longest >= CHUNKED_FROM
-    if chunked and spec.chunks_ok(proj.dtype):
+    if chunked and portions is not None and spec.chunks_ok(proj.dtype):
         per = spec.heads * lib.ipex_linear_scratch_floats(spec.dim, spec.vdim)
         most = max(1, min(portions.chunks, SCRATCH_BYTES // (4 * per)))
         scratch = torch.empty(most * per, dtype=torch.float32, device=dev)

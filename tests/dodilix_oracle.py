@@ -296,9 +296,10 @@ def parallel_layer(heads=4, kv_heads=2, dim=32, vdim=24, chunk=21, rot=16, base=
                       "left_scale": left_scale, "right_scale": right_scale}}
 
 
-def random_weights(cfg, seed=0, sharp=2.5, rank=6):
+def random_weights(cfg, seed=0, sharp=2.5, rank=6, spread=1.0):
     """Checkpoint tensors of ``cfg`` (bf16-representable fp32): projections keep unit variance, queries are scaled by
-    ``sharp`` so that the attention is far from uniform; decays reach from a few tokens to hundreds."""
+    ``sharp`` so that the attention is far from uniform; decays reach from a few tokens to hundreds.  ``spread`` below 1: a
+    layer's experts have a part in common, so that a choice which a rounded input turns around changes little."""
     g = torch.Generator().manual_seed(seed)
     W, S = cfg["width"], cfg["streams"]
 
@@ -353,8 +354,14 @@ def random_weights(cfg, seed=0, sharp=2.5, rank=6):
         else:
             E = f["router"]["experts"]
             w[p + "mlp.router"] = mat(E, W, 2.0)
+            unit(p + "common.", f["expert"]["ff"])
             for e in range(E):
                 unit(f"{p}mlp.e{e}.", f["expert"]["ff"])
+                for c in ("gate", "up", "down"):
+                    own, common = w[f"{p}mlp.e{e}.{c}"], w[f"{p}common.{c}"]
+                    w[f"{p}mlp.e{e}.{c}"] = (spread * own + math.sqrt(1.0 - spread ** 2) * common).bfloat16().float()
+            for c in ("gate", "up", "down"):
+                del w[f"{p}common.{c}"]
             if f.get("shared"):
                 unit(p + "mlp.shared.", f["shared"]["ff"])
                 w[p + "mlp.shared.sg"] = mat(1, W)
