@@ -98,6 +98,74 @@ __global__ void __launch_bounds__(kThreads) qk_prepare_kernel(T* __restrict__ x,
                  [&](int i, float y) { v[i] = DT<T>::from_f(y); });
 }
 
+// The same 16 bytes at a time: LG lanes hold a head, a pack each (dim <= LG packs), partners meet in shuffles; a group works
+// on kHeads heads at once, whose loads are all in flight together.
+template <typename T, int LG>
+__global__ void __launch_bounds__(kThreads) qk_prepare_vec_kernel(T* __restrict__ x, int64_t ld, const int* __restrict__ slot,
+                                                                  const int* __restrict__ pos, const int* __restrict__ start,
+                                                                  Prepare p, int64_t rows, int heads, int dim) {
+  constexpr int N = Pack<T, true>::n, kHeads = 4;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t r0 = ((int64_t)blockIdx.x * (kThreads / LG) + threadIdx.x / LG) * kHeads;
+  const int lane = threadIdx.x % LG, hp = p.half / N;
+  const bool mine = lane * N < dim, first = lane < hp, turns = lane < 2 * hp;
+  T* v[kHeads];
+  float a[kHeads][N];
+  int64_t at[kHeads];
+#pragma unroll
+  for (int u = 0; u < kHeads; ++u) {
+    const int64_t r = r0 + u;
+    const int t = r < rows ? (int)(r / heads) : 0, h = r < rows ? (int)(r % heads) : 0;
+    v[u] = x + (int64_t)t * ld + (int64_t)h * dim + lane * N;
+    at[u] = (int64_t)(pos[t] - start[slot[t]]) * p.half + (first ? lane : lane - hp) * N;
+#pragma unroll
+    for (int j = 0; j < N; ++j) a[u][j] = 0.f;
+    if (r < rows && mine) load_pack<T, true>(v[u], a[u]);
+  }
+#pragma unroll
+  for (int u = 0; u < kHeads; ++u) {
+    float f = 1.f;
+    if (p.unit) {
+      float ss = 0.f;
+#pragma unroll
+      for (int j = 0; j < N; ++j) ss = fmaf(a[u][j], a[u][j], ss);
+#pragma unroll
+      for (int o = LG / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      f = 1.0f / sqrtf(ss / (float)dim + p.eps);
+    }
+    float b[N];
+    const int partner = !turns ? lane : first ? lane + hp : lane - hp;
+#pragma unroll
+    for (int j = 0; j < N; ++j) b[j] = __shfl_sync(0xffffffffu, a[u][j], partner, LG);
+    if (r0 + u < rows && mine) {
+      if (turns) {
+        const float sign = first ? -1.f : 1.f;
+#pragma unroll
+        for (int j = 0; j < N; j += 4) {
+          const float4 c = *reinterpret_cast<const float4*>(p.cosp + at[u] + j);
+          const float4 s = *reinterpret_cast<const float4*>(p.sinp + at[u] + j);
+          const float cs[4] = {c.x, c.y, c.z, c.w}, sn[4] = {s.x, s.y, s.z, s.w};
+#pragma unroll
+          for (int e = 0; e < 4; ++e) a[u][j + e] = a[u][j + e] * cs[e] + sign * b[j + e] * sn[e];
+        }
+      }
+      __align__(16) T o[N];
+#pragma unroll
+      for (int j = 0; j < N; ++j) o[j] = DT<T>::from_f(a[u][j] * f);
+      *reinterpret_cast<uint4*>(v[u]) = *reinterpret_cast<const uint4*>(o);
+    }
+  }
+}
+
+template <typename T, int LG>
+cudaError_t launch_prepare(void* x, int64_t ld, const int* slot, const int* pos, const int* start, const Prepare& p,
+                           int64_t rows, int heads, int dim, bool pdl, cudaStream_t st) {
+  const int64_t per = (int64_t)kThreads / LG * 4;
+  return launch_kernel(qk_prepare_vec_kernel<T, LG>, dim3((unsigned)((rows + per - 1) / per)), dim3(kThreads), 0, st, pdl,
+                       (T*)x, ld, slot, pos, start, p, rows, heads, dim);
+}
+
 // ---------------------------------------------------------------------------------------------- append
 struct AppendArgs {
   const void* k;        // T [tokens, ld] at head * dim
@@ -526,6 +594,14 @@ IPEX_API int ipex_qk_prepare(void* x, int64_t ld, const int* slot, const int* po
   return by_dtype(dtype, [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
     const Prepare p = {cosp, sinp, half, unit, eps};
+    constexpr int VN = 16 / (int)sizeof(T);
+    if (dim % VN == 0 && dim / VN <= 32 && half % VN == 0 && ld % VN == 0 &&
+        (((uintptr_t)x | (uintptr_t)cosp | (uintptr_t)sinp) & 15) == 0) {
+      cudaStream_t st = (cudaStream_t)stream;
+      if (dim / VN <= 8) return launch_prepare<T, 8>(x, ld, slot, pos, start, p, rows, heads, dim, pdl != 0, st);
+      if (dim / VN <= 16) return launch_prepare<T, 16>(x, ld, slot, pos, start, p, rows, heads, dim, pdl != 0, st);
+      return launch_prepare<T, 32>(x, ld, slot, pos, start, p, rows, heads, dim, pdl != 0, st);
+    }
     return launch_kernel(qk_prepare_kernel<T>, dim3((unsigned)blocks), dim3(kThreads), 0, (cudaStream_t)stream, pdl != 0,
                          (T*)x, ld, slot, pos, start, p, rows, heads, dim);
   });

@@ -529,14 +529,20 @@ __global__ void __launch_bounds__(kThreads, 1) linear_chunks_kernel(ChunkArgs s,
           split_tf32(S[m][2], fa.hi[1], fa.lo[1]);
           split_tf32(S[m][1], fa.hi[2], fa.lo[2]);
           split_tf32(S[m][3], fa.hi[3], fa.lo[3]);
+          FragB fb[4];
 #pragma unroll
           for (int n = 0; n < 4; ++n) {
             const float2 q = *reinterpret_cast<const float2*>(Q + (n * 8 + g) * ld + tile * 8 + 2 * t4);
-            FragB fb;
-            split_tf32(q.x, fb.hi[0], fb.lo[0]);
-            split_tf32(q.y, fb.hi[1], fb.lo[1]);
-            mac3(o[n], fa, fb);
+            split_tf32(q.x, fb[n].hi[0], fb[n].lo[0]);
+            split_tf32(q.y, fb[n].hi[1], fb[n].lo[1]);
           }
+          // four independent chains side by side
+#pragma unroll
+          for (int n = 0; n < 4; ++n) mma_tf32(o[n], fa.lo, fb[n].hi);
+#pragma unroll
+          for (int n = 0; n < 4; ++n) mma_tf32(o[n], fa.hi, fb[n].lo);
+#pragma unroll
+          for (int n = 0; n < 4; ++n) mma_tf32(o[n], fa.hi, fb[n].hi);
         }
       }
       // values as left operands, exact in one part
@@ -563,21 +569,35 @@ __global__ void __launch_bounds__(kThreads, 1) linear_chunks_kernel(ChunkArgs s,
 #pragma unroll
         for (int i = 0; i < 4; ++i) rd[(n * 8 + 2 * t4 + (i & 1)) * 36 + g + 8 * (i >> 1)] = o[n][i];
       // ---- S^T <- S^T diag(G) + V^T K
+      const int mine = min(per, tiles - dg * per);       // tiles of this warp that exist
+      float add[MT][4];
 #pragma unroll
-      for (int m = 0; m < MT; ++m) {
-        const int tile = dg * per + m;
-        if (m < per && tile < tiles) {
-          float add[4] = {0.f, 0.f, 0.f, 0.f};
+      for (int m = 0; m < MT; ++m)
 #pragma unroll
-          for (int k = 0; k < 4; ++k)
-            mac2(add, va[k], frag_b([&](int kk, int j) { return K[(k * 8 + kk) * ld + tile * 8 + j]; }, g, t4));
-          const float2 gd = *reinterpret_cast<const float2*>(G + tile * 8 + 2 * t4);
-          S[m][0] = fmaf(gd.x, S[m][0], add[0]);
-          S[m][1] = fmaf(gd.y, S[m][1], add[1]);
-          S[m][2] = fmaf(gd.x, S[m][2], add[2]);
-          S[m][3] = fmaf(gd.y, S[m][3], add[3]);
-        }
+        for (int i = 0; i < 4; ++i) add[m][i] = 0.f;
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        FragB fb[MT];
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+          if (m < mine)
+            fb[m] = frag_b([&](int kk, int j) { return K[(k * 8 + kk) * ld + (dg * per + m) * 8 + j]; }, g, t4);
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+          if (m < mine) mma_tf32(add[m], va[k], fb[m].lo);
+#pragma unroll
+        for (int m = 0; m < MT; ++m)
+          if (m < mine) mma_tf32(add[m], va[k], fb[m].hi);
       }
+#pragma unroll
+      for (int m = 0; m < MT; ++m)
+        if (m < mine) {
+          const float2 gd = *reinterpret_cast<const float2*>(G + (dg * per + m) * 8 + 2 * t4);
+          S[m][0] = fmaf(gd.x, S[m][0], add[m][0]);
+          S[m][1] = fmaf(gd.y, S[m][1], add[m][1]);
+          S[m][2] = fmaf(gd.x, S[m][2], add[m][2]);
+          S[m][3] = fmaf(gd.y, S[m][3], add[m][3]);
+        }
     }
     if (__syncthreads_or(!ok)) {               // the parts are in place, the stage is free again
       ok = false;
