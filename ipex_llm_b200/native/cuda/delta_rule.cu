@@ -772,8 +772,8 @@ __global__ void __launch_bounds__(kThreads) gated_norm_kernel(const float* __res
   const int64_t r = (int64_t)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
   if (r >= rows) return;
-  const int64_t t = r / heads;
-  const int h = (int)(r % heads);
+  const int64_t t = r <= 0x7fffffff ? (int64_t)((uint32_t)r / (uint32_t)heads) : r / heads;
+  const int h = (int)(r - t * heads);
   const float* src = o + r * V;
   const T* gt = gate + t * ldg + (int64_t)h * V;
   T* dst = out + t * ldo + (int64_t)h * V;

@@ -103,11 +103,11 @@ __global__ void __launch_bounds__(kThreads) qk_prepare_kernel(T* __restrict__ x,
 template <typename T, int LG>
 __global__ void __launch_bounds__(kThreads) qk_prepare_vec_kernel(T* __restrict__ x, int64_t ld, const int* __restrict__ slot,
                                                                   const int* __restrict__ pos, const int* __restrict__ start,
-                                                                  Prepare p, int64_t rows, int heads, int dim) {
+                                                                  Prepare p, uint32_t rows, uint32_t heads, int dim) {
   constexpr int N = Pack<T, true>::n, kHeads = 4;
   pdl_launch_dependents();
   pdl_wait();
-  const int64_t r0 = ((int64_t)blockIdx.x * (kThreads / LG) + threadIdx.x / LG) * kHeads;
+  const uint32_t r0 = (blockIdx.x * (kThreads / LG) + threadIdx.x / LG) * kHeads;
   const int lane = threadIdx.x % LG, hp = p.half / N;
   const bool mine = lane * N < dim, first = lane < hp, turns = lane < 2 * hp;
   T* v[kHeads];
@@ -115,8 +115,7 @@ __global__ void __launch_bounds__(kThreads) qk_prepare_vec_kernel(T* __restrict_
   int64_t at[kHeads];
 #pragma unroll
   for (int u = 0; u < kHeads; ++u) {
-    const int64_t r = r0 + u;
-    const int t = r < rows ? (int)(r / heads) : 0, h = r < rows ? (int)(r % heads) : 0;
+    const uint32_t r = r0 + u, t = r < rows ? r / heads : 0, h = r < rows ? r - t * heads : 0;
     v[u] = x + (int64_t)t * ld + (int64_t)h * dim + lane * N;
     at[u] = (int64_t)(pos[t] - start[slot[t]]) * p.half + (first ? lane : lane - hp) * N;
 #pragma unroll
@@ -163,7 +162,7 @@ cudaError_t launch_prepare(void* x, int64_t ld, const int* slot, const int* pos,
                            int64_t rows, int heads, int dim, bool pdl, cudaStream_t st) {
   const int64_t per = (int64_t)kThreads / LG * 4;
   return launch_kernel(qk_prepare_vec_kernel<T, LG>, dim3((unsigned)((rows + per - 1) / per)), dim3(kThreads), 0, st, pdl,
-                       (T*)x, ld, slot, pos, start, p, rows, heads, dim);
+                       (T*)x, ld, slot, pos, start, p, (uint32_t)rows, (uint32_t)heads, dim);
 }
 
 // ---------------------------------------------------------------------------------------------- append
@@ -595,7 +594,7 @@ IPEX_API int ipex_qk_prepare(void* x, int64_t ld, const int* slot, const int* po
     using T = std::remove_pointer_t<decltype(tag)>;
     const Prepare p = {cosp, sinp, half, unit, eps};
     constexpr int VN = 16 / (int)sizeof(T);
-    if (dim % VN == 0 && dim / VN <= 32 && half % VN == 0 && ld % VN == 0 &&
+    if (rows < (1u << 31) && dim % VN == 0 && dim / VN <= 32 && half % VN == 0 && ld % VN == 0 &&
         (((uintptr_t)x | (uintptr_t)cosp | (uintptr_t)sinp) & 15) == 0) {
       cudaStream_t st = (cudaStream_t)stream;
       if (dim / VN <= 8) return launch_prepare<T, 8>(x, ld, slot, pos, start, p, rows, heads, dim, pdl != 0, st);

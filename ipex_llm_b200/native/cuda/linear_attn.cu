@@ -58,7 +58,7 @@ struct Common {
 };
 
 __device__ __forceinline__ float channel_decay(float z, float inv_tau) {
-  const float log_sigmoid = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
+  const float log_sigmoid = fminf(z, 0.f) - logf(1.0f + expf(-fabsf(z)));    // the sum's rounding is an error of 2^-24 here
   return expf(log_sigmoid * inv_tau);
 }
 
