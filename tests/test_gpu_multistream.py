@@ -55,7 +55,7 @@ def padded(x, dtype, extra=0):
 # streams
 # ------------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", [F32, BF16, F16])
-@pytest.mark.parametrize("n,S,K", [(1, 1, 64), (3, 2, 192), (2, 3, 1028), (5, 4, 4096), (2, 4, 8192), (2, 2, 2060), (7, 5, 96),
+@pytest.mark.parametrize("n,S,K", [(1, 1, 64), (3, 2, 208), (2, 3, 1028), (5, 4, 4096), (2, 4, 8192), (2, 2, 2060), (7, 5, 96),
                                    (2, 2, 75), (1, 16, 40), (200, 2, 256), (2, 3, 9000)])
 def test_joint_between_sublayers(dtype, n, S, K):
     from ipex_llm_b200.ops import stream as St
@@ -110,7 +110,7 @@ def test_silu_gated_unit(dtype, M, ff, K):
           "from finished products", 2)
 
 
-@pytest.mark.parametrize("E,groups,keep,top,scale", [(8, 1, 1, 2, 1.0), (12, 4, 3, 4, 1.5), (16, 4, 1, 4, 0.7), (6, 6, 2, 2, 2.0),
+@pytest.mark.parametrize("E,groups,keep,top,scale", [(8, 1, 1, 2, 1.0), (15, 5, 3, 5, 1.25), (16, 4, 1, 4, 0.7), (6, 6, 2, 2, 2.0),
                                                      (64, 8, 3, 6, 2.5), (5, 1, 1, 5, 1.0), (10, 5, 5, 1, 1.0), (256, 8, 4, 8, 1.0)])
 def test_choice_of_experts(E, groups, keep, top, scale):
     """Soft-max scores, groups by their best expert, renormalised weights; group limits and renormalisation show."""
@@ -132,7 +132,7 @@ def test_choice_of_experts(E, groups, keep, top, scale):
 
 
 MOE = [  # width, ff, experts, top, groups, keep, scale, shared ff
-    (64, 32, 8, 2, 1, 1, 1.0, None), (192, 96, 12, 4, 4, 3, 1.5, 128), (96, 24, 6, 3, 3, 2, 0.7, 24), (40, 20, 4, 2, 2, 1, 2.0, 13),
+    (64, 32, 8, 2, 1, 1, 1.0, None), (176, 80, 15, 5, 5, 3, 1.25, 112), (96, 24, 6, 3, 3, 2, 0.7, 24), (40, 20, 4, 2, 2, 1, 2.0, 13),
     (50, 7, 5, 1, 1, 1, 1.0, 9), (128, 64, 16, 6, 4, 2, 2.5, 200), (256, 40, 4, 4, 1, 1, 1.0, 64)]
 
 
@@ -390,7 +390,7 @@ class Linear:
 
 LINEAR_SIZES = [  # heads, dim, vdim, rank
     (4, 16, 24, 6), (3, 32, 32, 16), (2, 128, 128, 16), (6, 24, 40, 5), (2, 10, 7, 1), (1, 200, 96, 33), (2, 256, 64, 64),
-    (2, 48, 300, 16), (4, 8, 16, 7), (4, 48, 64, 16), (1, 64, 256, 128)]
+    (2, 48, 300, 16), (4, 8, 16, 7), (5, 56, 72, 24), (1, 64, 256, 128)]
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16, F16])
