@@ -26,7 +26,8 @@ _UNSUPPORTED_KW = ("num_beams", "penalty_alpha", "num_return_sequences", "constr
 
 # engines of the package's own model classes, which run every size and weight format of their family
 _STREAM_ENGINES = {"latent": ("latent_engine", "LatentEngine"), "hybrid": ("hybrid_engine", "HybridEngine"),
-                   "multistream": ("multistream_engine", "MultiStreamEngine")}
+                   "multistream": ("multistream_engine", "MultiStreamEngine"),
+                   "parallel_block": ("parallel_block_engine", "ParallelBlockEngine")}
 
 
 def supports(model, kwargs) -> bool:

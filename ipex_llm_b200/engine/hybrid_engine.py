@@ -26,7 +26,7 @@ def _one_plus(norm):
 
 
 class HybridStack(StreamStack):
-    components = ("stream", "hybrid")
+    components = ("stream", "attention", "recurrent", "delta")
 
     def __init__(self, model):
         base = model.model

@@ -43,7 +43,7 @@ class Joint:
 
 
 class MultiStreamStack(StreamStack):
-    components = ("stream", "latent", "hybrid", "linear")
+    components = ("stream", "latent", "attention", "recurrent", "linear")
 
     def __init__(self, model):
         cfg, base = model.config, model.model
@@ -64,13 +64,6 @@ class MultiStreamStack(StreamStack):
             self._feed_forward_layer(L, blk)
             self.layers.append(L)
         self.lenders = {L.lender for L in self.layers if getattr(L, "lender", None) is not None}
-        self._rot = {}           # (base, pairs) -> (cos, sin)
-        self._rot_retired = []   # tables a captured graph may still read
-        self._positions = 0
-
-    def _store(self, shape) -> int:
-        self.shapes.append(shape)
-        return len(self.shapes) - 1
 
     def _latent_layer(self, L, m):
         dt = self.dtype
@@ -113,18 +106,6 @@ class MultiStreamStack(StreamStack):
                                   None if sh is None else sh.gate_up_rows.data.to(dt),
                                   None if sh is None else sh.down_rows.data.to(dt))
         self.kernel_launches_per_step += 4
-
-    def ensure_positions(self, n: int):
-        if n <= self._positions and self._rot:
-            return
-        n = max(2048, (n + 1023) // 1024 * 1024)
-        self._rot_retired.append(self._rot)
-        self._rot = {L.rot_key: N.rotary_table(n, *L.rot_key, self.device) for L in self.layers}
-        self._positions = n
-
-    def _rows(self, T: int, n: int):
-        """An activation of ``n`` columns whose rows start on 16-byte boundaries."""
-        return torch.empty(T, (n + 7) // 8 * 8, dtype=self.dtype, device=self.device)[:, :n]
 
     # -- mixers ---------------------------------------------------------------------------------------
     def _latent(self, L, h, slot, pos, cache, visible, portions, borrowed, pdl):

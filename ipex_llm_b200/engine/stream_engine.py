@@ -8,13 +8,14 @@ buffers, one CUDA-graph replay per token, the interface of ``DecoderEngine``).
 from __future__ import annotations
 
 import os
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 from typing import List, Optional, Sequence, Tuple
 
 import torch
 
 from ..native.lib import prepare_components
 from ..ops import cuda_ops, stream as K
+from ..ops.latent import rotary_table
 from ..ops.kv_cache import SlotCache
 from ..ops.linear import LowBitLinear
 from .decoder_engine import DecoderEngine, _W
@@ -46,8 +47,22 @@ class Portions:
     chunk_seq: torch.Tensor      # [chunks] portion of every chunk of CHUNK tokens
     seq_chunk: torch.Tensor      # [n + 1] first chunk of every portion
     chunks: int
+    lengths: Optional[List[int]] = None      # ``length`` on the host
+    _pool_rows: dict = field(default_factory=dict)
 
     CHUNK = 32
+
+    def pool_rows(self, pool: int):
+        """Where the blocks of ``pool`` tokens of every (whole) portion go when they are packed: first rows, multiples of eight
+        (int32, device), and the number of all rows."""
+        if pool not in self._pool_rows:
+            lengths = self.length.tolist() if self.lengths is None else self.lengths
+            first, n = [], 0
+            for m in lengths:
+                first.append(n)
+                n += (m // pool + 7) // 8 * 8
+            self._pool_rows[pool] = torch.tensor(first, dtype=torch.int32, device=self.row.device), max(n, 8)
+        return self._pool_rows[pool]
 
 
 def stack_for(model, cls) -> "StreamStack":
@@ -81,6 +96,9 @@ class StreamStack:
         self.layers: List[_Layer] = []
         self.shapes = []             # of the layers' cache storage
         self.final_norm = None
+        self._rot = {}               # (base, pairs) -> (cos, sin), of the layers' ``rot_key``
+        self._rot_retired = []       # tables a captured graph may still read
+        self._positions = 0
 
     @staticmethod
     def _dtype(mods):
@@ -91,7 +109,14 @@ class StreamStack:
         return torch.bfloat16
 
     def ensure_positions(self, n: int):
-        """Tables for positions below ``n`` (families whose layers have none need nothing)."""
+        """Rotation tables for positions below ``n`` (families whose layers have none need nothing)."""
+        keys = {L.rot_key for L in self.layers if getattr(L, "rot_key", None) is not None}
+        if not keys or (n <= self._positions and self._rot):
+            return
+        n = max(2048, (n + 1023) // 1024 * 1024)
+        self._rot_retired.append(self._rot)
+        self._rot = {key: rotary_table(n, *key, self.device) for key in keys}
+        self._positions = n
 
     # ------------------------------------------------------------------------------------------------
     # products
@@ -110,26 +135,36 @@ class StreamStack:
         """``x += a @ w.T``."""
         return self._linear(P, a, x, K.OUT_ADD, pdl=pdl)
 
-    def _linear(self, P: _Proj, h, out, mode, act=0, pdl=False, interleaved=True, w2=None, out2=None):
+    def _rows(self, T: int, n: int):
+        """An activation of ``n`` columns whose rows start on 16-byte boundaries."""
+        return torch.empty(T, (n + 7) // 8 * 8, dtype=self.dtype, device=self.device)[:, :n]
+
+    def _store(self, shape) -> int:
+        """Add storage to the cache's layers; returns its index."""
+        self.shapes.append(shape)
+        return len(self.shapes) - 1
+
+    def _linear(self, P: _Proj, h, out, mode, act=0, pdl=False, interleaved=True, w2=None, out2=None, args=K.NO_ARGS):
         """``act(h @ w.T + bias)`` into ``out`` (see ``OUT_*``); ``w2`` / ``out2``: further dense rows with fp32 results."""
         # (the tensor-core row product, which takes up to sixteen rows, wants gate and up rows in blocks)
         if self._few(P, h.shape[0]) and (interleaved or h.shape[0] <= 8):
-            return K.gemv_rows(P.w, h, out, mode, act=act, pdl=pdl, bias=P.bias, w2=w2, out2=out2, interleaved=interleaved)
+            return K.gemv_rows(P.w, h, out, mode, act=act, pdl=pdl, bias=P.bias, w2=w2, out2=out2, interleaved=interleaved,
+                               args=args)
         if w2 is not None and P.packed is None:
-            return K.gemm(h, P.w, out, mode, act, P.bias, interleaved, w2, out2)
+            return K.gemm(h, P.w, out, mode, act, P.bias, interleaved, w2, out2, args)
         if w2 is not None:
             if h.shape[0] <= K.rows_max(w2.shape[1], self.dtype):
                 K.gemv_rows(w2, h, out2, K.OUT_F32)
             else:
                 K.gemm(h, w2, out2, K.OUT_F32)
-        return self._product(P, h, out, mode, act, interleaved)
+        return self._product(P, h, out, mode, act, interleaved, args)
 
-    def _product(self, P: _Proj, h, out, mode, act=0, interleaved=True):
+    def _product(self, P: _Proj, h, out, mode, act=0, interleaved=True, args=K.NO_ARGS):
         if P.packed is None:
-            return K.gemm(h, P.w, out, mode, act, P.bias, interleaved)
-        w, M = P.packed, h.shape[0]
-        glu = act in (K.ACT_GELU_GLU, K.ACT_SILU_GLU)
-        y = out if mode == K.OUT_ACT and not glu else torch.empty(M, w.N, dtype=h.dtype, device=h.device)
+            return K.gemm(h, P.w, out, mode, act, P.bias, interleaved, args=args)
+        w, M, h = P.packed, h.shape[0], h.contiguous()
+        glu = act in K.GATED_ACTS
+        y = out if mode == K.OUT_ACT and not glu and out.is_contiguous() else torch.empty(M, w.N, dtype=h.dtype, device=h.device)
         if M <= cuda_ops.GEMV_MAX_M:
             per = cuda_ops._gemv_rows_per_call(w.K)
             for s in range(0, M, per):
@@ -137,11 +172,12 @@ class StreamStack:
         else:
             cuda_ops.gemm_lowbit(h, w.data, w.qtype, w.N, w.K, out=y)
         if glu:
-            return K.glu_rows(y, P.bias, out, act, interleaved)
+            return K.glu_rows(y, P.bias, out, act, interleaved, args)
         if P.bias is not None:
             K.bias_rows_(y, P.bias)
         if mode == K.OUT_ACT:
-            return K.relu2_(y) if act == K.ACT_RELU2 else y
+            out = y if y is out else out.copy_(y)
+            return K.act_rows_(out, act, args) if act in (K.ACT_RELU2, K.ACT_GELU_MUL) else out
         return K.add_stream_(out, y) if mode == K.OUT_ADD else out.copy_(y)
 
     # ------------------------------------------------------------------------------------------------
@@ -201,7 +237,7 @@ class StreamStack:
         longest = max(p0 + m for (_, p0, _), m in zip(portions, lens))
         self.ensure_positions(longest)
         whole = all(p0 == cache.first_row(s) for s, p0, _ in portions)
-        where = Portions(row, ln, max(lens), whole, owner, first_chunk, sum(per))
+        where = Portions(row, ln, max(lens), whole, owner, first_chunk, sum(per), lens)
         return self.run(tokens, slot, pos, cache, longest, portions=where, collect=collect)[0]
 
     # ------------------------------------------------------------------------------------------------

@@ -152,6 +152,8 @@ FAMILIES = {
     "letarax": Family(engine="hybrid"),
     # several 32-bit residual streams, latent attention, attention and linear attention side by side: likewise
     "dodilix": Family(engine="multistream"),
+    # mixer and feed-forward side by side, attention beside a state space, a generalized delta rule: likewise
+    "gegorax": Family(engine="parallel_block"),
     # LayerNorm families without a dedicated forward file: low-bit linears + the fused LayerNorm kernel
     "gpt_neox": Family(post=[("LayerNorm", C.layer_norm_forward)]),
     "bloom": Family(post=[("LayerNorm", C.layer_norm_forward)]),

@@ -39,8 +39,12 @@ COMPONENTS = {
     # what decoders with a 32-bit residual stream share, and what only some of them need
     "stream": ("elementwise.cu", "gemm_stream_tcgen05.cu", "gemv_dense.cu", "packed_prefill_tcgen05.cu", "stream_ops.cu"),
     "latent": ("latent_attn.cu",),
-    "hybrid": ("delta_rule.cu", "kv_attn.cu"),
+    "attention": ("kv_attn.cu",),
+    "recurrent": ("recurrent_ops.cu",),
+    "delta": ("delta_rule.cu",),
+    "general_delta": ("general_delta.cu",),
     "linear": ("linear_attn.cu",),
+    "ssd": ("ssd.cu",),
 }
 
 NVCC_ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]

@@ -13,8 +13,6 @@
 //                 W = (I + A)^-1 beta e^L K
 //   delta_chunks  second half, sequential over a sequence's chunks: U = Ub - W S, O = e^L Q S + P U with
 //                 P[t,i] = e^(L_t - L_i) (q_t . k_i) for i <= t, S <- e^L_end S + (e^(L_end - L) K)^T U
-//   delta_tail    the last inputs of the convolutions into the slot's ring
-//   gated_norm    o / rms(o) * w * silu(gate) behind delta_chunks
 //
 // The products of the chunked form run on the tensor cores with every fp32 operand split into two tf32 parts (three
 // products, about 22 bits), accumulated in fp32; the state itself is only ever added to in fp32.  The state's columns
@@ -25,6 +23,8 @@
 // state there, so a slot needs no clearing when it changes hands.
 #include <cooperative_groups.h>
 
+#include "common/short_conv.cuh"
+#include "common/state_cols.cuh"
 #include "common/tf32_pairs.cuh"
 #include "common/utils.cuh"
 #include "tcgen05_common.cuh"
@@ -66,46 +66,11 @@ struct Common {
 
 constexpr float kUnitEps = 1e-6f;
 
-// silu of a 16-bit model's convolution
-__device__ __forceinline__ float fast_silu(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
-
-// Channel c of the convolution after silu, at packed token t: token j of its portion, position p of its sequence.  w: the
-// channel's last tap.
-template <typename T, typename TW>
-__device__ __forceinline__ float conv_silu(const Common& a, int c, int t, int j, int p, int start, int slot,
-                                           const TW* w) {
-  const T* proj = reinterpret_cast<const T*>(a.proj) + (int64_t)t * a.ldp + c;
-  const T* ring = reinterpret_cast<const T*>(a.ring) + (int64_t)slot * a.taps * a.channels + c;
-  const int pm = p % a.taps, seen = min(a.taps, p - start + 1);
-  float s = 0.f;
-  for (int b0 = 0; b0 < a.taps; b0 += 4) {
-    T x[4];
-    float wv[4];
-#pragma unroll
-    for (int u = 0; u < 4; ++u) {
-      const int back = b0 + u;
-      x[u] = DT<T>::from_f(0.f);
-      wv[u] = 0.f;
-      if (back < a.taps) {                       // (rows from before the start are read and not used: `start` comes late)
-        const int r = pm - back;
-        x[u] = back <= j ? proj[-(int64_t)back * a.ldp] : ring[(int64_t)(r < 0 ? r + a.taps : r) * a.channels];
-        wv[u] = DT<TW>::to_f(w[-back]);
-      }
-    }
-#pragma unroll
-    for (int u = 0; u < 4; ++u)
-      if (b0 + u < seen) s = fmaf(DT<T>::to_f(x[u]), wv[u], s);
-  }
-  return silu(s);
-}
-
 // log of the decay and write strength of one token and head
 __device__ __forceinline__ float log_decay(float a, float dt_bias, float a_log) {
   const float z = a + dt_bias;
-  const float sp = z > 20.f ? z : log1pf(expf(z));
-  return -expf(a_log) * sp;
+  return -expf(a_log) * softplusf(z);
 }
-__device__ __forceinline__ float sigmoidf(float x) { return 1.0f / (1.0f + expf(-x)); }
 
 // ---------------------------------------------------------------------------------------------- token by token
 struct StepArgs {
@@ -119,25 +84,6 @@ struct StepArgs {
   int ring_write;         // one token per sequence: file its convolution inputs
   int prefetch;           // slots are final before the kernels in front of this one end: fetch states early
 };
-
-template <int N>
-__device__ __forceinline__ void load_cols(const float* p, float (&v)[N]) {
-  if constexpr (N == 4) {
-    const float4 x = *reinterpret_cast<const float4*>(p);
-    v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
-  } else if constexpr (N == 2) {
-    const float2 x = *reinterpret_cast<const float2*>(p);
-    v[0] = x.x; v[1] = x.y;
-  } else {
-    v[0] = *p;
-  }
-}
-template <int N>
-__device__ __forceinline__ void store_cols(float* p, const float (&v)[N]) {
-  if constexpr (N == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-  else if constexpr (N == 2) *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
-  else *p = v[0];
-}
 
 // A warp owns the state rows warp, warp + 8, ...; a lane CV neighbouring columns of the CTA's 32 CV.
 template <typename T, int NR, int CV>
@@ -338,51 +284,6 @@ struct ChunkArgs {
   int c0, c1;
   int vec;                  // rows of proj and ring can be read 16 bytes at a time
 };
-
-// Eight neighbouring channels of the convolution for four tokens: every input row is read once.  TP: taps, 0 if only
-// known at run time.  first: token (of the chunk) of the first output; ws [taps][ldws]: weights of these channels.
-template <typename T, int TP>
-__device__ __forceinline__ void conv_block(const Common& a, int c, int t0, int row0, int p0, int start, int slot, int n,
-                                           int first, const float* ws, int ldws, float (&acc)[4][8]) {
-  const int taps = TP > 0 ? TP : a.taps;
-  const T* proj = reinterpret_cast<const T*>(a.proj) + c;
-  const T* ring = reinterpret_cast<const T*>(a.ring) + (int64_t)slot * taps * a.channels + c;
-#pragma unroll
-  for (int j = 0; j < 4; ++j)
-#pragma unroll
-    for (int e = 0; e < 8; ++e) acc[j][e] = 0.f;
-  auto row = [&](int rr) {
-    const int rel = first - (taps - 1) + rr, p = p0 + rel, t = t0 + rel;
-    uint4 raw = make_uint4(0, 0, 0, 0);
-    if (p >= start && rel < n)
-      raw = *reinterpret_cast<const uint4*>(t >= row0 ? proj + (int64_t)t * a.ldp
-                                                      : ring + (int64_t)(p % taps) * a.channels);
-    return raw;
-  };
-  auto use = [&](int rr, const uint4& raw) {
-    const T* e8 = reinterpret_cast<const T*>(&raw);
-#pragma unroll
-    for (int j = 0; j < 4; ++j) {
-      const int i = rr - j;
-      if (i >= 0 && i < taps) {
-        const float4 w0 = *reinterpret_cast<const float4*>(ws + i * ldws);
-        const float4 w1 = *reinterpret_cast<const float4*>(ws + i * ldws + 4);
-        const float w[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
-#pragma unroll
-        for (int e = 0; e < 8; ++e) acc[j][e] = fmaf(DT<T>::to_f(e8[e]), w[e], acc[j][e]);
-      }
-    }
-  };
-  if constexpr (TP > 0) {
-    uint4 raw[TP + 3];
-#pragma unroll
-    for (int rr = 0; rr < TP + 3; ++rr) raw[rr] = row(rr);
-#pragma unroll
-    for (int rr = 0; rr < TP + 3; ++rr) use(rr, raw[rr]);
-  } else {
-    for (int rr = 0; rr < taps + 3; ++rr) use(rr, row(rr));
-  }
-}
 
 template <typename T, int TP>
 __global__ void __launch_bounds__(kThreads, 3) delta_prep_kernel(ChunkArgs s) {
@@ -751,65 +652,6 @@ __global__ void __launch_bounds__(kChunkThreads, 1) delta_chunks_kernel(ChunkArg
       }
 }
 
-template <typename T>
-__global__ void __launch_bounds__(kThreads) delta_tail_kernel(Common a) {
-  const int seq = blockIdx.y, len = a.seq_len[seq], row0 = a.seq_row[seq], n = min(len, a.taps);
-  const int c = blockIdx.x * kThreads + threadIdx.x, slot = a.slot[row0], p0 = a.pos[row0];
-  if (c >= a.channels) return;
-  T* ring = reinterpret_cast<T*>(a.ring) + (int64_t)slot * a.taps * a.channels + c;
-  const T* proj = reinterpret_cast<const T*>(a.proj) + c;
-  for (int j = len - n; j < len; ++j)
-    ring[(int64_t)((p0 + j) % a.taps) * a.channels] = proj[(int64_t)(row0 + j) * a.ldp];
-}
-
-// A warp per (token, head); VEC: four neighbouring columns per lane and step.
-template <typename T, bool VEC>
-__global__ void __launch_bounds__(kThreads) gated_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate,
-                                                              int64_t ldg, const T* __restrict__ w, T* __restrict__ out,
-                                                              int64_t ldo, int64_t rows, int heads, int V, float eps,
-                                                              float scale) {
-  constexpr int N = VEC ? 4 : 1;
-  const int64_t r = (int64_t)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
-  const int lane = threadIdx.x & 31;
-  if (r >= rows) return;
-  const int64_t t = r <= 0x7fffffff ? (int64_t)((uint32_t)r / (uint32_t)heads) : r / heads;
-  const int h = (int)(r - t * heads);
-  const float* src = o + r * V;
-  const T* gt = gate + t * ldg + (int64_t)h * V;
-  T* dst = out + t * ldo + (int64_t)h * V;
-  auto load = [&](const T* p, float (&v)[N]) {
-    if constexpr (VEC && sizeof(T) == 2) {
-      const uint2 raw = *reinterpret_cast<const uint2*>(p);
-#pragma unroll
-      for (int c = 0; c < N; ++c) v[c] = DT<T>::to_f(reinterpret_cast<const T*>(&raw)[c]);
-    } else {
-#pragma unroll
-      for (int c = 0; c < N; ++c) v[c] = DT<T>::to_f(p[c]);
-    }
-  };
-  float x[N], gv[N], wv[N], ss = 0.f;
-  for (int i = lane * N; i < V; i += 32 * N) {
-    load_cols<N>(src + i, x);
-#pragma unroll
-    for (int c = 0; c < N; ++c) ss = fmaf(x[c], x[c], ss);
-  }
-  const float inv = scale / sqrtf(warp_sum(ss) / (float)V + eps);
-  for (int i = lane * N; i < V; i += 32 * N) {
-    load_cols<N>(src + i, x);
-    load(gt + i, gv);
-    load(w + i, wv);
-    __align__(16) T y[N];
-#pragma unroll
-    for (int c = 0; c < N; ++c) y[c] = DT<T>::from_f(x[c] * inv * wv[c] * silu(gv[c]));
-    if constexpr (VEC && sizeof(T) == 2) {
-      *reinterpret_cast<uint2*>(dst + i) = *reinterpret_cast<const uint2*>(y);
-    } else {
-#pragma unroll
-      for (int c = 0; c < N; ++c) dst[i + c] = y[c];
-    }
-  }
-}
-
 bool sizes_ok(int heads, int kv_heads, int dim, int vdim, int taps) {
   return heads >= 1 && heads <= 65535 && kv_heads >= 1 && heads % kv_heads == 0 && dim >= 1 && dim <= 512 && vdim >= 1 &&
          vdim <= 65535 && taps >= 1;
@@ -954,35 +796,4 @@ IPEX_API int ipex_delta_chunks(const void* proj, int64_t ldp, const float* gates
     return cudaGetLastError();
   };
   return (int)(dtype == DT_F16 ? run((__half*)nullptr) : run((__nv_bfloat16*)nullptr));
-}
-
-// The last convolution inputs of every sequence into its slot's ring (after everything that reads the ring).
-IPEX_API int ipex_delta_tail(const void* proj, int64_t ldp, void* ring, const int* slot, const int* pos,
-                             const int* seq_row, const int* seq_len, int seqs, int channels, int taps, int dtype,
-                             void* stream) {
-  if (seqs < 1 || seqs > 65535 || channels < 1 || taps < 1) return (int)cudaErrorInvalidValue;
-  return by_dtype(dtype, [&](auto* tag) {
-    using T = std::remove_pointer_t<decltype(tag)>;
-    Common c = {};
-    c.proj = proj; c.ldp = ldp; c.ring = ring; c.slot = slot; c.pos = pos; c.seq_row = seq_row; c.seq_len = seq_len;
-    c.channels = channels; c.taps = taps;
-    delta_tail_kernel<T><<<dim3((channels + kThreads - 1) / kThreads, seqs), kThreads, 0, (cudaStream_t)stream>>>(c);
-    return cudaGetLastError();
-  });
-}
-
-// out[t, h, :] = scale * o / sqrt(mean(o^2) + eps) * w * silu(gate), o [tokens, heads, vdim] fp32
-IPEX_API int ipex_gated_norm(const float* o, const void* gate, int64_t ldg, const void* w, void* out, int64_t ldo,
-                             int tokens, int heads, int vdim, float eps, float scale, int dtype, void* stream) {
-  if (tokens < 1 || heads < 1 || vdim < 1) return (int)cudaErrorInvalidValue;
-  return by_dtype(dtype, [&](auto* tag) {
-    using T = std::remove_pointer_t<decltype(tag)>;
-    const int64_t rows = (int64_t)tokens * heads;
-    const bool vec = vdim % 4 == 0 && ldg % 4 == 0 && ldo % 4 == 0 && ((uintptr_t)o & 15) == 0 &&
-                     (((uintptr_t)gate | (uintptr_t)w | (uintptr_t)out) & 7) == 0;
-    auto kern = vec ? gated_norm_kernel<T, true> : gated_norm_kernel<T, false>;
-    kern<<<(unsigned)((rows + 7) / 8), kThreads, 0, (cudaStream_t)stream>>>(o, (const T*)gate, ldg, (const T*)w, (T*)out,
-                                                                            ldo, rows, heads, vdim, eps, scale);
-    return cudaGetLastError();
-  });
 }

@@ -3,7 +3,9 @@
 //     out = x[M, K] . W[N, K]^T (+ bias)  out_mode 0: 16-bit, optionally squared relu      1: added to an fp32 stream
 //                                         2: fp32 (router scores, logits)
 //     y = glu(row_scale * (x . W_gu^T))                    gate / up rows interleaved in 16-row tiles, N / 2 columns
-//     y = gelu_tanh(gate) * up or silu(gate) * up          gate / up rows interleaved in 8-row tiles, N / 2 columns
+//     y = gelu_tanh(gate) * up, silu(gate) * up or a       gate / up rows interleaved in 8-row tiles, N / 2 columns
+//         clamped unit
+//     y = gelu_tanh(x . W^T) * the token's row of a table
 //
 // A second matrix (w2) may ride along: its rows multiply the same x and leave as fp32 in an output of their own.
 //
@@ -30,12 +32,17 @@ struct Args {
   int* err;
   int64_t ldo;
   int M, N, K, groups;
-  int out_mode, act;        // act 1: squared relu (out_mode 0); 2: clamped gated unit; 3 / 4: gelu- / silu-gated unit
+  int out_mode, act;        // act 1: squared relu (out_mode 0); 2: clamped gated unit of scaled rows; 3 / 4 / 5: gelu- /
+                            // silu-gated / clamped unit; 6: gelu times the token's row of `mul`
   float limit, alpha;
   const void* bias;         // T [N] or null
   float* out2;              // fp32 [M, ldo2], results of the second matrix's N2 rows (0: there is none)
   int64_t ldo2;
   int N2;
+  int act_from;             // act 1: columns from this one on
+  const void* mul;          // act 6: T [mul_rows, ldm]
+  const int64_t* ids;       // ... and its rows, [M]
+  int64_t ldm, mul_rows;
 };
 
 template <int BT>
@@ -213,7 +220,7 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
           continue;
         }
         const float bn = a.bias != nullptr && n < a.N ? to_float<T>(reinterpret_cast<const T*>(a.bias)[n]) : 0.f;
-        if (a.act >= 3) {
+        if (a.act >= 3 && a.act <= 5) {
           // lanes with bit 3 clear hold gate rows, the lanes eight above them the matching up rows: the former finish
           // the even tokens of a pair, the latter the odd ones
           const int n_out = (tl.nb * kBM + qd * 32) / 2 + (lane >> 4) * 8 + (lane & 7);
@@ -224,9 +231,15 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
             const float s0 = __uint_as_float(v[j]) + bn, s1 = __uint_as_float(v[j + 1]) + bn;
             const float got = __shfl_xor_sync(0xffffffffu, upper ? s0 : s1, 8);
             const float gv = upper ? got : s0, uv = upper ? s1 : got;
-            const float e = a.act == 4 ? gv : 1.5957691216057308f * (gv + 0.044715f * gv * gv * gv);
-            if (writer && j + upper < lim)
-              out[(int64_t)j * a.ldo] = from_float<T>(__fdividef(gv, 1.0f + __expf(-e)) * uv);
+            float f;
+            if (a.act == 5) {
+              const float gc = fminf(gv, a.limit);
+              f = __fdividef(gc, 1.0f + __expf(-a.alpha * gc)) * (fminf(fmaxf(uv, -a.limit), a.limit) + 1.0f);
+            } else {
+              const float e = a.act == 4 ? gv : 1.5957691216057308f * (gv + 0.044715f * gv * gv * gv);
+              f = __fdividef(gv, 1.0f + __expf(-e)) * uv;
+            }
+            if (writer && j + upper < lim) out[(int64_t)j * a.ldo] = from_float<T>(f);
           }
         } else if (a.act == 2) {
           // lanes 0..15 hold gate rows, lanes 16..31 the matching up rows
@@ -243,12 +256,22 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
               out[(int64_t)j * a.ldo] = from_float<T>(g / (1.0f + __expf(-a.alpha * g)) * (u + 1.0f));
           }
         } else if (n < a.N) {
-          if (a.out_mode == 0) {
+          if (a.act == 6) {
+            T* out = reinterpret_cast<T*>(a.out) + r0 * a.ldo + n;
+            const T* mul = reinterpret_cast<const T*>(a.mul) + n;
+#pragma unroll
+            for (int j = 0; j < 32; ++j) {
+              if (j < lim) {
+                const int64_t id = a.ids[r0 + j], row = id < 0 ? 0 : id >= a.mul_rows ? a.mul_rows - 1 : id;
+                out[(int64_t)j * a.ldo] = from_float<T>(gelu_tanh(__uint_as_float(v[j]) + bn) * to_float<T>(mul[row * a.ldm]));
+              }
+            }
+          } else if (a.out_mode == 0) {
             T* out = reinterpret_cast<T*>(a.out) + r0 * a.ldo + n;
 #pragma unroll
             for (int j = 0; j < 32; ++j) {
               float f = __uint_as_float(v[j]) + bn;
-              if (a.act == 1) f = f > 0.f ? f * f : 0.f;
+              if (a.act == 1 && n >= a.act_from) f = f > 0.f ? f * f : 0.f;
               if (j < lim) out[(int64_t)j * a.ldo] = from_float<T>(f);
             }
           } else {
@@ -325,19 +348,22 @@ int dispatch(int bt, const void* x, int64_t ldx, int x_rows, const void* w, int6
 }  // namespace
 
 // See the head of this file.  M: rows of x; with `ranges` the groups' rows partition them.  w: [groups * N, K].  bt:
-// token tile (32 / 64 / 128 / 256).  row_scale only with act 2 (then out_mode 0 and N a multiple of 32).  act 3, 4: out_mode
-// 0, N a multiple of 16.  bias (may be null) has N entries of the operands' type; not with act 2 or ranges.
+// token tile (32 / 64 / 128 / 256).  row_scale only with act 2 (then out_mode 0 and N a multiple of 32).  act 1: columns from
+// act_from on.  act 3 to 5: out_mode 0, N a multiple of 16.  act 6: out_mode 0, no ranges, `mul` [mul_rows, ldm] and the
+// tokens' rows of it, ids [M].  bias (may be null) has N entries of the operands' type; not with act 2 or ranges.
 // w2 / out2 (N2 = 0: none): N2 more rows of the same row stride, results in fp32; not with ranges or act 2.
 // Strides of x and w multiples of 8 elements, bases 16-byte aligned.  Returns a cudaError_t, or -1 when the
 // tensor-map encoder rejects the operands.
 IPEX_API int ipex_gemm_stream(const void* x, int64_t ldx, const void* w, int64_t ldw, void* out, int64_t ldo,
                               const void* bias, const void* w2, int N2, float* out2, int64_t ldo2, const float* row_scale, const int* ranges, int groups, int M, int N, int K, int out_mode,
-                              int act, float limit, float alpha, int bt, int dtype, int* err, void* stream) {
+                              int act, float limit, float alpha, int act_from, const void* mul, int64_t ldm, int64_t mul_rows,
+                              const int64_t* ids, int bt, int dtype, int* err, void* stream) {
   if (M < 1 || N < 1 || K < 1 || groups < 1 || (ldx % 8) != 0 || (ldw % 8) != 0 || out_mode < 0 || out_mode > 2)
     return (int)cudaErrorInvalidValue;
   if ((groups > 1) != (ranges != nullptr) && ranges == nullptr) return (int)cudaErrorInvalidValue;
   if (act == 2 && (row_scale == nullptr || out_mode != 0 || (N % 32) != 0)) return (int)cudaErrorInvalidValue;
-  if (act < 0 || act > 4 || (act == 1 && out_mode != 0) || (act >= 3 && (out_mode != 0 || (N % 16) != 0)) ||
+  if (act < 0 || act > 6 || (act == 1 && out_mode != 0) || (act >= 3 && act <= 5 && (out_mode != 0 || (N % 16) != 0)) ||
+      (act == 6 && (out_mode != 0 || ranges != nullptr || mul == nullptr || ids == nullptr || mul_rows < 1)) ||
       (bias != nullptr && (act == 2 || ranges != nullptr)))
     return (int)cudaErrorInvalidValue;
   if ((reinterpret_cast<uintptr_t>(x) & 15) || (reinterpret_cast<uintptr_t>(w) & 15)) return (int)cudaErrorInvalidValue;
@@ -346,7 +372,7 @@ IPEX_API int ipex_gemm_stream(const void* x, int64_t ldx, const void* w, int64_t
                             (reinterpret_cast<uintptr_t>(w2) & 15))))
     return (int)cudaErrorInvalidValue;
   Args a = {out, row_scale, ranges, err, ldo, M, N, K, groups, out_mode, act, limit, alpha, bias,
-            out2, ldo2, N2};
+            out2, ldo2, N2, act_from, mul, ids, ldm, mul_rows};
   cudaStream_t st = (cudaStream_t)stream;
   if (dtype == DT_F16) return dispatch<__half>(bt, x, ldx, M, w, ldw, w2, a, st);
   if (dtype == DT_BF16) return dispatch<__nv_bfloat16>(bt, x, ldx, M, w, ldw, w2, a, st);

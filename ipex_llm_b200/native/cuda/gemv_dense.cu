@@ -3,13 +3,14 @@
 //   gemv_rows    y[M <= 8, N] = act( x . W[N, K]^T )   with x either activations in the weight dtype or the fp32
 //                residual stream, RMS-normed while it is staged in shared memory; the result (plus a bias) goes out in
 //                the weight dtype, is added to an fp32 residual, or leaves as fp32 with an optional tanh soft-cap
-//                (logits); gate and up rows may be joined to gelu_tanh(gate) * up or silu(gate) * up, and the rows of a
-//                second matrix may ride along with fp32 results (gates of a recurrence beside its projections)
+//                (logits); gate and up rows may be joined to gelu_tanh(gate) * up, silu(gate) * up or a clamped unit, results
+//                to gelu_tanh(.) * the token's row of a table, and the rows of a second matrix may ride along with fp32
+//                results (gates of a recurrence beside its projections)
 //   moe_router   norm + router scores in fp32 + sigmoid + top-k of one token per CTA; or, from finished rows, soft-max
 //                scores, group-limited top-k with renormalised weights, and the gate of a shared expert
-//   moe_glu      per (token, choice) slot: gated unit of the chosen expert - clamped, the routing weight applied to the
-//                expert's input, or silu; a shared expert of another size is one more choice
-//   moe_down     residual[t] += sum over the token's choices of down_e(y), or fp32 rows of the weighted sum
+//   moe_glu      per (token, choice) slot: gated unit of the chosen expert - clamped (with the routing weight applied to the
+//                expert's input, or not), or silu; a shared expert of another size is one more choice
+//   moe_down     residual[t] += sum over the token's choices of down_e(y), weighted or not, or fp32 rows of the weighted sum
 //
 // All products are fp32 FMAs over 16-byte weight loads: with up to eight rows the weights are the traffic, and eight
 // rows of FMAs still fit under the memory time.  A warp owns R weight rows and walks K in steps of 32 vectors with
@@ -112,15 +113,23 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
   return warp_sum(t);
 }
 
-// Stage `rows` rows: plain copy of T rows, or RMS norm of fp32 rows.  Zero fill up to kp.  Whole block; `red` holds one
-// float per warp.
+// Stage `rows` rows: plain copy of T rows, or fp32 rows converted (x_f32) or RMS-normed.  Zero fill up to kp.  Whole block;
+// `red` holds one float per warp.
 template <typename T>
 __device__ __forceinline__ void stage_rows(T* sx, int kp, const void* x, int64_t ldx, const T* norm_w, float eps,
-                                           int rows, int K, float* red) {
+                                           int rows, int K, float* red, bool x_f32 = false) {
   constexpr int VN = Vec<T>::n;
   const int warps = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   for (int m = 0; m < rows; ++m)
     for (int k = K + threadIdx.x; k < kp; k += blockDim.x) sx[(size_t)m * kp + k] = DT<T>::from_f(0.f);
+  if (norm_w == nullptr && x_f32) {
+    for (int m = 0; m < rows; ++m) {
+      const float* src = reinterpret_cast<const float*>(x) + (int64_t)m * ldx;
+      for (int k = threadIdx.x; k < K; k += blockDim.x) sx[(size_t)m * kp + k] = DT<T>::from_f(src[k]);
+    }
+    __syncthreads();
+    return;
+  }
   if (norm_w == nullptr) {
     for (int m = 0; m < rows; ++m) {
       T* dst = sx + (size_t)m * kp;
@@ -183,23 +192,36 @@ __device__ __forceinline__ void stage_rows(T* sx, int kp, const void* x, int64_t
 
 struct GemvRowsArgs {
   const void* w;         // [N, K], row stride ldw
-  const void* x;         // T [M, K] or fp32 [M, K] (norm_w != null), row stride ldx
+  const void* x;         // T [M, K] or fp32 [M, K] (norm_w != null or x_f32), row stride ldx
   const void* norm_w;    // T [K] or null
   void* out;             // out_mode 0: T [M, N]; 1: fp32, accumulated into; 2: fp32 written (soft-capped)
   int64_t ldw, ldx, ldo;
   float eps, softcap;
   int M, N, K, kp;
-  int out_mode, act;     // act 1: square of relu; 3 / 4: gelu_tanh / silu(gate) * up, N / 2 columns come out
+  int out_mode, act;     // act 1: square of relu; 3 / 4 / 5: gelu_tanh / silu(gate) * up / clamped unit, N / 2 columns come
+                         // out; 6: gelu_tanh times the token's row of `mul`
   int vec;
   const void* bias;      // T [N] or null
   const void* w2;        // rows N1 .. N (row stride ldw), or null (then N1 = N)
   float* out2;           // ... and their results, fp32
   int64_t ldo2;
   int N1;
-  int interleaved;       // act 3, 4: gate and up rows alternate in blocks of eight, else gate rows before up rows
+  int interleaved;       // act 3 to 5: gate and up rows alternate in blocks of eight, else gate rows before up rows
+  int act_from;          // act 1: rows from this one on
+  int x_f32;
+  float limit, alpha;    // act 5
+  const void* mul;       // act 6: T [mul_rows, ldm]
+  const int64_t* ids;    // ... and its rows, [M]
+  int64_t ldm, mul_rows;
 };
 
-__device__ __forceinline__ float finish(float v, int act) { return act == 1 ? (v > 0.f ? v * v : 0.f) : v; }
+__host__ __device__ __forceinline__ bool gated(int act) { return act >= 3 && act <= 5; }
+
+// clamped gated unit
+__device__ __forceinline__ float clamped_unit(float g, float u, float limit, float alpha) {
+  g = fminf(g, limit);
+  return g / (1.0f + expf(-alpha * g)) * (fminf(fmaxf(u, -limit), limit) + 1.0f);
+}
 
 template <typename T>
 __device__ __forceinline__ const T* weight_row(const GemvRowsArgs& a, int n) {
@@ -216,7 +238,8 @@ __device__ __forceinline__ float bias_of(const GemvRowsArgs& a, int n) {
 template <typename T>
 __device__ __forceinline__ void store_gated(const GemvRowsArgs& a, int m, int i, int ng, int nu, float g, float u) {
   const float z = g + bias_of<T>(a, ng);
-  const float v = (a.act == 4 ? silu(z) : gelu_tanh(z)) * (u + bias_of<T>(a, nu));
+  u += bias_of<T>(a, nu);
+  const float v = a.act == 5 ? clamped_unit(z, u, a.limit, a.alpha) : (a.act == 4 ? silu(z) : gelu_tanh(z)) * u;
   reinterpret_cast<T*>(a.out)[(int64_t)m * a.ldo + i] = DT<T>::from_f(v);
 }
 
@@ -226,7 +249,13 @@ __device__ __forceinline__ void store_row(const GemvRowsArgs& a, int m, int n, f
     a.out2[(int64_t)m * a.ldo2 + n - a.N1] = v;
     return;
   }
-  v = finish(v + bias_of<T>(a, n), a.act);
+  v += bias_of<T>(a, n);
+  if (a.act == 1 && n >= a.act_from) {
+    v = v > 0.f ? v * v : 0.f;
+  } else if (a.act == 6) {
+    const int64_t row = min(max(a.ids[m], (int64_t)0), a.mul_rows - 1);
+    v = gelu_tanh(v) * DT<T>::to_f(reinterpret_cast<const T*>(a.mul)[row * a.ldm + n]);
+  }
   if (a.out_mode == 0) {
     reinterpret_cast<T*>(a.out)[(int64_t)m * a.ldo + n] = DT<T>::from_f(v);
   } else {
@@ -253,7 +282,7 @@ __global__ void __launch_bounds__(kThreads) gemv_rows_kernel(GemvRowsArgs a) {
   if (a.vec && t0 < ntask && lane < R && row_of(t0, lane) < a.N)
     prefetch_l2_bulk(weight_row<T>(a, row_of(t0, lane)), (uint32_t)(a.K * sizeof(T)));
   pdl_wait();
-  stage_rows<T>(sx, a.kp, a.x, a.ldx, reinterpret_cast<const T*>(a.norm_w), a.eps, a.M, a.K, red);
+  stage_rows<T>(sx, a.kp, a.x, a.ldx, reinterpret_cast<const T*>(a.norm_w), a.eps, a.M, a.K, red, a.x_f32 != 0);
   for (int t = t0; t < ntask; t += gridDim.x * kWarps) {
     const T* w[R];
 #pragma unroll
@@ -314,9 +343,9 @@ __global__ void __launch_bounds__(kThreads) gemv_mma_kernel(GemvRowsArgs a, int 
     if (lane < 16 && row < a.N && bytes > 0) prefetch_l2_bulk(weight_row<T>(a, row) + k0, (uint32_t)bytes);
   }
   pdl_wait();
-  const bool staged = a.norm_w != nullptr;
+  const bool staged = a.norm_w != nullptr || a.x_f32;
   if (staged)
-    stage_rows<T>(sx, a.kp, a.x, a.ldx, reinterpret_cast<const T*>(a.norm_w), a.eps, a.M, a.K, red);
+    stage_rows<T>(sx, a.kp, a.x, a.ldx, reinterpret_cast<const T*>(a.norm_w), a.eps, a.M, a.K, red, a.x_f32 != 0);
   const T* xs[NT];
   bool xon[NT];
 #pragma unroll
@@ -369,7 +398,7 @@ __global__ void __launch_bounds__(kThreads) gemv_mma_kernel(GemvRowsArgs a, int 
       __syncthreads();
       // the group's warps share the sums: value (n, i) goes to warp (n * 4 + i) % split
       const float* grp = part + ((size_t)par * kWarps + warp / split * split) * (NT * 128);
-      if (a.act >= 3) {
+      if (gated(a.act)) {
 #pragma unroll
         for (int n = 0; n < NT; ++n)
 #pragma unroll
@@ -395,7 +424,7 @@ __global__ void __launch_bounds__(kThreads) gemv_mma_kernel(GemvRowsArgs a, int 
             const int row = tile * 16 + g + 8 * (i >> 1), m = n * 8 + 2 * t + (i & 1);
             if (tile < ntile && row < a.N && m < a.M) store_row<T>(a, m, row, v);
           }
-    } else if (a.act >= 3) {
+    } else if (gated(a.act)) {
 #pragma unroll
       for (int n = 0; n < NT; ++n)
 #pragma unroll
@@ -443,7 +472,7 @@ cudaError_t launch_gemv(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
 template <typename T, int M>
 cudaError_t pick_rows(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
   const int warps = sm_count() * kWarps;
-  if (a.act >= 3) return launch_gemv<T, M, 2, true>(a, pdl, st);
+  if (gated(a.act)) return launch_gemv<T, M, 2, true>(a, pdl, st);
   if (a.N >= 4 * warps) return launch_gemv<T, M, 4>(a, pdl, st);
   if (a.N >= warps) return launch_gemv<T, M, 2>(a, pdl, st);
   return launch_gemv<T, M, 1>(a, pdl, st);
@@ -453,7 +482,7 @@ template <typename T, int NT>
 cudaError_t launch_gemv_mma(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
   auto kern = gemv_mma_kernel<T, NT>;
   a.kp = (a.K + 31) / 32 * 32 + 32;        // 64 bytes of skew between rows: neighbouring tokens in different banks
-  const size_t smem = (size_t)2 * kWarps * NT * 128 * sizeof(float) + (a.norm_w != nullptr ? (size_t)a.M * a.kp * sizeof(T) : 0);
+  const size_t smem = (size_t)2 * kWarps * NT * 128 * sizeof(float) + (a.norm_w != nullptr || a.x_f32 ? (size_t)a.M * a.kp * sizeof(T) : 0);
   if (smem > 226 * 1024) return cudaErrorInvalidValue;
   if (smem > 40 * 1024) {                 // (static shared memory counts against the default limit too)
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -473,8 +502,8 @@ bool mma_from(const GemvRowsArgs& a) { return a.M >= g_mma_from; }
 template <typename T>
 cudaError_t pick_m(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
   if constexpr (sizeof(T) == 2) {
-    const bool direct = a.norm_w != nullptr || ((reinterpret_cast<uintptr_t>(a.x) & 15) == 0 && a.ldx % 8 == 0);
-    if (a.vec && direct && mma_from(a) && (a.act < 3 || a.interleaved)) {
+    const bool direct = a.norm_w != nullptr || a.x_f32 || ((reinterpret_cast<uintptr_t>(a.x) & 15) == 0 && a.ldx % 8 == 0);
+    if (a.vec && direct && mma_from(a) && (!gated(a.act) || a.interleaved)) {
       if (a.M <= 8) return launch_gemv_mma<T, 1>(a, pdl, st);
       return launch_gemv_mma<T, 2>(a, pdl, st);
     }
@@ -613,11 +642,13 @@ struct MoeArgs {
   int K, I, E, k, kp;
   int tile;                // gate / up rows in alternating tiles of this many rows; 0: gate rows then up rows
   int vec;
-  int act;                 // glu: 2 clamped, on weighted inputs; 4 silu(gate) * up
+  int act;                 // glu: 2 clamped, on weighted inputs; 4 silu(gate) * up; 5 clamped
   const void* ws;          // the shared expert, number E of idx: glu [2 Is, K], down [N, Is]
   int Is, vec_s, tile_s;
   int64_t ldy;             // row stride of the hidden units (at least I and Is)
-  int weighted;            // down: weights applied here, results written instead of added
+  int weighted;            // down: weights applied here
+  int add;                 // down: results added instead of written
+  float limit_s;           // clamp of the shared expert
 };
 
 template <typename T>
@@ -645,12 +676,10 @@ __global__ void __launch_bounds__(kThreads) moe_glu_kernel(MoeArgs a) {
     const T* w[2] = {W + (int64_t)g * a.K, W + (int64_t)u * a.K};
     float acc[1][2] = {};
     dot_rows<T, 1, 2>(w, sx, a.kp, a.K, vec, lane, acc);
-    if (lane == 0 && a.act == 4) {
-      reinterpret_cast<T*>(a.out)[(int64_t)slot * a.ldy + i] = DT<T>::from_f(silu(acc[0][0]) * acc[0][1]);
-    } else if (lane == 0) {
-      const float gv = fminf(acc[0][0] * rw, a.limit);
-      const float uv = fminf(fmaxf(acc[0][1] * rw, -a.limit), a.limit);
-      const float y = gv / (1.0f + expf(-a.alpha * gv)) * (uv + 1.0f);
+    if (lane == 0) {
+      const float y = a.act == 4   ? silu(acc[0][0]) * acc[0][1]
+                      : a.act == 5 ? clamped_unit(acc[0][0], acc[0][1], shared ? a.limit_s : a.limit, a.alpha)
+                                   : clamped_unit(acc[0][0] * rw, acc[0][1] * rw, a.limit, a.alpha);
       reinterpret_cast<T*>(a.out)[(int64_t)slot * a.ldy + i] = DT<T>::from_f(y);
     }
   }
@@ -686,8 +715,8 @@ __global__ void __launch_bounds__(kThreads) moe_down_kernel(MoeArgs a) {
       s1 = fmaf(f, acc[0][1], s1);
     }
     float* o = reinterpret_cast<float*>(a.out) + (int64_t)t * a.ldo + n;
-    if (lane == 0) o[0] = a.weighted ? s0 : o[0] + s0;
-    if (lane == 1 && n + 1 < N) o[1] = a.weighted ? s1 : o[1] + s1;
+    if (lane == 0) o[0] = a.add ? o[0] + s0 : s0;
+    if (lane == 1 && n + 1 < N) o[1] = a.add ? o[1] + s1 : s1;
   }
 }
 
@@ -728,15 +757,18 @@ IPEX_API int ipex_gemv_rows_max(int K, int dtype) {
 IPEX_API void ipex_gemv_rows_tune(int mma_from_rows) { g_mma_from = mma_from_rows; }
 
 // y = act(x . W^T + bias): see GemvRowsArgs.  M <= ipex_gemv_rows_max(K, dtype).  w2 / out2 (may be null): N2 more
-// rows with the same row stride whose results go to out2 [M, ldo2] in fp32.  act 3, 4: out_mode 0, N even (a multiple of
-// 16 when interleaved), no second matrix.
+// rows with the same row stride whose results go to out2 [M, ldo2] in fp32.  act 1: rows from act_from on.  act 3 to 5:
+// out_mode 0, N even (a multiple of 16 when interleaved), no second matrix.  act 6: out_mode 0, `mul` [mul_rows, ldm] and the
+// tokens' rows of it, ids [M].  x_f32: x is fp32 and converted (norm_w null).
 IPEX_API int ipex_gemv_rows(const void* w, int64_t ldw, const void* x, int64_t ldx, const void* norm_w, float eps,
                             const void* bias, void* out, int64_t ldo, const void* w2, int N2, float* out2, int64_t ldo2,
-                            int M, int N, int K, int out_mode, int act, int interleaved, float softcap, int dtype,
-                            int pdl, void* stream) {
+                            int M, int N, int K, int out_mode, int act, int interleaved, float softcap, int x_f32,
+                            int act_from, float limit, float alpha, const void* mul, int64_t ldm, int64_t mul_rows,
+                            const int64_t* ids, int dtype, int pdl, void* stream) {
   if (M < 1 || N < 1 || K < 1 || out_mode < 0 || out_mode > 2 || M > ipex_gemv_rows_max(K, dtype))
     return (int)cudaErrorInvalidValue;
-  if (act < 0 || act == 2 || act > 4 || (act >= 3 && (out_mode != 0 || (N % 2) || (interleaved && (N % 16)) || w2 != nullptr)) ||
+  if (act < 0 || act == 2 || act > 6 || (gated(act) && (out_mode != 0 || (N % 2) || (interleaved && (N % 16)) || w2 != nullptr)) ||
+      (act == 6 && (out_mode != 0 || mul == nullptr || ids == nullptr || mul_rows < 1)) || (x_f32 && norm_w != nullptr) ||
       (w2 != nullptr && (N2 < 1 || out2 == nullptr)))
     return (int)cudaErrorInvalidValue;
   return by_dtype(dtype, [&](auto* tag) {
@@ -745,6 +777,14 @@ IPEX_API int ipex_gemv_rows(const void* w, int64_t ldw, const void* x, int64_t l
     a.bias = bias;
     a.N1 = N;
     a.interleaved = interleaved;
+    a.x_f32 = x_f32;
+    a.act_from = act_from;
+    a.limit = limit;
+    a.alpha = alpha;
+    a.mul = mul;
+    a.ids = ids;
+    a.ldm = ldm;
+    a.mul_rows = mul_rows;
     if (w2 != nullptr) {
       a.w2 = w2;
       a.out2 = out2;
@@ -791,20 +831,20 @@ IPEX_API int ipex_moe_router_softmax(const void* h, int64_t ldh, const void* w, 
 
 // First half of the experts for `tokens` rows.  act 2: y[token * k + j] = g * sigmoid(alpha g) * (u + 1), g = min(gate,
 // limit), u = clamp(up, +-limit), gate / up of expert idx[token, j] on weight * norm(x).  act 4: silu(gate) * up of
-// finished rows x (norm_w null).  ws (may be null): the shared expert's rows, [2 Is, K]; tile / tile_s: see MoeArgs.
+// finished rows x (norm_w null); act 5: the clamped unit of them, the shared expert's with limit_s.  ws (may be null): the shared expert's rows, [2 Is, K]; tile / tile_s: see MoeArgs.
 IPEX_API int ipex_moe_glu_rows(const void* x, int64_t ldx, const void* norm_w, float eps, const void* w, const void* ws,
                                void* y, int64_t ldy, const float* weights, const int64_t* idx, int tokens, int K, int I,
-                               int Is, int E, int k, int act, float limit, float alpha, int tile, int tile_s, int dtype,
-                               int pdl, void* stream) {
+                               int Is, int E, int k, int act, float limit, float limit_s, float alpha, int tile, int tile_s,
+                               int dtype, int pdl, void* stream) {
   if (tokens < 1 || K < 1 || I < 1 || k < 1 || (int64_t)tokens * k > 65535 || tile < 0 || (tile > 0 && I % tile != 0) ||
-      Is < 0 || (Is > 0 && (ws == nullptr || act != 4)) || tile_s < 0 || (tile_s > 0 && Is % tile_s != 0) || ldy < I ||
-      ldy < Is || (act != 2 && act != 4) || (act == 2) != (norm_w != nullptr))
+      Is < 0 || (Is > 0 && (ws == nullptr || act == 2)) || tile_s < 0 || (tile_s > 0 && Is % tile_s != 0) || ldy < I ||
+      ldy < Is || (act != 2 && act != 4 && act != 5) || (act == 2) != (norm_w != nullptr))
     return (int)cudaErrorInvalidValue;
   return by_dtype(dtype, [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
     MoeArgs a = {};
     a.x = x; a.norm_w = norm_w; a.w = w; a.out = y; a.weights = weights; a.idx = idx; a.ldx = ldx; a.eps = eps;
-    a.limit = limit; a.alpha = alpha; a.K = K; a.I = I; a.E = E; a.k = k; a.kp = padded<T>(K); a.act = act;
+    a.limit = limit; a.limit_s = limit_s; a.alpha = alpha; a.K = K; a.I = I; a.E = E; a.k = k; a.kp = padded<T>(K); a.act = act;
     a.ws = ws; a.Is = Is; a.ldy = ldy; a.tile = tile; a.tile_s = tile_s;
     a.vec = vec_ok<T>(w, K, K);
     a.vec_s = ws != nullptr && vec_ok<T>(ws, K, K);
@@ -818,11 +858,11 @@ IPEX_API int ipex_moe_glu_rows(const void* x, int64_t ldx, const void* norm_w, f
   });
 }
 
-// Second half: out[token] += sum_j down_{idx[token, j]}(y[token * k + j]); with weights: out[token] = the weighted sum.
+// Second half: sum_j down_{idx[token, j]}(y[token * k + j]), weighted unless weights is null, added to out or (add 0) written.
 // ws (may be null): the shared expert's rows, [N, Is]; it is then the last of the k choices.
 IPEX_API int ipex_moe_down_rows(const void* y, int64_t ldy, const void* w, const void* ws, const float* weights, float* out,
-                                int64_t ldo, const int64_t* idx, int tokens, int N, int I, int Is, int E, int k, int dtype,
-                                int pdl, void* stream) {
+                                int64_t ldo, const int64_t* idx, int tokens, int N, int I, int Is, int E, int k, int add,
+                                int dtype, int pdl, void* stream) {
   if (tokens < 1 || tokens > 65535 || N < 1 || I < 1 || k < 1 || Is < 0 || (Is > 0 && (ws == nullptr || k < 2)) ||
       ldy < I || ldy < Is)
     return (int)cudaErrorInvalidValue;
@@ -831,7 +871,7 @@ IPEX_API int ipex_moe_down_rows(const void* y, int64_t ldy, const void* w, const
     MoeArgs a = {};
     a.y_in = y; a.w = w; a.out = out; a.idx = idx; a.ldo = ldo; a.K = N; a.I = I; a.E = E; a.k = k;
     a.kp = padded<T>(I > Is ? I : Is);
-    a.weights = weights; a.weighted = weights != nullptr; a.ws = ws; a.Is = Is; a.ldy = ldy;
+    a.weights = weights; a.weighted = weights != nullptr; a.add = add; a.ws = ws; a.Is = Is; a.ldy = ldy;
     a.vec = vec_ok<T>(w, I, I);
     a.vec_s = ws != nullptr && vec_ok<T>(ws, Is, Is);
     const size_t smem = (size_t)a.kp * k * sizeof(T);

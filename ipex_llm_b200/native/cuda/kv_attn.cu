@@ -1,10 +1,12 @@
-// Attention over cached keys and values of different sizes, sm_100a: everything earlier, a sliding window or the query's
-// own chunk of positions, with an optional sink (a score of 0 or one learned number per head), mixed values, rotated and
-// unit-normed queries and keys, and gated outputs.
+// Attention over cached keys and values of different sizes, sm_100a: everything earlier, a sliding window - alone or beside
+// pooled blocks of what has left it - or the query's own chunk of positions, with an optional sink (a score of 0 or one
+// learned number per head), mixed values, rotated and (unit- or weighted-) normed queries and keys, and gated outputs.
 //
-//   qk_prepare  rotation and unit norm of the query and key heads of many tokens in place (prompts, portions)
+//   qk_prepare  norm and rotation of the query and key heads of many tokens in place (prompts, portions)
 //   kv_append   keys and values of the new tokens into the cache, the values mixed with those of an earlier layer;
 //               for prompts also the transposed values that the tcgen05 prompt attention reads
+//   kv_pool     means of the keys and values of the blocks of tokens that a portion completes, into the cache's rows of
+//               blocks and, for prompts, where the prompt attention reads them
 //   kv_attn     attention of query tokens against what their slots hold: decoding (which prepares and appends its own
 //               row on the way), portions of prompts, and whole prompts of sizes or formats the tensor-core kernel does not take
 //
@@ -58,12 +60,16 @@ struct Prepare {
   int half;             // pairs (i, i + half) of a head turn
   int unit;             // divide by the root mean square
   float eps;
+  const float* wq;      // [dim] weight of the queries' norm, or null
+  const float* wk;      // ... and of the keys'
+  int q_heads;          // heads of x that are queries (qk_prepare)
 };
 
-// One vector by one warp; load(i) / store(i, value) for its elements.  The norm does not change under the rotation, so
-// it is taken first and every lane finishes its own pairs.
+// One vector by one warp; load(i) / store(i, value) for its elements.  The norm comes before the rotation, which does not
+// change it; every lane finishes its own pairs.  w: weight of the norm, or null.
 template <typename L, typename S>
-__device__ __forceinline__ void prepare_vector(const Prepare& p, int dim, int rel, float scale, int lane, L&& load, S&& store) {
+__device__ __forceinline__ void prepare_vector(const Prepare& p, int dim, int rel, float scale, int lane, const float* w,
+                                               L&& load, S&& store) {
   float f = scale;
   if (p.unit) {
     float ss = 0.f;
@@ -75,12 +81,13 @@ __device__ __forceinline__ void prepare_vector(const Prepare& p, int dim, int re
   }
   const float* cp = p.cosp + (int64_t)rel * p.half;
   const float* sp = p.sinp + (int64_t)rel * p.half;
+  auto at = [&](int i) { return w != nullptr ? load(i) * w[i] : load(i); };
   for (int i = lane; i < p.half; i += 32) {
-    const float u = load(i), v = load(i + p.half), c = cp[i], s = sp[i];
+    const float u = at(i), v = at(i + p.half), c = cp[i], s = sp[i];
     store(i, (u * c - v * s) * f);
     store(i + p.half, (v * c + u * s) * f);
   }
-  for (int i = 2 * p.half + lane; i < dim; i += 32) store(i, load(i) * f);
+  for (int i = 2 * p.half + lane; i < dim; i += 32) store(i, at(i) * f);
 }
 
 // A warp per (token, head) of x: rows of `ld`, heads behind one another.
@@ -94,7 +101,8 @@ __global__ void __launch_bounds__(kThreads) qk_prepare_kernel(T* __restrict__ x,
   if (r >= rows) return;
   const int t = (int)(r / heads), h = (int)(r % heads);
   T* v = x + (int64_t)t * ld + (int64_t)h * dim;
-  prepare_vector(p, dim, pos[t] - start[slot[t]], 1.0f, threadIdx.x & 31, [&](int i) { return DT<T>::to_f(v[i]); },
+  prepare_vector(p, dim, pos[t] - start[slot[t]], 1.0f, threadIdx.x & 31, h < p.q_heads ? p.wq : p.wk,
+                 [&](int i) { return DT<T>::to_f(v[i]); },
                  [&](int i, float y) { v[i] = DT<T>::from_f(y); });
 }
 
@@ -111,12 +119,14 @@ __global__ void __launch_bounds__(kThreads) qk_prepare_vec_kernel(T* __restrict_
   const int lane = threadIdx.x % LG, hp = p.half / N;
   const bool mine = lane * N < dim, first = lane < hp, turns = lane < 2 * hp;
   T* v[kHeads];
+  const float* wt[kHeads];
   float a[kHeads][N];
   int64_t at[kHeads];
 #pragma unroll
   for (int u = 0; u < kHeads; ++u) {
     const uint32_t r = r0 + u, t = r < rows ? r / heads : 0, h = r < rows ? r - t * heads : 0;
     v[u] = x + (int64_t)t * ld + (int64_t)h * dim + lane * N;
+    wt[u] = h < (uint32_t)p.q_heads ? p.wq : p.wk;
     at[u] = (int64_t)(pos[t] - start[slot[t]]) * p.half + (first ? lane : lane - hp) * N;
 #pragma unroll
     for (int j = 0; j < N; ++j) a[u][j] = 0.f;
@@ -132,6 +142,10 @@ __global__ void __launch_bounds__(kThreads) qk_prepare_vec_kernel(T* __restrict_
 #pragma unroll
       for (int o = LG / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
       f = 1.0f / sqrtf(ss / (float)dim + p.eps);
+    }
+    if (wt[u] != nullptr && mine) {
+#pragma unroll
+      for (int j = 0; j < N; ++j) a[u][j] *= wt[u][lane * N + j];
     }
     float b[N];
     const int partner = !turns ? lane : first ? lane + hp : lane - hp;
@@ -256,6 +270,58 @@ __global__ void __launch_bounds__(kThreads) kv_append_kernel(AppendArgs a) {
   }
 }
 
+// ---------------------------------------------------------------------------------------------- pooled blocks
+struct PoolArgs {
+  const void* kc;       // cache rows: slot * k_slot + head * k_head + position * dim
+  const void* vc;
+  void* pk;             // rows of blocks: slot * pk_slot + head * pk_head + block * dim
+  void* pv;
+  void* kp;             // prompts: T [rows, ld_kp], head h at h * dim, rows from pool_row[portion] on; or null
+  void* vt;             // ... and T [heads * vdim, ld_vt]
+  const int* slot;      // [tokens]
+  const int* pos;       // [tokens]
+  const int* start;     // [slots]
+  const int* seq_row;   // [portions]
+  const int* seq_len;   // [portions]
+  const int* pool_row;  // [portions], or null
+  int64_t k_slot, k_head, v_slot, v_head, pk_slot, pk_head, pv_slot, pv_head, ld_kp, ld_vt;
+  int pool, dim, vdim;
+};
+
+// Mean of a block's rows, in order; what the attention of a decoded token computes for the block it completes.
+template <typename T>
+__device__ __forceinline__ T block_mean(const T* rows, int dim, int pool) {
+  float s = 0.f;
+#pragma unroll 4
+  for (int j = 0; j < pool; ++j) s += DT<T>::to_f(rows[(int64_t)j * dim]);
+  return DT<T>::from_f(s / (float)pool);
+}
+
+// A warp per (block, head, portion).
+template <typename T>
+__global__ void __launch_bounds__(kThreads) kv_pool_kernel(PoolArgs a) {
+  const int seq = blockIdx.z, g = blockIdx.y, lane = threadIdx.x & 31;
+  const int row0 = a.seq_row[seq], len = a.seq_len[seq], slot = a.slot[row0], start = a.start[slot];
+  const int p0 = a.pos[row0] - start, b = p0 / a.pool + blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
+  if ((int64_t)(b + 1) * a.pool > p0 + len) return;
+  const int64_t first = start + (int64_t)b * a.pool;
+  const T* k = reinterpret_cast<const T*>(a.kc) + slot * a.k_slot + g * a.k_head + first * a.dim;
+  const T* v = reinterpret_cast<const T*>(a.vc) + slot * a.v_slot + g * a.v_head + first * a.vdim;
+  T* pk = reinterpret_cast<T*>(a.pk) + slot * a.pk_slot + g * a.pk_head + (int64_t)b * a.dim;
+  T* pv = reinterpret_cast<T*>(a.pv) + slot * a.pv_slot + g * a.pv_head + (int64_t)b * a.vdim;
+  const int64_t row = a.pool_row != nullptr ? a.pool_row[seq] + b : 0;
+  for (int i = lane; i < a.dim; i += 32) {
+    const T m = block_mean(k + i, a.dim, a.pool);
+    pk[i] = m;
+    if (a.kp != nullptr) reinterpret_cast<T*>(a.kp)[row * a.ld_kp + (int64_t)g * a.dim + i] = m;
+  }
+  for (int i = lane; i < a.vdim; i += 32) {
+    const T m = block_mean(v + i, a.vdim, a.pool);
+    pv[i] = m;
+    if (a.vt != nullptr) reinterpret_cast<T*>(a.vt)[((int64_t)g * a.vdim + i) * a.ld_vt + row] = m;
+  }
+}
+
 // ---------------------------------------------------------------------------------------------- attention
 struct AttnArgs {
   const void* q;        // T [tokens, ldq], head h at h * dim
@@ -278,6 +344,10 @@ struct AttnArgs {
   float gate_scale;
   Prepare prep;
   int prepare;          // with append: queries and the new key are rotated / normed here
+  int pool;             // > 0: beside the window, the blocks of this many tokens that lie wholly before it
+  void* pk;             // rows of blocks: slot * pk_slot + head * pk_head + block * dim
+  void* pv;
+  int64_t pk_slot, pk_head, pv_slot, pv_head;
 };
 
 template <typename T, int RT, bool VEC>
@@ -301,12 +371,17 @@ __global__ void __launch_bounds__(kThreads) kv_attn_kernel(AttnArgs a, int nrb) 
   const int slot = a.slot[tok], pos = a.pos[tok], start = a.start[slot];
   int lo = max(start, a.window > 0 ? pos - a.window + 1 : 0);
   if (a.chunk > 0) lo = max(lo, pos - (pos - start) % a.chunk);
-  const int n = pos + 1 - lo;
+  // keys 0 .. nb are blocks, the others tokens from position lo on
+  const int nb = a.pool > 0 ? max(0, pos - start - a.window + 1) / a.pool : 0;
+  const int n = nb + pos + 1 - lo;
   const int chunk = (n + nsplit - 1) / nsplit;
-  const int j0 = lo + min(n, split * chunk), j1 = lo + min(n, (split + 1) * chunk);
+  const int j0 = min(n, split * chunk), j1 = min(n, (split + 1) * chunk);
   T* kc = reinterpret_cast<T*>(a.kc) + (int64_t)slot * a.k_slot + (int64_t)g * a.k_head;
   T* vc = reinterpret_cast<T*>(a.vc) + (int64_t)slot * a.v_slot + (int64_t)g * a.v_head;
-  if (a.append && j1 == pos + 1 && j0 < j1) {
+  T* pk = reinterpret_cast<T*>(a.pk) + (int64_t)slot * a.pk_slot + (int64_t)g * a.pk_head;
+  T* pv = reinterpret_cast<T*>(a.pv) + (int64_t)slot * a.pv_slot + (int64_t)g * a.pv_head;
+  const bool newest = a.append && j1 == n && j0 < j1;
+  if (newest) {
     // this CTA owns the newest key: it files the row and reads it back like the others (every row block of the head
     // does, with the same values)
     const T* k = reinterpret_cast<const T*>(a.k) + (int64_t)tok * a.ldq + (int64_t)g * a.dim;
@@ -318,7 +393,7 @@ __global__ void __launch_bounds__(kThreads) kv_attn_kernel(AttnArgs a, int nrb) 
         for (int i = lane; i < a.dim; i += 32) sk[i] = DT<T>::to_f(k[i]);
         __syncwarp();
         T* dst = kc + (int64_t)pos * a.dim;
-        prepare_vector(a.prep, a.dim, pos - start, 1.0f, lane, [&](int i) { return sk[i]; },
+        prepare_vector(a.prep, a.dim, pos - start, 1.0f, lane, a.prep.wk, [&](int i) { return sk[i]; },
                        [&](int i, float y) { dst[i] = DT<T>::from_f(y); });
       }
     } else {
@@ -338,7 +413,7 @@ __global__ void __launch_bounds__(kThreads) kv_attn_kernel(AttnArgs a, int nrb) 
         for (int i = lane; i < a.dim; i += 32) dst[i] = warp < rows ? DT<T>::to_f(q[(int64_t)warp * a.dim + i]) : 0.f;
         __syncwarp();
         if (warp < rows)
-          prepare_vector(a.prep, a.dim, pos - start, a.scale, lane, [&](int i) { return dst[i]; },
+          prepare_vector(a.prep, a.dim, pos - start, a.scale, lane, a.prep.wq, [&](int i) { return dst[i]; },
                          [&](int i, float y) { dst[i] = y; });
       }
     } else {
@@ -349,6 +424,14 @@ __global__ void __launch_bounds__(kThreads) kv_attn_kernel(AttnArgs a, int nrb) 
     }
   }
   __syncthreads();
+  if (newest && a.pool > 0 && (pos - start + 1) % a.pool == 0) {
+    // the new token completes a block, which nobody sees yet
+    const int b = (pos - start) / a.pool, first = start + b * a.pool;
+    for (int i = tid; i < a.dim; i += kThreads)
+      pk[(int64_t)b * a.dim + i] = block_mean(kc + (int64_t)first * a.dim + i, a.dim, a.pool);
+    for (int i = tid; i < a.vdim; i += kThreads)
+      pv[(int64_t)b * a.vdim + i] = block_mean(vc + (int64_t)first * a.vdim + i, a.vdim, a.pool);
+  }
 
   const int nvk = a.dim / VN, nvv = a.vdim / VN;
   const int subsets = kThreads / nvv, vv = tid % nvv, sub = tid / nvv;
@@ -370,7 +453,10 @@ __global__ void __launch_bounds__(kThreads) kv_attn_kernel(AttnArgs a, int nrb) 
       for (int i = 0; i < 4 * RT; ++i) s[i] = 0.f;
       const T* kp[4];
 #pragma unroll
-      for (int u = 0; u < 4; ++u) kp[u] = kc + (int64_t)(t0 + min(tn - 1, warp * 16 + u * 4 + kg)) * a.dim;
+      for (int u = 0; u < 4; ++u) {
+        const int j = t0 + min(tn - 1, warp * 16 + u * 4 + kg);
+        kp[u] = j < nb ? pk + (int64_t)j * a.dim : kc + (int64_t)(lo + j - nb) * a.dim;
+      }
       for (int c = ks; c < nvk; c += 8) {
         float kf[4][VN];
 #pragma unroll
@@ -447,11 +533,13 @@ __global__ void __launch_bounds__(kThreads) kv_attn_kernel(AttnArgs a, int nrb) 
 #pragma unroll
         for (int i = 0; i < VN; ++i) acc[r][i] *= c;
       }
-      const T* vp = vc + (int64_t)t0 * a.vdim + vv * VN;
+      const T* vp = vc + ((int64_t)lo + t0 - nb) * a.vdim + vv * VN;
+      const T* vb = pv + (int64_t)t0 * a.vdim + vv * VN;
+      const int blocks = nb - t0;                // of this tile's keys
 #pragma unroll 4
       for (int j = sub; j < tn; j += subsets) {
         float vf[VN];
-        load_pack<T, VEC>(vp + (int64_t)j * a.vdim, vf);
+        load_pack<T, VEC>((j < blocks ? vb : vp) + (int64_t)j * a.vdim, vf);
 #pragma unroll
         for (int r = 0; r < RT; ++r) {
           const float p = ss[r * kTile + j];
@@ -581,18 +669,40 @@ IPEX_API int ipex_kv_append(const void* k, const void* v, int64_t ld, const void
   });
 }
 
+// Means of the blocks of `pool` tokens (counted from the sequence's start) that the portions complete, from the cache's rows
+// into its rows of blocks; kp / vt with pool_row (all null, or whole prompts): also [rows, ld_kp], [heads * vdim, ld_vt] from
+// row pool_row[portion] on.  longest: tokens of the longest portion.
+IPEX_API int ipex_kv_pool(const void* kc, int64_t k_slot, int64_t k_head, const void* vc, int64_t v_slot, int64_t v_head,
+                          void* pk, int64_t pk_slot, int64_t pk_head, void* pv, int64_t pv_slot, int64_t pv_head, void* kp,
+                          int64_t ld_kp, void* vt, int64_t ld_vt, const int* pool_row, const int* slot, const int* pos,
+                          const int* start, const int* seq_row, const int* seq_len, int seqs, int longest, int kv_heads,
+                          int dim, int vdim, int pool, int dtype, void* stream) {
+  if (seqs < 1 || seqs > 65535 || longest < 1 || kv_heads < 1 || kv_heads > 65535 || dim < 1 || vdim < 1 || pool < 1 ||
+      (kp == nullptr) != (vt == nullptr) || (kp == nullptr) != (pool_row == nullptr))
+    return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    const PoolArgs a = {kc, vc, pk, pv, kp, vt, slot, pos, start, seq_row, seq_len, pool_row, k_slot, k_head, v_slot, v_head,
+                        pk_slot, pk_head, pv_slot, pv_head, ld_kp, ld_vt, pool, dim, vdim};
+    const int blocks = longest / pool + 1;           // that a portion can complete
+    kv_pool_kernel<T><<<dim3((blocks + kThreads / 32 - 1) / (kThreads / 32), kv_heads, seqs), kThreads, 0, (cudaStream_t)stream>>>(a);
+    return cudaGetLastError();
+  });
+}
+
 // Queries and keys of many tokens in place, x [tokens, ld] with `heads` of `dim`: pairs (i, i + half) turn by the tables'
-// angles for the token's place in its sequence; unit: divided by sqrt(mean square + eps).
+// angles for the token's place in its sequence; before that, unit: divided by sqrt(mean square + eps), and times wq (the
+// first q_heads heads) or wk (the others), [dim] each, unless null.
 IPEX_API int ipex_qk_prepare(void* x, int64_t ld, const int* slot, const int* pos, const int* start, const float* cosp,
-                             const float* sinp, int half, int unit, float eps, int tokens, int heads, int dim, int dtype,
-                             int pdl, void* stream) {
+                             const float* sinp, int half, int unit, float eps, const float* wq, const float* wk, int q_heads,
+                             int tokens, int heads, int dim, int dtype, int pdl, void* stream) {
   if (tokens < 1 || heads < 1 || dim < 1 || half < 0 || 2 * half > dim || (half > 0 && (cosp == nullptr || sinp == nullptr)))
     return (int)cudaErrorInvalidValue;
   const int64_t rows = (int64_t)tokens * heads, blocks = (rows + kThreads / 32 - 1) / (kThreads / 32);
   if (blocks > 0x7fffffff) return (int)cudaErrorInvalidValue;
   return by_dtype(dtype, [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
-    const Prepare p = {cosp, sinp, half, unit, eps};
+    const Prepare p = {cosp, sinp, half, unit, eps, wq, wk, q_heads};
     constexpr int VN = 16 / (int)sizeof(T);
     if (rows < (1u << 31) && dim % VN == 0 && dim / VN <= 32 && half % VN == 0 && ld % VN == 0 &&
         (((uintptr_t)x | (uintptr_t)cosp | (uintptr_t)sinp) & 15) == 0) {
@@ -610,18 +720,21 @@ IPEX_API int ipex_qk_prepare(void* x, int64_t ld, const int* slot, const int* po
 // [max(start, pos - window + 1), pos] of their slots (window 0: unlimited; chunk > 0: those of the query's own chunk, counted
 // from start).  append: file the tokens' own rows k / v (same row stride as q, v mixed with vfirst) first - then no two
 // tokens may share a slot; otherwise the cache holds them.  prepare (with append): queries and new keys are rotated and
-// normed on the way (see ipex_qk_prepare).  nsplit: CTAs (1, 2, 4 or 8) the keys of a token are shared by.  sink: one more
+// normed on the way (see ipex_qk_prepare).  pool > 0 (with a window): beside it, the blocks of `pool` tokens that lie wholly
+// before it, from pk / pv; append files the block that a token completes.  nsplit: CTAs (1, 2, 4 or 8) the keys of a token are shared by.  sink: one more
 // score without a value in every softmax, 0 or sinks[head].  gate (may be null): outputs times gate_scale * sigmoid.
 IPEX_API int ipex_kv_attn(const void* q, const void* k, const void* v, int64_t ldq, const void* vfirst, int64_t ld_vf,
                           float lambda, void* kc, int64_t k_slot, int64_t k_head, void* vc, int64_t v_slot,
                           int64_t v_head, void* out, int64_t ldo, const int* slot, const int* pos, const int* start,
                           int tokens, int heads, int kv_heads, int dim, int vdim, int window, int chunk, int sink,
                           const float* sinks, const void* gate, int64_t ldg, float gate_scale, int append, int prepare,
-                          const float* cosp, const float* sinp, int half, int unit, float eps, int nsplit, float scale,
-                          int dtype, int pdl, void* stream) {
+                          const float* cosp, const float* sinp, int half, int unit, float eps, const float* wq,
+                          const float* wk, int pool, void* pk, int64_t pk_slot, int64_t pk_head, void* pv, int64_t pv_slot,
+                          int64_t pv_head, int nsplit, float scale, int dtype, int pdl, void* stream) {
   if (tokens < 1 || tokens > 65535 || kv_heads < 1 || heads % kv_heads != 0 || dim < 1 || vdim < 1 || window < 0 || chunk < 0 ||
       nsplit < 1 || nsplit > 8 || (nsplit & (nsplit - 1)))
     return (int)cudaErrorInvalidValue;
+  if (pool < 0 || (pool > 0 && (window < 1 || chunk > 0 || pk == nullptr || pv == nullptr))) return (int)cudaErrorInvalidValue;
   if (prepare && (!append || half < 0 || 2 * half > dim || (half > 0 && (cosp == nullptr || sinp == nullptr))))
     return (int)cudaErrorInvalidValue;
   return by_dtype(dtype, [&](auto* tag) {
@@ -629,8 +742,9 @@ IPEX_API int ipex_kv_attn(const void* q, const void* k, const void* v, int64_t l
     constexpr int VN = 16 / (int)sizeof(T);
     AttnArgs a = {q, k, v, vfirst, kc, vc, out, slot, pos, start, ldq, ld_vf, ldo, k_slot, k_head, v_slot, v_head,
                   lambda, scale, heads, kv_heads, dim, vdim, window, sink, append, chunk, sinks, gate, ldg, gate_scale,
-                  {cosp, sinp, half, unit, eps}, prepare};
-    const bool vec = dim % VN == 0 && vdim % VN == 0 && vdim / VN <= kThreads && (((uintptr_t)kc | (uintptr_t)vc) & 15) == 0;
+                  {cosp, sinp, half, unit, eps, wq, wk, heads}, prepare, pool, pk, pv, pk_slot, pk_head, pv_slot, pv_head};
+    const bool vec = dim % VN == 0 && vdim % VN == 0 && vdim / VN <= kThreads &&
+                     (((uintptr_t)kc | (uintptr_t)vc | (uintptr_t)pk | (uintptr_t)pv) & 15) == 0;
     cudaStream_t st = (cudaStream_t)stream;
     if (vec) return pick_rows<T, true>(a, tokens, nsplit, pdl != 0, st);
     if (vdim > kThreads) return cudaErrorInvalidValue;

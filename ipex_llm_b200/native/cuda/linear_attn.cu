@@ -20,6 +20,7 @@
 // What lies before a sequence's first token counts as zero, so a slot needs no clearing when it changes hands.
 #include <cooperative_groups.h>
 
+#include "common/state_cols.cuh"
 #include "common/tf32_pairs.cuh"
 #include "common/utils.cuh"
 #include "tcgen05_common.cuh"
@@ -74,25 +75,6 @@ struct StepArgs {
   int prefetch;           // slots are final before the kernels in front of this one end: fetch states early
   int staged;             // the head's rows of `up` fit shared memory
 };
-
-template <int N>
-__device__ __forceinline__ void load_cols(const float* p, float (&v)[N]) {
-  if constexpr (N == 4) {
-    const float4 x = *reinterpret_cast<const float4*>(p);
-    v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
-  } else if constexpr (N == 2) {
-    const float2 x = *reinterpret_cast<const float2*>(p);
-    v[0] = x.x; v[1] = x.y;
-  } else {
-    v[0] = *p;
-  }
-}
-template <int N>
-__device__ __forceinline__ void store_cols(float* p, const float (&v)[N]) {
-  if constexpr (N == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
-  else if constexpr (N == 2) *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]);
-  else *p = v[0];
-}
 
 // A warp owns the state rows warp, warp + 8, ...; a lane CV neighbouring columns of the CTA's 32 CV.
 template <typename T, int NR, int CV>

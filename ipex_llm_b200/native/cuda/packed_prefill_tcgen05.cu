@@ -1,6 +1,6 @@
 // Prompt attention over packed sequences on the 5th-generation tensor cores, sm_100a: multi-head latent attention, and
-// attention with plain key / value heads (shared by groups of query heads), over everything earlier, a window or the
-// query's own chunk, with or without a sink and an output gate.
+// attention with plain key / value heads (shared by groups of query heads), over everything earlier, a window (alone or
+// beside pooled blocks of the tokens before it) or the query's own chunk, with or without a sink and an output gate.
 //
 // Keys and values are expanded from the latents by two GEMMs before this kernel; a head's key is then made of two
 // parts that live in different tensors: `dim` values of its own and `rd` rotated values shared by all heads.  Neither
@@ -13,7 +13,8 @@
 // V^T is produced directly by a GEMM with W_uv as its row operand.  Sequences of different lengths are packed one
 // behind the other (no padding rows); a CTA owns 128 queries of one head of one sequence and walks the key tiles
 // inside the causal sliding window.  A V^T tile must start at a multiple of 8 tokens (16-byte TMA rule), so tiles are
-// laid out from the sequence's first row rounded down to 8 and the surplus keys are masked.
+// laid out from the sequence's first row rounded down to 8 and the surplus keys are masked.  Pooled blocks are keys and
+// values of their own tensors, in rows that start at multiples of 8; their tiles come first.
 //
 //   warp 8: TMA loads (separate rings for K and V^T)   warp 9: MMA issue, S(j+1) goes out before P(j) is waited for
 //   warps 0-7: two threads per query row: maximum, exp2, sum, P to shared memory, running output in registers
@@ -61,13 +62,16 @@ struct Args {
   const void* gate;       // T [tokens, ldg], head h at h * vd, or null: outputs times gate_scale * sigmoid(gate)
   int64_t ldg;
   float gate_scale;
+  int pool;               // > 0: beside the window, the blocks of this many tokens that lie wholly before it
+  const int* pool_row;    // [B] first row of every sequence's blocks, a multiple of 8
 };
 
 template <typename T, int DV>
 __global__ void __launch_bounds__(kThreads, 1)
 packed_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_constant__ CUtensorMap tm_qr,
                       const __grid_constant__ CUtensorMap tm_kn, const __grid_constant__ CUtensorMap tm_kr,
-                      const __grid_constant__ CUtensorMap tm_vt, Args a) {
+                      const __grid_constant__ CUtensorMap tm_vt, const __grid_constant__ CUtensorMap tm_kp,
+                      const __grid_constant__ CUtensorMap tm_vp, Args a) {
   constexpr int kVBytes = DV * kBKV * 2;
   constexpr uint32_t kTmemCols = 512;
   const int h = blockIdx.x, b = blockIdx.z, hk = h / a.group;
@@ -104,7 +108,10 @@ packed_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
   int j0 = 0;
   if (a.window > 0) j0 = max(0, qb * kBQ - a.window + 1 + koff) / kBKV;
   if (a.chunk > 0) j0 = max(j0, (qb * kBQ / a.chunk * a.chunk + koff) / kBKV);
-  const int nblk = nkv - j0;
+  // tiles of pooled blocks that some row sees, then those of tokens
+  const int npt = a.pool > 0 ? (max(0, qmax - a.window + 1) / a.pool + kBKV - 1) / kBKV : 0;
+  const int prow = a.pool > 0 ? a.pool_row[b] : 0;
+  const int nblk = npt + nkv - j0;
 
   if (threadIdx.x == 0) {
     mbar_init(q_full, 1);
@@ -139,11 +146,14 @@ packed_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
       int ks = 0, vs = 0;
       uint32_t kp = 0, vp = 0;
       for (int jj = 0; jj < nblk && ok; ++jj) {
-        const int krow = base + (j0 + jj) * kBKV;
+        const bool pooled = jj < npt;
+        const CUtensorMap* tk = pooled ? &tm_kp : &tm_kn;
+        const CUtensorMap* tv = pooled ? &tm_vp : &tm_vt;
+        const int krow = pooled ? prow + jj * kBKV : base + (j0 + jj - npt) * kBKV;
         if (!mbar_wait(&k_empty[ks], kp ^ 1, abort_flag)) { ok = false; report(a.err, 34); break; }
         uint8_t* dk = sK + ks * nb * kBlkBytes;
         mbar_expect_tx(&k_full[ks], nb * kBlkBytes);
-        for (int i = 0; i < a.nbn; ++i) tma_load_3d(dk + i * kBlkBytes, &tm_kn, i * 64, hk, krow, &k_full[ks]);
+        for (int i = 0; i < a.nbn; ++i) tma_load_3d(dk + i * kBlkBytes, tk, i * 64, hk, krow, &k_full[ks]);
         for (int i = 0; i < a.nbr; ++i) tma_load_2d(dk + (a.nbn + i) * kBlkBytes, &tm_kr, i * 64, krow, &k_full[ks]);
         if (++ks == a.kst) { ks = 0; kp ^= 1; }
         if (!mbar_wait(&v_empty[vs], vp ^ 1, abort_flag)) { ok = false; report(a.err, 34); break; }
@@ -151,7 +161,7 @@ packed_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
         mbar_expect_tx(&v_full[vs], kVBytes);
 #pragma unroll
         for (int i = 0; i < kBKV / 64; ++i)
-          tma_load_2d(dv + i * (DV * 128), &tm_vt, krow + i * 64, hk * a.vd, &v_full[vs]);
+          tma_load_2d(dv + i * (DV * 128), tv, krow + i * 64, hk * a.vd, &v_full[vs]);
         if (++vs == a.vst) { vs = 0; vp ^= 1; }
       }
       if (!ok) {
@@ -225,12 +235,15 @@ packed_prefill_kernel(const __grid_constant__ CUtensorMap tm_qn, const __grid_co
     bool ok = true;
     int first = a.window > 0 ? max(0, qpos - a.window + 1) : 0;
     if (a.chunk > 0) first = max(first, qpos / a.chunk * a.chunk);
+    const int seen = a.pool > 0 ? max(0, qpos - a.window + 1) / a.pool : 0;      // blocks that this row sees
     for (int jj = 0; jj < nblk; ++jj) {
       const uint32_t jp = jj & 1;
       if (!mbar_wait(&s_full[jj & 1], (jj >> 1) & 1, abort_flag)) { ok = false; break; }
       tcgen05_fence_after();
-      const int k0 = (j0 + jj) * kBKV - koff + hf * 64;      // key of this thread's first column
-      const int lim = qpos + 1 - k0, lo = first - k0;        // visible columns [lo, lim)
+      const bool pooled = jj < npt;
+      // key of this thread's first column, visible columns [lo, lim)
+      const int k0 = pooled ? jj * kBKV + hf * 64 : (j0 + jj - npt) * kBKV - koff + hf * 64;
+      const int lim = (pooled ? seen : qpos + 1) - k0, lo = pooled ? 0 : first - k0;
       uint32_t v0[32], v1[32];
       const uint32_t sb = tmem_base + lane_addr + (jj & 1) * kBKV + hf * 64;
       tmem_ld_32x32(sb, v0);
@@ -363,7 +376,8 @@ size_t smem_need(int nb, int dv, int kst, int vst) {
 
 template <typename T, int DV>
 int launch(const void* q, int64_t ldq, const void* k, int64_t ldk, const void* kr, int64_t ld_kr, const void* vt,
-           int64_t ld_vt, Args& a, int B, int H, int tokens, int max_len, cudaStream_t stream) {
+           int64_t ld_vt, const void* kp, int64_t ld_kp, const void* vp, int64_t ld_vp, int pool_rows, Args& a, int B, int H,
+           int tokens, int max_len, cudaStream_t stream) {
   const CUtensorMapDataType dt =
       std::is_same<T, __half>::value ? CU_TENSOR_MAP_DATA_TYPE_FLOAT16 : CU_TENSOR_MAP_DATA_TYPE_BFLOAT16;
   const int nb = a.nbn + a.nbr;
@@ -372,7 +386,7 @@ int launch(const void* q, int64_t ldq, const void* k, int64_t ldk, const void* k
   if (smem_need(nb, DV, 2, a.vst) > kSmemMax) a.kst = 1;
   const size_t smem = smem_need(nb, DV, a.kst, a.vst);
   if (smem > kSmemMax) return (int)cudaErrorInvalidValue;
-  CUtensorMap qn, qr, kn, krm, vm;
+  CUtensorMap qn, qr, kn, krm, vm, kpm, vpm;
   const T* qp = reinterpret_cast<const T*>(q);
   const int G = H / a.group;
   if (!encode_heads(&qn, dt, qp, a.dim, H, tokens, a.dim + a.rd, ldq) ||
@@ -384,11 +398,16 @@ int launch(const void* q, int64_t ldq, const void* k, int64_t ldk, const void* k
   if (a.nbr > 0 && (!encode_heads(&qr, dt, qp + a.dim, a.rd, H, tokens, a.dim + a.rd, ldq) ||
                     !encode_2d_sw128(&krm, dt, kr, (uint64_t)a.rd, (uint64_t)tokens, (uint64_t)ld_kr * 2, 64, kBKV)))
     return -1;
+  kpm = kn;
+  vpm = vm;
+  if (a.pool > 0 && (!encode_heads(&kpm, dt, kp, a.dim, G, pool_rows, a.dim, ld_kp) ||
+                     !encode_2d_sw128(&vpm, dt, vp, (uint64_t)pool_rows, (uint64_t)G * a.vd, (uint64_t)ld_vp * 2, 64, DV)))
+    return -1;
   auto kern = packed_prefill_kernel<T, DV>;
   cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return (int)e;
   dim3 grid(H, (max_len + kBQ - 1) / kBQ, B);
-  kern<<<grid, kThreads, smem, stream>>>(qn, qr, kn, krm, vm, a);
+  kern<<<grid, kThreads, smem, stream>>>(qn, qr, kn, krm, vm, kpm, vpm, a);
   return (int)cudaGetLastError();
 }
 
@@ -406,14 +425,18 @@ IPEX_API int ipex_packed_prefill_ok(int dim, int rd, int vd, int R, int dtype) {
 // the G key heads of `dim`, kr [tokens, ld_kr] the rotated part shared by all heads (rd = 0: none), vt [G * vd, ld_vt]
 // the values transposed.  Query head h uses key / value head h / (H / G).  seq_row / seq_len: device, [B]; max_len: the
 // largest length.  window 0: unlimited.  chunk > 0: keys of the query's own chunk only.  sink: every softmax has one more
-// score, 0 or sinks[head], whose value is nothing.  gate (may be null): [tokens, ldg], outputs times gate_scale *
+// score, 0 or sinks[head], whose value is nothing.  pool > 0 (with a window, rd = 0): beside the window the blocks of `pool`
+// tokens that lie wholly before it, keys kp [pool_rows, ld_kp] and transposed values vp [G * vd, ld_vp] in rows from
+// pool_row[sequence] (device, multiples of 8) on; rows that are no block must hold finite numbers.  gate (may be null): [tokens, ldg], outputs times gate_scale *
 // sigmoid(gate).  Strides multiples of 8 elements, bases 16-byte aligned.  Returns a cudaError_t, or -1 when the tensor-map encoder rejects
 // the operands.
 IPEX_API int ipex_packed_prefill(const void* q, int64_t ldq, const void* k, int64_t ldk, const void* kr, int64_t ld_kr,
                                  const void* vt, int64_t ld_vt, void* out, int64_t ldo, const int* seq_row,
                                  const int* seq_len, int B, int H, int G, int tokens, int max_len, int dim, int rd,
                                  int vd, int window, int chunk, int sink, const float* sinks, const void* gate,
-                                 int64_t ldg, float gate_scale, float scale, int dtype, int* err, void* stream) {
+                                 int64_t ldg, float gate_scale, int pool, const void* kp, int64_t ld_kp, const void* vp,
+                                 int64_t ld_vp, const int* pool_row, int pool_rows, float scale, int dtype, int* err,
+                                 void* stream) {
   if (!ipex_packed_prefill_ok(dim, rd, vd, 8, dtype) || B < 1 || B > 65535 || H < 1 || tokens < 1 || max_len < 1 ||
       window < 0 || chunk < 0 || (max_len + kBQ - 1) / kBQ > 65535 || G < 1 || H % G != 0)
     return (int)cudaErrorInvalidValue;
@@ -421,6 +444,10 @@ IPEX_API int ipex_packed_prefill(const void* q, int64_t ldq, const void* k, int6
       (gate != nullptr && (ldg % 8)))
     return (int)cudaErrorInvalidValue;
   if (((uintptr_t)q | (uintptr_t)k | (uintptr_t)kr | (uintptr_t)vt | (uintptr_t)out | (uintptr_t)gate) & 15)
+    return (int)cudaErrorInvalidValue;
+  if (pool < 0 || (pool > 0 && (window < 1 || chunk > 0 || rd > 0 || kp == nullptr || vp == nullptr || pool_row == nullptr ||
+                                pool_rows < 1 || (ld_kp % 8) || (ld_vp % 8) || ld_vp < pool_rows ||
+                                (((uintptr_t)kp | (uintptr_t)vp) & 15))))
     return (int)cudaErrorInvalidValue;
   Args a = {};
   a.out = out; a.seq_row = seq_row; a.seq_len = seq_len; a.err = err; a.ldo = ldo;
@@ -430,11 +457,15 @@ IPEX_API int ipex_packed_prefill(const void* q, int64_t ldq, const void* k, int6
   a.group = H / G;
   a.sink = sink;
   a.chunk = chunk; a.sinks = sinks; a.gate = gate; a.ldg = ldg; a.gate_scale = gate_scale;
+  a.pool = pool; a.pool_row = pool_row;
   a.scale_log2 = scale * 1.4426950408889634f;
   cudaStream_t st = (cudaStream_t)stream;
-  if (dtype == DT_F16)
-    return vd <= 64 ? launch<__half, 64>(q, ldq, k, ldk, kr, ld_kr, vt, ld_vt, a, B, H, tokens, max_len, st)
-                    : launch<__half, 128>(q, ldq, k, ldk, kr, ld_kr, vt, ld_vt, a, B, H, tokens, max_len, st);
-  return vd <= 64 ? launch<__nv_bfloat16, 64>(q, ldq, k, ldk, kr, ld_kr, vt, ld_vt, a, B, H, tokens, max_len, st)
-                  : launch<__nv_bfloat16, 128>(q, ldq, k, ldk, kr, ld_kr, vt, ld_vt, a, B, H, tokens, max_len, st);
+  auto run = [&](auto* tag, auto dv) {
+    return launch<std::remove_pointer_t<decltype(tag)>, decltype(dv)::value>(
+        q, ldq, k, ldk, kr, ld_kr, vt, ld_vt, kp, ld_kp, vp, ld_vp, pool_rows, a, B, H, tokens, max_len, st);
+  };
+  using D64 = std::integral_constant<int, 64>;
+  using D128 = std::integral_constant<int, 128>;
+  if (dtype == DT_F16) return vd <= 64 ? run((__half*)nullptr, D64{}) : run((__half*)nullptr, D128{});
+  return vd <= 64 ? run((__nv_bfloat16*)nullptr, D64{}) : run((__nv_bfloat16*)nullptr, D128{});
 }

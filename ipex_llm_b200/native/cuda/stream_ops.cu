@@ -1,7 +1,8 @@
 // Element-wise and routing kernels of decoders with a 32-bit residual stream, sm_100a: embedding (scaled, with an
 // optional bigram table, into one or several streams), RMS norm of the stream into the activation dtype, the joint of a
 // block that norms a sublayer's output before it is added, the joint of blocks between which several streams are mixed
-// (hyper-connections), tanh soft-cap of fp32 logits, biases and gated units behind library or packed products, and
+// (hyper-connections), the joint of a block whose sublayers' outputs are normed side by side, tanh soft-cap of fp32 logits,
+// biases, activations and gated units behind library or packed products, and
 // the data movement around a dense expert bank for prompts (choice of experts, slots grouped by expert on the device,
 // row gather, gated unit, combination), plus a plain tiled product for sizes the tensor-core kernels do not take and for
 // 32-bit models.
@@ -185,6 +186,49 @@ __global__ void add_norm_stream_kernel(float* __restrict__ x, int64_t ldx, const
   for (int k = tid; k < K; k += nt) dst[k] = DT<T>::from_f(xr[k] * inv * w_in[k]);
 }
 
+// x += sum over one or two y of norm(y) * w, and out = x, or norm(x) * w_in, in the activation dtype.  One CTA per row.
+struct SidesArgs {
+  float* x;
+  const float* y[2];    // [n, ldy] or null
+  const float* w[2];    // [K]
+  const float* w_in;    // [K], or null: out is x itself
+  void* out;            // T [n, ldo] or null
+  int64_t ldx, ldy, ldo;
+  int K;
+  float eps;
+};
+
+template <typename T>
+__global__ void add_sides_kernel(SidesArgs a) {
+  __shared__ float red[32], red2[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int tid = threadIdx.x, nt = blockDim.x;
+  float* x = a.x + (int64_t)blockIdx.x * a.ldx;
+  const float* y0 = a.y[0] != nullptr ? a.y[0] + (int64_t)blockIdx.x * a.ldy : nullptr;
+  const float* y1 = a.y[1] != nullptr ? a.y[1] + (int64_t)blockIdx.x * a.ldy : nullptr;
+  T* out = a.out != nullptr ? reinterpret_cast<T*>(a.out) + (int64_t)blockIdx.x * a.ldo : nullptr;
+  float s0 = 0.f, s1 = 0.f;
+  for (int k = tid; k < a.K; k += nt) {
+    if (y0 != nullptr) s0 = fmaf(y0[k], y0[k], s0);
+    if (y1 != nullptr) s1 = fmaf(y1[k], y1[k], s1);
+  }
+  if (y0 != nullptr) s0 = 1.0f / sqrtf(block_sum(s0, red) / (float)a.K + a.eps);
+  if (y1 != nullptr) s1 = 1.0f / sqrtf(block_sum(s1, red2) / (float)a.K + a.eps);
+  float ss = 0.f;
+  for (int k = tid; k < a.K; k += nt) {
+    float v = x[k];
+    if (y0 != nullptr) v = fmaf(y0[k] * s0, a.w[0][k], v);
+    if (y1 != nullptr) v = fmaf(y1[k] * s1, a.w[1][k], v);
+    if (y0 != nullptr || y1 != nullptr) x[k] = v;
+    if (a.w_in != nullptr) ss = fmaf(v, v, ss);
+    else if (out != nullptr) out[k] = DT<T>::from_f(v);
+  }
+  if (a.w_in == nullptr || out == nullptr) return;
+  const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)a.K + a.eps);
+  for (int k = tid; k < a.K; k += nt) out[k] = DT<T>::from_f(x[k] * inv * a.w_in[k]);      // (what this thread wrote)
+}
+
 // Several residual streams x [S, K] per token.  Behind a sublayer with output y all streams are mixed,
 // x_t <- sum_s mix[s, t] x_s + w_out[t] y  (y null: they stay), and the next sublayer's input is the norm of
 // sum_s w_in[s] x_s.  One CTA per token; with NV > 0 a thread keeps its part of all streams in registers.
@@ -317,17 +361,37 @@ __global__ void bias_rows_kernel(TY* __restrict__ y, int64_t ldy, const T* __res
   for (int n = threadIdx.x; n < N; n += blockDim.x) r[n] = DT<TY>::from_f(DT<TY>::to_f(r[n]) + DT<T>::to_f(bias[n]));
 }
 
-// out[r, i] = act(gate + bias) * (up + bias) from a row of 2 I products, act gelu_tanh or silu; interleaved: gate and up
-// alternate in blocks of eight
-template <typename TY, typename T, bool SILU>
+// out[r, i] = act(gate + bias) * (up + bias) from a row of 2 I products, act gelu_tanh (3), silu (4) or the clamped unit (5);
+// interleaved: gate and up alternate in blocks of eight
+template <typename TY, typename T, int ACT>
 __global__ void glu_products_kernel(const TY* __restrict__ gu, int64_t ld, const T* __restrict__ bias,
-                                     T* __restrict__ out, int64_t ldo, int I, int interleaved) {
+                                     T* __restrict__ out, int64_t ldo, int I, int interleaved, float limit, float alpha) {
   const TY* r = gu + (int64_t)blockIdx.x * ld;
   for (int i = threadIdx.x; i < I; i += blockDim.x) {
     const int g = interleaved ? (i >> 3) * 16 + (i & 7) : i, u = interleaved ? g + 8 : I + i;
     const float bg = bias != nullptr ? DT<T>::to_f(bias[g]) : 0.f, bu = bias != nullptr ? DT<T>::to_f(bias[u]) : 0.f;
     const float z = DT<TY>::to_f(r[g]) + bg;
-    out[(int64_t)blockIdx.x * ldo + i] = DT<T>::from_f((SILU ? silu(z) : gelu_tanh(z)) * (DT<TY>::to_f(r[u]) + bu));
+    const float v = DT<TY>::to_f(r[u]) + bu;
+    float y;
+    if constexpr (ACT == 5) {
+      const float g1 = fminf(z, limit);
+      y = g1 / (1.0f + expf(-alpha * g1)) * (fminf(fmaxf(v, -limit), limit) + 1.0f);
+    } else {
+      y = (ACT == 4 ? silu(z) : gelu_tanh(z)) * v;
+    }
+    out[(int64_t)blockIdx.x * ldo + i] = DT<T>::from_f(y);
+  }
+}
+
+// columns [from, N) of y in place: act 1 squared relu; 6 gelu_tanh times row ids[r] of mul
+template <typename TY, typename T>
+__global__ void act_rows_kernel(TY* __restrict__ y, int64_t ldy, int N, int from, int act, const T* __restrict__ mul,
+                                int64_t ldm, int64_t mul_rows, const int64_t* __restrict__ ids) {
+  TY* r = y + (int64_t)blockIdx.x * ldy;
+  const int64_t row = act == 6 ? min(max(ids[blockIdx.x], (int64_t)0), mul_rows - 1) : 0;
+  for (int n = from + threadIdx.x; n < N; n += blockDim.x) {
+    const float v = DT<TY>::to_f(r[n]);
+    r[n] = DT<TY>::from_f(act == 6 ? gelu_tanh(v) * DT<T>::to_f(mul[row * ldm + n]) : v > 0.f ? v * v : 0.f);
   }
 }
 
@@ -384,21 +448,28 @@ __global__ void sigmoid_topk_kernel(const float* __restrict__ logits, int64_t ld
   }
 }
 
-// fp32 router logits [tokens, E (+ 1)] -> weights and experts (softmax_grouped_topk); a warp per token.  gate: the logit
-// behind the experts' becomes gate[t] = sigmoid.
-__global__ void softmax_topk_kernel(const float* __restrict__ logits, int64_t ld, float* __restrict__ w,
-                                    int64_t* __restrict__ idx, float* __restrict__ gate, int tokens, int E, int groups,
-                                    int keep, int k, float scale) {
+// fp32 router logits [tokens, E (+ 1)] -> weights and experts (softmax_grouped_topk) in rows of ldk; a warp per token.  bias:
+// [E] or null, added to the logits.  gate: the logit behind the experts' becomes gate[t] = sigmoid.  always: choice k is expert
+// E with weight 1.
+__global__ void softmax_topk_kernel(const float* __restrict__ logits, int64_t ld, const float* __restrict__ bias,
+                                    float* __restrict__ w, int64_t* __restrict__ idx, int ldk, float* __restrict__ gate,
+                                    int always, int tokens, int E, int groups, int keep, int k, float scale) {
   extern __shared__ float sh[];
+  pdl_launch_dependents();
+  pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, wpb = blockDim.x >> 5;
   const int t = blockIdx.x * wpb + warp;
   if (t >= tokens) return;
   float* sc = sh + (size_t)warp * (E + groups);
   const float* row = logits + (int64_t)t * ld;
-  for (int e = lane; e < E; e += 32) sc[e] = row[e];
+  for (int e = lane; e < E; e += 32) sc[e] = bias != nullptr ? row[e] + bias[e] : row[e];
   if (gate != nullptr && lane == 0) gate[t] = 1.0f / (1.0f + expf(-row[E]));
   __syncwarp();
-  softmax_grouped_topk(sc, sc + E, E, groups, keep, k, scale, w + (int64_t)t * k, idx + (int64_t)t * k, lane);
+  if (always && lane == 0) {
+    w[(int64_t)t * ldk + k] = 1.f;
+    idx[(int64_t)t * ldk + k] = E;
+  }
+  softmax_grouped_topk(sc, sc + E, E, groups, keep, k, scale, w + (int64_t)t * ldk, idx + (int64_t)t * ldk, lane);
 }
 
 // (token, choice) slots grouped by expert, one CTA: order[pos] = slot, inverse[slot] = pos, ranges[e] = (first, count).
@@ -484,21 +555,22 @@ __global__ void combine_slots_kernel(const T* __restrict__ y, const int* __restr
   }
 }
 
-// out[t] = gate[t] * out[t] (gate null: 0) + sum_j w[t, j] y[inverse[t * k + j]]
+// out[t] = gate[t] * out[t] (gate null: 0, or with `add` 1) + sum_j w[t, j] y[inverse[t * k + j]]
 template <typename T>
 __global__ void combine_weighted_kernel(const T* __restrict__ y, const int* __restrict__ inverse,
                                         const float* __restrict__ w, const float* __restrict__ gate,
-                                        float* __restrict__ out, int N, int k) {
+                                        float* __restrict__ out, int N, int k, int add) {
   const int t = blockIdx.x;
   float* o = out + (int64_t)t * N;
-  const float g = gate != nullptr ? gate[t] : 0.f;
+  const bool keep = gate != nullptr || add;
+  const float g = gate != nullptr ? gate[t] : 1.f;
   constexpr int VN = 16 / (int)sizeof(T);
   if (N % VN == 0) {
     for (int n = threadIdx.x * VN; n < N; n += blockDim.x * VN) {
       float s[VN];
 #pragma unroll
       for (int i = 0; i < VN; i += 4) {
-        const float4 f = gate != nullptr ? *reinterpret_cast<const float4*>(o + n + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        const float4 f = keep ? *reinterpret_cast<const float4*>(o + n + i) : make_float4(0.f, 0.f, 0.f, 0.f);
         s[i] = g * f.x; s[i + 1] = g * f.y; s[i + 2] = g * f.z; s[i + 3] = g * f.w;
       }
       for (int j = 0; j < k; ++j) {
@@ -514,7 +586,7 @@ __global__ void combine_weighted_kernel(const T* __restrict__ y, const int* __re
     return;
   }
   for (int n = threadIdx.x; n < N; n += blockDim.x) {
-    float s = gate != nullptr ? g * o[n] : 0.f;
+    float s = keep ? g * o[n] : 0.f;
     for (int j = 0; j < k; ++j)
       s = fmaf(w[(int64_t)t * k + j], DT<T>::to_f(y[(int64_t)inverse[(int64_t)t * k + j] * N + n]), s);
     o[n] = s;
@@ -616,6 +688,35 @@ IPEX_API int ipex_add_norm_stream(float* x, int64_t ldx, const float* y, int64_t
   });
 }
 
+// x [n, K] += norm(y0) * w0 + norm(y1) * w1 (y0, y1 may be null; row stride ldy); out (may be null) = x in the activation
+// dtype, or norm(x) * w_in.  Weights fp32.
+IPEX_API int ipex_add_sides(float* x, int64_t ldx, const float* y0, const float* w0, const float* y1, const float* w1,
+                            int64_t ldy, const float* w_in, void* out, int64_t ldo, int n, int K, float eps, int dtype, int pdl,
+                            void* stream) {
+  if (n < 1 || K < 1 || (y0 != nullptr && w0 == nullptr) || (y1 != nullptr && w1 == nullptr)) return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    const SidesArgs a = {x, {y0, y1}, {w0, w1}, w_in, out, ldx, ldy, ldo, K, eps};
+    const int threads = K <= 512 ? 128 : K <= 2048 ? 256 : K <= 4096 ? 512 : 1024;
+    return launch_kernel(add_sides_kernel<T>, dim3(n), dim3(threads), 0, (cudaStream_t)stream, pdl != 0, a);
+  });
+}
+
+// Columns [from, N) of y [n, N] (the activation dtype, or fp32) in place: act 1 squared relu; 6 gelu_tanh times the row ids[i] of
+// mul [mul_rows, ldm].
+IPEX_API int ipex_act_rows(void* y, int64_t ldy, int y_f32, int n, int N, int from, int act, const void* mul, int64_t ldm,
+                           int64_t mul_rows, const int64_t* ids, int dtype, void* stream) {
+  if (n < 1 || N < 1 || from < 0 || (act != 1 && act != 6) || (act == 6 && (mul == nullptr || ids == nullptr || mul_rows < 1)))
+    return (int)cudaErrorInvalidValue;
+  return by_dtype(dtype, [&](auto* tag) {
+    using T = std::remove_pointer_t<decltype(tag)>;
+    cudaStream_t st = (cudaStream_t)stream;
+    if (y_f32) act_rows_kernel<float, T><<<n, 256, 0, st>>>((float*)y, ldy, N, from, act, (const T*)mul, ldm, mul_rows, ids);
+    else act_rows_kernel<T, T><<<n, 256, 0, st>>>((T*)y, ldy, N, from, act, (const T*)mul, ldm, mul_rows, ids);
+    return cudaGetLastError();
+  });
+}
+
 // y [n, N] (the bias's dtype, or fp32) += bias
 IPEX_API int ipex_bias_rows(void* y, int64_t ldy, int y_f32, const void* bias, int n, int N, int dtype, void* stream) {
   if (n < 1 || N < 1) return (int)cudaErrorInvalidValue;
@@ -627,19 +728,19 @@ IPEX_API int ipex_bias_rows(void* y, int64_t ldy, int y_f32, const void* bias, i
   });
 }
 
-// out [n, I] = act(gate + bias) * (up + bias) of gu [n, 2 I] (the activation dtype, or fp32); use_silu: silu, else gelu_tanh
+// out [n, I] = act(gate + bias) * (up + bias) of gu [n, 2 I] (the activation dtype, or fp32); act: see glu_products_kernel
 IPEX_API int ipex_glu_rows(const void* gu, int64_t ld, int gu_f32, const void* bias, void* out, int64_t ldo, int n, int I,
-                           int interleaved, int use_silu, int dtype, void* stream) {
-  if (n < 1 || I < 1 || (interleaved && I % 8 != 0)) return (int)cudaErrorInvalidValue;
+                           int interleaved, int act, float limit, float alpha, int dtype, void* stream) {
+  if (n < 1 || I < 1 || (interleaved && I % 8 != 0) || act < 3 || act > 5) return (int)cudaErrorInvalidValue;
   cudaStream_t st = (cudaStream_t)stream;
   return by_dtype(dtype, [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
     if (gu_f32) {
-      auto kern = use_silu ? glu_products_kernel<float, T, true> : glu_products_kernel<float, T, false>;
-      kern<<<n, 256, 0, st>>>((const float*)gu, ld, (const T*)bias, (T*)out, ldo, I, interleaved);
+      auto kern = act == 5 ? glu_products_kernel<float, T, 5> : act == 4 ? glu_products_kernel<float, T, 4> : glu_products_kernel<float, T, 3>;
+      kern<<<n, 256, 0, st>>>((const float*)gu, ld, (const T*)bias, (T*)out, ldo, I, interleaved, limit, alpha);
     } else {
-      auto kern = use_silu ? glu_products_kernel<T, T, true> : glu_products_kernel<T, T, false>;
-      kern<<<n, 256, 0, st>>>((const T*)gu, ld, (const T*)bias, (T*)out, ldo, I, interleaved);
+      auto kern = act == 5 ? glu_products_kernel<T, T, 5> : act == 4 ? glu_products_kernel<T, T, 4> : glu_products_kernel<T, T, 3>;
+      kern<<<n, 256, 0, st>>>((const T*)gu, ld, (const T*)bias, (T*)out, ldo, I, interleaved, limit, alpha);
     }
     return cudaGetLastError();
   });
@@ -699,15 +800,17 @@ IPEX_API int ipex_moe_sigmoid_topk(const float* logits, int64_t ld, float* w, in
 }
 
 // logits [tokens, E] (with `gate`, E + 1) -> weights and experts [tokens, k]: soft-max, the `keep` best of `groups` equal
-// groups, the k largest, divided by their sum and times scale; gate [tokens] (may be null): sigmoid of the last logit.
-IPEX_API int ipex_moe_softmax_grouped_topk(const float* logits, int64_t ld, float* w, int64_t* idx, float* gate, int tokens,
-                                           int E, int groups, int keep, int k, float scale, void* stream) {
+// groups, the k largest, divided by their sum and times scale; gate [tokens] (may be null): sigmoid of the last logit.  bias
+// [E] (may be null) is added to the logits.  w and idx have rows of ldk; always: choice k is expert E, weight 1.
+IPEX_API int ipex_moe_softmax_grouped_topk(const float* logits, int64_t ld, const float* bias, float* w, int64_t* idx, int ldk,
+                                           float* gate, int always, int tokens, int E, int groups, int keep, int k,
+                                           float scale, int pdl, void* stream) {
   if (tokens < 1 || E < 1 || E > 2500 || k < 1 || k > E || groups < 1 || E % groups || keep < 1 || keep > groups ||
-      k > E / groups * keep)
+      k > E / groups * keep || ldk < k + (always != 0))
     return (int)cudaErrorInvalidValue;
-  softmax_topk_kernel<<<(tokens + 3) / 4, 128, (size_t)4 * (E + groups) * sizeof(float), (cudaStream_t)stream>>>(
-      logits, ld, w, idx, gate, tokens, E, groups, keep, k, scale);
-  return (int)cudaGetLastError();
+  return (int)launch_kernel(softmax_topk_kernel, dim3((tokens + 3) / 4), dim3(128), (size_t)4 * (E + groups) * sizeof(float),
+                            (cudaStream_t)stream, pdl != 0, logits, ld, bias, w, idx, ldk, gate, always, tokens, E, groups, keep, k,
+                            scale);
 }
 
 // Expert ids must lie in [0, E).
@@ -748,13 +851,13 @@ IPEX_API int ipex_moe_combine_slots(const void* y, const int* inverse, float* re
   });
 }
 
-// out [tokens, N] fp32 = gate * out (gate null: 0) + sum_j w[t, j] y[inverse[t k + j]]
+// out [tokens, N] fp32 = gate * out (gate null: 0, or with `add` 1) + sum_j w[t, j] y[inverse[t k + j]]
 IPEX_API int ipex_moe_combine_weighted(const void* y, const int* inverse, const float* w, const float* gate, float* out,
-                                       int tokens, int N, int k, int dtype, void* stream) {
+                                       int tokens, int N, int k, int add, int dtype, void* stream) {
   if (tokens < 1 || N < 1 || k < 1 || (((uintptr_t)y | (uintptr_t)out) & 15)) return (int)cudaErrorInvalidValue;
   return by_dtype(dtype, [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
-    combine_weighted_kernel<T><<<tokens, 256, 0, (cudaStream_t)stream>>>((const T*)y, inverse, w, gate, out, N, k);
+    combine_weighted_kernel<T><<<tokens, 256, 0, (cudaStream_t)stream>>>((const T*)y, inverse, w, gate, out, N, k, add);
     return cudaGetLastError();
   });
 }

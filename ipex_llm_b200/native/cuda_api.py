@@ -68,34 +68,37 @@ COMPONENT_SIGS = {
     "stream": {
         "ipex_argmax": _SIGS["ipex_argmax"],
         "ipex_gemv_rows_max": [ci, ci],
-        "ipex_gemv_rows": [vp, i64, vp, i64, vp, cf, vp, vp, i64, vp, ci, vp, i64, ci, ci, ci, ci, ci, ci, cf, ci, ci,
-                           vp],
+        "ipex_gemv_rows": [vp, i64, vp, i64, vp, cf, vp, vp, i64, vp, ci, vp, i64, ci, ci, ci, ci, ci, ci, cf, ci, ci, cf, cf,
+                           vp, i64, i64, vp, ci, ci, vp],
         "ipex_moe_router_sigmoid": [vp, i64, vp, cf, vp, vp, vp, ci, ci, ci, ci, ci, ci, vp],
         "ipex_moe_router_softmax": [vp, i64, vp, vp, vp, ci, ci, ci, ci, ci, ci, ci, cf, ci, ci, vp],
-        "ipex_moe_glu_rows": [vp, i64, vp, cf, vp, vp, vp, i64, vp, vp, ci, ci, ci, ci, ci, ci, ci, cf, cf, ci, ci, ci, ci, vp],
-        "ipex_moe_down_rows": [vp, i64, vp, vp, vp, vp, i64, vp, ci, ci, ci, ci, ci, ci, ci, ci, vp],
+        "ipex_moe_glu_rows": [vp, i64, vp, cf, vp, vp, vp, i64, vp, vp, ci, ci, ci, ci, ci, ci, ci, cf, cf, cf, ci, ci,
+                              ci, ci, vp],
+        "ipex_moe_down_rows": [vp, i64, vp, vp, vp, vp, i64, vp, ci, ci, ci, ci, ci, ci, ci, ci, ci, vp],
         "ipex_embed_stream": [vp, vp, vp, vp, vp, i64, vp, vp, vp, ci, ci, i64, cf, i64, i64, i64, ci, ci, ci, vp],
         "ipex_norm_stream": [vp, i64, vp, ci, vp, i64, vp, ci, ci, cf, ci, ci, vp],
         "ipex_add_norm_stream": [vp, i64, vp, i64, vp, vp, vp, i64, ci, ci, cf, ci, ci, vp],
+        "ipex_add_sides": [vp, i64, vp, vp, vp, vp, i64, vp, vp, i64, ci, ci, cf, ci, ci, vp],
+        "ipex_act_rows": [vp, i64, ci, ci, ci, ci, ci, vp, i64, i64, vp, ci, vp],
         "ipex_bias_rows": [vp, i64, ci, vp, ci, ci, ci, vp],
         "ipex_hyper_joint": [vp, vp, i64, vp, vp, vp, vp, vp, i64, ci, ci, ci, cf, ci, ci, vp],
-        "ipex_glu_rows": [vp, i64, ci, vp, vp, i64, ci, ci, ci, ci, ci, vp],
+        "ipex_glu_rows": [vp, i64, ci, vp, vp, i64, ci, ci, ci, ci, cf, cf, ci, vp],
         "ipex_softcap_f32": [vp, i64, cf, vp],
         "ipex_add_stream": [vp, vp, i64, ci, vp],
         "ipex_relu2_inplace": [vp, i64, ci, vp],
         "ipex_moe_sigmoid_topk": [vp, i64, vp, vp, ci, ci, ci, vp],
-        "ipex_moe_softmax_grouped_topk": [vp, i64, vp, vp, vp, ci, ci, ci, ci, ci, cf, vp],
+        "ipex_moe_softmax_grouped_topk": [vp, i64, vp, vp, vp, ci, vp, ci, ci, ci, ci, ci, ci, cf, ci, vp],
         "ipex_moe_group_slots": [vp, ci, ci, vp, vp, vp, vp],
         "ipex_moe_gather_slots": [vp, vp, vp, vp, vp, ci, ci, ci, ci, vp],
         "ipex_moe_glu_from_gu": [vp, vp, vp, ci, ci, cf, cf, ci, ci, vp],
         "ipex_moe_combine_slots": [vp, vp, vp, ci, ci, ci, ci, vp],
-        "ipex_moe_combine_weighted": [vp, vp, vp, vp, vp, ci, ci, ci, ci, vp],
+        "ipex_moe_combine_weighted": [vp, vp, vp, vp, vp, ci, ci, ci, ci, ci, vp],
         "ipex_gemm_plain": [vp, vp, vp, vp, ci, ci, ci, ci, ci, ci, vp],
         "ipex_gemm_stream": [vp, i64, vp, i64, vp, i64, vp, vp, ci, vp, i64, vp, vp, ci, ci, ci, ci, ci, ci, cf, cf,
-                             ci, ci, vp, vp],
+                             ci, vp, i64, i64, vp, ci, ci, vp, vp],
         "ipex_packed_prefill_ok": [ci, ci, ci, ci, ci],
         "ipex_packed_prefill": [vp, i64, vp, i64, vp, i64, vp, i64, vp, i64, vp, vp, ci, ci, ci, ci, ci, ci, ci, ci,
-                                ci, ci, ci, vp, vp, i64, cf, cf, ci, vp, vp],
+                                ci, ci, ci, vp, vp, i64, cf, ci, vp, i64, vp, i64, vp, ci, cf, ci, vp, vp],
     },
     "latent": {
         "ipex_latent_prep": [vp, i64, vp, i64, vp, cf, vp, vp, vp, vp, vp, vp, vp, i64, i64, vp, ci, ci, ci, ci, ci, ci,
@@ -108,20 +111,43 @@ COMPONENT_SIGS = {
                              vp],
         "ipex_latent_uv": [vp, vp, vp, vp, i64, vp, i64, ci, ci, ci, ci, ci, ci, ci, vp],
     },
-    "hybrid": {
+    "attention": {
         "ipex_kv_append": [vp, vp, i64, vp, i64, cf, vp, i64, i64, vp, i64, i64, vp, i64, vp, vp, ci, ci, ci, ci, ci,
                            ci, vp],
-        "ipex_qk_prepare": [vp, i64, vp, vp, vp, vp, vp, ci, ci, cf, ci, ci, ci, ci, ci, vp],
+        "ipex_kv_pool": [vp, i64, i64, vp, i64, i64, vp, i64, i64, vp, i64, i64, vp, i64, vp, i64, vp, vp, vp, vp, vp, vp, ci, ci,
+                         ci, ci, ci, ci, ci, vp],
+        "ipex_qk_prepare": [vp, i64, vp, vp, vp, vp, vp, ci, ci, cf, vp, vp, ci, ci, ci, ci, ci, ci, vp],
         "ipex_kv_attn": [vp, vp, vp, i64, vp, i64, cf, vp, i64, i64, vp, i64, i64, vp, i64, vp, vp, vp, ci, ci, ci, ci,
-                         ci, ci, ci, ci, vp, vp, i64, cf, ci, ci, vp, vp, ci, ci, cf, ci, cf, ci, ci, vp],
+                         ci, ci, ci, ci, vp, vp, i64, cf, ci, ci, vp, vp, ci, ci, cf, vp, vp, ci, vp, i64, i64, vp, i64, i64, ci,
+                         cf, ci, ci, vp],
+    },
+    "recurrent": {
+        "ipex_ring_tail": [vp, i64, vp, vp, vp, vp, vp, ci, ci, ci, ci, vp],
+        "ipex_gated_norm": [vp, vp, i64, vp, ci, ci, vp, i64, ci, ci, ci, cf, cf, ci, vp],
+        "ipex_gated_group_norm": [vp, vp, i64, vp, vp, i64, ci, ci, ci, cf, ci, ci, vp],
+    },
+    "delta": {
         "ipex_delta_chunks_ok": [ci, ci],
         "ipex_delta_fused_ok": [ci],
         "ipex_delta_step": [vp, i64, ci, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, ci, vp, cf, vp, i64, vp, ci, ci,
                             ci, ci, ci, ci, ci, vp],
         "ipex_delta_chunks": [vp, i64, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, ci, vp, vp, ci, ci, vp, vp, ci, ci,
                               ci, ci, ci, ci, vp, vp],
-        "ipex_delta_tail": [vp, i64, vp, vp, vp, vp, vp, ci, ci, ci, ci, vp],
-        "ipex_gated_norm": [vp, vp, i64, vp, vp, i64, ci, ci, ci, cf, cf, ci, vp],
+    },
+    "general_delta": {
+        "ipex_general_chunks_ok": [ci, ci, ci, cf],
+        "ipex_general_fused_ok": [ci],
+        "ipex_general_step": [vp, i64, ci, vp, i64, vp, vp, vp, vp, vp, vp, vp, vp, vp, ci, vp, cf, vp, i64, vp, ci, ci, ci, ci,
+                              cf, ci, ci, vp],
+        "ipex_general_chunks": [vp, i64, vp, i64, vp, vp, vp, vp, vp, vp, vp, vp, vp, ci, vp, vp, ci, ci, vp, vp, ci, ci, ci,
+                                ci, cf, ci, vp, vp],
+    },
+    "ssd": {
+        "ipex_ssd_chunks_ok": [ci, ci, ci],
+        "ipex_ssd_step": [vp, i64, vp, i64, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, ci, vp, ci, ci, ci, ci, ci, ci, ci,
+                          vp],
+        "ipex_ssd_chunks": [vp, i64, vp, i64, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, vp, ci, vp, vp, ci, ci, vp, vp, vp,
+                            ci, ci, ci, ci, ci, ci, vp, vp],
     },
     "linear": {
         "ipex_linear_chunks_ok": [ci, ci, ci],
@@ -134,16 +160,20 @@ COMPONENT_SIGS = {
 }
 
 
+# scratch sizes of the chunked recurrences: (dim, vdim) -> floats
+_SCRATCH_FLOATS = {"delta": ("ipex_delta_scratch_floats",), "general_delta": ("ipex_general_scratch_floats",),
+                   "linear": ("ipex_linear_scratch_floats",), "ssd": ("ipex_ssd_group_floats", "ipex_ssd_head_floats")}
+
+
 def declare_component(lib: ctypes.CDLL, name: str):
     for fn_name, args in COMPONENT_SIGS[name].items():
         fn = getattr(lib, fn_name)
         fn.argtypes, fn.restype = args, ci
     if name == "stream":
         lib.ipex_gemv_rows_tune.argtypes, lib.ipex_gemv_rows_tune.restype = [ci], None
-    if name == "hybrid":
-        lib.ipex_delta_scratch_floats.argtypes, lib.ipex_delta_scratch_floats.restype = [ci, ci], i64
-    if name == "linear":
-        lib.ipex_linear_scratch_floats.argtypes, lib.ipex_linear_scratch_floats.restype = [ci, ci], i64
+    for fn_name in _SCRATCH_FLOATS.get(name, ()):
+        fn = getattr(lib, fn_name)
+        fn.argtypes, fn.restype = [ci, ci], i64
 
 
 def declare(lib: ctypes.CDLL):

@@ -12,6 +12,7 @@ import torch
 from ..native import cuda_api as api
 from ..native.lib import current_stream, ptr, stream_lib
 from .cuda_ops import error_flag
+from .recurrent import gated_norm, ring_tail
 from .stream import _dt
 
 SCRATCH_BYTES = 256 << 20        # of the chunked form; longer prompts run in several passes
@@ -37,7 +38,7 @@ class DeltaSpec:
         return self.channels + self.heads * self.vdim
 
     def chunks_ok(self, dtype) -> bool:
-        return dtype != torch.float32 and bool(stream_lib("hybrid").ipex_delta_chunks_ok(self.dim, self.vdim))
+        return dtype != torch.float32 and bool(stream_lib("delta").ipex_delta_chunks_ok(self.dim, self.vdim))
 
 
 class DeltaWeights:
@@ -55,7 +56,7 @@ def delta_mix(spec: DeltaSpec, w: DeltaWeights, proj, gates, slot, pos, cache, l
     output gates before their convolutions and activations) and ``gates [tokens, 2 heads]`` (write strengths, decays;
     fp32); the slots' states and convolution inputs move on.  ``portions``: how the tokens belong together, None when
     every token is another sequence's next one.  ``chunked`` overrides the choice of the form."""
-    lib, layer = stream_lib("hybrid"), cache.layers[layer_idx]
+    lib, layer = stream_lib("delta"), cache.layers[layer_idx]
     T, dt, st, dev = proj.shape[0], _dt(proj), current_stream(), proj.device
     sizes = (spec.heads, spec.kv_heads, spec.dim, spec.vdim, spec.taps, dt)
     common = (ptr(gates), ptr(w.conv), ptr(w.a_log), ptr(w.dt_bias), ptr(layer._v), ptr(layer._k), ptr(slot), ptr(pos),
@@ -86,8 +87,5 @@ def delta_mix(spec: DeltaSpec, w: DeltaWeights, proj, gates, slot, pos, cache, l
         else:
             api.check(lib.ipex_delta_step(ptr(proj), proj.stride(0), gate_at, *common, ptr(row), ptr(ln), n, None, 0.0, None,
                                           0, ptr(raw), *sizes, 0, st), "delta_step")
-        api.check(lib.ipex_delta_tail(ptr(proj), proj.stride(0), ptr(layer._v), ptr(slot), ptr(pos), ptr(row), ptr(ln), n,
-                                      spec.channels, spec.taps, dt, st), "delta_tail")
-    api.check(lib.ipex_gated_norm(ptr(raw), ptr(proj[:, gate_at:]), proj.stride(0), ptr(w.norm), ptr(out), out.stride(0), T,
-                                  spec.heads, spec.vdim, w.eps, 1.0, dt, st), "gated_norm")
-    return out
+        ring_tail(proj, layer._v, slot, pos, portions, spec.channels, spec.taps)
+    return gated_norm(raw, proj[:, gate_at:], w.norm, out, w.eps)

@@ -354,6 +354,17 @@ class KeyValueLayer(LatentLayer):
         return NormalLayer._alloc(self, bsz, heads, cap, dk, dv, dtype, device)
 
 
+class PooledLayer(KeyValueLayer):
+    """A key and a value per block of ``pool`` tokens and key head, counted from the sequence's first token: ``_k [slots,
+    heads, capacity // pool, dim]``, ``_v`` likewise.  A row counts once its block is complete."""
+
+    def open(self, slots, capacity, shape, dtype, device):
+        self._grow(slots, max(1, capacity // shape.pool), shape.heads, shape.dim, shape.vdim, dtype, device)
+
+    def reserve(self, extra_tokens: int):
+        pass
+
+
 class DeltaStateLayer(NormalLayer):
     """State of a recurrent layer, of one size however long the sequence is: ``_k [slots, heads, dim, vdim]`` in fp32,
     and the last inputs of its short convolutions, ``_v [slots, 1, taps, channels]`` (row = position mod taps; empty for
@@ -406,6 +417,15 @@ class KeyValueShape:
     dim: int
     vdim: int
     layer_cls = KeyValueLayer
+
+
+@dataclass(frozen=True)
+class PooledShape:
+    heads: int
+    dim: int
+    vdim: int
+    pool: int
+    layer_cls = PooledLayer
 
 
 @dataclass(frozen=True)

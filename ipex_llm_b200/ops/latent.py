@@ -130,7 +130,7 @@ def latent_prompt(spec: LatentSpec, qkv, w_uk, w_uv, kv_norm, cos, sin, slot, po
     rc = stream_lib().ipex_packed_prefill(ptr(qkv), qkv.stride(0), ptr(k), k.stride(0), ptr(kr), kr.stride(0), ptr(vt), ld,
                                           ptr(out), out.stride(0), ptr(seq_row), ptr(seq_len), seq_row.shape[0], H, H, T,
                                           max_len, spec.dim, spec.rot_dim, spec.v_dim, spec.window, 0, 0, None, ptr(g), ldg,
-                                          1.0, spec.scale, dt, ptr(error_flag(dev)), st)
+                                          1.0, 0, None, 0, None, 0, None, 0, spec.scale, dt, ptr(error_flag(dev)), st)
     if rc == -1:
         raise RuntimeError("ipex_llm_b200: the driver's tensor-map encoder rejected the attention operands")
     api.check(rc, "packed_prefill")

@@ -12,6 +12,7 @@ import torch
 from ..native import cuda_api as api
 from ..native.lib import current_stream, ptr, stream_lib
 from .cuda_ops import error_flag
+from .recurrent import gated_norm
 from .stream import _dt
 
 SCRATCH_BYTES = 256 << 20        # of the chunked form; longer prompts run in several passes
@@ -80,7 +81,4 @@ def linear_mix(spec: LinearSpec, w: LinearWeights, proj, low, slot, pos, cache, 
     else:
         api.check(lib.ipex_linear_step(ptr(proj), proj.stride(0), spec.gate_at, *common, ptr(row), ptr(ln), n, None, 0.0,
                                        0.0, None, 0, ptr(raw), *sizes, int(pdl) if portions is None else 0, st), "linear_step")
-    api.check(stream_lib("hybrid").ipex_gated_norm(ptr(raw), ptr(proj[:, spec.gate_at:]), proj.stride(0), ptr(w.norm), ptr(out),
-                                                   out.stride(0), T, spec.heads, spec.vdim, w.eps, spec.out_scale, dt, st),
-              "gated_norm")
-    return out
+    return gated_norm(raw, proj[:, spec.gate_at:], w.norm, out, w.eps, spec.out_scale)

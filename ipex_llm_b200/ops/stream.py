@@ -7,6 +7,8 @@ Every function launches on the current stream; there is no eager substitute.  Th
 from __future__ import annotations
 
 from contextlib import contextmanager
+from dataclasses import dataclass
+from typing import Optional
 
 import torch
 
@@ -17,6 +19,27 @@ from .cuda_ops import error_flag
 OUT_ACT, OUT_ADD, OUT_F32 = 0, 1, 2        # activation dtype / added to the stream / fp32
 ACT_NONE, ACT_RELU2 = 0, 1
 ACT_GLU, ACT_GELU_GLU, ACT_SILU_GLU = 2, 3, 4     # grouped GEMM only / gate and up rows in blocks of eight
+ACT_CLAMP_GLU, ACT_GELU_MUL = 5, 6               # likewise / gelu_tanh times the token's row of a table
+GATED_ACTS = (ACT_GELU_GLU, ACT_SILU_GLU, ACT_CLAMP_GLU)
+
+
+@dataclass(frozen=True)
+class ActArgs:
+    """Constants and operands of an activation: ``ACT_RELU2`` from column ``start`` on; ``limit`` and ``alpha`` of
+    ``ACT_CLAMP_GLU``; ``table [rows, N]`` (a view) and the tokens' rows ``ids`` (int64) of ``ACT_GELU_MUL``."""
+    start: int = 0
+    limit: float = 0.0
+    alpha: float = 0.0
+    table: Optional[torch.Tensor] = None
+    ids: Optional[torch.Tensor] = None
+
+    def c_args(self):
+        t = self.table
+        return (self.start, self.limit, self.alpha, ptr(t), 0 if t is None else t.stride(0), 0 if t is None else t.shape[0],
+                ptr(self.ids))
+
+
+NO_ARGS = ActArgs()
 
 
 def _dt(t) -> int:
@@ -43,18 +66,22 @@ def rows_max(K: int, dtype) -> int:
 
 
 def gemv_rows(w, x, out, mode: int, norm=None, eps: float = 0.0, act: int = 0, softcap: float = 0.0, pdl=False, bias=None,
-              w2=None, out2=None, interleaved=True):
+              w2=None, out2=None, interleaved=True, args: ActArgs = NO_ARGS):
     """``act(x @ w.T + bias)`` for a few rows.  ``norm``: ``x`` is the stream and is RMS-normed with this weight on the way
-    (inside the product for one or two rows; a CTA would spend longer on the norms of more rows than on its weights).
-    ``w2`` / ``out2``: more rows for the same ``x``, with fp32 results.  ``ACT_GELU_GLU`` / ``ACT_SILU_GLU``: ``w`` holds gate and up
-    rows (in blocks of eight, or not ``interleaved``), half as many columns come out."""
+    (inside the product for one or two rows; a CTA would spend longer on the norms of more rows than on its weights); rows
+    of the stream without ``norm`` are converted on the way.  ``w2`` / ``out2``: more rows for the same ``x``, with fp32
+    results.  ``GATED_ACTS``: ``w`` holds gate and up rows (in blocks of eight, or not ``interleaved``), half as many columns
+    come out."""
     M, N, K = x.shape[0], w.shape[0], w.shape[1]
     if norm is not None and M > 2 and w.dtype != torch.float32:
         x, norm = norm_stream(x, norm, eps, pdl=pdl), None
+    raw = norm is None and x.dtype != w.dtype
+    if raw and M * (K + 64) * w.element_size() > 160 * 1024:      # more than a CTA can stage
+        x, raw = add_sides(x, (), (), None, eps, w.dtype, pdl=pdl), False
     rc = stream_lib().ipex_gemv_rows(ptr(w), w.stride(0), ptr(x), x.stride(0), ptr(norm), eps, ptr(bias), ptr(out),
                                      out.stride(0), ptr(w2), 0 if w2 is None else w2.shape[0], ptr(out2),
                                      0 if out2 is None else out2.stride(0), M, N, K, mode, act, int(interleaved),
-                                     softcap, _dt(w), int(pdl), current_stream())
+                                     softcap, int(raw), *args.c_args(), _dt(w), int(pdl), current_stream())
     api.check(rc, "gemv_rows")
     return out
 
@@ -73,11 +100,11 @@ def _tile(rows: float, cols: int = 1 << 20) -> int:
     return bt
 
 
-def gemm(x, w, out, mode: int, act: int = 0, bias=None, interleaved=True, w2=None, out2=None):
+def gemm(x, w, out, mode: int, act: int = 0, bias=None, interleaved=True, w2=None, out2=None, args: ActArgs = NO_ARGS):
     """``x [M, K] @ w[N, K].T (+ bias)`` into ``out`` (see ``OUT_*``): the tcgen05 kernel, or the library product for
-    32-bit weights and rows that are no multiple of 16 bytes.  ``ACT_GELU_GLU``, ``w2`` / ``out2``: see ``gemv_rows``."""
+    32-bit weights and rows that are no multiple of 16 bytes.  Activations, ``w2`` / ``out2``: see ``gemv_rows``."""
     M, (N, K) = x.shape[0], w.shape
-    gated = act in (ACT_GELU_GLU, ACT_SILU_GLU)
+    gated = act in GATED_ACTS
     if gemm_ok(x, w) and not (gated and not interleaved):
         both = w2 is not None and gemm_ok(x, w2) and w2.stride(0) == w.stride(0)
         if w2 is not None and not both:
@@ -85,8 +112,8 @@ def gemm(x, w, out, mode: int, act: int = 0, bias=None, interleaved=True, w2=Non
         rc = stream_lib().ipex_gemm_stream(ptr(x), x.stride(0), ptr(w), w.stride(0), ptr(out), out.stride(0), ptr(bias),
                                            ptr(w2 if both else None), w2.shape[0] if both else 0,
                                            ptr(out2 if both else None), out2.stride(0) if both else 0, None, None, 1, M, N,
-                                           K, mode, act, 0.0, 0.0, _tile(M, N), _dt(w), ptr(error_flag(x.device)),
-                                           current_stream())
+                                           K, mode, act, args.limit, args.alpha, args.start, *args.c_args()[3:], _tile(M, N),
+                                           _dt(w), ptr(error_flag(x.device)), current_stream())
         if rc == -1:
             raise RuntimeError("ipex_llm_b200: the driver's tensor-map encoder rejected the GEMM operands")
         api.check(rc, "gemm_stream")
@@ -95,14 +122,12 @@ def gemm(x, w, out, mode: int, act: int = 0, bias=None, interleaved=True, w2=Non
         gemm(x, w2, out2, OUT_F32)
     with _true_fp32():
         if gated:
-            return glu_rows(torch.matmul(x.float(), w.float().t()), bias, out, act, interleaved)
+            return glu_rows(torch.matmul(x.float(), w.float().t()), bias, out, act, interleaved, args)
         if mode == OUT_ACT:
             torch.matmul(x, w.t(), out=out) if out.is_contiguous() else out.copy_(torch.matmul(x, w.t()))
             if bias is not None:
                 bias_rows_(out, bias)
-            if act == ACT_RELU2:
-                relu2_(out)
-            return out
+            return act_rows_(out, act, args) if act in (ACT_RELU2, ACT_GELU_MUL) else out
         if x.dtype == torch.float32:
             out.addmm_(x, w.t(), beta=1.0 if mode == OUT_ADD else 0.0)
         else:
@@ -119,13 +144,23 @@ def bias_rows_(y, bias):
     return y
 
 
-def glu_rows(gu, bias, out, act: int, interleaved=True):
+def glu_rows(gu, bias, out, act: int, interleaved=True, args: ActArgs = NO_ARGS):
     """``act(gate + bias) * (up + bias)`` of finished products ``gu [n, 2 I]`` (the dtype of ``out``, or fp32)."""
     rc = stream_lib().ipex_glu_rows(ptr(gu), gu.stride(0), int(gu.dtype == torch.float32), ptr(bias), ptr(out),
-                                    out.stride(0), gu.shape[0], gu.shape[1] // 2, int(interleaved),
-                                    int(act == ACT_SILU_GLU), _dt(out), current_stream())
+                                    out.stride(0), gu.shape[0], gu.shape[1] // 2, int(interleaved), act, args.limit,
+                                    args.alpha, _dt(out), current_stream())
     api.check(rc, "glu_rows")
     return out
+
+
+def act_rows_(y, act: int, args: ActArgs = NO_ARGS):
+    """``ACT_RELU2`` or ``ACT_GELU_MUL`` on finished products ``y [n, N]``, in place."""
+    start, _, _, *table = args.c_args()
+    dtype = y.dtype if args.table is None else args.table.dtype
+    rc = stream_lib().ipex_act_rows(ptr(y), y.stride(0), int(y.dtype == torch.float32), y.shape[0], y.shape[1], start, act, *table,
+                                    _dt(dtype), current_stream())
+    api.check(rc, "act_rows")
+    return y
 
 
 def relu2_(x):
@@ -183,6 +218,19 @@ def add_norm_stream(x, y, w_out, w_in, eps: float, dtype, pdl=False):
     rc = stream_lib().ipex_add_norm_stream(ptr(x), x.stride(0), ptr(y), y.stride(0), ptr(w_out), ptr(w_in), ptr(h),
                                            x.shape[1], x.shape[0], x.shape[1], eps, _dt(dtype), int(pdl), current_stream())
     api.check(rc, "add_norm_stream")
+    return h
+
+
+def add_sides(x, ys, ws, w_in, eps: float, dtype, pdl=False):
+    """``x += sum of norm(y) * w`` over up to two fp32 ``ys``, then ``norm(x) * w_in`` in ``dtype``, or ``x`` itself (``w_in``
+    None): the joint behind sublayers whose outputs are normed side by side.  The weights are fp32."""
+    n, K = x.shape
+    h = torch.empty(n, (K + 7) // 8 * 8, dtype=dtype, device=x.device)[:, :K]
+    y0, y1 = [*ys, None, None][:2]
+    w0, w1 = [*ws, None, None][:2]
+    rc = stream_lib().ipex_add_sides(ptr(x), x.stride(0), ptr(y0), ptr(w0), ptr(y1), ptr(w1), 0 if y0 is None else y0.stride(0),
+                                     ptr(w_in), ptr(h), h.stride(0), n, K, eps, _dt(dtype), int(pdl), current_stream())
+    api.check(rc, "add_sides")
     return h
 
 

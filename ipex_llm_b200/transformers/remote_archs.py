@@ -337,7 +337,8 @@ def _minicpm3(c: dict):
 # Architectures that neither transformers nor a remote modeling file implements: the package's own model classes.  Their
 # raw checkpoints carry an ``architecture`` field instead of a ``model_type`` (one written back by ``save_pretrained`` or
 # ``save_low_bit`` has both, and loads through the Auto classes the module registers).
-NATIVE_ARCHS: Dict[str, str] = {"Dobetar": "dobetar", "Dodilix": "dodilix", "Letarax": "letarax"}
+NATIVE_ARCHS: Dict[str, str] = {"Dobetar": "dobetar", "Dodilix": "dodilix", "Gegorax": "gegorax",
+                                "Letarax": "letarax"}
 
 
 def register_native_archs():

@@ -196,11 +196,11 @@ def kernels(z, prompt: int, peaks):
     add(f"delta_chunks (4 kernels) T={T}", us, nb, fl, f"rwkv5 {like:.1f} us",
         max(16.0 * T * dH * dV / hbm, 4.0 * T * dH * dV * dV / tf) / like)
     from ..native.lib import ptr, stream_lib
-    lib = stream_lib("hybrid")
-    per = dH * lib.ipex_delta_scratch_floats(dD, dV)
+    lib = stream_lib("recurrent")
+    per = dH * stream_lib("delta").ipex_delta_scratch_floats(dD, dV)
     rows.append({"kernel": f"delta scratch, MB for T={T}", "us": round(nc * per * 4 / 1e6, 1)})
     raw = torch.empty(T, dH, dV, device=dev)
-    us = _graph_us(lambda i: lib.ipex_gated_norm(ptr(raw), ptr(projs[i][:, dl.channels:]), dl.rows, ptr(w.norm), ptr(out),
+    us = _graph_us(lambda i: lib.ipex_gated_norm(ptr(raw), ptr(projs[i][:, dl.channels:]), dl.rows, ptr(w.norm), 0, 0, ptr(out),
                                                  out.stride(0), T, dH, dV, 1e-6, 1.0, 1, S.current_stream()), 4)
     add(f"gated_norm T={T}", us, 8.0 * T * dH * dV)
     cuda_ops.check_error_flag(torch.device("cuda", 0))

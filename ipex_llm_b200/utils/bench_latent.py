@@ -257,7 +257,7 @@ def kernels(z, prompt: int, peaks):
         us = _graph_us(lambda i: L.stream_lib().ipex_packed_prefill(
             L.ptr(qs[i]), ldq, L.ptr(ks[i]), H * z["dim"], L.ptr(kr), z["rd"], L.ptr(vt), T, L.ptr(out), H * z["vd"],
             L.ptr(row), L.ptr(ln), 1, H, H, T, T, z["dim"], z["rd"], z["vd"], win, 0, 0, None, None, 0,
-            1.0, 0.05, 1, L.ptr(err),
+            1.0, 0, None, 0, None, 0, None, 0, 0.05, 1, L.ptr(err),
             L.current_stream()), n)
         w = win or T
         pairs = T * min(w, T) - min(w, T) * (min(w, T) - 1) / 2
