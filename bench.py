@@ -1,7 +1,8 @@
 #!/usr/bin/env python
 """Headline benchmark: decode latency / throughput of low-bit Llama models on B200.
 
-    python bench.py --gpus N --steps K --warmup W [--config 7b|70b-tp|7b-spec|mixtral-pp|qlora-dp|latent|hybrid|multistream]
+    python bench.py --gpus N --steps K --warmup W [--config 7b|70b-tp|7b-spec|mixtral-pp|qlora-dp|latent|hybrid|multistream|
+                                                      parallel-block]
                     [--batch B]
                     [--model llama2-7b|llama3-70b] [--impl ours|reference|constructed]
 
@@ -12,7 +13,8 @@ fine-tuning of Llama-2-13B nf4, data parallel, sequence 512, micro-batch 4 per G
 throughput of the latent-attention decoder (Dobetar, bf16) at three sizes, beside a Llama-architecture model of equal
 size (``value`` is the largest size's decode throughput at batch 1, ``config.sizes`` holds the rest); ``hybrid`` the same
 for the decoder of attention and recurrent layers (Letarax); ``multistream`` for the decoder with several residual streams
-(Dodilix), beside the two before it.
+(Dodilix), beside the two before it; ``parallel-block`` for the decoder whose mixer and feed-forward stand side by side
+(Gegorax), beside the two before it.
 
 One "step" is one decode step (one new token for every sequence of the batch) after a prompt pass of
 ``--prompt`` random tokens.  ``ms_per_step`` is therefore the reference harness's "2+ avg latency (ms/token)"
@@ -166,6 +168,11 @@ def other_config(args):
         res = bench_multistream.run(["--iters", str(max(16, args.steps)), "--prompt", str(args.prompt or 2048)], timed=timed)
         extra = {"metric": "multi-stream decoder, decode tokens/s at batch 1", "scaling": "strong", "dtype": "bf16",
                  "parallelism": "single"}
+    elif args.config == "parallel-block":
+        from ipex_llm_b200.utils import bench_parallel_block
+        res = bench_parallel_block.run(["--iters", str(max(16, args.steps)), "--prompt", str(args.prompt or 2048)], timed=timed)
+        extra = {"metric": "parallel-block decoder, decode tokens/s at batch 1", "scaling": "strong", "dtype": "bf16",
+                 "parallelism": "single"}
     else:
         from ipex_llm_b200.utils import bench_speculative
         res = bench_speculative.run(["--new-tokens", str(max(32, args.steps))], timed=timed)
@@ -270,7 +277,7 @@ def main():
                     help="reference: the unmodified reference (unavailable offline); constructed: its semantics on "
                          "stock cuBLAS + NCCL (baseline/constructed.py)")
     ap.add_argument("--config", default="auto", choices=["auto", "7b", "70b-tp", "7b-spec", "mixtral-pp", "qlora-dp",
-                                                           "latent", "hybrid", "multistream"])
+                                                           "latent", "hybrid", "multistream", "parallel-block"])
     ap.add_argument("--model", default="auto")
     ap.add_argument("--batch", type=int, default=None)
     ap.add_argument("--prompt", type=int, default=None)
@@ -291,7 +298,7 @@ def main():
         runpy.run_path(sys.argv[0], run_name="__main__")
         return 0
     args.warmup = max(args.warmup, 3)
-    if args.config in ("mixtral-pp", "qlora-dp", "7b-spec", "latent", "hybrid", "multistream"):
+    if args.config in ("mixtral-pp", "qlora-dp", "7b-spec", "latent", "hybrid", "multistream", "parallel-block"):
         return other_config(args)
     if args.config == "7b" and args.model == "auto":
         args.model = "llama2-7b"

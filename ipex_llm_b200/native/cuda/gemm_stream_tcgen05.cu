@@ -255,18 +255,22 @@ gemm_stream_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_consta
             if (writer && j < lim)
               out[(int64_t)j * a.ldo] = from_float<T>(g / (1.0f + __expf(-a.alpha * g)) * (u + 1.0f));
           }
-        } else if (n < a.N) {
-          if (a.act == 6) {
-            T* out = reinterpret_cast<T*>(a.out) + r0 * a.ldo + n;
-            const T* mul = reinterpret_cast<const T*>(a.mul) + n;
+        } else if (a.act == 6) {
+          // a lane looks up one token's row for the whole warp; all loads before the first store
+          const int64_t id = a.ids[r0 + min(lane, lim - 1)], row = id < 0 ? 0 : id >= a.mul_rows ? a.mul_rows - 1 : id;
+          const T* mul = reinterpret_cast<const T*>(a.mul) + min(n, a.N - 1);
+          T* out = reinterpret_cast<T*>(a.out) + r0 * a.ldo + n;
+          T e[32];
 #pragma unroll
-            for (int j = 0; j < 32; ++j) {
-              if (j < lim) {
-                const int64_t id = a.ids[r0 + j], row = id < 0 ? 0 : id >= a.mul_rows ? a.mul_rows - 1 : id;
-                out[(int64_t)j * a.ldo] = from_float<T>(gelu_tanh(__uint_as_float(v[j]) + bn) * to_float<T>(mul[row * a.ldm]));
-              }
-            }
-          } else if (a.out_mode == 0) {
+          for (int j = 0; j < 32; ++j) e[j] = mul[__shfl_sync(0xffffffffu, row, j) * a.ldm];
+#pragma unroll
+          for (int j = 0; j < 32; ++j) {
+            const float z = __uint_as_float(v[j]) + bn, y = 1.5957691216057308f * (z + 0.044715f * z * z * z);
+            if (n < a.N && j < lim)
+              out[(int64_t)j * a.ldo] = from_float<T>(__fdividef(z, 1.0f + __expf(-y)) * to_float<T>(e[j]));
+          }
+        } else if (n < a.N) {
+          if (a.out_mode == 0) {
             T* out = reinterpret_cast<T*>(a.out) + r0 * a.ldo + n;
 #pragma unroll
             for (int j = 0; j < 32; ++j) {

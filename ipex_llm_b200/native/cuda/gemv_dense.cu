@@ -320,6 +320,15 @@ __device__ __forceinline__ void mma16816(float (&c)[4], uint32_t a0, uint32_t a1
                  : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
+// eight fp32 values in T
+template <typename T>
+__device__ __forceinline__ uint4 converted(const float* p) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  __align__(16) T o[8] = {DT<T>::from_f(a.x), DT<T>::from_f(a.y), DT<T>::from_f(a.z), DT<T>::from_f(a.w),
+                          DT<T>::from_f(b.x), DT<T>::from_f(b.y), DT<T>::from_f(b.z), DT<T>::from_f(b.w)};
+  return *reinterpret_cast<const uint4*>(o);
+}
+
 // 16-bit weights on the tensor cores, NT * 8 tokens: a tile is 16 weight rows (the A operand, straight from global
 // memory), `split` warps of the CTA share its K range and meet once per tile in shared memory.  The k order inside a
 // 32-wide block is permuted alike for both operands, so that a lane's fragment is one 16-byte load: lane (g, t) holds
@@ -343,10 +352,11 @@ __global__ void __launch_bounds__(kThreads) gemv_mma_kernel(GemvRowsArgs a, int 
     if (lane < 16 && row < a.N && bytes > 0) prefetch_l2_bulk(weight_row<T>(a, row) + k0, (uint32_t)bytes);
   }
   pdl_wait();
-  const bool staged = a.norm_w != nullptr || a.x_f32;
+  const bool staged = a.norm_w != nullptr;
   if (staged)
-    stage_rows<T>(sx, a.kp, a.x, a.ldx, reinterpret_cast<const T*>(a.norm_w), a.eps, a.M, a.K, red, a.x_f32 != 0);
+    stage_rows<T>(sx, a.kp, a.x, a.ldx, reinterpret_cast<const T*>(a.norm_w), a.eps, a.M, a.K, red);
   const T* xs[NT];
+  const float* xf[NT];           // rows of the 32-bit stream, converted on the way
   bool xon[NT];
 #pragma unroll
   for (int n = 0; n < NT; ++n) {
@@ -354,6 +364,7 @@ __global__ void __launch_bounds__(kThreads) gemv_mma_kernel(GemvRowsArgs a, int 
     xon[n] = m < a.M;
     xs[n] = (staged ? sx + (size_t)(xon[n] ? m : 0) * a.kp
                     : reinterpret_cast<const T*>(a.x) + (int64_t)(xon[n] ? m : 0) * a.ldx) + t * 8;
+    xf[n] = reinterpret_cast<const float*>(a.x) + (int64_t)(xon[n] ? m : 0) * a.ldx + t * 8;
   }
   int par = 0;
   for (int base = blockIdx.x * tpc; base < ntile; base += gridDim.x * tpc, par ^= 1) {
@@ -377,7 +388,8 @@ __global__ void __launch_bounds__(kThreads) gemv_mma_kernel(GemvRowsArgs a, int 
           const bool in = kb + u < kb1 && k + t * 8 < a.K;
 #pragma unroll
           for (int n = 0; n < NT; ++n) {
-            const uint4 x = in && xon[n] ? *reinterpret_cast<const uint4*>(xs[n] + k) : make_uint4(0, 0, 0, 0);
+            uint4 x = make_uint4(0, 0, 0, 0);
+            if (in && xon[n]) x = a.x_f32 ? converted<T>(xf[n] + k) : *reinterpret_cast<const uint4*>(xs[n] + k);
             mma16816<T>(acc[0][n], r0[u].x, r1[u].x, r0[u].y, r1[u].y, x.x, x.y);
             mma16816<T>(acc[1][n], r0[u].z, r1[u].z, r0[u].w, r1[u].w, x.z, x.w);
           }
@@ -482,7 +494,7 @@ template <typename T, int NT>
 cudaError_t launch_gemv_mma(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
   auto kern = gemv_mma_kernel<T, NT>;
   a.kp = (a.K + 31) / 32 * 32 + 32;        // 64 bytes of skew between rows: neighbouring tokens in different banks
-  const size_t smem = (size_t)2 * kWarps * NT * 128 * sizeof(float) + (a.norm_w != nullptr || a.x_f32 ? (size_t)a.M * a.kp * sizeof(T) : 0);
+  const size_t smem = (size_t)2 * kWarps * NT * 128 * sizeof(float) + (a.norm_w != nullptr ? (size_t)a.M * a.kp * sizeof(T) : 0);
   if (smem > 226 * 1024) return cudaErrorInvalidValue;
   if (smem > 40 * 1024) {                 // (static shared memory counts against the default limit too)
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -502,7 +514,7 @@ bool mma_from(const GemvRowsArgs& a) { return a.M >= g_mma_from; }
 template <typename T>
 cudaError_t pick_m(GemvRowsArgs& a, bool pdl, cudaStream_t st) {
   if constexpr (sizeof(T) == 2) {
-    const bool direct = a.norm_w != nullptr || a.x_f32 || ((reinterpret_cast<uintptr_t>(a.x) & 15) == 0 && a.ldx % 8 == 0);
+    const bool direct = a.norm_w != nullptr || ((reinterpret_cast<uintptr_t>(a.x) & 15) == 0 && a.ldx % (a.x_f32 ? 4 : 8) == 0);
     if (a.vec && direct && mma_from(a) && (!gated(a.act) || a.interleaved)) {
       if (a.M <= 8) return launch_gemv_mma<T, 1>(a, pdl, st);
       return launch_gemv_mma<T, 2>(a, pdl, st);

@@ -83,7 +83,7 @@ struct StepArgs {
 
 // A warp owns the state rows warp, warp + 8, ...; a lane CV neighbouring columns of the CTA's 32 CV.
 template <typename T, int NR, int CV>
-__global__ void __launch_bounds__(kThreads, NR * CV <= 32 ? 2 : 1) general_step_kernel(StepArgs s) {
+__global__ void __launch_bounds__(kThreads, NR * CV <= 64 ? 2 : 1) general_step_kernel(StepArgs s) {
   constexpr int VS = 32 * CV;
   extern __shared__ __align__(16) float sm[];
   const Common& a = s.c;
@@ -307,74 +307,170 @@ struct ChunkArgs {
 };
 
 constexpr int kLdM = 36;      // row stride of the 32 x 32 matrices
-size_t prep_smem(const Scratch& L, int rank) {
-  return ((size_t)4 * kC * (L.Dp + 4) + (size_t)kC * (L.slices * kVS + 8) + 7 * kC * kLdM + 4 * (L.Dp + 1) + 2 * kC +
-          (size_t)kC * rank + (size_t)rank * (L.Dp + 1)) * sizeof(float);
-}
+constexpr int kR = 64;        // columns of the decays' projection at a time
+// Shared memory of general_prep: four arrays of 32 rows; what the decays' projection needs, later the 32 x 32 matrices; sums.
+struct PrepLayout {
+  int ld, ldv, ldu, lds;      // row strides: the arrays, v (in T), up (in T), low
+  int mats, tot, floats;
+  __host__ __device__ PrepLayout(const Scratch& L)
+      : ld(L.Dp + 4), ldv(L.slices * kVS + 8), ldu(kR + 8), lds(kR + 4) {
+    mats = 4 * kC * ld + kC * ldv / 2;
+    const int proj = L.Dp * ldu / 2 + kC * lds, matrices = 7 * kC * kLdM;
+    tot = mats + (proj > matrices ? proj : matrices);
+    floats = tot + 4 * (L.Dp + 1) + kC;
+  }
+};
+size_t prep_smem(const Scratch& L) { return (size_t)PrepLayout(L).floats * sizeof(float); }
 size_t chunk_smem(const Scratch& L, int stages) {
   return ((size_t)(L.Dm + kC) * L.ldu + (size_t)stages * L.stage()) * sizeof(float);
 }
 
-template <typename T>
-__global__ void __launch_bounds__(kThreads) general_prep_kernel(ChunkArgs s) {
+__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(tc5::smem_u32(dst)), "l"(src) : "memory");
+}
+
+// NZ: 64-channel tiles of a head.
+template <typename T, int NZ>
+__global__ void __launch_bounds__(kThreads, NZ == 1 ? 3 : NZ == 2 ? 2 : 1) general_prep_kernel(ChunkArgs s) {
   extern __shared__ __align__(16) float sm[];
   const Common& a = s.c;
   const int D = a.dim, V = a.vdim, h = blockIdx.y, chunk = s.c0 + blockIdx.x, rank = a.rank;
   const Scratch L(D, V);
-  const int Dp = L.Dp, Vp = L.slices * kVS, ld = Dp + 4, ldv = Vp + 8;
+  const PrepLayout PL(L);
+  const int Dp = L.Dp, Vp = L.slices * kVS, ld = PL.ld, ldv = PL.ldv;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
   float* sq = sm;                        // [32][Dp + 4]: r, then q
   float* sk = sq + kC * ld;              // k, then g
   float* sp = sk + kC * ld;              // running sum of the decays' logarithms, then p
   float* sb = sp + kC * ld;              // rates, then b
-  float* sv = sb + kC * ld;              // [32][Vp + 8]
-  float* mA = sv + kC * ldv;             // 32 x 32 matrices
+  T* sv = reinterpret_cast<T*>(sb + kC * ld);                // [32][Vp + 8]
+  float* mA = sm + PL.mats;              // 32 x 32 matrices
   float* mM = mA + kC * kLdM;
   float* mE = mM + kC * kLdM;
   float* mH = mE + kC * kLdM;
   float* mT = mH + kC * kLdM;
   float* mTM = mT + kC * kLdM;
   float* mHT = mTM + kC * kLdM;
-  float* tot = mHT + kC * kLdM;          // [4][Dp + 1]: logarithms of eight tokens' decays
+  T* sup = reinterpret_cast<T*>(mA);     // before them: [Dp][kR + 8] of `up`, ...
+  float* slow = mA + L.Dp * PL.ldu / 2;  // ... [32][kR + 4] of tanh(low)
+  float* tot = sm + PL.tot;              // [4][Dp + 1]: logarithms of eight tokens' decays
   float* sik = tot + 4 * (Dp + 1);       // [32] 1 / |k|
-  float* sone = sik + kC;                // [32] (padding)
-  float* slow = sone + kC;               // [32][rank]
-  float* sup = slow + kC * rank;         // [rank][Dp + 1]
   const int seq = s.chunk_seq[chunk], row0 = a.seq_row[seq], off = (chunk - s.seq_chunk[seq]) * kC;
   const int n = min(kC, a.seq_len[seq] - off), t0 = row0 + off;
   float* out = s.scratch + ((int64_t)(chunk - s.c0) * a.heads + h) * L.floats();
   const T* proj = reinterpret_cast<const T*>(a.proj) + (int64_t)t0 * a.ldp;
-
-  // ---- operands (zeros behind the sequence's end and past the sizes)
-  const T* up = reinterpret_cast<const T*>(a.up) + (int64_t)h * D * rank;
-  for (int i = tid; i < D * rank; i += kThreads) sup[i % rank * (Dp + 1) + i / rank] = DT<T>::to_f(up[i]);
-  for (int i = tid; i < kC * rank; i += kThreads) {
-    const int t = i / rank;
-    slow[i] = t < n ? tanhf(a.low[(int64_t)(t0 + t) * a.ldl + i - t * rank]) : 0.f;
-  }
   const int rc = h * D, kcol = a.heads * D + rc, vcol = 2 * a.heads * D + h * V, acol = a.heads * (2 * D + V) + rc;
   const bool vec = D % 8 == 0 && V % 8 == 0 && a.ldp % 8 == 0 && (reinterpret_cast<uintptr_t>(a.proj) & 15) == 0;
-  if (vec) {
-    const int nd = D / 8, nvv = Vp / 8, per = 3 * nd + nvv;
-    for (int i = tid; i < kC * per; i += kThreads) {
-      const int t = i / per, c = i % per;
-      const int what = min(c / nd, 3), e0 = (c - what * nd) * 8;
-      uint4 raw = make_uint4(0, 0, 0, 0);
-      const bool on = t < n && (what < 3 || e0 < V);
-      if (on)
-        raw = *reinterpret_cast<const uint4*>(proj + (int64_t)t * a.ldp +
-                                              (what == 0 ? rc : what == 1 ? kcol : what == 2 ? acol : vcol) + e0);
-      const T* e = reinterpret_cast<const T*>(&raw);
-      float* dst = what == 0 ? sq + t * ld + e0 : what == 1 ? sk + t * ld + e0 : what == 2 ? sb + t * ld + e0 : sv + t * ldv + e0;
-      float x[8];
-#pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        x[j] = DT<T>::to_f(e[j]);
-        if (what == 2) x[j] = on ? sigmoidf(x[j] + a.rate_bias[rc + e0 + j]) : 0.f;
-      }
-#pragma unroll
-      for (int j = 0; j < 8; j += 4) *reinterpret_cast<float4*>(dst + j) = make_float4(x[j], x[j + 1], x[j + 2], x[j + 3]);
+
+  // ---- operands (zeros behind the sequence's end and past the sizes): the first loads are in flight during the projection
+  constexpr int kEarly = NZ <= 2 ? 4 * NZ : 8;
+  const int nd = D / 8, per = 3 * nd + Vp / 8;
+  uint4 early[kEarly];
+  auto fetch = [&](int i) {
+    const int t = i / per, c = i % per, what = min(c / max(nd, 1), 3), e0 = (c - what * nd) * 8;
+    uint4 raw = make_uint4(0, 0, 0, 0);
+    if (i < kC * per && t < n && (what < 3 || e0 < V))
+      raw = *reinterpret_cast<const uint4*>(proj + (int64_t)t * a.ldp +
+                                            (what == 0 ? rc : what == 1 ? kcol : what == 2 ? acol : vcol) + e0);
+    return raw;
+  };
+  auto file = [&](int i, const uint4& raw) {
+    if (i >= kC * per) return;
+    const int t = i / per, c = i % per, what = min(c / nd, 3), e0 = (c - what * nd) * 8;
+    if (what == 3) {
+      *reinterpret_cast<uint4*>(sv + t * ldv + e0) = raw;
+      return;
     }
+    const T* e = reinterpret_cast<const T*>(&raw);
+    float* dst = (what == 0 ? sq : what == 1 ? sk : sb) + t * ld + e0;
+    float x[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) x[j] = DT<T>::to_f(e[j]);
+    if (what == 2) {
+      const float4 b0 = *reinterpret_cast<const float4*>(a.rate_bias + rc + e0);
+      const float4 b1 = *reinterpret_cast<const float4*>(a.rate_bias + rc + e0 + 4);
+      const float b[8] = {b0.x, b0.y, b0.z, b0.w, b1.x, b1.y, b1.z, b1.w};
+#pragma unroll
+      for (int j = 0; j < 8; ++j) x[j] = t < n ? sigmoidf(x[j] + b[j]) : 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < 8; j += 4) *reinterpret_cast<float4*>(dst + j) = make_float4(x[j], x[j + 1], x[j + 2], x[j + 3]);
+  };
+  if (vec) {
+#pragma unroll
+    for (int u = 0; u < kEarly; ++u) early[u] = fetch(tid + u * kThreads);
+  }
+  // ---- z = up tanh(low): `up` is exact in one tf32 part; a warp has every eighth tile of eight channels, both row tiles
+  float z[NZ][2][4];
+#pragma unroll
+  for (int j = 0; j < NZ; ++j)
+#pragma unroll
+    for (int m = 0; m < 2; ++m)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) z[j][m][i] = 0.f;
+  const T* up = reinterpret_cast<const T*>(a.up) + (int64_t)h * D * rank;
+  for (int r0 = 0; r0 < rank; r0 += kR) {
+    const int nr = min(kR, rank - r0), nk = (nr + 7) / 8 * 8;
+    if (r0 > 0) __syncthreads();
+    if (rank % 8 == 0 && (reinterpret_cast<uintptr_t>(up) & 15) == 0) {
+      const int nv = nk / 8;
+      for (int i = tid; i < D * nv; i += kThreads) {
+        const int d = i / nv, c = (i - d * nv) * 8;
+        cp_async16(sup + d * PL.ldu + c, up + (int64_t)d * rank + r0 + c);
+      }
+      for (int i = D * nk + tid; i < Dp * nk; i += kThreads) sup[i / nk * PL.ldu + i % nk] = DT<T>::from_f(0.f);
+    } else {
+      for (int i = tid; i < Dp * nk; i += kThreads) {
+        const int d = i / nk, c = i - d * nk;
+        sup[d * PL.ldu + c] = d < D && c < nr ? up[(int64_t)d * rank + r0 + c] : DT<T>::from_f(0.f);
+      }
+    }
+    for (int i = tid; i < kC * nk; i += kThreads) {
+      const int t = i / nk, c = i - t * nk;
+      slow[t * PL.lds + c] = t < n && c < nr ? tanhf(a.low[(int64_t)(t0 + t) * a.ldl + r0 + c]) : 0.f;
+    }
+    asm volatile("cp.async.commit_group;\ncp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    for (int k0 = 0; k0 < nk; k0 += 8) {
+      FragA fa[2];
+#pragma unroll
+      for (int m = 0; m < 2; ++m) fa[m] = frag_a([&](int r, int k) { return slow[(m * 16 + r) * PL.lds + k0 + k]; }, g, t4);
+#pragma unroll
+      for (int j = 0; j < NZ; ++j) {
+        const int n0 = (j * 8 + warp) * 8;
+        if (n0 < Dp) {
+          const T* b = sup + (n0 + g) * PL.ldu + k0 + t4;
+          const uint32_t fb[2] = {__float_as_uint(DT<T>::to_f(b[0])), __float_as_uint(DT<T>::to_f(b[4]))};
+#pragma unroll
+          for (int m = 0; m < 2; ++m) {
+            mma_tf32(z[j][m], fa[m].lo, fb);
+            mma_tf32(z[j][m], fa[m].hi, fb);
+          }
+        }
+      }
+    }
+  }
+  // ---- logarithms of the decays
+#pragma unroll
+  for (int j = 0; j < NZ; ++j) {
+    const int n0 = (j * 8 + warp) * 8;
+    if (n0 < Dp) {
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int d = n0 + 2 * t4 + i;
+        const float b = d < D ? a.bias[rc + d] : 0.f;
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          const int t = g + 8 * q;
+          sp[t * ld + d] = t < n && d < D ? -a.c * sigmoidf(z[j][q >> 1][(q & 1) * 2 + i] + b) : 0.f;
+        }
+      }
+    }
+  }
+  if (vec) {
+#pragma unroll
+    for (int u = 0; u < kEarly; ++u) file(tid + u * kThreads, early[u]);
+    for (int i = tid + kEarly * kThreads; i < kC * per; i += kThreads) file(i, fetch(i));
   } else {
     for (int i = tid; i < kC * Dp; i += kThreads) {
       const int t = i / Dp, d = i % Dp;
@@ -386,28 +482,18 @@ __global__ void __launch_bounds__(kThreads) general_prep_kernel(ChunkArgs s) {
     }
     for (int i = tid; i < kC * Vp; i += kThreads) {
       const int t = i / Vp, c = i % Vp;
-      sv[t * ldv + c] = t < n && c < V ? DT<T>::to_f(proj[(int64_t)t * a.ldp + vcol + c]) : 0.f;
+      sv[t * ldv + c] = t < n && c < V ? proj[(int64_t)t * a.ldp + vcol + c] : DT<T>::from_f(0.f);
     }
   }
   __syncthreads();
-  // ---- logarithms of the decays, summed over the eight tokens of an item; lengths of the keys
+  // ---- ... summed over the eight tokens of an item; lengths of the keys
   for (int i = tid; i < Dp * (kC / 8); i += kThreads) {
-    const int d = i % Dp, b8 = i / Dp, tb = b8 * 8;
-    float z[8];
-    const float b = d < D ? a.bias[rc + d] : 0.f;
-#pragma unroll
-    for (int t = 0; t < 8; ++t) z[t] = b;
-    if (d < D)
-      for (int r = 0; r < rank; ++r) {
-        const float u = sup[r * (Dp + 1) + d];
-#pragma unroll
-        for (int t = 0; t < 8; ++t) z[t] = fmaf(slow[(tb + t) * rank + r], u, z[t]);
-      }
+    const int d = i % Dp, b8 = i / Dp;
     float run = 0.f;
 #pragma unroll
     for (int t = 0; t < 8; ++t) {
-      if (tb + t < n && d < D) run -= a.c * sigmoidf(z[t]);
-      sp[(tb + t) * ld + d] = run;
+      run += sp[(b8 * 8 + t) * ld + d];
+      sp[(b8 * 8 + t) * ld + d] = run;
     }
     tot[b8 * (Dp + 1) + d] = run;
   }
@@ -552,13 +638,12 @@ __global__ void __launch_bounds__(kThreads) general_prep_kernel(ChunkArgs s) {
     // a warp keeps its row tile of [T; H T; (T M)^T] and walks the columns
     for (int m = 0; m < 6; ++m) {
       const int kind = m >> 1, m0 = (m & 1) * 16;
+      const float* mat = kind == 0 ? mT : kind == 1 ? mHT : mTM;
+      const int rs = kind == 2 ? 1 : kLdM, cs = kind == 2 ? kLdM : 1;
       FragA fm[4];
 #pragma unroll
       for (int f = 0; f < 4; ++f)
-        fm[f] = frag_a([&](int r, int k) {
-          return kind == 0 ? mT[(m0 + r) * kLdM + f * 8 + k] : kind == 1 ? mHT[(m0 + r) * kLdM + f * 8 + k]
-                                                                         : mTM[(f * 8 + k) * kLdM + m0 + r];
-        }, g, t4);
+        fm[f] = frag_a([&](int r, int k) { return mat[(m0 + r) * rs + (f * 8 + k) * cs]; }, g, t4);
       for (int n0 = warp * 8; n0 < Dp; n0 += kThreads / 4) {
         Acc x;
         x.zero();
@@ -614,8 +699,8 @@ __global__ void __launch_bounds__(kThreads) general_prep_kernel(ChunkArgs s) {
       }, g, t4);
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        const float* v = sv + (f * 8 + t4) * ldv + ng * 32 + j * 8 + g;
-        const uint32_t fb[2] = {__float_as_uint(v[0]), __float_as_uint(v[4 * ldv])};
+        const T* v = sv + (f * 8 + t4) * ldv + ng * 32 + j * 8 + g;
+        const uint32_t fb[2] = {__float_as_uint(DT<T>::to_f(v[0])), __float_as_uint(DT<T>::to_f(v[4 * ldv]))};
         mma_tf32(acc[j], fa.hi, fb);
         mma_tf32(low[j], fa.lo, fb);
       }
@@ -843,7 +928,7 @@ Common common_args(const void* proj, int64_t ldp, const float* low, int64_t ldl,
 // Can the chunked form take these sizes and decays of at least exp(-c)?
 IPEX_API int ipex_general_chunks_ok(int dim, int vdim, int rank, float c) {
   const Scratch L(dim, vdim);
-  return dim >= 1 && dim <= 256 && vdim >= 1 && rank >= 1 && c >= 0.f && c * kC <= kMaxLog && prep_smem(L, rank) <= kSmemMax &&
+  return dim >= 1 && dim <= 256 && vdim >= 1 && rank >= 1 && c >= 0.f && c * kC <= kMaxLog && prep_smem(L) <= kSmemMax &&
          chunk_smem(L, 1) <= kSmemMax;
 }
 IPEX_API int64_t ipex_general_scratch_floats(int dim, int vdim) { return Scratch(dim, vdim).floats(); }
@@ -895,10 +980,11 @@ IPEX_API int ipex_general_chunks(const void* proj, int64_t ldp, const float* low
                    chunk_seq, seq_chunk, scratch, raw, err, c0, c1};
     cudaStream_t st = (cudaStream_t)stream;
     const Scratch L(dim, vdim);
-    const size_t ps = prep_smem(L, rank);
-    cudaError_t e = cudaFuncSetAttribute(general_prep_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ps);
+    const size_t ps = prep_smem(L);
+    auto prep = dim <= 64 ? general_prep_kernel<T, 1> : dim <= 128 ? general_prep_kernel<T, 2> : general_prep_kernel<T, 4>;
+    cudaError_t e = cudaFuncSetAttribute(prep, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ps);
     if (e != cudaSuccess) return e;
-    general_prep_kernel<T><<<dim3(c1 - c0, heads), kThreads, ps, st>>>(s);
+    prep<<<dim3(c1 - c0, heads), kThreads, ps, st>>>(s);
     e = cudaGetLastError();
     if (e != cudaSuccess) return e;
     int stages = 3;

@@ -224,7 +224,7 @@ struct ChunkArgs {
   int vec;                  // rows of proj and ring can be read 16 bytes at a time
 };
 
-// Convolution and silu of `width` neighbouring channels of a chunk from channel c0 on; put(token, channel - c0, value).  ws:
+// Convolution and silu of `width` neighbouring channels of a chunk from channel c0 on; put(token, channel - c0, n values).  ws:
 // room for [taps][width] and a bias row.
 template <typename T, int TP, typename F>
 __device__ __forceinline__ void conv_chunk(const Common& a, bool vec, int c0, int width, int t0, int row0, int off, int p0,
@@ -232,26 +232,43 @@ __device__ __forceinline__ void conv_chunk(const Common& a, bool vec, int c0, in
   const int tid = threadIdx.x;
   const T* w = reinterpret_cast<const T*>(a.conv) + (int64_t)c0 * a.taps;
   float* bs = ws + a.taps * width;
-  for (int i = tid; i < width * a.taps; i += kThreads) ws[i % a.taps * width + i / a.taps] = DT<T>::to_f(w[i]);
-  for (int i = tid; i < width; i += kThreads) bs[i] = a.conv_b[c0 + i];
+  const int nt = blockDim.x;
+  for (int i = tid; i < width; i += nt) {
+    for (int j = 0; j < a.taps; ++j) ws[j * width + i] = DT<T>::to_f(w[i * a.taps + j]);
+    bs[i] = a.conv_b[c0 + i];
+  }
   __syncthreads();
   if (vec) {
     const int nvec = width / 8;
-    for (int i = tid; i < nvec * (kC / 4); i += kThreads) {
+    for (int i = tid; i < nvec * (kC / 4); i += nt) {
       const int c = (i % nvec) * 8, first = (i / nvec) * 4;
       float acc[4][8];
       conv_block<T, TP>(a, c0 + c, t0, row0, p0, start, slot, n, first, ws + c, width, acc, bs + c);
 #pragma unroll
-      for (int j = 0; j < 4; ++j)
+      for (int j = 0; j < 4; ++j) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) put(first + j, c + e, first + j < n ? fast_silu(acc[j][e]) : 0.f);
+        for (int e = 0; e < 8; ++e) acc[j][e] = first + j < n ? fast_silu(acc[j][e]) : 0.f;
+        put(first + j, c, acc[j], std::integral_constant<int, 8>{});
+      }
     }
   } else {
-    for (int i = tid; i < kC * width; i += kThreads) {
+    for (int i = tid; i < kC * width; i += nt) {
       const int t = i / width, c = i % width;
-      put(t, c, t < n ? conv_silu<T>(a, c0 + c, t0 + t, off + t, p0 + t, start, slot, w + (int64_t)c * a.taps + a.taps - 1, bs[c])
-                      : 0.f);
+      const float v = t < n ? conv_silu<T>(a, c0 + c, t0 + t, off + t, p0 + t, start, slot, w + (int64_t)c * a.taps + a.taps - 1, bs[c])
+                            : 0.f;
+      put(t, c, &v, std::integral_constant<int, 1>{});
     }
+  }
+}
+
+// n neighbouring values (n = 8: 16-byte aligned)
+template <int N>
+__device__ __forceinline__ void put_values(float* dst, const float* v) {
+  if constexpr (N == 8) {
+    *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]);
+    *reinterpret_cast<float4*>(dst + 4) = make_float4(v[4], v[5], v[6], v[7]);
+  } else {
+    dst[0] = v[0];
   }
 }
 
@@ -277,10 +294,10 @@ __global__ void __launch_bounds__(kThreads) ssd_groups_kernel(ChunkArgs s) {
       sB[t * ld + d] = sC[t * ld + d] = 0.f;
     }
   conv_chunk<T, TP>(a, s.vec != 0, bc, D, t0, row0, off, p0, start, slot, n, ws,
-                    [&](int t, int c, float v) { sB[t * ld + c] = v; });
+                    [&](int t, int c, const float* v, auto k) { put_values<decltype(k)::value>(sB + t * ld + c, v); });
   __syncthreads();
   conv_chunk<T, TP>(a, s.vec != 0, bc + a.groups * D, D, t0, row0, off, p0, start, slot, n, ws,
-                    [&](int t, int c, float v) { sC[t * ld + c] = v; });
+                    [&](int t, int c, const float* v, auto k) { put_values<decltype(k)::value>(sC + t * ld + c, v); });
   __syncthreads();
   for (int i = tid; i < kC * Dp; i += kThreads) {
     const int t = i / Dp, d = i % Dp;
@@ -298,6 +315,7 @@ __global__ void __launch_bounds__(kThreads) ssd_groups_kernel(ChunkArgs s) {
   for (int i = 0; i < 4; ++i) out[L.cb() + (m0 + g + 8 * (i >> 1)) * L.ldp + n0 + 2 * t4 + (i & 1)] = x.get(i);
 }
 
+// 64 to 256 threads
 template <typename T, int TP>
 __global__ void __launch_bounds__(kThreads) ssd_heads_kernel(ChunkArgs s) {
   extern __shared__ __align__(16) float sm[];      // [taps + 1][vdim] convolution weights
@@ -308,7 +326,7 @@ __global__ void __launch_bounds__(kThreads) ssd_heads_kernel(ChunkArgs s) {
   const Common& a = s.c;
   const int V = a.vdim, h = blockIdx.y, chunk = s.c0 + blockIdx.x, gi = h / (a.heads / a.groups);
   const Scratch L(a.dim, V);
-  const int tid = threadIdx.x, lane = tid & 31;
+  const int tid = threadIdx.x, nt = blockDim.x, lane = tid & 31;
   const int seq = s.chunk_seq[chunk], row0 = a.seq_row[seq], off = (chunk - s.seq_chunk[seq]) * kC;
   const int n = min(kC, a.seq_len[seq] - off), t0 = row0 + off;
   const int slot = a.slot[row0], start = a.start[slot], p0 = a.pos[row0] + off;
@@ -335,15 +353,19 @@ __global__ void __launch_bounds__(kThreads) ssd_heads_kernel(ChunkArgs s) {
   }
   const int Vp = L.slices * kVS;
   if (Vp > V)
-    for (int i = tid; i < kC * (Vp - V); i += kThreads) {
+    for (int i = tid; i < kC * (Vp - V); i += nt) {
       const int t = i / (Vp - V), c = V + i % (Vp - V);
       out[L.x(c / kVS) + t * L.ldv + c % kVS] = 0.f;
     }
-  conv_chunk<T, TP>(a, s.vec != 0, h * V, V, t0, row0, off, p0, start, slot, n, sm, [&](int t, int c, float v) {
-    out[L.x(c / kVS) + t * L.ldv + c % kVS] = rounded<T>(v);
+  conv_chunk<T, TP>(a, s.vec != 0, h * V, V, t0, row0, off, p0, start, slot, n, sm, [&](int t, int c, const float* v, auto k) {
+    constexpr int N = decltype(k)::value;
+    float x[N];
+#pragma unroll
+    for (int e = 0; e < N; ++e) x[e] = rounded<T>(v[e]);
+    put_values<N>(out + L.x(c / kVS) + t * L.ldv + c % kVS, x);
   });
   // (conv_chunk's barrier: the sums are in place)
-  for (int i = tid; i < kC * kC; i += kThreads) {
+  for (int i = tid; i < kC * kC; i += nt) {
     const int t = i >> 5, j = i & 31;
     out[t * L.ldp + j] = j <= t ? cb[t * L.ldp + j] * sD[j] * expf((float)(sL[t] - sL[j])) : 0.f;
   }
@@ -353,13 +375,13 @@ size_t groups_smem(const Scratch& L, int D, int taps) {
   return ((size_t)2 * kC * (L.Dp + 4) + (size_t)(taps + 1) * D) * sizeof(float);
 }
 size_t chunk_smem(const Scratch& L, int stages) {
-  return ((size_t)stages * L.stage() + 2 * 4 * kC * 36) * sizeof(float);
+  return ((size_t)stages * L.stage() + 4 * kC * 36) * sizeof(float);
 }
 
 // CTA = 32 state columns of one head of one sequence.  Warp (vt, dg): columns 16 vt .. + 15, channel tiles of share dg; S^T
 // in accumulator fragments.  The four shares' read-outs meet in shared memory.
-template <int MT>
-__global__ void __launch_bounds__(kThreads, 1) ssd_chunks_kernel(ChunkArgs s, int stages) {
+template <int MT, int PER_SM>
+__global__ void __launch_bounds__(kThreads, PER_SM) ssd_chunks_kernel(ChunkArgs s, int stages) {
   extern __shared__ __align__(16) float sm[];
   __shared__ __align__(8) uint64_t full[4];
   __shared__ int abort_word;
@@ -374,7 +396,7 @@ __global__ void __launch_bounds__(kThreads, 1) ssd_chunks_kernel(ChunkArgs s, in
   if (ca >= cb) return;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
   const int vt = warp & 1, dg = warp >> 1;
-  float* red = sm + stages * L.stage();        // [2][4][32][36]
+  float* red = sm + stages * L.stage();        // [4][32][36]
   const int row0 = a.seq_row[seq], len = a.seq_len[seq];
   const int slot = a.slot[row0], start = a.start[slot], p0 = a.pos[row0];
   float* st = a.state + (((int64_t)slot * a.heads + h) * D) * V + v0;
@@ -474,7 +496,7 @@ __global__ void __launch_bounds__(kThreads, 1) ssd_chunks_kernel(ChunkArgs s, in
           for (int n = 0; n < 4; ++n)
             if (n >= k) mac2(o[n], va[k], frag_b([&](int kk, int j) { return P[(n * 8 + j) * L.ldp + k * 8 + kk]; }, g, t4));
         }
-      float* rd = red + ((at & 1) * 4 + dg) * (kC * 36) + vt * 16;
+      float* rd = red + dg * (kC * 36) + vt * 16;
 #pragma unroll
       for (int n = 0; n < 4; ++n)
 #pragma unroll
@@ -520,7 +542,7 @@ __global__ void __launch_bounds__(kThreads, 1) ssd_chunks_kernel(ChunkArgs s, in
     }
     if (tid == 0) fetch(c + stages);
     const int off = (c - first) * kC;
-    const float* rd = red + (at & 1) * 4 * (kC * 36);
+    const float* rd = red;
 #pragma unroll
     for (int i = 0; i < kC * kVS / kThreads; ++i) {
       const int t = warp + 8 * i;
@@ -528,6 +550,7 @@ __global__ void __launch_bounds__(kThreads, 1) ssd_chunks_kernel(ChunkArgs s, in
                       (rd[(2 * kC + t) * 36 + lane] + rd[(3 * kC + t) * 36 + lane]);
       if (off + t < len && lane < nv) s.raw[((int64_t)(row0 + off + t) * a.heads + h) * V + v0 + lane] = fmaf(skip, xs[i], y);
     }
+    __syncthreads();                           // the sums are read
   }
   if (!ok) {                                   // copies in flight still write to this CTA's memory
     if (tid == 0)
@@ -649,13 +672,18 @@ IPEX_API int ipex_ssd_chunks(const void* proj, int64_t ldp, const float* dt, int
     prep_g<<<dim3(c1 - c0, groups), kThreads, gs, st>>>(s);
     e = cudaGetLastError();
     if (e != cudaSuccess) return e;
-    prep_h<<<dim3(c1 - c0, heads), kThreads, hs, st>>>(s);
+    const int items = vdim / 8 * (kC / 4), ht = items <= 64 ? 64 : items <= 128 ? 128 : kThreads;
+    prep_h<<<dim3(c1 - c0, heads), ht, hs, st>>>(s);
     e = cudaGetLastError();
     if (e != cudaSuccess) return e;
+    // more CTAs than SMs: two per SM with fewer stages each
+    const bool pairs = dim <= 128 && (int64_t)L.slices * heads * seqs > 148;
     int stages = 4;
-    while (stages > 1 && chunk_smem(L, stages) > kSmemMax) --stages;
+    while (stages > 1 && chunk_smem(L, stages) > (pairs ? kSmemMax / 2 : kSmemMax)) --stages;
     const size_t cs = chunk_smem(L, stages);
-    auto kern = dim <= 64 ? ssd_chunks_kernel<2> : dim <= 128 ? ssd_chunks_kernel<4> : ssd_chunks_kernel<8>;
+    auto kern = dim <= 64    ? (pairs ? ssd_chunks_kernel<2, 2> : ssd_chunks_kernel<2, 1>)
+                : dim <= 128 ? (pairs ? ssd_chunks_kernel<4, 2> : ssd_chunks_kernel<4, 1>)
+                             : ssd_chunks_kernel<8, 1>;
     e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)cs);
     if (e != cudaSuccess) return e;
     kern<<<dim3(L.slices, heads, seqs), kThreads, cs, st>>>(s, stages);

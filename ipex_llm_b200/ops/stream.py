@@ -76,7 +76,7 @@ def gemv_rows(w, x, out, mode: int, norm=None, eps: float = 0.0, act: int = 0, s
     if norm is not None and M > 2 and w.dtype != torch.float32:
         x, norm = norm_stream(x, norm, eps, pdl=pdl), None
     raw = norm is None and x.dtype != w.dtype
-    if raw and M * (K + 64) * w.element_size() > 160 * 1024:      # more than a CTA can stage
+    if raw and (M > 8 or K % 8) and M * (K + 64) * w.element_size() > 160 * 1024:      # more than a CTA can stage
         x, raw = add_sides(x, (), (), None, eps, w.dtype, pdl=pdl), False
     rc = stream_lib().ipex_gemv_rows(ptr(w), w.stride(0), ptr(x), x.stride(0), ptr(norm), eps, ptr(bias), ptr(out),
                                      out.stride(0), ptr(w2), 0 if w2 is None else w2.shape[0], ptr(out2),
